@@ -14,3 +14,4 @@ from .supevik import SupevikConfig  # noqa: F401  (registers the architecture)
 from .fogapel import FogapelConfig  # noqa: F401  (registers the architecture)
 from .zosipel import ZosipelConfig  # noqa: F401  (registers the architecture)
 from .divadra import DivadraConfig  # noqa: F401  (registers the architecture)
+from .ditazen import DitazenConfig  # noqa: F401  (registers the architecture)

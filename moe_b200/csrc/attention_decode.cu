@@ -104,6 +104,7 @@ struct GateOut {
     const float* gate;
     int gate_ld;
     int dv;
+    int per_head;          // one logit a head, gate[t * gate_ld + h], instead of one a column
 };
 template <typename T>
 __device__ __forceinline__ void write_head_column(T* out, const GateOut go, int t, int nh, int h, int hd, int d,
@@ -116,7 +117,7 @@ __device__ __forceinline__ void write_head_column(T* out, const GateOut go, int 
     if (go.gate) {
         T r;
         st_f(&r, val);
-        val = ld_f(&r) * (1.0f / (1.0f + expf(-go.gate[(size_t)t * go.gate_ld + (size_t)h * go.dv + d])));
+        val = ld_f(&r) * (1.0f / (1.0f + expf(-go.gate[(size_t)t * go.gate_ld + (go.per_head ? (size_t)h : (size_t)h * go.dv + d)])));
     }
     st_f(out + ((size_t)t * nh + h) * go.dv + d, val);
 }
@@ -208,7 +209,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     if (s < 0) {                                         // padding row: zeros (unfused: by the merge kernel)
         if (FUSED && split == 0 && h0 == 0)
             for (int i = threadIdx.x; i < group * HD; i += blockDim.x)
-                write_head_column((T*)fa.out, GateOut{nullptr, 0, fa.dv}, t, nh, kvh * group + i / HD, HD, i % HD, 0.f);
+                write_head_column((T*)fa.out, GateOut{nullptr, 0, fa.dv, 0}, t, nh, kvh * group + i / HD, HD, i % HD, 0.f);
         return;
     }
     if (FUSED) __syncthreads();
@@ -405,7 +406,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             ll += f * __ldcg(base + (size_t)sp * REC + HD + 1);
             a += f * __ldcg(base + (size_t)sp * REC + d);
         }
-        write_head_column((T*)fa.out, GateOut{fa.gate, fa.gate_ld, fa.dv}, t, nh, h, HD, d,
+        write_head_column((T*)fa.out, GateOut{fa.gate, fa.gate_ld, fa.dv, 0}, t, nh, h, HD, d,
                           a / attn_denominator(mm, ll, av.sink, attn_sink_value(av, h)));
     }
 }
@@ -557,7 +558,7 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ partial, T* _
     const int rec = hd + 2;
     if (seq_of_token[t] < 0) {
         for (int d = threadIdx.x; d < hd; d += blockDim.x)
-            write_head_column(out, GateOut{nullptr, 0, go.dv}, t, nh, h, hd, d, 0.f);
+            write_head_column(out, GateOut{nullptr, 0, go.dv, 0}, t, nh, h, hd, d, 0.f);
         return;
     }
     const float* base = partial + ((size_t)t * nh + h) * nsplit * rec;
@@ -858,7 +859,7 @@ template <typename T>
 int launch(const void* q, const void* k_cache, const void* v_cache, void* out, float* partial,
            const int* seq_of_token, const int* pos, const int* slots, const int* tables, int table_stride, int ring,
            int page_size, int num_pages, int num_tokens, int nh, int nkv, int hd, int window, float scale, int nsplit,
-           int* status, cudaStream_t stream, const FusedArgs* fused = nullptr, const GateOut go = GateOut{nullptr, 0, 0},
+           int* status, cudaStream_t stream, const FusedArgs* fused = nullptr, const GateOut go = GateOut{nullptr, 0, 0, 0},
            const AttnVariant av = AttnVariant{0, 0.f, 0, nullptr}) {
     const int group = nh / nkv;
     dim3 grid(nsplit, nkv, num_tokens);
@@ -965,7 +966,8 @@ MOE_API void moe_set_decode_grouped(int enabled) { g_decode_grouped = enabled ? 
 
 // q: [T, nh, hd]; out: [T, nh * hd]; partial: T * nh * nsplit * (hd + 2) floats of scratch.
 // With dv > 0 out is [T, nh * dv]: the first dv columns of every head, times the sigmoid of the
-// 32-bit gate logits gate[t * gate_ld + h * dv + d] if gate is given.
+// 32-bit gate logits gate[t * gate_ld + h * dv + d] if gate is given (a negative gate_ld: one logit a head,
+// gate[t * -gate_ld + h]).
 MOE_API int moe_attention_decode(const void* q, const void* k_cache, const void* v_cache, void* out, float* partial,
                                  int dt, const int* seq_of_token, const int* pos, const int* slots,
                                  const int* tables, int table_stride, int ring, int page_size, int num_pages,
@@ -974,7 +976,7 @@ MOE_API int moe_attention_decode(const void* q, const void* k_cache, const void*
                                  int sink, const float* sink_vals, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (dv < 0 || dv > hd || (gate && dv == 0)) return (int)cudaErrorInvalidValue;
-    const GateOut go{gate, gate_ld, dv};
+    const GateOut go{gate, gate_ld < 0 ? -gate_ld : gate_ld, dv, gate_ld < 0};
     const AttnVariant av{chunk, softcap, sink, sink_vals};
     if (hd % 16 != 0 || hd > MAX_HD || hd <= 0 || nkv <= 0 || nh <= 0 || nh > 65535 || nh % nkv != 0 || nsplit < 1 ||
         nsplit > 65535 || nkv > 65535 || num_tokens > 65535 || !q || !k_cache || !v_cache || !out || !partial)

@@ -6,13 +6,22 @@
 // the attention itself runs over the cached latents alone: every query head reads the same single
 // record c as key AND as value, with queries W_uk_h^T q_h of r numbers, and the head's values are
 // formed from the r numbers that come out.  The two per-head products are grouped products (a group
-// a head) over rows laid out head by head, hence the transposes here.
-//   latent_prepare    from the 32-bit projection row [q heads | latent]: c = x / sqrt(mean(x^2) + eps) * w
-//                     over the latent, written as the step's key record of width D >= r (zero-filled)
-//                     and, optionally, appended to the paged cache; the queries are written head by
-//                     head, q_t[h][t][0..d).
+// a head) over rows laid out head by head, hence the transposes here.  A head may have a ROTATED part of
+// `rot` dimensions beside the d: its key is one vector per position that all heads share and follows
+// the latent in the record, [c | rotated key part], and a query is [W_uk_h^T q_h | rotated query part].
+//   latent_prepare    KEYS: from the 32-bit projection row, c = x / sqrt(mean(x^2) + eps) * w over the
+//                     latent, then the key part after it rotated by the token's position, written as the
+//                     step's key record of width D >= r + rot (zero-filled) and, optionally, appended to the
+//                     paged cache; the same norm over a latent of the queries, if they have one, rounded
+//                     to the activation dtype for the product that follows.
+//                     QUERIES: from 32-bit rows of heads [unrotated | rot], the rotation and the layout: token
+//                     by token as records q[t][h][0..D) (zero-filled), or the unrotated part head by head,
+//                     q_t[h][t][0..d), with the rotated part put into the records' columns from r on.
+//                     Either half may be left out.
 //   heads_transpose   dst[b][a][0..wd) = src[a][b][0..n) (zero-filled beyond n), any of the two
-//                     storage types on either side.
+//                     storage types on either side, optionally times sigmoid(gate[b][a]).
+// The rotation turns pairs (i, i + rot/2) or, interleaved, (2i, 2i + 1) by pos * freq[i], cos and sin times
+// a factor.
 //
 // DIFFERENTIAL attention.  Every head runs two softmax attentions ("maps") over the same values and
 // joins them:  o = a1 - lambda a2;  o <- o / sqrt(mean(o^2) + eps) * mult;  o <- o * sigmoid(g_h),
@@ -55,71 +64,155 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, const float* v) {
     *reinterpret_cast<uint2*>(p) = x;
 }
 
+constexpr int LATENT_MAX_ROT = 512;
+
+struct LatentArgs {
+    const int* pos;
+    const int* seq_of_token;
+    // keys
+    const float* proj;        // [T, ld] the projection row: the latent from column lat_at, its rotated part after it
+    int ld, lat_at, r;
+    const float* w;           // [r]
+    float eps;
+    const float* cq_w;        // [q_rank] the norm weight of the queries' latent (columns 0 ... q_rank); null: none
+    int q_rank;
+    // queries
+    const float* q32;         // [T, ldq] heads of dq + rot; null: none
+    int ldq, nh, dq;
+    int q_major;              // records token by token; else head by head and the rotated part into q_rec
+    // the rotation
+    const float* freq;
+    int rot, interleaved;
+    float mscale;
+    int num_tokens, D;
+};
+
 // One block a token.
 template <typename OT>
 __global__ void __launch_bounds__(256)
-latent_prepare_kernel(const float* __restrict__ proj, int ld, const int* __restrict__ pos,
-                      const int* __restrict__ seq_of_token, const float* __restrict__ w, float eps, int num_tokens,
-                      int nh, int d, int r, int D, OT* __restrict__ q_t, OT* __restrict__ k_new,
-                      const LatentCommit c, int* status, int vec4, int q_major) {
+latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__ q_rec, OT* __restrict__ k_new,
+                      OT* __restrict__ cq, const LatentCommit c, int* status, int vec4) {
     __shared__ float red[32];
-    const int t = blockIdx.x;
+    __shared__ __align__(16) float ang[LATENT_MAX_ROT];        // cos[rot / 2], sin[rot / 2]
+    const int t = blockIdx.x, rot = a.rot, half = rot / 2, D = a.D, r = a.r;
     pdl_sync();
-    const float* row = proj + (size_t)t * ld;
-    const float* lat = row + (size_t)nh * d;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < r; i += blockDim.x) ss += lat[i] * lat[i];
-    ss = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(ss / (float)r + eps);
-    OT* cd = nullptr;
-    OT* cv = nullptr;
-    if (c.k_cache) {
-        const int s = seq_of_token[t];
-        const int p = pos[t];
-        if (s >= 0 && !(c.ring > 0 && p < c.seq_end[s] - c.ring)) {
-            const CachePos cp = cache_pos(p, c.ring, c.tables + (size_t)c.slots[s] * c.table_stride, c.page_size,
-                                          c.num_pages, status);
-            const size_t at = cache_index(cp, 0, 1, c.page_size, D);
-            cd = (OT*)c.k_cache + at;
-            if (c.v_cache && c.v_cache != c.k_cache) cv = (OT*)c.v_cache + at;
+    if (rot > 0) {
+        const float p = (float)a.pos[t];
+        for (int i = threadIdx.x; i < half; i += blockDim.x) {
+            float sn, cs;
+            sincosf(p * a.freq[i], &sn, &cs);
+            ang[i] = cs * a.mscale, ang[half + i] = sn * a.mscale;
+        }
+        __syncthreads();
+    }
+    // element j of the rotated vector whose rotated part starts at v
+    auto turned = [&](const float* v, int j) {
+        const int i = a.interleaved ? j >> 1 : (j < half ? j : j - half);
+        const bool second = a.interleaved ? (j & 1) != 0 : j >= half;
+        const float lo = v[a.interleaved ? 2 * i : i], hi = v[a.interleaved ? 2 * i + 1 : i + half];
+        return second ? rot_hi(lo, hi, ang[i], ang[half + i]) : rot_lo(lo, hi, ang[i], ang[half + i]);
+    };
+    if (k_new) {
+        const float* row = a.proj + (size_t)t * a.ld;
+        const float* lat = row + a.lat_at;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < r; i += blockDim.x) ss += lat[i] * lat[i];
+        ss = block_sum(ss, red);
+        const float inv = 1.0f / sqrtf(ss / (float)r + a.eps);
+        OT* cd = nullptr;
+        OT* cv = nullptr;
+        if (c.k_cache) {
+            const int s = a.seq_of_token[t];
+            const int p = a.pos[t];
+            if (s >= 0 && !(c.ring > 0 && p < c.seq_end[s] - c.ring)) {
+                const CachePos cp = cache_pos(p, c.ring, c.tables + (size_t)c.slots[s] * c.table_stride, c.page_size,
+                                              c.num_pages, status);
+                const size_t at = cache_index(cp, 0, 1, c.page_size, D);
+                cd = (OT*)c.k_cache + at;
+                if (c.v_cache && c.v_cache != c.k_cache) cv = (OT*)c.v_cache + at;
+            }
+        }
+        OT* kd = k_new + (size_t)t * D;
+        for (int i = threadIdx.x; i < D; i += blockDim.x) {
+            const float x = i < r ? lat[i] * inv * a.w[i] : i < r + rot ? turned(lat + r, i - r) : 0.f;
+            st_f(kd + i, x);
+            if (cd) st_f(cd + i, x);
+            if (cv) st_f(cv + i, x);
+        }
+        if (a.cq_w) {
+            float sq = 0.f;
+            for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) sq += row[i] * row[i];
+            sq = block_sum(sq, red);
+            const float qi = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps);
+            for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x)
+                st_f(cq + (size_t)t * a.q_rank + i, row[i] * qi * a.cq_w[i]);
         }
     }
-    OT* kd = k_new + (size_t)t * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) {
-        const float x = i < r ? lat[i] * inv * w[i] : 0.f;
-        st_f(kd + i, x);
-        if (cd) st_f(cd + i, x);
-        if (cv) st_f(cv + i, x);
-    }
-    if (q_major) {       // the queries token by token, q[t][h][0..D), zero-filled beyond d
+    if (!a.q32) return;
+    const int nh = a.nh, dq = a.dq, hd = dq + rot;
+    const float* row = a.q32 + (size_t)t * a.ldq;
+    if (a.q_major) {     // the queries token by token, q[t][h][0..D), zero-filled beyond dq + rot
         OT* qd = q_t + (size_t)t * nh * D;
-        if (vec4 && D % 4 == 0) {
+        if (vec4) {
             for (int i = threadIdx.x * 4; i < nh * D; i += blockDim.x * 4) {
-                const int h = i / D, j = i % D;
+                const int h = i / D, j = i - h * D;
+                const float* head = row + (size_t)h * hd;
                 float v[4] = {0.f, 0.f, 0.f, 0.f};
-                if (j < d) ld4(row + (size_t)h * d + j, v);
+                if (j < dq) {
+                    ld4(head + j, v);
+                } else if (j < hd) {
+                    const float* rp = head + dq;
+                    const int jj = j - dq;
+                    ld4(rp + jj, v);
+                    if (a.interleaved) {
+                        const int i0 = jj >> 1;
+#pragma unroll
+                        for (int e = 0; e < 2; e++) {
+                            const float lo = v[2 * e], hi = v[2 * e + 1], cs = ang[i0 + e], sn = ang[half + i0 + e];
+                            v[2 * e] = rot_lo(lo, hi, cs, sn), v[2 * e + 1] = rot_hi(lo, hi, cs, sn);
+                        }
+                    } else {
+                        const bool second = jj >= half;
+                        const int i0 = second ? jj - half : jj;
+                        float o[4];
+                        ld4(rp + (second ? i0 : i0 + half), o);
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const float cs = ang[i0 + e], sn = ang[half + i0 + e];
+                            v[e] = second ? rot_hi(o[e], v[e], cs, sn) : rot_lo(v[e], o[e], cs, sn);
+                        }
+                    }
+                }
                 st4(qd + i, v);
             }
         } else {
             for (int i = threadIdx.x; i < nh * D; i += blockDim.x) {
-                const int h = i / D, j = i % D;
-                st_f(qd + i, j < d ? row[(size_t)h * d + j] : 0.f);
+                const int h = i / D, j = i - h * D;
+                const float* head = row + (size_t)h * hd;
+                st_f(qd + i, j < dq ? head[j] : j < hd ? turned(head + dq, j - dq) : 0.f);
             }
         }
         return;
     }
-    if (vec4) {          // d and the row pitch are multiples of four, both pointers aligned to four elements
-        for (int i = threadIdx.x * 4; i < nh * d; i += blockDim.x * 4) {
-            const int h = i / d, j = i % d;
+    if (rot > 0) {       // the records' columns from r on; the ones before come from the per-head product
+        const int tail = D - r;
+        for (int i = threadIdx.x; i < nh * tail; i += blockDim.x) {
+            const int h = i / tail, j = i - h * tail;
+            st_f(q_rec + ((size_t)t * nh + h) * D + r + j, j < rot ? turned(row + (size_t)h * hd + dq, j) : 0.f);
+        }
+    }
+    if (vec4) {
+        for (int i = threadIdx.x * 4; i < nh * dq; i += blockDim.x * 4) {
+            const int h = i / dq, j = i - h * dq;
             float v[4];
-            ld4(row + i, v);
-            st4(q_t + ((size_t)h * num_tokens + t) * d + j, v);
+            ld4(row + (size_t)h * hd + j, v);
+            st4(q_t + ((size_t)h * a.num_tokens + t) * dq + j, v);
         }
         return;
     }
-    for (int i = threadIdx.x; i < nh * d; i += blockDim.x) {
-        const int h = i / d, j = i % d;
-        st_f(q_t + ((size_t)h * num_tokens + t) * d + j, row[i]);
+    for (int i = threadIdx.x; i < nh * dq; i += blockDim.x) {
+        const int h = i / dq, j = i - h * dq;
+        st_f(q_t + ((size_t)h * a.num_tokens + t) * dq + j, row[(size_t)h * hd + j]);
     }
 }
 
@@ -136,10 +229,11 @@ __device__ __forceinline__ void st2(__nv_bfloat16* p, const float* v) {
     *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
 }
 
-// VEC = 4: n, wd and both pitches are multiples of four and both pointers aligned to four elements.
+// VEC = 4: n, wd and all pitches are multiples of four and both pointers aligned to four elements.
 template <typename ST, typename DT, int VEC>
 __global__ void heads_transpose_kernel(const ST* __restrict__ src, long long s_outer, long long s_inner, int A, int B,
-                                       int n, int wd, DT* __restrict__ dst) {
+                                       int n, int wd, DT* __restrict__ dst, int ldd, const float* __restrict__ gate,
+                                       int gate_ld) {
     pdl_sync();
     const int wv = wd / VEC;
     const long long total = (long long)A * B * wv;
@@ -149,13 +243,15 @@ __global__ void heads_transpose_kernel(const ST* __restrict__ src, long long s_o
     const long long ba = i / wv;
     const int a = (int)(ba % A), b = (int)(ba / A);
     const ST* from = src + (size_t)a * s_outer + (size_t)b * s_inner + j;
-    DT* to = dst + ba * wd + j;
+    DT* to = dst + ba * ldd + j;
+    const float f = gate ? 1.0f / (1.0f + expf(-gate[(size_t)b * gate_ld + a])) : 1.0f;
     if (VEC == 4) {
         float v[4] = {0.f, 0.f, 0.f, 0.f};
         if (j < n) ld4(from, v);
+        v[0] *= f, v[1] *= f, v[2] *= f, v[3] *= f;
         st4(to, v);
     } else {
-        st_f(to, j < n ? ld_f(from) : 0.f);
+        st_f(to, j < n ? ld_f(from) * f : 0.f);
     }
 }
 
@@ -224,42 +320,55 @@ __global__ void add_row_kernel(float* __restrict__ x, const float* __restrict__ 
 
 }  // namespace
 
-// proj: [T, ld] 32-bit: nh * d query columns, then r latent columns.  q_t: [nh, T, d], or with q_major
-// [T, nh, D] zero-filled beyond d (d <= D); k_new: [T, D].
-MOE_API int moe_latent_prepare(const float* proj, int ld, const int* pos, const int* seq_of_token, const float* w,
-                               float eps, int num_tokens, int nh, int d, int r, int D, void* q_t, void* k_new,
+// Keys (k_new given): proj [T, ld] 32-bit with the latent's r columns from lat_at, then `rot` columns of the
+// rotated key part; k_new: [T, D], D >= r + rot; with cq_w the columns 0 ... q_rank are normed into cq [T, q_rank].
+// Queries (q32 given): [T, ldq] 32-bit, nh heads of dq + rot; q_major: q_t is [T, nh, D], zero-filled beyond
+// dq + rot <= D; else q_t is [nh, T, dq] and, with rot > 0, columns r ... D of q_rec [T, nh, D] are written.
+MOE_API int moe_latent_prepare(const float* proj, int ld, int lat_at, int r, const float* w, float eps, const float* cq_w,
+                               int q_rank, void* cq, const float* q32, int ldq, int nh, int dq, int q_major,
+                               const float* freq, int rot, int interleaved, float mscale, const int* pos,
+                               const int* seq_of_token, int num_tokens, int D, void* q_t, void* q_rec, void* k_new,
                                int out_dt, void* k_cache, void* v_cache, const int* seq_end, const int* slots,
                                const int* tables, int table_stride, int ring, int page_size, int num_pages,
-                               int* status, int q_major, cudaStream_t stream) {
+                               int* status, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
-    if (nh <= 0 || d <= 0 || r <= 0 || D < r || ld < nh * d + r || !proj || !w || !q_t || !k_new || (q_major && d > D))
+    if (rot < 0 || rot % 2 || rot > LATENT_MAX_ROT || (rot > 0 && (!freq || !pos)) || r <= 0 || D < r + rot)
         return (int)cudaErrorInvalidValue;
-    if (k_cache && (!seq_end || !slots || !tables || !seq_of_token || !pos)) return (int)cudaErrorInvalidValue;
+    if (!k_new && !q32) return (int)cudaErrorInvalidValue;
+    if (k_new && (!proj || !w || lat_at < 0 || ld < lat_at + r + rot)) return (int)cudaErrorInvalidValue;
+    if (cq_w && (!k_new || !cq || q_rank <= 0 || q_rank > lat_at)) return (int)cudaErrorInvalidValue;
+    if (q32 && (nh <= 0 || dq <= 0 || ldq < nh * (dq + rot) || !q_t || (q_major && dq + rot > D) || (!q_major && rot > 0 && !q_rec)))
+        return (int)cudaErrorInvalidValue;
+    if (k_cache && (!k_new || !seq_end || !slots || !tables || !seq_of_token || !pos)) return (int)cudaErrorInvalidValue;
     const LatentCommit c{k_cache, v_cache, seq_end, slots, tables, table_stride, ring, page_size, num_pages};
-    const int vec4 = d % 4 == 0 && ld % 4 == 0 && (uintptr_t)proj % 16 == 0 &&
-                     (uintptr_t)q_t % (out_dt == DT_F32 ? 16 : 8) == 0;
+    const LatentArgs a{pos, seq_of_token, proj, ld, lat_at, r, w, eps, cq_w, q_rank, q32, ldq, nh, dq, q_major,
+                       freq, rot, interleaved, mscale, num_tokens, D};
+    const int vec4 = dq % 4 == 0 && ldq % 4 == 0 && (uintptr_t)q32 % 16 == 0 && rot % (interleaved ? 4 : 8) == 0 &&
+                     (!q_major || D % 4 == 0) && (uintptr_t)q_t % (out_dt == DT_F32 ? 16 : 8) == 0;
     if (out_dt == DT_F32)
-        return launch_pdl(latent_prepare_kernel<float>, num_tokens, 256, 0, stream, proj, ld, pos, seq_of_token, w, eps,
-                          num_tokens, nh, d, r, D, (float*)q_t, (float*)k_new, c, status, vec4, q_major);
-    return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, 256, 0, stream, proj, ld, pos, seq_of_token, w,
-                      eps, num_tokens, nh, d, r, D, (__nv_bfloat16*)q_t, (__nv_bfloat16*)k_new, c, status, vec4, q_major);
+        return launch_pdl(latent_prepare_kernel<float>, num_tokens, 256, 0, stream, a, (float*)q_t, (float*)q_rec,
+                          (float*)k_new, (float*)cq, c, status, vec4);
+    return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, 256, 0, stream, a, (__nv_bfloat16*)q_t,
+                      (__nv_bfloat16*)q_rec, (__nv_bfloat16*)k_new, (__nv_bfloat16*)cq, c, status, vec4);
 }
 
-// src: element (a, b, j) at a * s_outer + b * s_inner + j, j < n; dst: dense [B, A, wd].
+// src: element (a, b, j) at a * s_outer + b * s_inner + j, j < n; dst: [B, A, wd] with rows of ldd elements (dense
+// otherwise); gate: 32-bit logits [B, A], rows of gate_ld, or null.
 MOE_API int moe_heads_transpose(const void* src, int src_dt, long long s_outer, long long s_inner, int A, int B, int n,
-                                int wd, void* dst, int dst_dt, cudaStream_t stream) {
+                                int wd, void* dst, int dst_dt, int ldd, const float* gate, int gate_ld,
+                                cudaStream_t stream) {
     const long long total = (long long)A * B * wd;
     if (total <= 0) return 0;
-    if (n < 0 || n > wd || !src || !dst) return (int)cudaErrorInvalidValue;
+    if (n < 0 || n > wd || ldd < wd || !src || !dst || (gate && gate_ld < A)) return (int)cudaErrorInvalidValue;
     const size_t se = src_dt == DT_F32 ? 4 : 2, de = dst_dt == DT_F32 ? 4 : 2;
-    const bool vec = n % 4 == 0 && wd % 4 == 0 && s_outer % 4 == 0 && s_inner % 4 == 0 &&
+    const bool vec = n % 4 == 0 && wd % 4 == 0 && ldd % 4 == 0 && s_outer % 4 == 0 && s_inner % 4 == 0 &&
                      (uintptr_t)src % (4 * se) == 0 && (uintptr_t)dst % (4 * de) == 0;
     const unsigned blocks = (unsigned)(((vec ? total / 4 : total) + 255) / 256);
 #define TR(ST_, DT_)                                                                                                \
     return vec ? launch_pdl(heads_transpose_kernel<ST_, DT_, 4>, blocks, 256, 0, stream, (const ST_*)src, s_outer,      \
-                            s_inner, A, B, n, wd, (DT_*)dst)                                                        \
+                            s_inner, A, B, n, wd, (DT_*)dst, ldd, gate, gate_ld)                                        \
                : launch_pdl(heads_transpose_kernel<ST_, DT_, 1>, blocks, 256, 0, stream, (const ST_*)src, s_outer,      \
-                            s_inner, A, B, n, wd, (DT_*)dst)
+                            s_inner, A, B, n, wd, (DT_*)dst, ldd, gate, gate_ld)
     if (src_dt == DT_F32) {
         if (dst_dt == DT_F32) TR(float, float);
         TR(float, __nv_bfloat16);

@@ -12,8 +12,8 @@
 //                   Optionally the keys and values are appended to the paged cache in the same
 //                   launch (whole prompts and single-token steps).
 //   gate_pack       out[t, h * dv + j] = ctx[t, h, j] * sigmoid(gate[t, h * dv + j]) (gate logits
-//                   are columns of the same projection row; null: no gate), which also drops the
-//                   padding columns.
+//                   are columns of the same projection row, or one a head, gate[t, h]; null: no gate),
+//                   which also drops the padding columns.
 // Norm, angles, rotation and the gate are 32-bit; only the stores round to the activation dtype.
 #include "common.cuh"
 
@@ -260,7 +260,7 @@ __device__ __forceinline__ float sigmoid32(float x) { return 1.0f / (1.0f + expf
 // One thread per four consecutive columns of a head (VEC) or per element.
 template <typename OT, bool VEC>
 __global__ void gate_pack_kernel(const OT* __restrict__ ctx, const float* __restrict__ gate, int ld, long long total,
-                                 int nh, int dv, int D, OT* __restrict__ out) {
+                                 int nh, int dv, int D, OT* __restrict__ out, int per_head) {
     pdl_sync();
     const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * (VEC ? 4 : 1);
     if (i >= total) return;
@@ -269,32 +269,36 @@ __global__ void gate_pack_kernel(const OT* __restrict__ ctx, const float* __rest
     const int c = (int)(i % w), h = c / dv, j = c % dv;
     if (VEC) {
         float4 x = prep_load4(ctx + ((size_t)t * nh + h) * D + j);
-        if (gate) {
+        if (gate && per_head) {
+            const float g = sigmoid32(gate[(size_t)t * ld + h]);
+            x.x *= g, x.y *= g, x.z *= g, x.w *= g;
+        } else if (gate) {
             const float4 g = *reinterpret_cast<const float4*>(gate + (size_t)t * ld + c);
             x.x *= sigmoid32(g.x), x.y *= sigmoid32(g.y), x.z *= sigmoid32(g.z), x.w *= sigmoid32(g.w);
         }
         prep_store4(out + i, x.x, x.y, x.z, x.w);
     } else {
         float x = ld_f(ctx + ((size_t)t * nh + h) * D + j);
-        if (gate) x *= sigmoid32(gate[(size_t)t * ld + c]);
+        if (gate) x *= sigmoid32(gate[(size_t)t * ld + (per_head ? h : c)]);
         st_f(out + i, x);
     }
 }
 
-// ctx: [T, nh, D]; gate: first gate logit of token 0 (row pitch ld, 32-bit) or null; out: [T, nh * dv].
+// ctx: [T, nh, D]; gate: first gate logit of token 0 (row pitch ld, 32-bit; one a column, or one a head with
+// per_head) or null; out: [T, nh * dv].
 MOE_API int moe_gate_pack(const void* ctx, const float* gate, int ld, int num_tokens, int nh, int dv, int D, void* out,
-                          int dt, cudaStream_t stream) {
+                          int dt, int per_head, cudaStream_t stream) {
     const long long total = (long long)num_tokens * nh * dv;
     if (total <= 0) return 0;
     if (D < dv) return (int)cudaErrorInvalidValue;
     const size_t esz = dt == DT_F32 ? 4 : 2;
-    const bool vec = dv % 4 == 0 && D % 4 == 0 && ld % 4 == 0 && ((uintptr_t)gate % 16) == 0 &&
+    const bool vec = dv % 4 == 0 && D % 4 == 0 && (per_head || (ld % 4 == 0 && ((uintptr_t)gate % 16) == 0)) &&
                      ((uintptr_t)ctx % (4 * esz)) == 0 && ((uintptr_t)out % (4 * esz)) == 0;
     const long long threads = vec ? total / 4 : total;
     const unsigned blocks = (unsigned)((threads + 255) / 256);
 #define PACK(OT_, VEC_)                                                                                        \
     return launch_pdl(gate_pack_kernel<OT_, VEC_>, blocks, 256, 0, stream, (const OT_*)ctx, gate, ld, total, nh, dv, \
-                      D, (OT_*)out)
+                      D, (OT_*)out, per_head)
     if (dt == DT_F32) {
         if (vec) PACK(float, true);
         PACK(float, false);

@@ -14,7 +14,7 @@
 //   warps 2-5   epilogue: tensor memory -> registers -> global memory
 //
 // Modes
-//   PLAIN    out[t, n] = f(acc (+ bias[n])); out is float32 or bfloat16; f is the identity, or relu(.)^2 with ACT_RELU2
+//   PLAIN    out[t, n] = f(acc (+ bias[n])); out is float32 or bfloat16; f is the identity, or plain_act (ACT_RELU2, ACT_GELU)
 //   SWIGLU   W holds gate rows [0, I) and up rows [I, 2I) per group; two accumulators;
 //            out[t, j] = silu(gate) * up  (reference: src/model.rs:26-35)
 // Groups (routed experts): rows of X are partitioned by group_offsets[G + 1]; group g

@@ -12,8 +12,9 @@
 //                   a step's first row is the sequence's state, which the block of that row then
 //                   replaces by the step's last token (it is the state's only reader).
 //   pair_norm_mean  out = (rmsnorm(a) * wa + rmsnorm(b) * wb) / 2, both norms over the model's width.
-//   relu2           out = relu(in)^2 element by element, rounded to the activation dtype (where the
-//                   tensor-core product's epilogue does not form it).
+//   plain_act       an ungated feed-forward's activation (plain_act in common.cuh) element by element,
+//                   rounded to the activation dtype (where the tensor-core product's epilogue does not
+//                   form it).
 //   table_route     a token's experts are row `token id` of an integer table; each weighs 1 / top.
 // All arithmetic is 32-bit; only stores into activation buffers round.
 #include "common.cuh"
@@ -178,12 +179,11 @@ pair_norm_mean_kernel(const float* __restrict__ a, const float* __restrict__ wa,
 }
 
 template <typename OT>
-__global__ void relu2_kernel(const float* __restrict__ in, OT* __restrict__ out, long long n) {
+__global__ void plain_act_kernel(const float* __restrict__ in, OT* __restrict__ out, long long n, int act) {
     pdl_sync();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
-    const float v = fmaxf(in[i], 0.f);
-    st_f(out + i, v * v);
+    st_f(out + i, plain_act(act, in[i]));
 }
 
 __global__ void table_route_kernel(const int* __restrict__ table, int width, const int* __restrict__ tokens,
@@ -291,11 +291,11 @@ MOE_API int moe_pair_norm_mean(const float* a, const float* wa, const float* b, 
     return launch_pdl(pair_norm_mean_kernel, dim3(num_tokens), 256, 0, stream, a, wa, b, wb, eps, hidden, out);
 }
 
-MOE_API int moe_relu2(const float* in, void* out, int out_dt, long long n, cudaStream_t stream) {
+MOE_API int moe_plain_act(const float* in, void* out, int out_dt, long long n, int act, cudaStream_t stream) {
     if (n <= 0) return 0;
     const unsigned blocks = (unsigned)((n + 255) / 256);
-    if (out_dt == DT_F32) return launch_pdl(relu2_kernel<float>, dim3(blocks), 256, 0, stream, in, (float*)out, n);
-    return launch_pdl(relu2_kernel<__nv_bfloat16>, dim3(blocks), 256, 0, stream, in, (__nv_bfloat16*)out, n);
+    if (out_dt == DT_F32) return launch_pdl(plain_act_kernel<float>, dim3(blocks), 256, 0, stream, in, (float*)out, n, act);
+    return launch_pdl(plain_act_kernel<__nv_bfloat16>, dim3(blocks), 256, 0, stream, in, (__nv_bfloat16*)out, n, act);
 }
 
 // table: [vocab, width >= top] int32; topk_idx / topk_w: [T, top].

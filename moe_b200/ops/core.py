@@ -18,7 +18,7 @@ DT_F32, DT_BF16 = 0, 1
 # the gate's activation of a gated feed-forward (ACT_* in csrc/common.cuh)
 GLU_ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_sigmoid": 2}
 # what an ungated product's output may pass in the tensor-core kernel's epilogue
-PLAIN_ACTS = {"relu2": 3}
+PLAIN_ACTS = {"relu2": 3, "gelu": 4}
 
 
 class KernelError(RuntimeError):
@@ -37,11 +37,13 @@ def lib():
             "moe_embed": [P, I, P, P, I, I, I, P, P, P, P, F, P],
             "moe_dyt": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P, P],
             "moe_heads_prepare": [P, I, P, P, P, P, F, P, I, F, I, I, I, I, I, I, P, P, P, LL, LL, I, P, P, P, P, P, I, I, I, I, P, P],
-            "moe_gate_pack": [P, P, I, I, I, I, I, P, I, P],
-            "moe_latent_prepare": [P, I, P, P, P, F, I, I, I, I, I, P, P, I, P, P, P, P, P, I, I, I, I, P, I, P],
-            "moe_heads_transpose": [P, I, LL, LL, I, I, I, I, P, I, P],
+            "moe_gate_pack": [P, P, I, I, I, I, I, P, I, I, P],
+            "moe_latent_prepare": [P, I, I, I, P, F, P, I, P, P, I, I, I, I, P, I, I, F, P, P, I, I, P, P, P, I, P, P, P, P,
+                                   P, I, I, I, I, P, P],
+            "moe_heads_transpose": [P, I, LL, LL, I, I, I, I, P, I, I, P, I, P],
             "moe_diff_combine": [P, P, I, I, I, I, I, F, F, F, P, I, P],
             "moe_add_row": [P, P, P, LL, I, P],
+            "moe_layernorm": [P, P, P, P, P, P, P, I, I, I, F, I, P, P],
             "moe_rmsnorm": [P, P, P, P, P, P, I, I, I, F, I, P, P],
             "moe_rmsnorm_combine": [P, P, P, P, I, P, P, P, P, P, P, I, I, I, F, I, P, P],
             "moe_add_inplace": [P, P, LL, P],
@@ -80,10 +82,13 @@ def lib():
             "moe_seq_conv": [I, P, LL, P, P, P, P, P, P, LL, P, P, P, P, P, I, I, LL, P, P, P, P, I, I, I, I, P],
             "moe_embed_pair": [P, P, I, P, F, P, P, I, I, I, I, I, I, P, P, P, P, P, P, P, P],
             "moe_pair_norm_mean": [P, P, P, P, F, I, I, P, P],
-            "moe_relu2": [P, P, I, LL, P],
+            "moe_plain_act": [P, P, I, LL, I, P],
             "moe_table_route": [P, I, P, P, P, P, I, I, I, I, P, P, P, P],
             "moe_ssd_scan": [P, LL, P, LL, P, P, P, P, LL, P, P, I, I, I, I, I, P, I, I, P, P, P],
             "moe_ssd_finish": [P, P, LL, P, F, P, I, I, I, P, I, P],
+            "moe_delta_prepare": [P, LL, I, I, P, I, P, LL, P, P, P, P, P, I, I, I, I, I, F, F, I, P, P, P],
+            "moe_delta_step": [P, P, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P],
+            "moe_delta_scan": [P, P, P, LL, P, P, I, I, I, I, I, P, P],
         }
         for name, argtypes in sig.items():
             fn = getattr(L, name)
@@ -244,6 +249,33 @@ def rmsnorm(x, weight, eps, *, delta=None, rows=None, out32=None, out16=None, wr
                           1 if (write_back and rows is None) else 0, _p(status), _stream()), "rmsnorm")
 
 
+def layernorm(x, weight, eps, *, bias=None, delta=None, rows=None, out32=None, out16=None, write_back=True, status=None):
+    """y = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight (+ bias) with v = x[r] (+ delta[r]), for r
+    in rows (or every row); ``delta``, ``write_back`` and the outputs as in ``rmsnorm``."""
+    _chk(x, "x", torch.float32, 2), _chk(weight, "weight", torch.float32, 1)
+    S, H = x.shape
+    n_out = S if rows is None else rows.numel()
+    if weight.numel() != H:
+        raise KernelError("layernorm: weight size")
+    if bias is not None:
+        _chk(bias, "bias", torch.float32, 1)
+        if bias.numel() != H:
+            raise KernelError("layernorm: bias size")
+    if delta is not None:
+        _chk(delta, "delta", torch.float32, 2)
+        if delta.shape != x.shape:
+            raise KernelError("layernorm: delta shape")
+    if rows is not None:
+        _chk(rows, "rows", torch.int32, 1)
+    for o, dt in ((out32, torch.float32), (out16, torch.bfloat16)):
+        if o is not None:
+            _chk(o, "out", dt, 2)
+            if o.shape[0] < n_out or o.shape[1] != H:
+                raise KernelError("layernorm: output shape")
+    _ok(lib().moe_layernorm(_p(x), _p(delta), _p(weight), _p(bias), _p(rows), _p(out32), _p(out16), n_out, S, H, float(eps),
+                            1 if (write_back and rows is None) else 0, _p(status), _stream()), "layernorm")
+
+
 def rmsnorm_combine(x, cd, weight, eps, *, rows=None, out32=None, out16=None, write_back=True, status=None) -> bool:
     """``rmsnorm`` whose delta is still the uncombined output of routed experts (``cd``: y,
     pos_of_pair, topk_w, top_k, shared, shared_gate): combined inside the norm's kernel.  False,
@@ -348,32 +380,71 @@ def heads_prepare(proj, pos, seq_of_token, *, nh, nkv, d, dv, width, q, k, v, q_
 
 def gate_pack(ctx, out, *, nh, dv, width, gate=None):
     """out[t, h * dv + j] = ctx[t, h, j] * sigmoid(gate[t, h * dv + j]); ``gate``: a column slice
-    [T, nh * dv] of a float32 projection (unit stride along the row), or None for the packing alone."""
+    [T, nh * dv], or [T, nh] (one logit a head), of a float32 projection (unit stride along the row), or
+    None for the packing alone."""
     _chk(ctx, "ctx"), _chk(out, "out", dims=2)
     T = out.shape[0]
     if ctx.numel() < T * nh * width or out.shape[1] != nh * dv or out.dtype != ctx.dtype:
         raise KernelError("gate_pack: shapes or dtypes")
-    ld = 0
+    ld, per_head = 0, False
     if gate is not None:
-        if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape != (T, nh * dv):
+        per_head = gate.dim() == 2 and gate.shape[1] == nh and dv != 1
+        if (gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1
+                or tuple(gate.shape) != (T, nh if per_head else nh * dv)):
             raise KernelError("gate_pack: gate shape, dtype or layout")
         ld = gate.stride(0)
-    _ok(lib().moe_gate_pack(_p(ctx), _p(gate), ld, T, nh, dv, width, _p(out), _dt(out), _stream()), "gate_pack")
+    _ok(lib().moe_gate_pack(_p(ctx), _p(gate), ld, T, nh, dv, width, _p(out), _dt(out), 1 if per_head else 0, _stream()),
+        "gate_pack")
 
 
-def latent_prepare(proj, batch, *, nh, d, r, width, weight, eps, q_t, k_new, commit=None, status=None,
-                   token_major=False):
-    """From a step's 32-bit projection rows [q heads (nh x d) | latent (r)]: the latent divided by its
-    root mean square, times ``weight``, into ``k_new`` [T, width] (zero-filled beyond r) and, with
-    ``commit`` (a cache view), appended to that cache layer; the queries head by head into ``q_t``
-    [nh, T, d], or with ``token_major`` token by token into ``q_t`` [T, nh, width] (zero-filled
-    beyond d)."""
-    _chk(proj, "proj", torch.float32, 2), _chk(weight, "latent norm weight", torch.float32, 1)
-    T = proj.shape[0]
-    _chk(q_t, "q_t"), _chk(k_new, "k_new")
-    if (proj.shape[1] < nh * d + r or weight.numel() != r or q_t.numel() != nh * T * (width if token_major else d)
-            or k_new.numel() != T * width or q_t.dtype != k_new.dtype or width < r or (token_major and width < d)):
-        raise KernelError("latent_prepare: shapes or dtypes")
+def latent_prepare(proj, batch, *, r, width, nh=0, d=0, weight=None, eps=0.0, q_t=None, k_new=None, commit=None, status=None,
+                   token_major=False, lat_at=None, q32=None, q_rec=None, rot=0, freq=None, interleaved=False, mscale=1.0,
+                   cq=None, cq_weight=None):
+    """Lays out latent attention's keys and queries from 32-bit projection rows.
+
+    Keys (``k_new`` given): ``proj`` [T, >= lat_at + r + rot] holds the latent from column ``lat_at`` (default nh x
+    (d + rot): behind the queries).  The latent divided by its root mean square, times ``weight``, then the ``rot``
+    columns after it turned by the token's position, go into ``k_new`` [T, width] (zero-filled) and, with ``commit``
+    (a cache view), into that cache layer.  With ``cq`` [T, q_rank] and ``cq_weight`` the first q_rank columns are
+    normed in the same way and rounded into ``cq``.
+
+    Queries (``q_t`` given): from ``q32`` (default ``proj``), heads of d + rot columns.  With ``token_major`` into
+    ``q_t`` [T, nh, width] (the last rot columns of a head turned, zero-filled); else the d columns head by head into
+    ``q_t`` [nh, T, d] and the turned ones into columns r ... of ``q_rec`` [T, nh, width].
+
+    The rotation: pairs (i, i + rot/2), or (2i, 2i + 1) with ``interleaved``, by pos * ``freq``[i], cos and sin times
+    ``mscale``."""
+    keys, queries = k_new is not None, q_t is not None
+    if not keys and not queries:
+        raise KernelError("latent_prepare: nothing to do")
+    hd = d + rot
+    lat_at = nh * hd if lat_at is None else int(lat_at)
+    out = k_new if keys else q_t
+    T = batch.num_tokens if hasattr(batch, "num_tokens") else proj.shape[0]
+    if keys:
+        _chk(proj, "proj", torch.float32, 2), _chk(weight, "latent norm weight", torch.float32, 1), _chk(k_new, "k_new")
+        T = proj.shape[0]
+        if proj.shape[1] < lat_at + r + rot or weight.numel() != r or k_new.numel() != T * width or width < r + rot:
+            raise KernelError("latent_prepare: shapes or dtypes")
+    if cq is not None:
+        _chk(cq, "cq", dims=2), _chk(cq_weight, "query latent norm weight", torch.float32, 1)
+        if not keys or cq.shape[0] != T or cq_weight.numel() != cq.shape[1] or cq.shape[1] > lat_at or cq.dtype != out.dtype:
+            raise KernelError("latent_prepare: the queries' latent")
+    if queries:
+        q32 = proj if q32 is None else q32
+        _chk(q32, "q32", torch.float32, 2), _chk(q_t, "q_t")
+        T = q32.shape[0]
+        if (q32.shape[1] < nh * hd or q_t.numel() != nh * T * (width if token_major else d) or q_t.dtype != out.dtype
+                or (token_major and width < hd)):
+            raise KernelError("latent_prepare: shapes or dtypes")
+        if rot and not token_major:
+            _chk(q_rec, "q_rec", dims=3)
+            if tuple(q_rec.shape) != (T, nh, width) or q_rec.dtype != out.dtype:
+                raise KernelError("latent_prepare: the records' shape or dtype")
+    if rot:
+        _chk(freq, "freq", torch.float32, 1)
+        if freq.numel() < rot // 2:
+            raise KernelError("latent_prepare: frequency table too short")
     kc = vc = se = sl = tb = None
     ts = ring = ps = npg = 0
     if commit is not None:
@@ -382,21 +453,30 @@ def latent_prepare(proj, batch, *, nh, d, r, width, weight, eps, q_t, k_new, com
             raise KernelError("latent_prepare: the cache layer differs from the latent in dtype or shape")
         kc, vc, se, sl, tb = commit.k, commit.v, batch.seq_end, batch.slots, g.table
         ts, ring, ps, npg = g.table.stride(0), g.ring, g.page_size, g.num_pages
-    _ok(lib().moe_latent_prepare(_p(proj), proj.stride(0), _p(batch.pos), _p(batch.seq_of_token), _p(weight), float(eps),
-                                 T, nh, d, r, width, _p(q_t), _p(k_new), _dt(k_new), _p(kc), _p(vc), _p(se), _p(sl),
-                                 _p(tb), ts, ring, ps, npg, _p(status), 1 if token_major else 0, _stream()),
-        "latent_prepare")
+    _ok(lib().moe_latent_prepare(_p(proj) if keys else None, proj.stride(0) if keys else 0, lat_at, r,
+                                 _p(weight), float(eps), _p(cq_weight) if cq is not None else None,
+                                 cq.shape[1] if cq is not None else 0, _p(cq), _p(q32) if queries else None,
+                                 q32.stride(0) if queries else 0, nh, d, 1 if token_major else 0, _p(freq) if rot else None,
+                                 int(rot), 1 if interleaved else 0, float(mscale), _p(batch.pos), _p(batch.seq_of_token), T,
+                                 width, _p(q_t), _p(q_rec), _p(k_new), _dt(out), _p(kc), _p(vc), _p(se), _p(sl), _p(tb),
+                                 ts, ring, ps, npg, _p(status), _stream()), "latent_prepare")
 
 
-def heads_transpose(src, dst, *, n):
+def heads_transpose(src, dst, *, n, gate=None):
     """dst[b, a, :n] = src[a, b, :n], zero beyond n; src: [A, B, >= n] with unit stride along the last
-    axis (any pitch of the other two), dst: dense [B, A, wd >= n]; float32 or bfloat16 on either side."""
-    if (src.dim() != 3 or dst.dim() != 3 or not dst.is_contiguous() or src.stride(2) != 1 or src.shape[2] < n
-            or dst.shape[2] < n or (dst.shape[0], dst.shape[1]) != (src.shape[1], src.shape[0])):
+    axis (any pitch of the other two), dst: [B, A, wd >= n] dense but for the pitch of its rows; float32 or
+    bfloat16 on either side.  ``gate``: float32 logits [B, A] (a column slice is fine); row (b, a) is multiplied by
+    sigmoid(gate[b, a])."""
+    if (src.dim() != 3 or dst.dim() != 3 or dst.stride(2) != 1 or dst.stride(0) != dst.shape[1] * dst.stride(1)
+            or src.stride(2) != 1 or src.shape[2] < n or dst.shape[2] < n
+            or (dst.shape[0], dst.shape[1]) != (src.shape[1], src.shape[0])):
         raise KernelError("heads_transpose: shapes")
     A, B = src.shape[0], src.shape[1]
+    if gate is not None and (gate.dtype != torch.float32 or tuple(gate.shape) != (B, A) or gate.stride(1) != 1):
+        raise KernelError("heads_transpose: the gate must be float32 [B, A]")
     _ok(lib().moe_heads_transpose(_p(src), _dt(src), src.stride(0), src.stride(1), A, B, int(n), dst.shape[2], _p(dst),
-                                  _dt(dst), _stream()), "heads_transpose")
+                                  _dt(dst), dst.stride(1), _p(gate), gate.stride(0) if gate is not None else 0, _stream()),
+        "heads_transpose")
 
 
 def diff_combine(ctx, out, *, nh, dv, width, lam, eps, mult, gate=None):
@@ -866,8 +946,9 @@ def _head_blocks(nh: int, nkv: int, group_view=None, dtype=None) -> int:
     return nkv * (1 if group == 1 else -(-group // 2))
 
 
-def _gate_args(out, T, nh, hd, gate, dv):
-    """(gate pointer, its row pitch, dv) of a merge that writes [T, nh * dv] instead of [T, nh * hd]."""
+def _gate_args(out, T, nh, hd, gate, dv, per_head=False):
+    """(gate pointer, its row pitch, dv) of a merge that writes [T, nh * dv] instead of [T, nh * hd]; ``per_head``:
+    the merge also takes one logit a head."""
     if not dv:
         if gate is not None:
             raise KernelError("attention: a gate needs the value width dv")
@@ -876,22 +957,26 @@ def _gate_args(out, T, nh, hd, gate, dv):
         raise KernelError("attention: dv or the packed output's size")
     if gate is None:
         return None, 0, int(dv)
-    if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (T, nh * dv):
+    if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1:
         raise KernelError("attention: gate shape, dtype or layout")
-    return gate.data_ptr(), gate.stride(0), int(dv)
+    if tuple(gate.shape) == (T, nh * dv):
+        return gate.data_ptr(), gate.stride(0), int(dv)
+    if tuple(gate.shape) != (T, nh) or not per_head:
+        raise KernelError("attention: gate shape, dtype or layout")
+    return gate.data_ptr(), -gate.stride(0), int(dv)           # (a negative pitch: one logit a head)
 
 
 def attention_decode(q, view, batch, out, *, nh, window, scale, status, gate=None, dv=0, chunk=0, softcap=0.0,
                      sink=False):
     """Attention of one new token per sequence over the cache alone (its own key already
     appended); split along the keys and merged.  With ``dv`` the merge writes [T, nh * dv], the
-    first dv columns of every head, times sigmoid(``gate``) (a float32 column slice [T, nh * dv])
-    if given."""
+    first dv columns of every head, times sigmoid(``gate``) (a float32 column slice [T, nh * dv], or
+    [T, nh]: one logit a head) if given."""
     g = view.group
     T = batch.num_tokens
     if q.dtype != g.dtype or out.dtype != q.dtype:
         raise KernelError("attention: dtypes of queries, cache and output must agree")
-    gp, gld, gdv = _gate_args(out, T, nh, g.head_dim, gate, dv)
+    gp, gld, gdv = _gate_args(out, T, nh, g.head_dim, gate, dv, per_head=True)
     nsplit = decode_splits(q.device, T, _head_blocks(nh, g.num_kv_heads, g, q.dtype), getattr(batch, "max_end", 0))
     partial = torch.empty(T * nh * nsplit * (g.head_dim + 2), dtype=torch.float32, device=q.device)
     _ok(lib().moe_attention_decode(_p(q), _p(view.k), _p(view.v), _p(out), _p(partial), _dt(q),
@@ -1242,12 +1327,18 @@ def pair_norm_mean(a, wa, b, wb, eps, out):
     _ok(lib().moe_pair_norm_mean(_p(a), _p(wa), _p(b), _p(wb), float(eps), T, H, _p(out), _stream()), "pair_norm_mean")
 
 
-def relu2(x, out):
-    """out = relu(x)^2, rounded to ``out``'s dtype."""
+def plain_act(x, out, act):
+    """out = act(x) element by element, rounded to ``out``'s dtype; ``act`` is one of ``PLAIN_ACTS``: "relu2" is
+    relu(x)^2, "gelu" x times the normal distribution's probability below x."""
     _chk(x, "x", torch.float32), _chk(out, "out")
     if out.numel() != x.numel():
-        raise KernelError("relu2: sizes differ")
-    _ok(lib().moe_relu2(_p(x), _p(out), _dt(out), x.numel(), _stream()), "relu2")
+        raise KernelError("plain_act: sizes differ")
+    _ok(lib().moe_plain_act(_p(x), _p(out), _dt(out), x.numel(), PLAIN_ACTS[act], _stream()), "plain_act")
+
+
+def relu2(x, out):
+    """out = relu(x)^2, rounded to ``out``'s dtype."""
+    plain_act(x, out, "relu2")
 
 
 def table_route(table, batch, top_k, num_experts, topk_idx, topk_w, status):
@@ -1317,3 +1408,70 @@ def ssd_finish(y, z, norm_w, eps, batch, out, *, norm_groups):
         raise KernelError("ssd_finish: shapes")
     _ok(lib().moe_ssd_finish(_p(y), _p(z), z.stride(0), _p(norm_w), float(eps), _p(batch.seq_of_token), T, inner,
                              int(norm_groups), _p(out), _dt(out), _stream()), "ssd_finish")
+
+
+def _delta_state(state, offset, floats):
+    if not state.is_cuda or state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1:
+        raise KernelError("delta: the state must be float32 rows (a column slice is fine)")
+    if offset + floats > state.shape[1]:
+        raise KernelError("delta: the state's row is too short")
+    return state.data_ptr() + 4 * int(offset)
+
+
+def delta_prepare(proj, taps_w, a_log, dt_bias, state, batch, out, step, *, heads, kv_heads, d, dv, b_at, a_at, eps, q_scale,
+                  offset=0):
+    """From 32-bit projection rows [q (kv_heads x d) | k (kv_heads x d) | v (heads x dv) | ...] with the columns of b
+    and a (one a value head) from ``b_at`` and ``a_at``: the causal convolution of q, k and v (``taps_w`` float32 [taps,
+    channels]; earlier rows come from the step or from ``state``, whose rows hold (taps - 1) * channels floats from
+    ``offset``) and silu; query and key heads divided by sqrt(sum(x^2) + eps), queries also times ``q_scale``, into ``out``
+    float32 [T, channels]; sigmoid(b) and -exp(a_log) softplus(a + dt_bias) into ``step`` float32 [T, 2 heads].  In a step
+    of one token a sequence the convolution's state is moved on here; else the caller runs ``conv_state_update``."""
+    _chk(proj, "proj", torch.float32, 2), _chk(taps_w, "taps", torch.float32, 2), _chk(out, "out", torch.float32, 2)
+    _chk(a_log, "A_log", torch.float32, 1), _chk(dt_bias, "dt_bias", torch.float32, 1), _chk(step, "step", torch.float32, 2)
+    T, channels, taps = proj.shape[0], 2 * kv_heads * d + heads * dv, taps_w.shape[0]
+    if (taps_w.shape[1] != channels or tuple(out.shape) != (T, channels) or tuple(step.shape) != (T, 2 * heads)
+            or a_log.numel() != heads or dt_bias.numel() != heads or proj.shape[1] < max(channels, b_at + heads, a_at + heads)):
+        raise KernelError("delta_prepare: shapes")
+    st = _delta_state(state, offset, (taps - 1) * channels) if taps > 1 else None
+    _ok(lib().moe_delta_prepare(_p(proj), proj.stride(0), int(b_at), int(a_at), _p(taps_w), taps, st,
+                                state.stride(0) if taps > 1 else 0, _p(a_log), _p(dt_bias), _p(batch.seq_of_token),
+                                _p(batch.cu_seqlens), _p(batch.slots), T, heads, kv_heads, d, dv, float(eps), float(q_scale),
+                                1 if (batch.all_decode and taps > 1) else 0, _p(out), _p(step), _stream()), "delta_prepare")
+
+
+def _delta_chk(qkv, step, heads, kv_heads, d, dv):
+    _chk(qkv, "qkv", torch.float32, 2), _chk(step, "step", torch.float32, 2)
+    T = qkv.shape[0]
+    if qkv.shape[1] != 2 * kv_heads * d + heads * dv or tuple(step.shape) != (T, 2 * heads) or heads % kv_heads:
+        raise KernelError("delta: shapes")
+    return T
+
+
+def delta_step(qkv, step, state, gate, norm_w, norm_eps, batch, out, *, heads, kv_heads, d, dv, offset=0) -> bool:
+    """One token a sequence of the gated delta rule on what ``delta_prepare`` left, with the head norm (RMS, times
+    ``norm_w`` [heads * dv]) and silu(``gate``) behind it, into ``out`` [T, heads * dv]; ``state`` rows hold heads * d * dv
+    floats from ``offset``.  False, with nothing launched, for sizes the kernel does not take."""
+    T = _delta_chk(qkv, step, heads, kv_heads, d, dv)
+    _chk(norm_w, "norm weight", torch.float32, 1), _chk(out, "out", dims=2)
+    if (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * dv)
+            or tuple(out.shape) != (T, heads * dv) or norm_w.numel() != heads * dv):
+        raise KernelError("delta_step: shapes")
+    code = lib().moe_delta_step(_p(qkv), _p(step), _delta_state(state, offset, heads * d * dv), state.stride(0), _p(gate),
+                                gate.stride(0), _p(norm_w), float(norm_eps), _p(batch.seq_of_token), _p(batch.cu_seqlens),
+                                _p(batch.slots), T, batch.num_seqs, heads, kv_heads, d, dv, _p(out), _dt(out), _stream())
+    if code == -1:
+        return False
+    _ok(code, "delta_step")
+    return True
+
+
+def delta_scan(qkv, step, state, batch, o, *, heads, kv_heads, d, dv, offset=0):
+    """Per sequence and value head, tokens in order: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, on
+    what ``delta_prepare`` left; o: float32 [T, heads * dv]."""
+    T = _delta_chk(qkv, step, heads, kv_heads, d, dv)
+    _chk(o, "o", torch.float32, 2)
+    if tuple(o.shape) != (T, heads * dv):
+        raise KernelError("delta_scan: shapes")
+    _ok(lib().moe_delta_scan(_p(qkv), _p(step), _delta_state(state, offset, heads * d * dv), state.stride(0),
+                             _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs, heads, kv_heads, d, dv, _p(o), _stream()),
+        "delta_scan")

@@ -133,7 +133,7 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swiglu: bool
     """out = x @ w[g].T (PLAIN) or act(x @ gate.T) * (x @ up.T) (SwiGLU, w rows = gate then up; ``act``
     is the gate's activation, one of ``core.GLU_ACTS``, ``act_param`` its constant if it has one).
 
-    Without ``swiglu``, ``act`` may name a function of the output itself (``core.PLAIN_ACTS``: "relu2").
+    Without ``swiglu``, ``act`` may name a function of the output itself (``core.PLAIN_ACTS``: "relu2", "gelu").
 
     x: [M, K] bf16 (row pitch a multiple of 8); w: [N', K] or [G, N', K] bf16 contiguous;
     out: [M, N] float32 or bfloat16 with N = N' (PLAIN) or N' / 2 (SwiGLU).

@@ -66,24 +66,28 @@ class DenseSwiGLU(Part):
         return linear(rt, swiglu_linear(rt, h.act, self.w_gu, self.activation, self.limit), self.w_down)
 
 
-def relu2_linear(rt, a, w_up, out=None):
-    """relu(a Wu^T)^2 in the compute dtype: in the tensor-core product's epilogue (on the 32-bit
-    accumulator) where that kernel takes the product, else the product's 32-bit output and then the
-    activation."""
+def act_linear(rt, a, w_up, act, out=None):
+    """act(a Wu^T) in the compute dtype (``act``: one of ``core.PLAIN_ACTS``): in the tensor-core product's
+    epilogue (on the 32-bit accumulator) where that kernel takes the product, else the product's 32-bit
+    output and then the activation."""
     if out is None:
         out = torch.empty((a.shape[0], w_up.shape[0]), dtype=rt.compute_dtype, device=a.device)
     if rt.is_bf16 and a.dtype == torch.bfloat16 and w_up.dtype == torch.bfloat16:
         from ..ops import tc
 
-        if tc.gemm_tc(a, w_up, out, status=rt.status, act="relu2"):
+        if tc.gemm_tc(a, w_up, out, status=rt.status, act=act):
             return out
-    core.relu2(linear(rt, a, w_up), out)
+    core.plain_act(linear(rt, a, w_up), out, act)
     return out
 
 
+def relu2_linear(rt, a, w_up, out=None):
+    return act_linear(rt, a, w_up, "relu2", out)
+
+
 class DenseMLP(Part):
-    """y = Wd f(Wu n), no gate; ``activation`` names f: "relu2" is relu(z)^2.  The activation is 32-bit
-    arithmetic on the first product's 32-bit output; the bfloat16 path rounds its result."""
+    """y = Wd f(Wu n), no gate; ``activation`` names f: "relu2" is relu(z)^2, "gelu" the exact (erf) GELU.  The
+    activation is 32-bit arithmetic on the first product's 32-bit output; the bfloat16 path rounds its result."""
 
     category, kind = "ffn", "dense_mlp"
     graph_safe = True
@@ -95,8 +99,8 @@ class DenseMLP(Part):
         self.hidden = int(self.params["hidden_size"])
         self.size = int(self.params["size"])
         self.activation = str(self.params.get("activation", "relu2"))
-        if self.activation != "relu2":
-            raise ValueError(f"dense feed-forward: activation '{self.activation}' is none of ['relu2']")
+        if self.activation not in core.PLAIN_ACTS:
+            raise ValueError(f"dense feed-forward: activation '{self.activation}' is none of {sorted(core.PLAIN_ACTS)}")
 
     def tensors(self):
         n = self.names
@@ -111,7 +115,7 @@ class DenseMLP(Part):
         self.w_down = tensors[self.names["down"]].contiguous()
 
     def forward(self, rt, h, batch):
-        return linear(rt, relu2_linear(rt, h.act, self.w_up), self.w_down)
+        return linear(rt, act_linear(rt, h.act, self.w_up, self.activation), self.w_down)
 
 
 class CombineDelta(LazyDelta):

@@ -1,8 +1,9 @@
 """Norms of the residual stream.
 
 RMSNorm: s = 1/sqrt(mean(x^2) + eps), out = x * s * w (src/model.rs:211-216).
+LayerNorm: out = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w (+ b).
 DynamicTanh: out = tanh(alpha x) * w + b with a scalar alpha; no statistic of x enters.
-Both add a pending delta to the 32-bit stream inside their kernel before they normalise it."""
+All add a pending delta to the 32-bit stream inside their kernel before they normalise it."""
 from __future__ import annotations
 
 import torch
@@ -100,6 +101,58 @@ class RMSNorm(Part):
         return Activations(act=out16 if rt.is_bf16 else out32, f32=out32)
 
 
+class LayerNorm(Part):
+    """Centred and scaled by the row's own mean and variance, times a weight; ``bias``: plus a shift.
+    ``scale``: a constant factor on the output (a model whose logits carry a factor puts it on the norm
+    in front of the output projection); it is folded into weight and shift when bound."""
+
+    category, kind = "norm", "layernorm"
+    graph_safe = True
+    default_names = {"weight": "weight", "bias": "bias"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.size = int(self.params["size"])
+        self.eps = float(self.params["eps"])
+        self.has_bias = bool(self.params.get("bias", False))
+        self.scale = float(self.params.get("scale", 1.0))
+
+    def tensors(self):
+        t = {self.names["weight"]: TensorSpec((self.size,), init="ones", vector=True)}
+        if self.has_bias:
+            t[self.names["bias"]] = TensorSpec((self.size,), init="zeros", vector=True)
+        return t
+
+    def describe(self):
+        return (f"LayerNorm eps {self.eps:g}" + ("" if self.has_bias else ", no bias")
+                + (f", output x {self.scale:g}" if self.scale != 1.0 else ""))
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        self.weight = (tensors[self.names["weight"]].to(torch.float32) * self.scale).contiguous()
+        self.bias = (tensors[self.names["bias"]].to(torch.float32) * self.scale).contiguous() if self.has_bias else None
+
+    def normed32(self, rt, t):
+        out = rt.empty(t.shape, torch.float32)
+        core.layernorm(t, self.weight, self.eps, bias=self.bias, out32=out, write_back=False, status=rt.status)
+        return out
+
+    def forward(self, rt, x, delta=None, rows=None, want32=False, write_back=True) -> Activations:
+        n = x.shape[0] if rows is None else rows.numel()
+        out32 = out16 = None
+        if rt.is_bf16:
+            out16 = rt.empty((n, self.size), torch.bfloat16)
+            if want32:
+                out32 = rt.empty((n, self.size), torch.float32)
+        else:
+            out32 = rt.empty((n, self.size), torch.float32)
+        if isinstance(delta, LazyDelta):
+            delta = delta.materialize(rt)
+        core.layernorm(x, self.weight, self.eps, bias=self.bias, delta=delta, rows=rows, out32=out32, out16=out16,
+                       write_back=write_back, status=rt.status)
+        return Activations(act=out16 if rt.is_bf16 else out32, f32=out32)
+
+
 class DynamicTanh(Part):
     """tanh(alpha * x) * weight + shift.  Where the delta it is handed is the output of a sublayer
     that has a Dynamic Tanh of its own in front of the residual sum (``PostNormDelta`` of kind
@@ -185,4 +238,5 @@ class ChannelScale(Part):
 
 register_part("scale", "channel_scale", ChannelScale)
 register_part("norm", "rmsnorm", RMSNorm)
+register_part("norm", "layernorm", LayerNorm)
 register_part("norm", "dyt", DynamicTanh)

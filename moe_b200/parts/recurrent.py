@@ -249,6 +249,110 @@ class SSDMixer(Part):
         return linear(rt, out, self.wo)
 
 
+class DeltaMixer(Part):
+    """The gated delta rule: a matrix-valued state per head that forgets by one decay number and is
+    corrected towards each token's value.
+
+    With n_t the layer's input, H value heads of dv on G query/key heads of d (value head h reads query/key
+    head h // (H // G)):
+        q, k, v = silu(conv(Wq n)), silu(conv(Wk n)), silu(conv(Wv n))      conv: causal over time, per channel,
+            ``taps`` factors a channel (tensors [channels, taps], the last one multiplies the token's own row)
+        q, k <- divided by sqrt(sum(x^2) + 1e-6) over the head;  q also times d^(-1/2)
+        beta = sigmoid(Wb n),  g = exp(-exp(A_log) softplus(Wa n + dt_bias))             one number a value head
+        S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q                 S [d, dv], zero at the start
+    and out = Wo ((o / rms(o over each head)) * norm_weight * silu(Wg n)), one norm weight of dv for all heads.
+
+    What a sequence carries from step to step is of fixed size: the convolutions' last taps - 1 inputs and
+    S of every value head, both 32-bit.  Everything but the projections is 32-bit arithmetic in both dtypes;
+    the bfloat16 path rounds the input of the two projections.  A step of one token a sequence is one
+    product, ``delta_prepare``, ``delta_step`` (recurrence, head norm and gate) and one product."""
+
+    category, kind = "mixer", "delta"
+    graph_safe = True
+    UNIT_EPS = 1e-6
+    default_names = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b",
+                     "a": "a", "a_log": "A_log", "dt_bias": "dt_bias", "gate": "g", "norm": "norm", "o": "o"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.hidden = int(p["hidden_size"])
+        self.nh, self.nkv = int(p["num_heads"]), int(p["num_kv_heads"])
+        self.d, self.dv = int(p["head_dim"]), int(p["value_dim"])
+        self.taps = int(p["taps"])
+        self.eps = float(p["eps"])                     # of the per-head norm of the output
+        if self.nh % self.nkv:
+            raise ValueError("delta: num_heads must be a multiple of num_kv_heads")
+        if not (0 < self.d <= 256 and self.dv > 0 and 1 <= self.taps <= 16):
+            raise ValueError(f"delta: heads of {self.d}, {self.taps} taps; the kernels take up to 256 and 1 to 16")
+        self.qk, self.inner = self.nkv * self.d, self.nh * self.dv
+        self.channels = 2 * self.qk + self.inner
+
+    def tensors(self):
+        n, W = self.names, self.hidden
+        return {
+            n["q"]: TensorSpec((self.qk, W)), n["k"]: TensorSpec((self.qk, W)), n["v"]: TensorSpec((self.inner, W)),
+            n["q_conv"]: TensorSpec((self.qk, self.taps)), n["k_conv"]: TensorSpec((self.qk, self.taps)),
+            n["v_conv"]: TensorSpec((self.inner, self.taps)),
+            n["b"]: TensorSpec((self.nh, W)), n["a"]: TensorSpec((self.nh, W)),
+            n["a_log"]: TensorSpec((self.nh,), init="zeros", vector=True),
+            n["dt_bias"]: TensorSpec((self.nh,), init="zeros", vector=True),
+            n["gate"]: TensorSpec((self.inner, W)),
+            n["norm"]: TensorSpec((self.dv,), init="ones", vector=True),
+            n["o"]: TensorSpec((W, self.inner)),
+        }
+
+    def describe(self):
+        return (f"gated delta rule ({self.nh} heads of {self.dv} on {self.nkv} query/key heads of {self.d}, state "
+                f"{self.d}x{self.dv} a head, convolution of {self.taps} taps)")
+
+    def kv_request(self):
+        return None
+
+    def state_request(self):
+        # [the convolutions' last taps - 1 inputs (to a multiple of four floats) | S of every value head]
+        return StateRequest((self._state_at() + self.nh * self.d * self.dv,), torch.float32)
+
+    def _state_at(self):
+        return -(-((self.taps - 1) * self.channels) // 4) * 4
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        n = self.names
+        ws = [tensors[n[r]] for r in ("q", "k", "v", "gate", "b", "a")]
+        dt = ws[0].dtype if all(w.dtype == ws[0].dtype for w in ws) else torch.float32
+        rows = sum(w.shape[0] for w in ws)
+        # (rows of zeros up to a multiple of eight: rows of the output stay 16-byte units)
+        ws.append(torch.zeros((-rows % 8, self.hidden), dtype=dt, device=ws[0].device))
+        self.w_in = torch.cat([w.to(dt) for w in ws], dim=0).contiguous()
+        self.gate_at = self.channels
+        self.b_at, self.a_at = self.channels + self.inner, self.channels + self.inner + self.nh
+        self.taps_w = torch.cat([tensors[n[r + "_conv"]].to(torch.float32) for r in ("q", "k", "v")], dim=0).t().contiguous()
+        self.a_log = tensors[n["a_log"]].to(torch.float32).contiguous()
+        self.dt_bias = tensors[n["dt_bias"]].to(torch.float32).contiguous()
+        self.norm_w = tensors[n["norm"]].to(torch.float32).repeat(self.nh).contiguous()
+        self.wo = tensors[n["o"]].contiguous()
+
+    def forward(self, rt, h, batch, cache_view, state):
+        T, C, I = batch.num_tokens, self.channels, self.inner
+        proj = linear(rt, h.act, self.w_in)                       # float32 [T, q | k | v | gate | b | a]
+        sizes = dict(heads=self.nh, kv_heads=self.nkv, d=self.d, dv=self.dv)
+        qkv = torch.empty((T, C), dtype=torch.float32, device=proj.device)
+        step = torch.empty((T, 2 * self.nh), dtype=torch.float32, device=proj.device)
+        core.delta_prepare(proj, self.taps_w, self.a_log, self.dt_bias, state, batch, qkv, step, b_at=self.b_at,
+                           a_at=self.a_at, eps=self.UNIT_EPS, q_scale=self.d ** -0.5, **sizes)
+        if self.taps > 1 and not batch.all_decode:
+            core.conv_state_update(proj, state, batch, taps=self.taps, channels=C)
+        gate = proj[:, self.gate_at:self.gate_at + I]
+        y = rt.empty((T, I))
+        at = dict(offset=self._state_at(), **sizes)
+        if not (batch.all_decode and core.delta_step(qkv, step, state, gate, self.norm_w, self.eps, batch, y, **at)):
+            o = torch.empty((T, I), dtype=torch.float32, device=proj.device)
+            core.delta_scan(qkv, step, state, batch, o, **at)
+            core.wkv_finish(o, gate, self.norm_w, self.eps, batch, y, heads=self.nh, d=self.dv)
+        return linear(rt, y, self.wo)
+
+
 class _SubTensors:
     """The tensors of a part that lives inside another: local names with the inner prefix taken off."""
 
@@ -380,4 +484,5 @@ class SideBySideMixer(Part):
 
 
 register_part("mixer", "ssd", SSDMixer)
+register_part("mixer", "delta", DeltaMixer)
 register_part("mixer", "side_by_side", SideBySideMixer)

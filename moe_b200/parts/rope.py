@@ -32,10 +32,17 @@ class RotaryEncoding(Part):
         if self.rotary_dim % 2:
             raise ValueError("rotary_dim must be even")
         self.interleaved = bool(self.params.get("interleaved", False))
+        # the table formed in float64 and rounded to float32 once, instead of the reference's float32 exponents
+        self.float64 = bool(self.params.get("float64", False))
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
-        self.inv_freq = rotary_inv_freq(self.theta, self.rotary_dim).to(rt.device)
+        if self.float64:
+            i = torch.arange(self.rotary_dim // 2, dtype=torch.float64)
+            table = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / self.rotary_dim).to(torch.float32)
+        else:
+            table = rotary_inv_freq(self.theta, self.rotary_dim)
+        self.inv_freq = table.to(rt.device)
 
     def describe(self):
         return (f"rope theta {self.theta:.0f}" + (f" on {self.rotary_dim} dims" if self.params.get("partial") else "")
@@ -91,7 +98,7 @@ class YarnRotary(RotaryEncoding):
         self.inv_freq = self.frequencies().to(rt.device)
 
     def describe(self):
-        return f"rope theta {self.theta:.0f} on {self.rotary_dim} dims, YaRN x{self.factor:g} from {self.original:g}"
+        return f"rope theta {self.theta:.0f} on {self.rotary_dim} dims, YaRN x{self.factor:g} from {self.original:g}" + (", pairs (2i, 2i+1)" if self.interleaved else "")
 
     def cos_sin_scale(self) -> float:
         return 0.1 * math.log(self.factor) + 1.0
