@@ -1346,6 +1346,269 @@ def run_zosipel(args):
     return 0
 
 
+# Ditazen at sizes that resemble a real model's layers, and beside each the library's closest model at
+# equal size: Zosipel with as many layers (run as often with the same weights), latent layers of the same
+# heads, head sizes and records, differential attention where Ditazen has its delta layers, and one expert
+# that every token takes with as many weights as Ditazen's feed-forward.  w2048 has records of 128 numbers
+# a position, w4096 of 256.
+DITAZEN_SHAPES = {
+    "w2048": dict(width=2048, heads=16, dim=96, rot=32, vdim=128, rank=96, q_rank=768, window=1024, d_heads=32, d_kv=16, d_dim=128,
+                  d_vdim=128, conv=4, ff=5632, order=("latent_attention", "latent_attention_2", "latent_attention_2", "delta"),
+                  vocab=32768),
+    "w4096": dict(width=4096, heads=32, dim=128, rot=64, vdim=128, rank=192, q_rank=1536, window=2048, d_heads=64, d_kv=32, d_dim=128,
+                  d_vdim=128, conv=4, ff=11008, order=("latent_attention", "latent_attention_2", "delta"), vocab=32768),
+}
+
+
+def ditazen_config(sh):
+    lat = {"heads": sh["heads"], "dim": sh["dim"], "rot_dim": sh["rot"], "vdim": sh["vdim"], "kv_rank": sh["rank"],
+           "scale": (sh["dim"] + sh["rot"]) ** -0.5}
+    mixers = {
+        "latent_attention": dict(lat, mask={"size": sh["window"]}, rot={"base": 5e5, "dims": sh["rot"]}),
+        "latent_attention_2": dict(lat, q_rank=sh["q_rank"], rot={
+            "base": 5e5, "dims": sh["rot"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}),
+        "delta": {"heads": sh["d_heads"], "kv_heads": sh["d_kv"], "dim": sh["d_dim"], "vdim": sh["d_vdim"], "conv": sh["conv"]},
+    }
+    layers = [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": sh["ff"]}} for t in sh["order"]]
+    layers += [dict(l, weights_of=j) for j, l in enumerate(layers)]
+    return {"architecture": "Ditazen", "vocab": sh["vocab"], "width": sh["width"], "norm": {"eps": 1e-5}, "logit_scale": 1.0,
+            "layers": layers}
+
+
+def ditazen_zosipel_config(sh):
+    lat = {"heads": sh["heads"], "dim": sh["dim"] + sh["rot"], "vdim": sh["vdim"], "kv_rank": sh["rank"] + sh["rot"],
+           "scale": (sh["dim"] + sh["rot"]) ** -0.5}
+    att = {"heads": sh["heads"], "kv_heads": sh["heads"] // 4, "dim": 64, "vdim": 128, "scale": 0.125, "softcap": 30.0, "diff": 0.3,
+           "mask": {"size": sh["window"]},
+           "rot": {"dims": 64, "base": 5e5, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "router": {"experts": 1, "top": 1}, "expert": {"ff": sh["ff"] * 2 // 3 // 64 * 64}}
+    n = len(sh["order"])
+    return {"architecture": "Zosipel", "vocab": sh["vocab"], "width": sh["width"], "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": n, "times": 2},
+            "layers": [{"type": "attention" if t == "delta" else "latent_attention", "mixer": att if t == "delta" else lat, "mlp": moe}
+                       for t in sh["order"]]}
+
+
+def ditazen_kernels(sh, pk):
+    """The new design's own kernels beside the like kernels of the library's other models, each alone at 8,192
+    tokens of 4 sequences (what a call reads and writes exceeds L2), as fractions of the measured copy
+    bandwidth (attention and products: of the measured bf16 peak, counting the products the mechanism needs);
+    then the recurrence and the attention of one token of 64 sequences (at a context of 2,048; calls whose
+    kernels are shorter than the host's work to launch them are replayed from a CUDA graph)."""
+    import torch
+
+    from moe_b200.cache.kv import KVCache, KVRequest
+    from moe_b200.ops import core, tc
+    from moe_b200.parts.feedforward import act_linear
+    from moe_b200.parts.latent import record_width
+
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    import gpu_util as G
+
+    dev, bf = "cuda:0", torch.bfloat16
+    B, n = 4, 2048
+    T, W = B * n, sh["width"]
+    H, d, rot, rk, qr, win = sh["heads"], sh["dim"], sh["rot"], sh["rank"], sh["q_rank"], sh["window"]
+    D = record_width(rk + rot, rk + rot, True)
+    status = core.new_status(dev)
+    r = lambda *s: torch.randn(*s, device=dev)
+    out = {}
+
+    def row(name, ms, nbytes=None, flops=None):
+        e = {"us": round(ms * 1e3, 1)}
+        if nbytes:
+            e["of_copy_peak"] = round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3)
+        if flops:
+            e["tflops"] = round(flops / ms / 1e9, 0)
+            e["of_bf16_peak"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 3)
+        out[name] = e
+
+    batch = G.make_batch(dev, list(range(1, B + 1)), [0] * B, [n] * B)
+    b1 = G.make_batch(dev, [1], [0], [n])
+    one = G.make_batch(dev, list(range(1, 65)), [n] * 64, [1] * 64)
+    # ---- norms --------------------------------------------------------------------------------------------
+    x, delta, w = r(T, W), r(T, W) / 100, r(W)
+    o16 = torch.empty((T, W), dtype=bf, device=dev)
+    nb = T * W * (4 + 4 + 4 + 2)
+    row("layernorm (sum + norm)", _median_ms(lambda: core.layernorm(x, w, 1e-5, delta=delta, out16=o16, status=status)), nb)
+    row("like: rmsnorm (sum + norm)", _median_ms(lambda: core.rmsnorm(x, w, 1e-5, delta=delta, out16=o16, status=status)), nb)
+    # ---- between projection and attention -----------------------------------------------------------------
+    freq = torch.rand(rot // 2, device=dev)
+    turn = dict(rot=rot, freq=freq, mscale=1.1)
+    q, k_new = torch.empty((T, H, D), dtype=bf, device=dev), torch.empty((T, 1, D), dtype=bf, device=dev)
+    cols = H * (rk + rot) + rk + rot
+    proj = r(T, -(-(cols + H) // 8) * 8)
+    wn, cw = r(rk), r(qr)
+    nb = T * (cols * 4 + (H + 1) * D * 2)
+    row("latent_prepare (records and queries, halves turned)", _median_ms(lambda: core.latent_prepare(
+        proj, batch, nh=H, d=rk, r=rk, width=D, weight=wn, eps=1e-5, q_t=q, k_new=k_new, token_major=True, status=status, **turn)), nb)
+    q32 = r(T, H * (rk + rot))
+    row("latent_prepare (queries, neighbours turned)", _median_ms(lambda: core.latent_prepare(
+        None, batch, q32=q32, nh=H, d=rk, r=rk, width=D, q_t=q, token_major=True, interleaved=True, status=status, **turn)),
+        T * H * ((rk + rot) * 4 + D * 2))
+    proj2 = r(T, -(-(qr + rk + rot + H) // 8) * 8)
+    cq = torch.empty((T, qr), dtype=bf, device=dev)
+    row("latent_prepare (records and the queries' latent)", _median_ms(lambda: core.latent_prepare(
+        proj2, batch, r=rk, width=D, weight=wn, eps=1e-5, k_new=k_new, lat_at=qr, cq=cq, cq_weight=cw, interleaved=True,
+        status=status, **turn)), T * ((qr + rk + rot) * 4 + (qr + D) * 2))
+    lproj = r(T, H * D + D)
+    wd_ = r(D)
+    row("like: latent_prepare without a rotation (records and queries)", _median_ms(lambda: core.latent_prepare(
+        lproj, batch, nh=H, d=D, r=D, width=D, weight=wd_, eps=1e-5, q_t=q, k_new=k_new, token_major=True, status=status)),
+        T * (H + 1) * D * 6)
+    # ---- attention of whole prompts -----------------------------------------------------------------------
+    seen = sum(min(p + 1, win) for p in range(n)) * B
+    causal = n * (n + 1) // 2 * B
+    lq, lk = torch.randn(T, H, D, device=dev).to(bf), torch.randn(T, 1, D, device=dev).to(bf)
+    ctx = torch.empty((T, H, D), dtype=bf, device=dev)
+
+    def prompt(window):
+        kw = dict(nh=H, window=window, scale=d ** -0.5, status=status)
+        if not tc.attention_prefill(lq, lk, lk, batch, ctx, nkv=1, hd=D, **kw):
+            cache = KVCache({0: KVRequest(1, D, None, values_are_keys=True)}, {0: None}, max_tokens=64, max_slots=1, dtype=bf, device=dev)
+            core.attention_tiled(lq, lk, lk, cache.view(0), batch, ctx, use_local=True, **kw)
+
+    row("attention of prompts over records, window", _median_ms(lambda: prompt(win)), flops=2.0 * seen * H * (2 * rk + rot))
+    row("attention of prompts over records, causal", _median_ms(lambda: prompt(None)), flops=2.0 * causal * H * (2 * rk + rot))
+    sinks = r(H)
+    zq, zk, zctx = (torch.randn(T, m, 128, device=dev).to(bf) for m in (H, 1, H))
+    row("like: tcgen05 attention over latents of 128, causal, a sink a head", _median_ms(lambda: tc.attention_prefill(
+        zq, zk, zk, batch, zctx, nh=H, nkv=1, hd=128, window=None, scale=0.1, status=status, sink=sinks)), flops=4.0 * causal * H * 128)
+    gk, gv = (torch.randn(T, H // 4, 128, device=dev).to(bf) for _ in range(2))
+    row("like: tcgen05 attention, 4 heads a kv head of 128, window", _median_ms(lambda: tc.attention_prefill(
+        zq, gk, gv, batch, zctx, nh=H, nkv=H // 4, hd=128, window=win, scale=0.1, status=status)), flops=4.0 * seen * H * 128)
+    # ---- after attention ----------------------------------------------------------------------------------
+    packed = torch.empty((T, H * rk), dtype=bf, device=dev)
+    row("gate_pack (a gate a head)", _median_ms(lambda: core.gate_pack(ctx, packed, nh=H, dv=rk, width=D, gate=proj[:, cols:cols + H])),
+        T * H * (rk * 4 + 4))
+    p128 = torch.empty((T, H * 128), dtype=bf, device=dev)
+    gl = r(T, H * 128)
+    row("like: gate_pack (a gate a column)", _median_ms(lambda: core.gate_pack(zctx, p128, nh=H, dv=128, width=128, gate=gl)),
+        T * H * 128 * 8)
+    # ---- the delta mixer ----------------------------------------------------------------------------------
+    dh, dk, dd, dv, taps = sh["d_heads"], sh["d_kv"], sh["d_dim"], sh["d_vdim"], sh["conv"]
+    ch, inner = 2 * dk * dd + dh * dv, dh * dv
+    dproj = r(T, ch + inner + 2 * dh)
+    sizes = dict(heads=dh, kv_heads=dk, d=dd, dv=dv)
+    off = (taps - 1) * ch
+    state = torch.zeros((66, off + dh * dd * dv), device=dev)
+    tw, alog, dtb = r(taps, ch), r(dh) - 1, r(dh) - 1
+    qkv, stp = torch.empty((T, ch), device=dev), torch.empty((T, 2 * dh), device=dev)
+
+    def prep(b, p, o, s):
+        core.delta_prepare(p, tw, alog, dtb, state, b, o, s, b_at=ch + inner, a_at=ch + inner + dh, eps=1e-6, q_scale=dd ** -0.5, **sizes)
+
+    row("delta_prepare (convolution + silu + unit norms + steps)", _median_ms(lambda: prep(batch, dproj, qkv, stp)), T * (ch * 8 + dh * 16))
+    bias = r(ch)
+    row("like: seq_conv with bias and silu", _median_ms(lambda: core.seq_conv(
+        [dict(u=dproj[:, :ch], w=tw, bias=bias, offset=0, out32=qkv)], state, batch, taps=taps, channels=ch, act="silu")), T * ch * 8)
+    prep(batch, dproj, qkv, stp)
+    o = torch.empty((T, inner), device=dev)
+    macs = 3.0 * inner * dd                               # the recurrence's multiply-adds a token
+    ms = _median_ms(lambda: core.delta_scan(qkv, stp, state, batch, o, offset=off, **sizes))
+    row("delta_scan (4 sequences of 2,048 tokens)", ms, T * (ch + inner) * 4, flops=2.0 * T * macs)
+    out["delta_scan (4 sequences of 2,048 tokens)"]["us_per_token_of_a_sequence"] = round(ms * 1e3 / n, 3)
+    row("delta_scan (one sequence of 2,048 tokens)", _median_ms(lambda: core.delta_scan(qkv[:n], stp[:n], state, b1, o[:n], offset=off, **sizes)),
+        n * (ch + inner) * 4, flops=2.0 * n * macs)
+    N = dd
+    xbc, dtr, dsk = r(T, inner + 2 * N), r(T, dh), r(dh)
+    sst = torch.zeros((66, dh * N * dv), device=dev)
+    ms = _median_ms(lambda: core.ssd_scan(xbc, dtr, dtb, alog, dsk, sst, batch, o, heads=dh, groups=1, n=N, dv=dv))
+    row("like: ssd_scan (4 sequences of 2,048 tokens)", ms, T * (2 * inner + 2 * N) * 4, flops=4.0 * T * inner * N)
+    row("like: ssd_scan (one sequence of 2,048 tokens)", _median_ms(lambda: core.ssd_scan(
+        xbc[:n], dtr[:n], dtb, alog, dsk, sst, b1, o[:n], heads=dh, groups=1, n=N, dv=dv)), n * (2 * inner + 2 * N) * 4, flops=4.0 * n * inner * N)
+    y, gate, nw = torch.empty((T, inner), dtype=bf, device=dev), dproj[:, ch:ch + inner], r(inner)
+    row("wkv_finish (head norm + gate)", _median_ms(lambda: core.wkv_finish(o, gate, nw, 1e-5, batch, y, heads=dh, d=dv)), T * inner * 10)
+    row("delta_step (one token of 64 sequences: the state read and written, head norm, gate)", _graph_ms(lambda: core.delta_step(
+        qkv[:64], stp[:64], state, gate[:64], nw, 1e-5, one, y[:64], offset=off, **sizes)), 64 * inner * dd * 8)
+    row("like: ssd_scan (one token of 64 sequences: the state read and written)", _graph_ms(lambda: core.ssd_scan(
+        xbc[:64], dtr[:64], dtb, alog, dsk, sst, one, o[:64], heads=dh, groups=1, n=N, dv=dv)), 64 * inner * N * 8)
+    # ---- the feed-forward's first product and activation ---------------------------------------------------
+    a16 = torch.randn(T, W, device=dev).to(bf)
+    wup = (torch.randn(sh["ff"], W, device=dev) / 32).to(bf)
+    act = torch.empty((T, sh["ff"]), dtype=bf, device=dev)
+    fl = 2.0 * T * sh["ff"] * W
+    row("up product with the exact gelu", _median_ms(lambda: act_linear(_Rt(status), a16, wup, "gelu", act)), flops=fl)
+    row("like: up product with the squared relu", _median_ms(lambda: act_linear(_Rt(status), a16, wup, "relu2", act)), flops=fl)
+    # ---- one token of 64 sequences at a context of 2,048: the cache read once -------------------------------
+    S, ctxlen = 64, 2048
+
+    def decode_case(nh, nkv, hd, window, latent, dv=0, gate=None, **kw):
+        cache = KVCache({0: KVRequest(nkv, hd, window, values_are_keys=latent)}, {0: None}, max_tokens=S * (ctxlen + 64),
+                        max_slots=S + 1, dtype=bf, device=dev)
+        cache.groups[0].storage.normal_()
+        slots = [cache.acquire() for _ in range(S)]
+        for s_ in slots:
+            G.give_pages(cache, s_, ctxlen + 1)
+        step = G.make_batch(dev, slots, [ctxlen] * S, [1] * S)
+        q_ = torch.randn(S, nh, hd, device=dev).to(bf)
+        o_ = torch.empty((S, nh * (dv or hd)), dtype=bf, device=dev)
+        ms = _graph_ms(lambda: core.attention_decode(q_, cache.view(0), step, o_, nh=nh, window=window, scale=0.1, status=status,
+                                                     dv=dv, gate=gate, **kw))
+        return ms, S * min(window or ctxlen + 1, ctxlen + 1) * nkv * hd * 2 * (1 if latent else 2)
+
+    row("decode attention over records, causal, a gate a head", *decode_case(H, 1, D, None, True, dv=rk, gate=proj[:S, cols:cols + H]))
+    row("decode attention over records, window, a gate a head", *decode_case(H, 1, D, win, True, dv=rk, gate=proj[:S, cols:cols + H]))
+    row("like: decode attention over latents of 128, a sink a head", *decode_case(H, 1, 128, None, True, sink=sinks))
+    core.check_status(status)
+    return out
+
+
+def _model_rates(cfg, args):
+    """Prefill of one prompt and decode of 1, 8 and 64 sequences with random weights of ``cfg``."""
+    import torch
+
+    import moe_b200
+
+    model = moe_b200.random_model(cfg, seed=0, dtype="bfloat16", device="cuda:0")
+    V = cfg["vocab"]
+    r = {"parameters": int(model.num_parameters)}
+    eng = moe_b200.Engine(model, max_tokens=64 * (512 + args.steps + 64) + 4096, max_slots=64)
+    ids = [(i * 7 + 13) % V for i in range(PREFILL_TOKENS)]
+
+    def prefill():
+        s = eng.new_sequence()
+        eng.step([s], [ids], check=False)
+        eng.release(s)
+
+    ms = _median_ms(prefill)
+    r["prefill_2048"] = {"ms": round(ms, 3), "tokens_per_s": round(PREFILL_TOKENS / ms * 1e3, 0)}
+    for B in (1, 8, 64):
+        slots = [eng.new_sequence() for _ in range(B)]
+        eng.step(slots, [ids[:PROMPT_LEN]] * B, check=False)
+        for i in range(args.warmup):
+            eng.step(slots, [[i % V]] * B, check=False)
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        for i in range(args.steps):
+            eng.step(slots, [[(i + 5) % V]] * B, check=False)
+        b.record()
+        torch.cuda.synchronize()
+        eng.rt.check()
+        ms = a.elapsed_time(b) / args.steps
+        r[f"decode_b{B}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(B / ms * 1e3, 0)}
+        for s in slots:
+            eng.release(s)
+    del eng, model
+    torch.cuda.empty_cache()
+    return r
+
+
+def run_ditazen(args):
+    """``--workload ditazen``: prefill and decode of the Ditazen design at two sizes, the closest existing
+    model at equal size beside it, and the new kernels beside their counterparts.  One JSON line per
+    shape; not the benchmark record."""
+    pk = peaks()
+    for name in [args.shape] if args.shape in DITAZEN_SHAPES else list(DITAZEN_SHAPES):
+        sh = DITAZEN_SHAPES[name]
+        res = {"workload": "ditazen", "shape": name, "sizes": sh, "dtype": "bfloat16", "data": "synthetic, random weights",
+               "peaks": pk, "ditazen": _model_rates(ditazen_config(sh), args), "zosipel": _model_rates(ditazen_zosipel_config(sh), args),
+               "kernels_at_8192_tokens": ditazen_kernels(sh, pk)}
+        print(json.dumps(res), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1359,12 +1622,12 @@ def main():
     ap.add_argument("--batch", type=int, default=8, help="with --profile-step decode: sequences in the batch")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="with --profile-step: the path whose kernels are wanted")
-    ap.add_argument("--shape", choices=["a2.7b", "57b"] + sorted(set(SUPEVIK_SHAPES) | set(FOGAPEL_SHAPES) | set(ZOSIPEL_SHAPES) | set(DIVADRA_SHAPES)), default="a2.7b",
-                    help="with --sweep: the layer sizes; with --workload supevik, fogapel, zosipel or divadra: one of its shapes (default: all)")
+    ap.add_argument("--shape", choices=["a2.7b", "57b"] + sorted(set(SUPEVIK_SHAPES) | set(FOGAPEL_SHAPES) | set(ZOSIPEL_SHAPES) | set(DIVADRA_SHAPES) | set(DITAZEN_SHAPES)), default="a2.7b",
+                    help="with --sweep: the layer sizes; with --workload supevik, fogapel, zosipel, divadra or ditazen: one of its shapes (default: all)")
     ap.add_argument("--prompt-len", type=int, default=0, help="with --sweep: tokens in each prompt (default 512)")
-    ap.add_argument("--workload", choices=["fp32-32k", "long-prompt", "supevik", "fogapel", "zosipel", "divadra"], default=None,
+    ap.add_argument("--workload", choices=["fp32-32k", "long-prompt", "supevik", "fogapel", "zosipel", "divadra", "ditazen"], default=None,
                     help="fp32-32k: the true 32-bit path at a context of 32,768; long-prompt: one bfloat16 prompt of "
-                         "--prompt-len tokens [32768] run in pieces; supevik, fogapel, zosipel, divadra: that design at two sizes beside "
+                         "--prompt-len tokens [32768] run in pieces; supevik, fogapel, zosipel, divadra, ditazen: that design at two sizes beside "
                          "the closest model at equal size (each prints its own line, no benchmark record)")
     ap.add_argument("--unequal", action="store_true", help="with --sweep: prompts of unequal lengths, 256 to 2,048 tokens")
     ap.add_argument("--sweep", default=None, help="comma-separated batch sizes: print decode throughput for each "
@@ -1392,6 +1655,8 @@ def main():
         return run_zosipel(args)
     if args.workload == "divadra":
         return run_divadra(args)
+    if args.workload == "ditazen":
+        return run_ditazen(args)
     return run_ours(args)
 
 
