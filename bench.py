@@ -1409,7 +1409,7 @@ def ditazen_kernels(sh, pk):
     B, n = 4, 2048
     T, W = B * n, sh["width"]
     H, d, rot, rk, qr, win = sh["heads"], sh["dim"], sh["rot"], sh["rank"], sh["q_rank"], sh["window"]
-    D = record_width(rk + rot, rk + rot, True)
+    D = record_width(rk + rot, True)
     status = core.new_status(dev)
     r = lambda *s: torch.randn(*s, device=dev)
     out = {}

@@ -624,7 +624,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 template <int HD>
-__global__ void __launch_bounds__(WARPS * 32, 4)
+__global__ void __launch_bounds__(WARPS * 32, HD <= 128 ? 4 : 2)
 attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                            const __nv_bfloat16* __restrict__ v_cache, float* __restrict__ partial,
                            const int* __restrict__ seq_of_token, const int* __restrict__ pos,
@@ -814,6 +814,8 @@ attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
 
 // Heads of a group at or above which the tensor-core kernel above takes a bfloat16 step.
 constexpr int GROUPED_MIN_HEADS = 8;
+// ... and for records of 192 and 256, which the kernels above stream at a lower rate
+constexpr int GROUPED_MIN_HEADS_WIDE = 3;
 
 template <int HD>
 int launch_grouped(const void* q, const void* k_cache, const void* v_cache, float* partial, const int* seq_of_token,
@@ -873,14 +875,14 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, f
     if (fused && !fast) return -1;
     if constexpr (sizeof(T) == 2) {
         // many heads on one key/value head: scores and weighted sum on the tensor cores
-        if (!fused && aligned && group >= GROUPED_MIN_HEADS && (hd == 64 || hd == 128) && page_size == GT_KEYS &&
-            ring % GT_KEYS == 0 && moe_decode_grouped_enabled()) {
-            const int rc = hd == 64 ? launch_grouped<64>(q, k_cache, v_cache, partial, seq_of_token, pos, slots, tables,
-                                                        table_stride, ring, num_pages, num_tokens, nh, nkv, window, scale,
-                                                        nsplit, status, stream, av)
-                                    : launch_grouped<128>(q, k_cache, v_cache, partial, seq_of_token, pos, slots, tables,
-                                                         table_stride, ring, num_pages, num_tokens, nh, nkv, window, scale,
-                                                         nsplit, status, stream, av);
+        if (!fused && aligned && page_size == GT_KEYS && ring % GT_KEYS == 0 && moe_decode_grouped_enabled() &&
+            (((hd == 64 || hd == 128) && group >= GROUPED_MIN_HEADS) ||
+             ((hd == 192 || hd == 256) && group >= GROUPED_MIN_HEADS_WIDE))) {
+#define GROUPED(HD_)                                                                                                   \
+    launch_grouped<HD_>(q, k_cache, v_cache, partial, seq_of_token, pos, slots, tables, table_stride, ring, num_pages, \
+                        num_tokens, nh, nkv, window, scale, nsplit, status, stream, av)
+            const int rc = hd == 64 ? GROUPED(64) : hd == 128 ? GROUPED(128) : hd == 192 ? GROUPED(192) : GROUPED(256);
+#undef GROUPED
             if (rc) return rc;
             return launch_pdl(attn_decode_merge_kernel<T>, dim3(num_tokens, nh), 128, 0, stream, (const float*)partial,
                               (T*)out, seq_of_token, nh, hd, nsplit, go, av);

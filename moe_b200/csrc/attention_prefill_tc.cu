@@ -1,5 +1,6 @@
 // Attention of a step of several tokens a sequence on the 5th-generation tensor cores (tcgen05),
-// head sizes 64 and 128: whole prompts, and sequences that go on from the cache.
+// head sizes 64 and 128 (192 and 256 where the values are the keys): whole prompts, and sequences that go on
+// from the cache.
 //
 // Same formulas as attention_prefill.cu (reference: src/model.rs:794-827): causal, optional window
 // [p + 1 - w, p] (or the chunk of p, capped scores and a softmax with a sink: AttnVariant in
@@ -32,6 +33,15 @@
 // tile j.  The MMAs of one thread run in the order they were issued: S of tile j + 2, which
 // overwrites P of tile j, is issued after P V of tile j and needs no barrier of its own.
 // Every barrier wait is bounded (ST_WAIT_TIMEOUT).
+//
+// SHARED: the values are the keys (attention over one record a position that all heads share).  A tile is
+// then fetched once and is the operand of both products, K-major in the first and MN-major in the second; its
+// stage is free again after P V, and the shared memory that the values would take leaves room for records of
+// 192 and 256 (two stages) and a third stage for smaller ones.
+//
+// The output is [T, nh, HD], or with dv > 0 packed to [T, nh * dv], the first dv columns of every head (only
+// those are computed), times the sigmoid of one gate logit a head: rounded to bfloat16 before the gate is
+// multiplied in, as the merge of a single-token step rounds it.
 #include <cuda.h>
 
 #include <mutex>
@@ -184,7 +194,13 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int HD>
+struct PackedOut {
+    int dv;                  // 0: whole records
+    const float* gate;       // one 32-bit logit a head, row pitch ld; null: none
+    int ld;
+};
+
+template <int HD, bool SHARED>
 __global__ void __launch_bounds__(320, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmKc,
@@ -192,10 +208,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                        const int* __restrict__ cu_seqlens, const int* __restrict__ seq_start,
                        const int* __restrict__ slots, const int* __restrict__ tables, int table_stride, int ring,
                        int num_pages, int num_seqs, int nh, int nkv, int window, float scale_log2, int* status,
-                       const AttnVariant av) {
+                       const AttnVariant av, const PackedOut po) {
     constexpr int CH = HD / 64;                      // 128-byte chunks of a row
     constexpr int TILE_BYTES = CH * 128 * 128;       // a 128-row operand tile
-    constexpr int STAGE_BYTES = 2 * TILE_BYTES;      // K, then V
+    constexpr int STAGE_BYTES = (SHARED ? 1 : 2) * TILE_BYTES;      // K, then V (SHARED: one tile for both)
+    constexpr int NST = SHARED && HD <= 128 ? 3 : 2;                // stages of keys
+    static_assert(SHARED || HD <= 128, "keys and values of their own: heads of up to 128");
     extern __shared__ uint8_t smem_raw[];
     __shared__ int s_seq, s_tile;
     __shared__ volatile int s_abort;
@@ -239,22 +257,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t sQ = base;
     auto sK = [&](int st) { return base + TILE_BYTES + st * STAGE_BYTES; };
-    auto sV = [&](int st) { return base + TILE_BYTES + st * STAGE_BYTES + TILE_BYTES; };
-    const uint32_t bars = base + TILE_BYTES + 2 * STAGE_BYTES;
+    auto sV = [&](int st) { return base + TILE_BYTES + st * STAGE_BYTES + (SHARED ? 0 : TILE_BYTES); };
+    const uint32_t bars = base + TILE_BYTES + NST * STAGE_BYTES;
     const uint32_t q_full = bars;
     auto k_full = [&](int st) { return bars + 8u * (1 + st); };
-    auto k_empty = [&](int st) { return bars + 8u * (3 + st); };
+    auto k_empty = [&](int st) { return bars + 8u * (4 + st); };
     auto v_full = [&](int st) { return bars + 8u * (15 + st); };
     auto v_empty = [&](int st) { return bars + 8u * (17 + st); };
-    auto s_full = [&](int b) { return bars + 8u * (5 + b); };
+    auto s_full = [&](int b) { return bars + 8u * (7 + b); };
     const uint32_t p_full = bars + 8u * 9, pv_done = bars + 8u * 10;
     auto x_bar = [&](int q) { return bars + 8u * (11 + q); };
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
-        for (int i = 0; i < 2; i++) {
+        for (int i = 0; i < NST; i++) {
             mbar_init(k_full(i), 1);
             mbar_init(k_empty(i), 1);
+        }
+        for (int i = 0; i < 2; i++) {
             mbar_init(v_full(i), 1);
             mbar_init(v_empty(i), 1);
             mbar_init(s_full(i), 1);
@@ -300,14 +320,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                 }
             };
             auto load_k = [&](int it) {
-                const int st = it & 1;
-                if (!mbar_wait(k_empty(st), ((it >> 1) & 1) ^ 1, &s_abort, status, 0x41)) return false;
+                const int st = it % NST, pb = it & 1;
+                if (!mbar_wait(k_empty(st), ((it / NST) & 1) ^ 1, &s_abort, status, 0x41)) return false;
                 if (it < nc) find_pages(it);
                 mbar_expect_tx(k_full(st), TILE_BYTES);
                 for (int c = 0; c < CH; c++) {
                     if (it < nc) {
-                        tma_load_2d(sK(st) + c * 16384, &tmKc, c * 64, page_row[st][0], k_full(st));
-                        tma_load_2d(sK(st) + c * 16384 + 8192, &tmKc, c * 64, page_row[st][1], k_full(st));
+                        tma_load_2d(sK(st) + c * 16384, &tmKc, c * 64, page_row[pb][0], k_full(st));
+                        tma_load_2d(sK(st) + c * 16384 + 8192, &tmKc, c * 64, page_row[pb][1], k_full(st));
                     } else {
                         tma_load_3d(sK(st) + c * 16384, &tmK, c * 64, kvh, tok0 + (t_lo + it - nc) * KT, k_full(st));
                     }
@@ -330,37 +350,42 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                 nv = it + 1;
                 return true;
             };
-            ok = load_k(0);
-            for (int it = 0; it < n_tiles && ok; it++) {
-                if (it + 1 < n_tiles) ok = load_k(it + 1);
-                if (ok) ok = load_v(it);
+            if (SHARED) {
+                for (int it = 0; it < n_tiles && ok; it++) ok = load_k(it);
+            } else {
+                ok = load_k(0);
+                for (int it = 0; it < n_tiles && ok; it++) {
+                    if (it + 1 < n_tiles) ok = load_k(it + 1);
+                    if (ok) ok = load_v(it);
+                }
             }
             if (!ok) {
                 atomicOr(status, ST_WAIT_TIMEOUT);
                 s_abort = 1;
-                for (int i = max(0, nk - 2); i < nk; i++)       // copies in flight must land
-                    mbar_wait(k_full(i & 1), (i >> 1) & 1, nullptr, status, 0x43);
+                for (int i = max(0, nk - NST); i < nk; i++)       // copies in flight must land
+                    mbar_wait(k_full(i % NST), (i / NST) & 1, nullptr, status, 0x43);
                 for (int i = max(0, nv - 2); i < nv; i++) mbar_wait(v_full(i & 1), (i >> 1) & 1, nullptr, status, 0x43);
             }
         }
     } else if (warp == 1) {
         // ---- MMA issuer ----------------------------------------------------------------------------
         if (lane == 0) {
-            constexpr uint32_t idesc_s = instr_desc(KT, 0), idesc_pv = instr_desc(HD, 1);
+            constexpr uint32_t idesc_s = instr_desc(KT, 0);
+            const uint32_t idesc_pv = instr_desc(po.dv > 0 ? (po.dv + 15) & ~15 : HD, 1);      // only the columns that are kept
             bool ok = mbar_wait(q_full, 0, &s_abort, status, 0x44);
             auto issue_s = [&](int it) {           // scores of tile `it` into buffer it & 1
-                const int b = it & 1;
-                if (!mbar_wait(k_full(b), (it >> 1) & 1, &s_abort, status, 0x45)) return false;
+                const int b = it & 1, kb = it % NST;
+                if (!mbar_wait(k_full(kb), (it / NST) & 1, &s_abort, status, 0x45)) return false;
                 // (buffer b held P of tile it - 2: its P V product was issued before this, and the
                 // MMAs run in order)
                 tc_fence_after();
 #pragma unroll
                 for (int ks = 0; ks < HD / 16; ks++) {
                     const uint32_t off = (ks / 4) * 16384 + (ks % 4) * 32;
-                    umma_ss(tmem + COL_S + b * KT, desc_k_major(sQ + off), desc_k_major(sK(b) + off), idesc_s, ks > 0);
+                    umma_ss(tmem + COL_S + b * KT, desc_k_major(sQ + off), desc_k_major(sK(kb) + off), idesc_s, ks > 0);
                 }
                 umma_commit(s_full(b));
-                umma_commit(k_empty(b));           // the key tile is free when these MMAs have read it
+                if (!SHARED) umma_commit(k_empty(kb));           // the key tile is free when these MMAs have read it
                 return true;
             };
             if (ok) ok = issue_s(0);
@@ -368,7 +393,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                 if (it + 1 < n_tiles) ok = issue_s(it + 1);
                 if (!ok) break;
                 const int st = it & 1;
-                ok = mbar_wait(v_full(st), (it >> 1) & 1, &s_abort, status, 0x47) && mbar_wait(p_full, it & 1, &s_abort, status, 0x48);
+                const int vb = SHARED ? it % NST : st;
+                ok = (SHARED || mbar_wait(v_full(st), (it >> 1) & 1, &s_abort, status, 0x47)) && mbar_wait(p_full, it & 1, &s_abort, status, 0x48);
                 if (!ok) break;
                 tc_fence_after();
                 const uint32_t tp = tmem + COL_S + st * KT;      // P lies where the tile's scores were
@@ -377,11 +403,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 #pragma unroll
                     for (int ks = 0; ks < KT / 16; ks++)         // 16 keys per step: 8 columns of packed P
                         umma_ts(tmem + COL_O, tp + (ks / 2) * 32 + term * 16 + (ks % 2) * 8,
-                                desc_mn_major(sV(st) + ks * 2048), idesc_pv,
+                                desc_mn_major(sV(vb) + ks * 2048), idesc_pv,
                                 (it | term | ks) != 0);          // the output row accumulates over all tiles
                 }
                 umma_commit(pv_done);
-                umma_commit(v_empty(st));
+                umma_commit(SHARED ? k_empty(vb) : v_empty(st));
             }
             if (!ok) {
                 atomicOr(status, ST_WAIT_TIMEOUT);
@@ -550,19 +576,29 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             tc_fence_after();
             const float lsum = x_sum[0][r] + x_sum[1][r];
             const float inv = sigmoid_w ? 1.f : lsum > 0.f ? 1.f / lsum : 0.f;
-            uint4* dst = reinterpret_cast<uint4*>(out + ((size_t)(tok0 + min(row, len - 1)) * nh + head) * HD +
-                                                  half * (HD / 2));
+            const size_t item = (size_t)(tok0 + min(row, len - 1)) * nh + head;
+            const int ncols = po.dv > 0 ? po.dv : HD;
+            const float gate = po.gate ? 1.0f / (1.0f + expf(-po.gate[(size_t)(tok0 + min(row, len - 1)) * po.ld + head])) : 1.0f;
+            uint4* dst = reinterpret_cast<uint4*>(out + item * ncols + half * (HD / 2));
 #pragma unroll
             for (int c = 0; c < HD / 64; c++) {
                 float t[32];
                 tmem_ld32_issue(to + c * 32, t);               // (every lane of the warp takes part in the load)
                 tmem_ld_wait();
                 if (row < len) {
+                    if (po.gate) {
+#pragma unroll
+                        for (int d = 0; d < 32; d++) t[d] = __bfloat162float(__float2bfloat16_rn(t[d] * inv)) * gate;
+                    } else {
+#pragma unroll
+                        for (int d = 0; d < 32; d++) t[d] *= inv;
+                    }
 #pragma unroll
                     for (int d = 0; d < 32; d += 8) {
+                        if (half * (HD / 2) + c * 32 + d >= ncols) break;
                         uint4 v;
-                        v.x = pack_bf16(t[d] * inv, t[d + 1] * inv), v.y = pack_bf16(t[d + 2] * inv, t[d + 3] * inv);
-                        v.z = pack_bf16(t[d + 4] * inv, t[d + 5] * inv), v.w = pack_bf16(t[d + 6] * inv, t[d + 7] * inv);
+                        v.x = pack_bf16(t[d], t[d + 1]), v.y = pack_bf16(t[d + 2], t[d + 3]);
+                        v.z = pack_bf16(t[d + 4], t[d + 5]), v.w = pack_bf16(t[d + 6], t[d + 7]);
                         dst[(c * 32 + d) / 8] = v;
                     }
                 }
@@ -628,53 +664,67 @@ struct CacheArgs {
     int table_stride, ring, num_pages;
 };
 
-template <int HD>
+template <int HD, bool SHARED>
 int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CacheArgs& c, void* out,
            const int* cu_seqlens, int num_seqs, int num_tokens, int nh, int nkv, int window, float scale, int* status,
-           const AttnVariant av, cudaStream_t stream) {
+           const AttnVariant av, const PackedOut po, cudaStream_t stream) {
     constexpr int TILE_BYTES = (HD / 64) * 128 * 128;
-    const int smem = 5 * TILE_BYTES + 1024 + 192;
+    const int smem = (SHARED ? (HD <= 128 ? 4 : 3) : 5) * TILE_BYTES + 1024 + 192;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(((num_tokens + QT - 1) / QT + num_seqs) * nh);
-    return launch_pdl(attn_prefill_tc_kernel<HD>, grid, 320, (size_t)smem, stream, tmQ, tmK, tmV, c.tmK, c.tmV,
+    return launch_pdl(attn_prefill_tc_kernel<HD, SHARED>, grid, 320, (size_t)smem, stream, tmQ, tmK, tmV, c.tmK, c.tmV,
                       (__nv_bfloat16*)out, cu_seqlens, c.seq_start, c.slots, c.tables, c.table_stride, c.ring,
-                      c.num_pages, num_seqs, nh, nkv, window, scale * 1.4426950408889634f, status, av);
+                      c.num_pages, num_seqs, nh, nkv, window, scale * 1.4426950408889634f, status, av, po);
 }
 
 int run(const void* q, const void* k, const void* v, CacheArgs& c, void* out, const int* cu_seqlens, int num_seqs,
         int num_tokens, int nh, int nkv, int hd, int window, float scale, int* status, const AttnVariant av,
-        cudaStream_t stream) {
+        const PackedOut po, bool shared, cudaStream_t stream) {
     CUtensorMap tmQ, tmK, tmV;
     if (!make_map(&tmQ, q, num_tokens, nh, hd) || !make_map(&tmK, k, num_tokens, nkv, hd) ||
         !make_map(&tmV, v, num_tokens, nkv, hd))
         return -1;
     if (!c.seq_start) c.tmK = tmK, c.tmV = tmV;         // never used: no tile comes from the cache
-    if (hd == 64)
-        return launch<64>(tmQ, tmK, tmV, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, window, scale, status, av, stream);
-    return launch<128>(tmQ, tmK, tmV, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, window, scale, status, av, stream);
+#define RUN(HD_, S_)                                                                                                   \
+    return launch<HD_, S_>(tmQ, tmK, tmV, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, window, scale, status, av, po, stream)
+    if (shared) {
+        if (hd == 64) RUN(64, true);
+        if (hd == 128) RUN(128, true);
+        if (hd == 192) RUN(192, true);
+        RUN(256, true);
+    }
+    if (hd == 64) RUN(64, false);
+    RUN(128, false);
+#undef RUN
+}
+
+// heads of 64 and 128, and of 192 and 256 where the values are the keys; packed output in rows of whole 16-byte units
+bool takes(int hd, bool shared, int dv, const float* gate) {
+    return (hd == 64 || hd == 128 || (shared && (hd == 192 || hd == 256))) && dv % 8 == 0 && !(gate && dv == 0);
 }
 
 }  // namespace
 
-// q: [T, nh, hd], k, v: [T, nkv, hd], out: [T, nh * hd], all bfloat16, 16-byte aligned; sequences
-// start at position 0.  Returns -1 (nothing launched) for a head size or an alignment this kernel
+// q: [T, nh, hd], k, v: [T, nkv, hd], out: [T, nh * hd], all bfloat16, 16-byte aligned; with
+// dv > 0 out: [T, nh * dv], times sigmoid(gate[t * gate_ld + h]) if gate is given; sequences start at position 0.  Returns -1 (nothing launched) for a head size or an alignment this kernel
 // does not take: the caller then uses moe_attention_prefill_bf16.
 MOE_API int moe_attention_prefill_tc(const void* q, const void* k, const void* v, void* out, const int* cu_seqlens,
                                      int num_seqs, int num_tokens, int nh, int nkv, int hd, int window, float scale,
-                                     int* status, int chunk, float softcap, int sink,
-        const float* sink_vals, cudaStream_t stream) {
+                                     int* status, int chunk, float softcap, int sink, const float* sink_vals, int dv,
+                                     const float* gate, int gate_ld, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
-    if (nkv <= 0 || nh % nkv != 0 || nh > 65535) return (int)cudaErrorInvalidValue;
-    if (hd != 64 && hd != 128) return -1;
+    if (nkv <= 0 || nh % nkv != 0 || nh > 65535 || dv < 0 || dv > hd) return (int)cudaErrorInvalidValue;
+    const bool shared = k == v;
+    if (!takes(hd, shared, dv, gate)) return -1;
     if ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out) & 15) != 0) return -1;
     CacheArgs c{};
     return run(q, k, v, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, hd, window, scale, status,
-               AttnVariant{chunk, softcap, sink, sink_vals}, stream);
+               AttnVariant{chunk, softcap, sink, sink_vals}, PackedOut{dv, gate, gate_ld}, shared, stream);
 }
 
 // The same for sequences that go on from the cache: sequence i held seq_start[i] tokens before the
@@ -687,12 +737,13 @@ MOE_API int moe_attention_cached_tc(const void* q, const void* k, const void* v,
                                     const void* v_cache, void* out, const int* cu_seqlens, const int* seq_start,
                                     const int* slots, const int* tables, int table_stride, int ring, int page_size,
                                     int num_pages, int num_seqs, int num_tokens, int nh, int nkv, int hd, int window,
-                                    float scale, int* status, int chunk, float softcap, int sink,
-        const float* sink_vals, cudaStream_t stream) {
+                                    float scale, int* status, int chunk, float softcap, int sink, const float* sink_vals,
+                                    int dv, const float* gate, int gate_ld, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
-    if (nkv <= 0 || nh % nkv != 0 || nh > 65535 || num_pages <= 0) return (int)cudaErrorInvalidValue;
+    if (nkv <= 0 || nh % nkv != 0 || nh > 65535 || num_pages <= 0 || dv < 0 || dv > hd) return (int)cudaErrorInvalidValue;
     if (!seq_start || !slots || !tables || !k_cache || !v_cache) return (int)cudaErrorInvalidValue;
-    if (hd != 64 && hd != 128) return -1;
+    const bool shared = k == v && k_cache == v_cache;
+    if (!takes(hd, shared, dv, gate)) return -1;
     if (page_size != 64 || ring % 64 != 0 || (long long)num_pages * nkv * 64 > 0x7fffffffLL) return -1;
     if ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) != 0)
         return -1;
@@ -703,5 +754,5 @@ MOE_API int moe_attention_cached_tc(const void* q, const void* k, const void* v,
         !make_cache_map(&c.tmV, v_cache, (long long)num_pages * nkv * 64, hd))
         return -1;
     return run(q, k, v, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, hd, window, scale, status,
-               AttnVariant{chunk, softcap, sink, sink_vals}, stream);
+               AttnVariant{chunk, softcap, sink, sink_vals}, PackedOut{dv, gate, gate_ld}, shared, stream);
 }

@@ -937,11 +937,11 @@ def decode_splits(device, num_tokens: int, nkv: int, max_end: int = 0) -> int:
 
 def _head_blocks(nh: int, nkv: int, group_view=None, dtype=None) -> int:
     """Blocks along the heads of the decode attention's grid: a kv head's query heads two at a time, or,
-    where the tensor-core kernel for groups of eight and more heads takes the step (bfloat16, records of
-    64 or 128, pages of 64), sixteen at a time."""
+    where the tensor-core kernel for groups of many heads takes the step (bfloat16, pages of 64, eight and more
+    heads on records of 64 or 128, three and more on 192 or 256), sixteen at a time."""
     group = max(1, nh // max(nkv, 1))
-    if (group_view is not None and dtype == torch.bfloat16 and group >= 8 and group_view.head_dim in (64, 128)
-            and group_view.page_size == 64 and group_view.ring % 64 == 0):
+    if (group_view is not None and dtype == torch.bfloat16
+            and group >= {64: 8, 128: 8, 192: 3, 256: 3}.get(group_view.head_dim, 1 << 30) and group_view.page_size == 64 and group_view.ring % 64 == 0):
         return nkv * -(-group // 16)
     return nkv * (1 if group == 1 else -(-group // 2))
 

@@ -35,9 +35,9 @@ def lib():
 
         L.moe_attention_prefill_bf16.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P]
         L.moe_attention_prefill_bf16.restype = c_int
-        L.moe_attention_prefill_tc.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P, I, c_float, I, P, P]
+        L.moe_attention_prefill_tc.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P, I, c_float, I, P, I, P, I, P]
         L.moe_attention_prefill_tc.restype = c_int
-        L.moe_attention_cached_tc.argtypes = [P] * 10 + [I] * 10 + [c_float, P, I, c_float, I, P, P]
+        L.moe_attention_cached_tc.argtypes = [P] * 10 + [I] * 10 + [c_float, P, I, c_float, I, P, I, P, I, P]
         L.moe_attention_cached_tc.restype = c_int
         L.moe_tc_set_pdl.argtypes = [c_int]
         L.moe_tc_set_pdl.restype = None
@@ -200,27 +200,32 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swiglu: bool
 
 
 def attention_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, batch, out: torch.Tensor, *, nh: int, nkv: int,
-                      hd: int, window, scale: float, status=None, chunk=0, softcap=0.0, sink=False) -> bool:
+                      hd: int, window, scale: float, status=None, chunk=0, softcap=0.0, sink=False, dv: int = 0,
+                      gate=None) -> bool:
     """Causal (optionally windowed) attention of whole prompts on the tensor cores; every
     sequence of ``batch`` must start at position 0.  False if the head size is not taken.
-    Head sizes 64 and 128 run on tcgen05 (``attention_prefill_tc.cu``), 16 and 32 on mma.sync.
-    ``chunk``, ``softcap``, ``sink``: as in ``core.attention_generic``; only the tcgen05 kernel
-    takes them."""
-    if q.dtype != torch.bfloat16 or hd not in (16, 32, 64, 128):
+    Head sizes 64 and 128 (and, where ``v`` is ``k``, 192 and 256) run on tcgen05
+    (``attention_prefill_tc.cu``), 16 and 32 on mma.sync.
+    ``chunk``, ``softcap``, ``sink``: as in ``core.attention_generic``; ``dv``, ``gate``: ``out`` is [T, nh * dv],
+    the first dv columns (a multiple of 8) of every head, times sigmoid(``gate``) (a float32 column slice [T, nh])
+    if given.  Only the tcgen05 kernel takes these."""
+    wide = hd in (192, 256) and k.data_ptr() == v.data_ptr()
+    if q.dtype != torch.bfloat16 or not (hd in (16, 32, 64, 128) or wide):
         return False
     variant = core._variant(chunk, softcap, sink)
-    plain = variant == (0, 0.0, 0, None)
-    if not plain and not (hd in (64, 128) and status is not None and _ATTN_TC):
+    plain = variant == (0, 0.0, 0, None) and not dv and gate is None
+    on_tc = (hd in (64, 128) or wide) and status is not None and _ATTN_TC
+    if not on_tc and (not plain or wide):
         return False
-    if hd in (64, 128) and status is not None and _ATTN_TC:
+    if on_tc:
         code = lib().moe_attention_prefill_tc(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(),
                                               batch.cu_seqlens.data_ptr(), batch.num_seqs, batch.num_tokens, nh, nkv,
                                               hd, int(window or 0), float(scale), status.data_ptr(), *variant,
-                                              core._stream())
+                                              *_packed(out, batch.num_tokens, nh, hd, dv, gate), core._stream())
         if code != -1:
             core._ok(code, "attention_prefill_tc")
             return True
-        if not plain:
+        if not plain or wide:
             return False
     code = lib().moe_attention_prefill_bf16(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(),
                                             batch.cu_seqlens.data_ptr(), batch.num_seqs, batch.num_tokens, nh, nkv,
@@ -232,25 +237,43 @@ def attention_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, batch, 
 
 
 def attention_cached(q: torch.Tensor, k_new: torch.Tensor, v_new: torch.Tensor, view, batch, out: torch.Tensor, *,
-                     nh: int, window, scale: float, status, chunk=0, softcap=0.0, sink=False) -> bool:
+                     nh: int, window, scale: float, status, chunk=0, softcap=0.0, sink=False, dv: int = 0,
+                     gate=None) -> bool:
     """Causal (optionally windowed) attention of a step whose sequences go on from the cache, on
     tcgen05: the keys before the step from the pages of ``view`` (one layer's cache), the step's own
     from ``k_new`` / ``v_new``.  False, with nothing launched, for what the kernel does not take
-    (head sizes other than 64 and 128, another dtype or page size)."""
+    (head sizes other than 64 and 128 or, where the values are the keys, 192 and 256; another dtype or page
+    size).  ``dv``, ``gate``: as in ``attention_prefill``."""
     g = view.group
     hd = g.head_dim
-    if q.dtype != torch.bfloat16 or g.dtype != torch.bfloat16 or hd not in (64, 128) or not _ATTN_TC:
+    if q.dtype != torch.bfloat16 or g.dtype != torch.bfloat16 or hd not in (64, 128, 192, 256) or not _ATTN_TC:
         return False
     code = lib().moe_attention_cached_tc(q.data_ptr(), k_new.data_ptr(), v_new.data_ptr(), view.k.data_ptr(),
                                          view.v.data_ptr(), out.data_ptr(), batch.cu_seqlens.data_ptr(),
                                          batch.seq_start.data_ptr(), batch.slots.data_ptr(), g.table.data_ptr(),
                                          g.table.stride(0), g.ring, g.page_size, g.num_pages, batch.num_seqs,
                                          batch.num_tokens, nh, g.num_kv_heads, hd, int(window or 0), float(scale),
-                                         status.data_ptr(), *core._variant(chunk, softcap, sink), core._stream())
+                                         status.data_ptr(), *core._variant(chunk, softcap, sink),
+                                         *_packed(out, batch.num_tokens, nh, hd, dv, gate), core._stream())
     if code == -1:
         return False
     core._ok(code, "attention_cached_tc")
     return True
+
+
+def _packed(out, T: int, nh: int, hd: int, dv: int, gate):
+    """(dv, gate pointer, its row pitch) of an attention whose output is packed to [T, nh * dv]."""
+    if not dv:
+        if gate is not None:
+            raise core.KernelError("attention: a gate needs the value width dv")
+        return 0, None, 0
+    if not 0 < dv <= hd or out.numel() < T * nh * dv:
+        raise core.KernelError("attention: dv or the packed output's size")
+    if gate is None:
+        return int(dv), None, 0
+    if gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (T, nh):
+        raise core.KernelError("attention: the gate must be float32 [T, nh]")
+    return int(dv), gate.data_ptr(), gate.stride(0)
 
 
 def gather_rows(src: torch.Tensor, rows: torch.Tensor, n: int, status) -> torch.Tensor:

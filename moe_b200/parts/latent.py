@@ -51,8 +51,15 @@ from ..cache.kv import KVRequest
 from ..config.spec import PartSpec
 from ..ops import core
 from ..ops.linear import grouped_linear, linear
-from .attention import record_width
 from .base import Part, TensorSpec, make_part, register_part
+
+
+def record_width(n: int, bf16: bool) -> int:
+    """Width of a cached record of n numbers: in bfloat16 the tensor-core attention over records that are key
+    and value takes 64, 128, 192 and 256, everything takes multiples of 16."""
+    if bf16 and n <= 256:
+        return -(-n // 64) * 64
+    return -(-n // 16) * 16
 
 
 class LatentAttention(Part):
@@ -150,7 +157,7 @@ class LatentAttention(Part):
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
         n, H, d, dv, r, rot, Q = self.names, self.nh, self.hd, self.vd, self.rank, self.rot, self.q_inputs
-        self.width = D = record_width(self.record, self.record, rt.is_bf16)
+        self.width = D = record_width(self.record, rt.is_bf16)
         self.fold_q, self.fold_o = self._folds()
         self.position.bind(tensors, rt)
         table = self.position.rotary_table()[0] if rot else None
@@ -244,26 +251,37 @@ class LatentAttention(Part):
             # (the merge of the key splits multiplies by the gate and packs the heads)
             core.attention_decode(q, cache_view, batch, packed, gate=gate, dv=r, **kw)
             return linear(rt, packed, self.wo)
-        ctx = rt.empty((T, H, D))
+        ctx, done = None, False
+        if not batch.all_decode and rt.is_bf16:
+            from ..ops import tc
+
+            # (the tensor-core kernel may multiply by the gate and pack the heads itself)
+            forms = [(packed, dict(dv=r, gate=gate))] if packed is not None and r % 8 == 0 else []
+            for out, form in forms + [(None, {})]:
+                if out is None:
+                    out = ctx = rt.empty((T, H, D))
+                if getattr(batch, "has_padding", False):
+                    out.zero_()      # rows of no sequence are written by no attention kernel
+                if batch.all_fresh:
+                    done = tc.attention_prefill(q, k_new, k_new, batch, out, nkv=1, hd=D, **form, **kw)
+                else:
+                    done = tc.attention_cached(q, k_new, k_new, cache_view, batch, out, **form, **kw)
+                if done:
+                    break
+        if ctx is None and not done:
+            ctx = rt.empty((T, H, D))
+            if getattr(batch, "has_padding", False) and not batch.all_decode:
+                ctx.zero_()
         if batch.all_decode:
             core.attention_decode(q, cache_view, batch, ctx.view(T, H * D), **kw)
         else:
-            if getattr(batch, "has_padding", False):
-                ctx.zero_()      # rows of no sequence are written by no attention kernel
-            done = False
-            if rt.is_bf16:
-                from ..ops import tc
-
-                if batch.all_fresh:
-                    done = tc.attention_prefill(q, k_new, k_new, batch, ctx, nkv=1, hd=D, **kw)
-                else:
-                    done = tc.attention_cached(q, k_new, k_new, cache_view, batch, ctx, **kw)
             if not done and not core.attention_tiled(q, k_new, k_new, cache_view, batch, ctx, use_local=True, **kw):
                 core.attention_generic(q, k_new, k_new, cache_view, batch, ctx, use_local=True, **kw)
             if not early:
                 core.kv_commit(k_new, k_new, cache_view, batch, rt.status)
         if packed is not None:
-            core.gate_pack(ctx, packed, nh=H, dv=r, width=D, gate=gate)
+            if ctx is not None:
+                core.gate_pack(ctx, packed, nh=H, dv=r, width=D, gate=gate)
             return linear(rt, packed, self.wo)
         if self.fold_o:
             return linear(rt, ctx.view(T, H * D), self.wo)

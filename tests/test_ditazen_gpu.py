@@ -306,10 +306,11 @@ PASTS = [([0, 0, 0], [5, 70, 131]),                       # fresh sequences only
 
 
 @pytest.mark.parametrize("window", [None, 1, 64, 75, 200])
-@pytest.mark.parametrize("H,D", [(5, 64), (6, 128), (17, 128), (3, 192), (4, 256), (16, 256)])
-def test_steps_of_several_tokens_over_shared_records(H, D, window):
+@pytest.mark.parametrize("H,D,dv", [(5, 64, 40), (6, 128, 96), (17, 128, 8), (3, 192, 136), (4, 256, 248), (16, 256, 192), (2, 144, 0)])
+def test_steps_of_several_tokens_over_shared_records(H, D, dv, window):
     """Whole prompts and sequences that go on from the cache, all heads on one record that is key and value:
-    the tensor-core kernel where it takes the record's width, else the kernel that the layer falls back to."""
+    the tensor-core kernel where it takes the record's width, once with whole records as its output and once
+    packed to dv columns a head times the head's gate; else the kernel that the layer falls back to."""
     from moe_b200.cache import KVCache, KVRequest
     from moe_b200.ops import core, tc
 
@@ -333,10 +334,19 @@ def test_steps_of_several_tokens_over_shared_records(H, D, window):
         q, kn = torch.cat(Q).to(DEV).contiguous(), torch.cat([k[a:] for k, a in zip(K, before)]).to(DEV).contiguous()
         out = torch.full((q.shape[0], H, D), float("nan"), dtype=dt, device=DEV)
         kw = dict(nh=H, window=window, scale=scale, status=st)
-        done = (tc.attention_cached(q, kn, kn, cache.view(0), batch, out, **kw) if any(before)
-                else tc.attention_prefill(q, kn, kn, batch, out, nkv=1, hd=D, **kw))
-        assert done == (D in (64, 128))
-        if not done:
+
+        def on_tensor_cores(o, **form):
+            return (tc.attention_cached(q, kn, kn, cache.view(0), batch, o, **form, **kw) if any(before)
+                    else tc.attention_prefill(q, kn, kn, batch, o, nkv=1, hd=D, **form, **kw))
+
+        done = on_tensor_cores(out)
+        assert done == (D in (64, 128, 192, 256))
+        packed = None
+        if done:
+            logits = torch.randn(q.shape[0], H + 1)
+            packed = torch.full((q.shape[0], H * dv), float("nan"), dtype=dt, device=DEV)
+            assert on_tensor_cores(packed, dv=dv, gate=dev(logits)[:, 1:])
+        else:
             assert core.attention_tiled(q, kn, kn, cache.view(0), batch, out, use_local=True, **kw)
         core.check_status(st)
         o = 0
@@ -345,7 +355,11 @@ def test_steps_of_several_tokens_over_shared_records(H, D, window):
             s = torch.einsum("thd,jd->htj", Q[i].double(), k) * scale
             seen = plain.seen_mask(a + b, window)[a:]
             p = torch.softmax(s.masked_fill(~seen, float("-inf")), dim=-1)
-            close(out[o:o + b], torch.einsum("htj,jd->thd", p, k), 2e-2)
+            ref = torch.einsum("htj,jd->thd", p, k)
+            close(out[o:o + b], ref, 2e-2)
+            if packed is not None:
+                g = torch.sigmoid(logits[o:o + b, 1:].double())
+                close(packed[o:o + b].view(b, H, dv), ref[:, :, :dv] * g[:, :, None], 2e-2)
             o += b
 
 
