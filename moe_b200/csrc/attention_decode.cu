@@ -30,6 +30,7 @@ static inline int moe_decode_grouped_enabled() { return g_decode_grouped; }
 namespace {
 
 constexpr int MAX_HD = 256;
+constexpr int WIDE_HD = 1024;      // wider records (moe_attention_decode only) take the general kernel, one head at a time
 constexpr int WARPS = 4;
 
 template <typename T>
@@ -411,9 +412,9 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     }
 }
 
-// The general kernel: one lane per key row, any head size that is a multiple of 16.
-constexpr int GHS = 4;
-template <typename T>
+// The general kernel: one lane per key row, any head size that is a multiple of 16 up to MD; GHS heads of a
+// group are worked on at once.
+template <typename T, int GHS, int MD>
 __global__ void __launch_bounds__(WARPS * 32)
 attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                         float* __restrict__ partial, const int* __restrict__ seq_of_token,
@@ -448,12 +449,12 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
         for (int i = threadIdx.x; i < gh * hd; i += blockDim.x)
             qs[i] = ld_f(q + ((size_t)t * nh + kvh * group + h0 + i / hd) * hd + i % hd);
         __syncthreads();
-        float m[GHS], l[GHS], acc[GHS][MAX_HD / 32];
+        float m[GHS], l[GHS], acc[GHS][MD / 32];
 #pragma unroll
         for (int g = 0; g < GHS; g++) {
             m[g] = -INFINITY, l[g] = 0.f;
 #pragma unroll
-            for (int i = 0; i < MAX_HD / 32; i++) acc[g][i] = 0.f;
+            for (int i = 0; i < MD / 32; i++) acc[g][i] = 0.f;
         }
         for (int j0 = k_begin + warp * 32; j0 < k_end; j0 += WARPS * 32) {
             const int j = j0 + lane;
@@ -493,7 +494,7 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                     l[g] = l[g] * alpha + warp_sum(pr[g]);
                     m[g] = m_new;
 #pragma unroll
-                    for (int i = 0; i < MAX_HD / 32; i++) acc[g][i] *= alpha;
+                    for (int i = 0; i < MD / 32; i++) acc[g][i] *= alpha;
                 } else {
                     pr[g] = 0.f;
                 }
@@ -501,9 +502,9 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
 #pragma unroll 4
             for (int jj = 0; jj < n_valid; jj++) {
                 const T* vj = (const T*)__shfl_sync(0xffffffffu, (unsigned long long)vp, jj);
-                float vv[MAX_HD / 32];
+                float vv[MD / 32];
 #pragma unroll
-                for (int i = 0; i < MAX_HD / 32; i++) {
+                for (int i = 0; i < MD / 32; i++) {
                     const int d = lane + 32 * i;
                     vv[i] = (i < dpl && d < hd) ? ld_f(vj + d) : 0.f;
                 }
@@ -512,7 +513,7 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                     if (g < gh) {
                         const float pj = __shfl_sync(0xffffffffu, pr[g], jj);
 #pragma unroll
-                        for (int i = 0; i < MAX_HD / 32; i++) acc[g][i] = fmaf(pj, vv[i], acc[g][i]);
+                        for (int i = 0; i < MD / 32; i++) acc[g][i] = fmaf(pj, vv[i], acc[g][i]);
                     }
                 }
             }
@@ -522,7 +523,7 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             if (g < gh) {
                 float* r = red + ((size_t)warp * GHS + g) * rec;
 #pragma unroll
-                for (int i = 0; i < MAX_HD / 32; i++) {
+                for (int i = 0; i < MD / 32; i++) {
                     const int d = lane + 32 * i;
                     if (d < hd) r[d] = acc[g][i];
                 }
@@ -919,10 +920,14 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, f
             default: FAST_G(32); break;
         }
     } else {
-        const size_t smem = ((size_t)GHS * hd + (size_t)WARPS * GHS * (hd + 2)) * sizeof(float);
-        rc = launch_pdl(attn_decode_rows_kernel<T>, grid, WARPS * 32, smem, stream, (const T*)q, (const T*)k_cache,
-                        (const T*)v_cache, partial, seq_of_token, pos, slots, tables, table_stride, ring, page_size,
-                        num_pages, nh, nkv, hd, window, scale, status, av);
+        const int at_once = hd <= MAX_HD ? 4 : 1;
+        const size_t smem = ((size_t)at_once * hd + (size_t)WARPS * at_once * (hd + 2)) * sizeof(float);
+#define ROWS(G_, MD_)                                                                                                  \
+    launch_pdl(attn_decode_rows_kernel<T, G_, MD_>, grid, WARPS * 32, smem, stream, (const T*)q, (const T*)k_cache,    \
+               (const T*)v_cache, partial, seq_of_token, pos, slots, tables, table_stride, ring, page_size, num_pages, nh, \
+               nkv, hd, window, scale, status, av)
+        rc = at_once == 4 ? ROWS(4, MAX_HD) : ROWS(1, WIDE_HD);
+#undef ROWS
     }
 #undef FAST
 #undef FAST_G
@@ -980,7 +985,7 @@ MOE_API int moe_attention_decode(const void* q, const void* k_cache, const void*
     if (dv < 0 || dv > hd || (gate && dv == 0)) return (int)cudaErrorInvalidValue;
     const GateOut go{gate, gate_ld < 0 ? -gate_ld : gate_ld, dv, gate_ld < 0};
     const AttnVariant av{chunk, softcap, sink, sink_vals};
-    if (hd % 16 != 0 || hd > MAX_HD || hd <= 0 || nkv <= 0 || nh <= 0 || nh > 65535 || nh % nkv != 0 || nsplit < 1 ||
+    if (hd % 16 != 0 || hd > WIDE_HD || hd <= 0 || nkv <= 0 || nh <= 0 || nh > 65535 || nh % nkv != 0 || nsplit < 1 ||
         nsplit > 65535 || nkv > 65535 || num_tokens > 65535 || !q || !k_cache || !v_cache || !out || !partial)
         return (int)cudaErrorInvalidValue;
     // cache rows are read 16 bytes at a time; q and out at least by whole elements

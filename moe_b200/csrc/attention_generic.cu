@@ -15,12 +15,12 @@
 //
 // One warp per (token, head): lanes take one key each for the scores and one
 // slice of the head dimension each for the weighted sum.  Any number of heads
-// and groups; head_dim a multiple of 16 up to 256.
+// and groups; head_dim a multiple of 16 up to 1,024.
 #include "common.cuh"
 
 namespace {
 
-constexpr int MAX_HD = 256;
+constexpr int WIDE_HD = 1024;
 
 __device__ __forceinline__ float dot_row(const float* kp, const float* qs, int hd) {
     float s = 0.f;
@@ -47,7 +47,7 @@ __device__ __forceinline__ float dot_row(const __nv_bfloat16* kp, const float* q
     return s;
 }
 
-template <typename T>
+template <typename T, int MAX_HD>
 __global__ void __launch_bounds__(32)
 attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const T* __restrict__ v_new,
                     const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
@@ -130,19 +130,21 @@ MOE_API int moe_attention_generic(const void* q, const void* k_new, const void* 
                                   int chunk, float softcap, int sink, const float* sink_vals, cudaStream_t stream) {
     const AttnVariant av{chunk, softcap, sink, sink_vals};
     if (num_tokens <= 0) return 0;
-    if (hd % 16 != 0 || hd > MAX_HD || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535)
+    if (hd % 16 != 0 || hd > WIDE_HD || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535)
         return (int)cudaErrorInvalidValue;
     dim3 grid(num_tokens, nh);
-    if (dt == DT_F32)
-        attn_generic_kernel<float><<<grid, 32, 0, stream>>>(
-            (const float*)q, (const float*)k_new, (const float*)v_new, (const float*)k_cache, (const float*)v_cache,
-            (float*)out, seq_of_token, pos, seq_start, cu_seqlens, slots, tables, table_stride, ring, page_size,
-            num_pages, nh, nkv, hd, window, scale, use_local, status, av);
-    else
-        attn_generic_kernel<__nv_bfloat16><<<grid, 32, 0, stream>>>(
-            (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_new, (const __nv_bfloat16*)v_new,
-            (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (__nv_bfloat16*)out, seq_of_token, pos,
-            seq_start, cu_seqlens, slots, tables, table_stride, ring, page_size, num_pages, nh, nkv, hd, window,
-            scale, use_local, status, av);
+#define GENERIC(T_, MD_)                                                                                               \
+    attn_generic_kernel<T_, MD_><<<grid, 32, 0, stream>>>(                                                             \
+        (const T_*)q, (const T_*)k_new, (const T_*)v_new, (const T_*)k_cache, (const T_*)v_cache, (T_*)out, seq_of_token, \
+        pos, seq_start, cu_seqlens, slots, tables, table_stride, ring, page_size, num_pages, nh, nkv, hd, window, scale,  \
+        use_local, status, av)
+    if (dt == DT_F32) {
+        if (hd <= 256) GENERIC(float, 256);
+        else GENERIC(float, WIDE_HD);
+    } else {
+        if (hd <= 256) GENERIC(__nv_bfloat16, 256);
+        else GENERIC(__nv_bfloat16, WIDE_HD);
+    }
+#undef GENERIC
     return launch_status();
 }

@@ -65,6 +65,7 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, const float* v) {
 }
 
 constexpr int LATENT_MAX_ROT = 512;
+constexpr int CQ_UNITS = 2;        // 16-byte units of the queries' latent a thread keeps in registers
 
 struct LatentArgs {
     const int* pos;
@@ -91,7 +92,7 @@ struct LatentArgs {
 template <typename OT>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__ q_rec, OT* __restrict__ k_new,
-                      OT* __restrict__ cq, const LatentCommit c, int* status, int vec4) {
+                      OT* __restrict__ cq, const LatentCommit c, int* status, int vec4, int cq_vec) {
     __shared__ float red[32];
     __shared__ __align__(16) float ang[LATENT_MAX_ROT];        // cos[rot / 2], sin[rot / 2]
     const int t = blockIdx.x, rot = a.rot, half = rot / 2, D = a.D, r = a.r;
@@ -113,11 +114,35 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
         return second ? rot_hi(lo, hi, ang[i], ang[half + i]) : rot_lo(lo, hi, ang[i], ang[half + i]);
     };
     if (k_new) {
+        // Both latents' loads are on their way before either sum is formed; the queries' latent stays in
+        // registers (four elements a unit) where it fits, and both sums share their barriers.
         const float* row = a.proj + (size_t)t * a.ld;
         const float* lat = row + a.lat_at;
-        float ss = 0.f;
+        float4 cu[CQ_UNITS];
+        const bool cq_regs = cq_vec && a.q_rank <= 4 * CQ_UNITS * (int)blockDim.x;
+        float ss = 0.f, sq = 0.f;
+        if (a.cq_w && cq_regs) {
+#pragma unroll
+            for (int u = 0; u < CQ_UNITS; u++) {
+                const int i = (threadIdx.x + u * blockDim.x) * 4;
+                cu[u] = i < a.q_rank ? *reinterpret_cast<const float4*>(row + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
         for (int i = threadIdx.x; i < r; i += blockDim.x) ss += lat[i] * lat[i];
-        ss = block_sum(ss, red);
+        if (a.cq_w) {
+            if (cq_regs) {
+#pragma unroll
+                for (int u = 0; u < CQ_UNITS; u++)
+                    sq += cu[u].x * cu[u].x, sq += cu[u].y * cu[u].y, sq += cu[u].z * cu[u].z, sq += cu[u].w * cu[u].w;
+            } else {
+                for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) sq += row[i] * row[i];
+            }
+        }
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+        ss = warp_sum(ss), sq = warp_sum(sq);
+        if (lane == 0) red[warp] = ss, red[16 + warp] = sq;
+        __syncthreads();
+        ss = warp_sum(lane < nw ? red[lane] : 0.f), sq = warp_sum(lane < nw ? red[16 + lane] : 0.f);
         const float inv = 1.0f / sqrtf(ss / (float)r + a.eps);
         OT* cd = nullptr;
         OT* cv = nullptr;
@@ -140,12 +165,21 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
             if (cv) st_f(cv + i, x);
         }
         if (a.cq_w) {
-            float sq = 0.f;
-            for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) sq += row[i] * row[i];
-            sq = block_sum(sq, red);
             const float qi = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps);
-            for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x)
-                st_f(cq + (size_t)t * a.q_rank + i, row[i] * qi * a.cq_w[i]);
+            OT* cr = cq + (size_t)t * a.q_rank;
+            if (cq_regs) {
+#pragma unroll
+                for (int u = 0; u < CQ_UNITS; u++) {
+                    const int i = (threadIdx.x + u * blockDim.x) * 4;
+                    if (i < a.q_rank) {
+                        const float4 w = *reinterpret_cast<const float4*>(a.cq_w + i);
+                        const float v[4] = {cu[u].x * qi * w.x, cu[u].y * qi * w.y, cu[u].z * qi * w.z, cu[u].w * qi * w.w};
+                        st4(cr + i, v);
+                    }
+                }
+            } else {
+                for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) st_f(cr + i, row[i] * qi * a.cq_w[i]);
+            }
         }
     }
     if (!a.q32) return;
@@ -345,11 +379,15 @@ MOE_API int moe_latent_prepare(const float* proj, int ld, int lat_at, int r, con
                        freq, rot, interleaved, mscale, num_tokens, D};
     const int vec4 = dq % 4 == 0 && ldq % 4 == 0 && (uintptr_t)q32 % 16 == 0 && rot % (interleaved ? 4 : 8) == 0 &&
                      (!q_major || D % 4 == 0) && (uintptr_t)q_t % (out_dt == DT_F32 ? 16 : 8) == 0;
+    const int al = out_dt == DT_F32 ? 16 : 8;
+    const int cq_vec = cq_w && q_rank % 4 == 0 && ld % 4 == 0 && ((uintptr_t)proj | (uintptr_t)cq_w) % 16 == 0 && (uintptr_t)cq % al == 0;
+    // keys alone are little work a token: smaller blocks, more of them on an SM
+    const int threads = q32 || num_tokens < 512 ? 256 : 128;
     if (out_dt == DT_F32)
-        return launch_pdl(latent_prepare_kernel<float>, num_tokens, 256, 0, stream, a, (float*)q_t, (float*)q_rec,
-                          (float*)k_new, (float*)cq, c, status, vec4);
-    return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, 256, 0, stream, a, (__nv_bfloat16*)q_t,
-                      (__nv_bfloat16*)q_rec, (__nv_bfloat16*)k_new, (__nv_bfloat16*)cq, c, status, vec4);
+        return launch_pdl(latent_prepare_kernel<float>, num_tokens, threads, 0, stream, a, (float*)q_t, (float*)q_rec,
+                          (float*)k_new, (float*)cq, c, status, vec4, cq_vec);
+    return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, a, (__nv_bfloat16*)q_t,
+                      (__nv_bfloat16*)q_rec, (__nv_bfloat16*)k_new, (__nv_bfloat16*)cq, c, status, vec4, cq_vec);
 }
 
 // src: element (a, b, j) at a * s_outer + b * s_inner + j, j < n; dst: [B, A, wd] with rows of ldd elements (dense

@@ -238,7 +238,8 @@ MOE_API int moe_attention_tiled(const void* q, const void* k_new, const void* v_
                                 const float* sink_vals, cudaStream_t stream) {
     if (num_tokens <= 0 || num_seqs <= 0) return 0;
     const AttnVariant av{chunk, softcap, sink, sink_vals};
-    if (hd % 16 != 0 || hd > 256 || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return (int)cudaErrorInvalidValue;
+    if (hd > 256) return -1;
+    if (hd % 16 != 0 || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return (int)cudaErrorInvalidValue;
     if (page_size != BK || (ring % BK) != 0) return -1;
     const size_t align = dt == DT_F32 ? 16 : 8;          // rows are read four elements at a time
     if (((uintptr_t)q | (uintptr_t)k_new | (uintptr_t)v_new | (uintptr_t)k_cache | (uintptr_t)v_cache) % align) return -1;

@@ -11,7 +11,7 @@
 //                   In a step of one token a sequence the same launch moves the convolution's state on.
 //   delta_step      one token a sequence: the recurrence with the state read once and written once, and
 //                   the output's norm and gate behind it, a block a (head, sequence).
-//   delta_scan      several tokens a sequence, one after the other, the state in registers.
+//   delta_scan      several tokens a sequence, four at a time, the state in registers.
 // Everything here is 32-bit arithmetic; only the normed, gated output of delta_step is rounded.
 #include "common.cuh"
 
@@ -239,146 +239,261 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
              su[c] * inv * norm_w[(size_t)h * dv + c] * silu32(gate[(size_t)t * ldg + (size_t)h * dv + c]));
 }
 
-// ---- several tokens a sequence, one after the other ----------------------------------------------------
-// grid (ceil(dv / 64), heads, sequences), KP * 16 threads: thread (kp = tid % KP, cg = tid / KP) holds rows
-// kp * RPT ... of four neighbouring columns of S in registers (rows beyond d stay zero).  A run of TOK tokens is
-// staged in shared memory as [k | q | the block's columns of v | beta | decay] a token, the next run's loads in
-// flight while this one is worked on.  From one token to the next only S is carried, so the chain is: product
-// with k, its sum over the KP threads, u, the update; the product with q hangs off it.
-constexpr int DS_CPT = 4, DS_CG = 16, DS_COLS = DS_CPT * DS_CG;
+// ---- several tokens a sequence: four at a time ------------------------------------------------------------
+// With b_i the sum of the decays' logarithms from a group's first token to its i-th, S the state before the group,
+// and the index pairs j < i (or j <= i) inside the group,
+//     u_i = beta_i v_i - beta_i e^(b_i) S^T k_i - sum_(j<i) beta_i e^(b_i - b_j) (k_i . k_j) u_j
+//     o_i = e^(b_i) S^T q_i + sum_(j<=i) e^(b_i - b_j) (q_i . k_j) u_j
+//     S   <- e^(b_4) S + sum_j k_j (e^(b_4 - b_j) u_j)^T
+// which is the recurrence written out: every exponent is <= 0, only the order of additions differs.  Against
+// one token at a time the products with S are eight independent sums instead of two with an update between
+// them, their sums over the threads are formed together, and the state is multiplied by a decay once.
+//
+// grid (ceil(dv / 32), heads, sequences), 128 threads: thread (kp = tid % 16, cg = tid / 16) holds rows kp * RPT ...
+// of four neighbouring columns of S in registers (rows beyond d stay zero).  A run of sixteen tokens is staged
+// in shared memory as [k | q | the block's columns of v] a token (cp.async, two buffers; rows beyond the
+// sequence's last token are zeros with beta 0 and decay 1: they change nothing); warp w forms the scalars of the
+// run's group w.  Within a run the groups follow one another without a block barrier.
+constexpr int DG = 4, DRUN = 16, DKP = 16, DCG = 8, DCOLS = 4 * DCG, DTHREADS = DKP * DCG;
 
-template <int RPT, int KP, int TOK>
-__global__ void __launch_bounds__(KP * DS_CG)
+__device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes, bool on) {
+    const unsigned at = (unsigned)__cvta_generic_to_shared(dst);
+    const int n = on ? bytes : 0;
+    if (bytes == 16)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(at), "l"(src), "r"(n) : "memory");
+    else
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(at), "l"(src), "r"(n) : "memory");
+}
+
+// VEC: rows of q, k and v start on 16-byte boundaries and hold whole 16-byte units.
+template <int RPT, bool VEC>
+__global__ void __launch_bounds__(DTHREADS)
 delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
-    constexpr int NP = RPT * KP, THREADS = KP * DS_CG;
-    constexpr int PER_TOK = 2 * NP + DS_COLS + 2;
-    constexpr int ROWLEN = (PER_TOK + 3) & ~3;
-    constexpr int XPT = (PER_TOK + THREADS - 1) / THREADS;
-    extern __shared__ __align__(16) float sm[];               // [TOK][ROWLEN]
-    const int tid = threadIdx.x, kp = tid % KP, cg = tid / KP;
+    constexpr int NP = RPT * DKP;
+    constexpr int ROWLEN = 2 * NP + DCOLS;
+    extern __shared__ __align__(16) float sm[];               // [2][DRUN][ROWLEN] | steps [2][2][DRUN] | scalars [4][32] | u [DG][DCOLS]
+    float* s_step = sm + 2 * DRUN * ROWLEN;
+    float* s_coef = s_step + 4 * DRUN;
+    float* s_u = s_coef + 4 * 32;
+    const int tid = threadIdx.x, kp = tid % DKP, cg = tid / DKP, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, s = blockIdx.z, g = h / (p.H / p.G), d = p.d, dv = p.dv;
-    const int c0 = blockIdx.x * DS_COLS, col = c0 + cg * DS_CPT;
+    const int c0 = blockIdx.x * DCOLS, col = c0 + cg * 4;
+    for (int i = tid; i < 2 * DRUN * ROWLEN; i += DTHREADS) sm[i] = 0.f;         // columns that no copy writes stay zero
     pdl_sync();
     const int tok0 = p.cu_seqlens[s], cnt = p.cu_seqlens[s + 1] - tok0;
     if (cnt <= 0) return;
-    const int channels = 2 * p.G * d + p.H * dv;
+    const int channels = 2 * p.G * d + p.H * dv, ncols = min(DCOLS, dv - c0);
     float* S = p.state + (size_t)p.slots[s] * p.state_pitch + (size_t)h * d * dv;
-    const bool vec = dv % 4 == 0 && ((uintptr_t)S) % 16 == 0;
-    float sreg[RPT][DS_CPT];
+    const bool vec_state = dv % 4 == 0 && ((uintptr_t)S) % 16 == 0;
+    float sreg[RPT][4];
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
         const int n = kp * RPT + m;
-        if (vec && n < d && col < dv) {
+        if (vec_state && n < d && col < dv) {
             const float4 t4 = *reinterpret_cast<const float4*>(S + (size_t)n * dv + col);
             sreg[m][0] = t4.x, sreg[m][1] = t4.y, sreg[m][2] = t4.z, sreg[m][3] = t4.w;
         } else {
 #pragma unroll
-            for (int c = 0; c < DS_CPT; c++) sreg[m][c] = (n < d && col + c < dv) ? S[(size_t)n * dv + col + c] : 0.f;
+            for (int c = 0; c < 4; c++) sreg[m][c] = (n < d && col + c < dv) ? S[(size_t)n * dv + col + c] : 0.f;
         }
     }
-    // what this thread brings into shared memory of every token; where each element comes from is worked out once
-    const float* src[XPT];
-    long long pitch[XPT];
-#pragma unroll
-    for (int e = 0; e < XPT; e++) {
-        const int x = tid + e * THREADS;
-        src[e] = nullptr, pitch[e] = channels;
-        if (x < NP) {
-            if (x < d) src[e] = p.qkv + (size_t)tok0 * channels + (size_t)(p.G + g) * d + x;
-        } else if (x < 2 * NP) {
-            if (x - NP < d) src[e] = p.qkv + (size_t)tok0 * channels + (size_t)g * d + (x - NP);
-        } else if (x < 2 * NP + DS_COLS) {
-            const int c = c0 + x - 2 * NP;
-            if (c < dv) src[e] = p.qkv + (size_t)tok0 * channels + (size_t)2 * p.G * d + (size_t)h * dv + c;
-        } else if (x < PER_TOK) {
-            src[e] = p.step + (size_t)tok0 * 2 * p.H + (x - 2 * NP - DS_COLS) * p.H + h, pitch[e] = 2 * p.H;
+    const float* base = p.qkv + (size_t)tok0 * channels;
+    const float* sbase = p.step + (size_t)tok0 * 2 * p.H + h;
+    const int k_at = (p.G + g) * d, q_at = g * d, v_at = 2 * p.G * d + h * dv + c0;
+    auto stage = [&](int t0, int buf) {
+        float* dst = sm + buf * DRUN * ROWLEN;
+        constexpr int W = VEC ? 4 : 1;
+        const int kw = d / W, vw = ncols / W, per = 2 * kw + vw;
+        for (int i = tid; i < DRUN * per; i += DTHREADS) {
+            const int tt = i / per, e = i - tt * per;
+            const bool on = t0 + tt < cnt;
+            const float* row = base + (size_t)min(t0 + tt, cnt - 1) * channels;
+            if (e < kw) cp_zfill(dst + tt * ROWLEN + e * W, row + k_at + e * W, 4 * W, on);
+            else if (e < 2 * kw) cp_zfill(dst + tt * ROWLEN + NP + (e - kw) * W, row + q_at + (e - kw) * W, 4 * W, on);
+            else cp_zfill(dst + tt * ROWLEN + 2 * NP + (e - 2 * kw) * W, row + v_at + (e - 2 * kw) * W, 4 * W, on);
         }
-    }
-    float ahead[TOK][XPT];
-    auto fetch = [&](int t0) {
-        const int nt = min(TOK, cnt - t0);
-#pragma unroll
-        for (int tt = 0; tt < TOK; tt++) {
-            const long long r = t0 + min(tt, nt - 1);
-#pragma unroll
-            for (int e = 0; e < XPT; e++) ahead[tt][e] = src[e] ? src[e][r * pitch[e]] : 0.f;
+        if (tid < 2 * DRUN) {
+            const int tt = tid % DRUN, which = tid / DRUN;
+            cp_zfill(s_step + (buf * 2 + which) * DRUN + tt, sbase + (size_t)min(t0 + tt, cnt - 1) * 2 * p.H + which * p.H, 4, t0 + tt < cnt);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0);
-    const bool b0 = (kp & 1) != 0, b1 = (kp & 2) != 0;
-    // sums over the KP threads of a column group: afterwards every thread holds one column's, chosen by its
-    // lowest two bits (each thread drops the columns another one carries on)
-    auto reduce = [&](const float (&a)[2][DS_CPT]) {
-        const float p0 = a[0][0] + a[1][0], p1 = a[0][1] + a[1][1], p2 = a[0][2] + a[1][2], p3 = a[0][3] + a[1][3];
-        float v0 = (b0 ? p2 : p0) + __shfl_xor_sync(0xffffffffu, b0 ? p0 : p2, 1);
-        const float v1 = (b0 ? p3 : p1) + __shfl_xor_sync(0xffffffffu, b0 ? p1 : p3, 1);
-        v0 = (b1 ? v1 : v0) + __shfl_xor_sync(0xffffffffu, b1 ? v0 : v1, 2);
+    __syncthreads();                                  // the zeros are there before any copy writes
+    stage(0, 0);
+    const bool b0 = (kp & 1) != 0, b1 = (kp & 2) != 0, b2 = (kp & 4) != 0, b3 = (kp & 8) != 0;
+    const int my_col = (b0 ? 2 : 0) + (b1 ? 1 : 0);
+    for (int t0 = 0, buf = 0; t0 < cnt; t0 += DRUN, buf ^= 1) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                              // this run is there, and the one before is no longer read
+        if (t0 + DRUN < cnt) stage(t0 + DRUN, buf ^ 1);
+        const float* run = sm + buf * DRUN * ROWLEN;
+        {
+            // the scalars of group `warp`: products of its keys and queries, then everything made of them
+            const float* row = run + warp * DG * ROWLEN;
+            float dots[16];                           // [0 ... 5] k_i . k_j, j < i;  [6 ... 15] q_i . k_j, j <= i
 #pragma unroll
-        for (int off = 4; off < KP; off <<= 1) v0 += __shfl_xor_sync(0xffffffffu, v0, off);
-        return v0;
-    };
-    const int lane = tid & 31, group = lane & ~(KP - 1), my_col = (b0 ? 2 : 0) + (b1 ? 1 : 0);
-    for (int t0 = 0; t0 < cnt; t0 += TOK) {
-        const int nt = min(TOK, cnt - t0);
-        __syncthreads();                     // the run before is no longer read
+            for (int i = 0; i < 16; i++) dots[i] = 0.f;
+            for (int e = lane * 4; e < NP; e += 128) {
+                float4 k4[DG], q4[DG];
 #pragma unroll
-        for (int tt = 0; tt < TOK; tt++)
+                for (int i = 0; i < DG; i++) {
+                    k4[i] = *reinterpret_cast<const float4*>(row + i * ROWLEN + e);
+                    q4[i] = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + e);
+                }
+                int x = 0;
 #pragma unroll
-            for (int e = 0; e < XPT; e++) {
-                const int x = tid + e * THREADS;
-                if (x < PER_TOK) sm[tt * ROWLEN + x] = x == PER_TOK - 1 ? expf(ahead[tt][e]) : ahead[tt][e];
+                for (int i = 1; i < DG; i++)
+#pragma unroll
+                    for (int j = 0; j < i; j++, x++)
+                        dots[x] = fmaf(k4[i].x, k4[j].x, fmaf(k4[i].y, k4[j].y, fmaf(k4[i].z, k4[j].z, fmaf(k4[i].w, k4[j].w, dots[x]))));
+#pragma unroll
+                for (int i = 0; i < DG; i++)
+#pragma unroll
+                    for (int j = 0; j <= i; j++, x++)
+                        dots[x] = fmaf(q4[i].x, k4[j].x, fmaf(q4[i].y, k4[j].y, fmaf(q4[i].z, k4[j].z, fmaf(q4[i].w, k4[j].w, dots[x]))));
             }
+            // sixteen sums over the warp; lane l ends with number l & 15
+            float v8[8], v4[4], v2[2];
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                const bool up = (lane & 8) != 0;
+                v8[i] = (up ? dots[8 + i] : dots[i]) + __shfl_xor_sync(0xffffffffu, up ? dots[i] : dots[8 + i], 8);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const bool up = (lane & 4) != 0;
+                v4[i] = (up ? v8[4 + i] : v8[i]) + __shfl_xor_sync(0xffffffffu, up ? v8[i] : v8[4 + i], 4);
+            }
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const bool up = (lane & 2) != 0;
+                v2[i] = (up ? v4[2 + i] : v4[i]) + __shfl_xor_sync(0xffffffffu, up ? v4[i] : v4[2 + i], 2);
+            }
+            const bool up = (lane & 1) != 0;
+            float dot = (up ? v2[1] : v2[0]) + __shfl_xor_sync(0xffffffffu, up ? v2[0] : v2[1], 1);
+            dot += __shfl_xor_sync(0xffffffffu, dot, 16);
+            // [0 ... 3] beta_i  [4 ... 7] beta_i e^(b_i)  [8 ... 11] e^(b_i)  [12 ... 15] e^(b_4 - b_i)  [16 ... 21] beta_i e^(b_i - b_j) k_i . k_j
+            // [22 ... 31] e^(b_i - b_j) q_i . k_j
+            const float* be = s_step + buf * 2 * DRUN + warp * DG;
+            const float* lg = be + DRUN;
+            const float bs[DG] = {lg[0], lg[0] + lg[1], lg[0] + lg[1] + lg[2], lg[0] + lg[1] + lg[2] + lg[3]};
+            const int n = lane & 15;
+            if (lane < 16) {
+                const int i = n & 3;
+                const float ei = expf(i == 0 ? bs[0] : i == 1 ? bs[1] : i == 2 ? bs[2] : bs[3]);
+                float rest = 0.f;                     // b_4 - b_i, added up and not subtracted
+                for (int e = i + 1; e < DG; e++) rest += lg[e];
+                s_coef[warp * 32 + n] = n < 4 ? be[i] : n < 8 ? be[i] * ei : n < 12 ? ei : expf(rest);
+            } else {
+                // pair number n: j < i of the keys, then j <= i of queries and keys
+                const int i = n < 6 ? (n < 1 ? 1 : n < 3 ? 2 : 3) : (n < 7 ? 0 : n < 9 ? 1 : n < 12 ? 2 : 3);
+                const int j = n < 6 ? n - i * (i - 1) / 2 : n - 6 - i * (i + 1) / 2;
+                float decay = 0.f;                    // b_i - b_j, the same
+                for (int e = j + 1; e <= i; e++) decay += lg[e];
+                s_coef[warp * 32 + 16 + n] = dot * expf(decay) * (n < 6 ? be[i] : 1.f);
+            }
+        }
         __syncthreads();
-        if (t0 + TOK < cnt) fetch(t0 + TOK);
-#pragma unroll 2
-        for (int tt = 0; tt < nt; tt++) {
-            const float* row = sm + tt * ROWLEN;
-            const float beta = row[2 * NP + DS_COLS], decay = row[2 * NP + DS_COLS + 1];
-            float kr[RPT];
-            float acc[2][DS_CPT] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        const int groups = (min(DRUN, cnt - t0) + DG - 1) / DG;
+        for (int gr = 0; gr < groups; gr++) {
+            const float* row = run + gr * DG * ROWLEN + kp * RPT;
+            float kr[DG][RPT];
+            float hk[DG][4], hq[DG][4];
+#pragma unroll
+            for (int i = 0; i < DG; i++)
+#pragma unroll
+                for (int c = 0; c < 4; c++) hk[i][c] = 0.f, hq[i][c] = 0.f;
 #pragma unroll
             for (int m0 = 0; m0 < RPT; m0 += 4) {
-                const float4 k4 = *reinterpret_cast<const float4*>(row + kp * RPT + m0);
-                kr[m0] = k4.x, kr[m0 + 1] = k4.y, kr[m0 + 2] = k4.z, kr[m0 + 3] = k4.w;
 #pragma unroll
-                for (int z = 0; z < 4; z++)
+                for (int i = 0; i < DG; i++) {
+                    const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + m0);
+                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0);
+                    kr[i][m0] = k4.x, kr[i][m0 + 1] = k4.y, kr[i][m0 + 2] = k4.z, kr[i][m0 + 3] = k4.w;
+                    const float qi[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
-                    for (int c = 0; c < DS_CPT; c++) {
-                        sreg[m0 + z][c] *= decay;
-                        acc[z & 1][c] = fmaf(kr[m0 + z], sreg[m0 + z][c], acc[z & 1][c]);
-                    }
+                    for (int z = 0; z < 4; z++)
+#pragma unroll
+                        for (int c = 0; c < 4; c++) {
+                            hk[i][c] = fmaf(kr[i][m0 + z], sreg[m0 + z][c], hk[i][c]);
+                            hq[i][c] = fmaf(qi[z], sreg[m0 + z][c], hq[i][c]);
+                        }
+                }
             }
-            const float mine = beta * (row[2 * NP + cg * DS_CPT + my_col] - reduce(acc));
-            // the column's u from the thread of the group that holds it: column c = 2 * bit0 + bit1 of its number
-            float u[DS_CPT];
+            // Sums over the sixteen threads of a column group.  On the way every thread drops what another one
+            // carries on: bits 0 and 1 of kp pick the column, bit 2 the product with the keys or the queries.
+            float r2[2 * DG][2], r1[2 * DG], rr[DG];
 #pragma unroll
-            for (int c = 0; c < DS_CPT; c++) u[c] = __shfl_sync(0xffffffffu, mine, group + ((c >> 1) | ((c & 1) << 1)));
-            float oc[2][DS_CPT] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            for (int i = 0; i < DG; i++)
 #pragma unroll
-            for (int m0 = 0; m0 < RPT; m0 += 4) {
-                const float4 q4 = *reinterpret_cast<const float4*>(row + NP + kp * RPT + m0);
-                const float qi[4] = {q4.x, q4.y, q4.z, q4.w};
+                for (int c = 0; c < 2; c++) {
+                    r2[i][c] = (b0 ? hk[i][2 + c] : hk[i][c]) + __shfl_xor_sync(0xffffffffu, b0 ? hk[i][c] : hk[i][2 + c], 1);
+                    r2[DG + i][c] = (b0 ? hq[i][2 + c] : hq[i][c]) + __shfl_xor_sync(0xffffffffu, b0 ? hq[i][c] : hq[i][2 + c], 1);
+                }
 #pragma unroll
-                for (int z = 0; z < 4; z++)
+            for (int i = 0; i < 2 * DG; i++)
+                r1[i] = (b1 ? r2[i][1] : r2[i][0]) + __shfl_xor_sync(0xffffffffu, b1 ? r2[i][0] : r2[i][1], 2);
 #pragma unroll
-                    for (int c = 0; c < DS_CPT; c++) {
-                        sreg[m0 + z][c] = fmaf(kr[m0 + z], u[c], sreg[m0 + z][c]);
-                        oc[z & 1][c] = fmaf(qi[z], sreg[m0 + z][c], oc[z & 1][c]);
-                    }
+            for (int i = 0; i < DG; i++) {
+                rr[i] = (b2 ? r1[DG + i] : r1[i]) + __shfl_xor_sync(0xffffffffu, b2 ? r1[i] : r1[DG + i], 4);
+                rr[i] += __shfl_xor_sync(0xffffffffu, rr[i], 8);
             }
-            const float ov = reduce(oc);
-            if (kp < 4 && col + my_col < dv) o[(size_t)(tok0 + t0 + tt) * p.H * dv + (size_t)h * dv + col + my_col] = ov;
+            float cf[32];
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                const float4 c4 = *reinterpret_cast<const float4*>(s_coef + gr * 32 + i * 4);
+                cf[4 * i] = c4.x, cf[4 * i + 1] = c4.y, cf[4 * i + 2] = c4.z, cf[4 * i + 3] = c4.w;
+            }
+            // (threads of the queries' half go through the same motions with their own sums; their u is not used)
+            float u[DG];
+            const float* vrow = run + gr * DG * ROWLEN + 2 * NP + cg * 4 + my_col;
+            u[0] = cf[0] * vrow[0] - cf[4] * rr[0];
+            u[1] = cf[1] * vrow[ROWLEN] - cf[5] * rr[1] - cf[16] * u[0];
+            u[2] = cf[2] * vrow[2 * ROWLEN] - cf[6] * rr[2] - cf[17] * u[0] - cf[18] * u[1];
+            u[3] = cf[3] * vrow[3 * ROWLEN] - cf[7] * rr[3] - cf[19] * u[0] - cf[20] * u[1] - cf[21] * u[2];
+#pragma unroll
+            for (int i = 0; i < DG; i++) {
+                if (!b2 && !b3) s_u[i * DCOLS + cg * 4 + my_col] = cf[12 + i] * u[i];
+                const float other = __shfl_xor_sync(0xffffffffu, u[i], 4);
+                u[i] = b2 ? other : u[i];
+            }
+            __syncwarp();                             // a column group's sixteen threads lie in one warp
+            if (b2 && !b3 && col + my_col < dv) {
+                const float out[DG] = {cf[8] * rr[0] + cf[22] * u[0], cf[9] * rr[1] + cf[23] * u[0] + cf[24] * u[1],
+                                       cf[10] * rr[2] + cf[25] * u[0] + cf[26] * u[1] + cf[27] * u[2],
+                                       cf[11] * rr[3] + cf[28] * u[0] + cf[29] * u[1] + cf[30] * u[2] + cf[31] * u[3]};
+                const int t = t0 + gr * DG;
+#pragma unroll
+                for (int i = 0; i < DG; i++)
+                    if (t + i < cnt) o[(size_t)(tok0 + t + i) * p.H * dv + (size_t)h * dv + col + my_col] = out[i];
+            }
+            float uw[DG][4];
+#pragma unroll
+            for (int i = 0; i < DG; i++) {
+                const float4 u4 = *reinterpret_cast<const float4*>(s_u + i * DCOLS + cg * 4);
+                uw[i][0] = u4.x, uw[i][1] = u4.y, uw[i][2] = u4.z, uw[i][3] = u4.w;
+            }
+            __syncwarp();                             // read by all before the next group's are written
+#pragma unroll
+            for (int m = 0; m < RPT; m++)
+#pragma unroll
+                for (int c = 0; c < 4; c++) {
+                    float x = cf[11] * sreg[m][c];
+#pragma unroll
+                    for (int i = 0; i < DG; i++) x = fmaf(kr[i][m], uw[i][c], x);
+                    sreg[m][c] = x;
+                }
         }
     }
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
         const int n = kp * RPT + m;
         if (n >= d) continue;
-        if (vec && col < dv) {
+        if (vec_state && col < dv) {
             *reinterpret_cast<float4*>(S + (size_t)n * dv + col) = make_float4(sreg[m][0], sreg[m][1], sreg[m][2], sreg[m][3]);
         } else {
 #pragma unroll
-            for (int c = 0; c < DS_CPT; c++)
+            for (int c = 0; c < 4; c++)
                 if (col + c < dv) S[(size_t)n * dv + col + c] = sreg[m][c];
         }
     }
@@ -463,13 +578,25 @@ MOE_API int moe_delta_scan(const float* qkv, const float* step, float* state, lo
         state_pitch < (long long)H * d * dv || H > 65535 || num_seqs > 65535)
         return (int)cudaErrorInvalidValue;
     const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv};
-    const dim3 grid((dv + DS_COLS - 1) / DS_COLS, H, num_seqs);
-#define SCAN(RPT_, KP_, TOK_)                                                                                          \
-    return launch_pdl(delta_scan_kernel<RPT_, KP_, TOK_>, grid, dim3(KP_ * DS_CG),                                     \
-                      (size_t)(TOK_) * ((2 * RPT_ * KP_ + DS_COLS + 2 + 3) / 4 * 4) * sizeof(float), stream, p, o)
-    if (d <= 32) SCAN(4, 8, 16);
-    if (d <= 64) SCAN(8, 8, 16);
-    if (d <= 128) SCAN(16, 8, 16);
-    SCAN(16, 16, 16);
+    const dim3 grid((dv + DCOLS - 1) / DCOLS, H, num_seqs);
+    const bool vec = d % 4 == 0 && dv % 4 == 0 && aligned16(qkv);
+#define SCAN_V(RPT_, V_)                                                                                               \
+    do {                                                                                                               \
+        constexpr size_t smem = (size_t)(2 * DRUN * (2 * RPT_ * DKP + DCOLS) + 4 * DRUN + 4 * 32 + DG * DCOLS) * sizeof(float); \
+        if (smem > 48 * 1024) {                                                                                        \
+            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                       \
+        }                                                                                                              \
+        return launch_pdl(delta_scan_kernel<RPT_, V_>, grid, dim3(DTHREADS), smem, stream, p, o);                      \
+    } while (0)
+#define SCAN(RPT_)                                                                                                     \
+    do {                                                                                                               \
+        if (vec) SCAN_V(RPT_, true);                                                                                   \
+        SCAN_V(RPT_, false);                                                                                           \
+    } while (0)
+    if (d <= 64) SCAN(4);
+    if (d <= 128) SCAN(8);
+    SCAN(16);
 #undef SCAN
+#undef SCAN_V
 }

@@ -377,6 +377,53 @@ wkv_finish_kernel(const float* __restrict__ o, const float* __restrict__ gate, l
     }
 }
 
+// The same with the head in registers: LPH lanes a head, UNITS 16-byte units a lane (heads of a multiple of four
+// numbers, rows on 16-byte boundaries); output and gate are on their way before the sum is formed.
+template <typename OT, int LPH, int UNITS>
+__global__ void __launch_bounds__(256)
+wkv_finish_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ldg,
+                      const float* __restrict__ norm_w, float eps, const int* __restrict__ seq_of_token, int num_tokens,
+                      int heads, int d, OT* __restrict__ out) {
+    pdl_sync();
+    const int lane = threadIdx.x % LPH;
+    const long long item = (long long)blockIdx.x * (256 / LPH) + threadIdx.x / LPH;
+    const bool there = item < (long long)num_tokens * heads;
+    const int t = there ? (int)(item / heads) : 0, head = there ? (int)(item - (long long)t * heads) : 0;
+    const bool live = there && seq_of_token[t] >= 0;
+    const size_t base = (size_t)t * heads * d + (size_t)head * d;
+    float4 x[UNITS], g[UNITS];
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < UNITS; u++) {
+        const int e = (u * LPH + lane) * 4;
+        const bool on = live && e < d;
+        x[u] = on ? *reinterpret_cast<const float4*>(o + base + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        g[u] = on ? *reinterpret_cast<const float4*>(gate + (size_t)t * ldg + (size_t)head * d + e) : x[u];
+    }
+#pragma unroll
+    for (int u = 0; u < UNITS; u++)
+        ss = fmaf(x[u].x, x[u].x, fmaf(x[u].y, x[u].y, fmaf(x[u].z, x[u].z, fmaf(x[u].w, x[u].w, ss))));
+#pragma unroll
+    for (int off = LPH / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+    const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+#pragma unroll
+    for (int u = 0; u < UNITS; u++) {
+        const int e = (u * LPH + lane) * 4;
+        if (!there || e >= d) continue;
+        const float4 w = *reinterpret_cast<const float4*>(norm_w + (size_t)head * d + e);
+        const float y[4] = {x[u].x * inv * w.x * (g[u].x / (1.0f + expf(-g[u].x))), x[u].y * inv * w.y * (g[u].y / (1.0f + expf(-g[u].y))),
+                            x[u].z * inv * w.z * (g[u].z / (1.0f + expf(-g[u].z))), x[u].w * inv * w.w * (g[u].w / (1.0f + expf(-g[u].w)))};
+        if constexpr (sizeof(OT) == 4) {
+            *reinterpret_cast<float4*>(out + base + e) = make_float4(y[0], y[1], y[2], y[3]);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
+            uint2 v;
+            v.x = *reinterpret_cast<const unsigned*>(&lo), v.y = *reinterpret_cast<const unsigned*>(&hi);
+            *reinterpret_cast<uint2*>(out + base + e) = v;
+        }
+    }
+}
+
 }  // namespace
 
 // h: [T, width] 32-bit; mu: [streams, width]; state: per slot `width` floats at the start of a row of
@@ -460,6 +507,23 @@ MOE_API int moe_wkv_finish(const float* o, const float* gate, long long ldg, con
         return (int)cudaErrorInvalidValue;
     const long long items = (long long)num_tokens * heads;
     const unsigned blocks = (unsigned)((items + 7) / 8);
+    if (d % 4 == 0 && d <= 256 && ldg % 4 == 0 && ((uintptr_t)o | (uintptr_t)gate | (uintptr_t)norm_w) % 16 == 0 &&
+        (uintptr_t)out % (out_dt == DT_F32 ? 16 : 8) == 0) {
+#define FIN(OT_, LPH_, U_)                                                                                             \
+    return launch_pdl(wkv_finish_vec_kernel<OT_, LPH_, U_>, dim3((unsigned)((items + 256 / LPH_ - 1) / (256 / LPH_))), 256, 0, \
+                      stream, o, gate, ldg, norm_w, eps, seq_of_token, num_tokens, heads, d, (OT_*)out)
+#define FIN_D(OT_)                                                                                                     \
+    do {                                                                                                               \
+        if (d <= 32) FIN(OT_, 8, 1);                                                                                   \
+        if (d <= 64) FIN(OT_, 16, 1);                                                                                  \
+        if (d <= 128) FIN(OT_, 32, 1);                                                                                 \
+        FIN(OT_, 32, 2);                                                                                               \
+    } while (0)
+        if (out_dt == DT_F32) FIN_D(float);
+        FIN_D(__nv_bfloat16);
+#undef FIN_D
+#undef FIN
+    }
     if (out_dt == DT_F32)
         return launch_pdl(wkv_finish_kernel<float>, dim3(blocks), 256, 0, stream, o, gate, ldg, norm_w, eps,
                           seq_of_token, num_tokens, heads, d, (float*)out);

@@ -56,7 +56,7 @@ from .base import Part, TensorSpec, make_part, register_part
 
 def record_width(n: int, bf16: bool) -> int:
     """Width of a cached record of n numbers: in bfloat16 the tensor-core attention over records that are key
-    and value takes 64, 128, 192 and 256, everything takes multiples of 16."""
+    and value takes 64, 128, 192 and 256, everything takes multiples of 16 (beyond 256 the plain kernels run)."""
     if bf16 and n <= 256:
         return -(-n // 64) * 64
     return -(-n // 16) * 16
@@ -90,10 +90,10 @@ class LatentAttention(Part):
         self.position = make_part("position", PartSpec(pos.pop("kind"), pos, spec.prefix))
         if self.rot and getattr(self.position, "rotary_dim", 0) != self.rot:
             raise ValueError("latent attention: the position encoding must turn exactly the rotated part of a head")
-        if not (self.nh > 0 and self.hd > 0 and self.vd > 0 and self.rank > 0 and 0 < self.rank + self.rot <= 256):
+        if not (self.nh > 0 and self.hd > 0 and self.vd > 0 and self.rank > 0 and 0 < self.rank + self.rot <= 1024):
             raise ValueError(f"latent attention: {self.nh} heads of {self.hd} / {self.vd} on a latent of {self.rank}"
                              + (f" and a rotated part of {self.rot}" if self.rot else "")
-                             + "; the attention kernels take records of up to 256")
+                             + "; the attention kernels take records of up to 1024")
         if self.window is not None and self.window <= 0:
             raise ValueError("window must be positive")
         self.record = self.rank + self.rot        # numbers a position

@@ -100,6 +100,9 @@ CONFIGS = {
         layer(windowed(3, 48, 64, 40, 136, size=100), ff=96),
         layer(causal(8, 64, 32, 64, 224, 40, scaling=(2.0, 64, 8.0, 1.0)), ff=96),
         layer(delta(2, 2, 200, 72, 4), ff=64)]),
+    # records wider than any tiled or tensor-core kernel takes
+    "huge": dict(vocab=77, width=64, eps=1e-5, logit_scale=1.0, layers=[
+        layer(windowed(5, 24, 12, 16, 300, size=90), ff=64), layer(causal(2, 32, 64, 40, 500, 30), ff=None)]),
     # one layer that sees everything: the tests make one far key stand out in it
     "far": dict(vocab=70, width=32, eps=1e-5, logit_scale=1.0, layers=[
         layer(causal(2, 16, 8, 16, 24, 20, scale=1.0), ff=48)]),

@@ -83,8 +83,8 @@ def test_parts_refuse_what_the_kernels_do_not_take():
     from moe_b200.config.spec import PartSpec
     from moe_b200.parts.base import make_part
 
-    base = {"hidden_size": 32, "num_heads": 2, "head_dim": 8, "kv_rank": 240, "scale": 1.0, "eps": 1e-5}
-    with pytest.raises(ValueError, match="records of up to 256"):
+    base = {"hidden_size": 32, "num_heads": 2, "head_dim": 8, "kv_rank": 1010, "scale": 1.0, "eps": 1e-5}
+    with pytest.raises(ValueError, match="records of up to 1024"):
         make_part("mixer", PartSpec("latent_attention", dict(base, rot_dim=32, position={"kind": "rotary", "theta": 1e4, "rotary_dim": 32})))
     with pytest.raises(ValueError, match="exactly the rotated part"):
         make_part("mixer", PartSpec("latent_attention", dict(base, rot_dim=8, position={"kind": "rotary", "theta": 1e4, "rotary_dim": 4})))

@@ -21,7 +21,7 @@ pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 DEV = "cuda:0"
 DTYPES = ["float32", "bfloat16"]
-NAMES = ["mix", "lean", "ones", "sharp", "wide", "large", "memory"]
+NAMES = ["mix", "lean", "ones", "sharp", "wide", "large", "huge", "memory"]
 F = torch.float64
 
 
@@ -253,7 +253,8 @@ def test_one_gate_a_head_on_the_packed_heads(bf16, H, dv, D):
 @pytest.mark.parametrize("window", [None, 1, 9, 64, 70, 300])
 @pytest.mark.parametrize("dt,H,dv,D", [(torch.float32, 3, 40, 48), (torch.float32, 4, 33, 64), (torch.bfloat16, 6, 96, 128),
                                        (torch.bfloat16, 16, 96, 128), (torch.bfloat16, 9, 48, 64), (torch.bfloat16, 4, 130, 144),
-                                       (torch.bfloat16, 20, 192, 256), (torch.bfloat16, 3, 250, 256)])
+                                       (torch.bfloat16, 20, 192, 256), (torch.bfloat16, 3, 250, 256), (torch.bfloat16, 3, 300, 320),
+                                       (torch.float32, 2, 510, 512)])
 def test_single_tokens_over_shared_records_with_a_gate_a_head(dt, H, dv, D, window):
     """All heads on one record that is key and value; the merge keeps dv columns and multiplies by the head's
     gate.  A key that towers over all others stands at the window's last place, or one before it."""
@@ -530,7 +531,7 @@ def test_decoding_from_the_first_token_on_and_a_prompt_against_its_replay(root, 
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mix", "ones", "wide", "lean"])
+@pytest.mark.parametrize("name", ["mix", "ones", "wide", "lean", "huge"])
 @pytest.mark.parametrize("sizes", [[2], [3], [63, 2], [64], [65, 1, 1, 7], [129]])
 def test_portions_of_several_sizes(root, name, dtype, sizes):
     d, eng = engine_of(root, name, dtype)
