@@ -65,7 +65,6 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, const float* v) {
 }
 
 constexpr int LATENT_MAX_ROT = 512;
-constexpr int CQ_UNITS = 2;        // 16-byte units of the queries' latent a thread keeps in registers
 
 struct LatentArgs {
     const int* pos;
@@ -88,8 +87,9 @@ struct LatentArgs {
     int num_tokens, D;
 };
 
-// One block a token.
-template <typename OT>
+// One block a token.  CQ_UNITS: 16-byte units of the queries' latent a thread keeps in registers (0: there is none, so
+// that the other forms do not pay for its registers).
+template <typename OT, int CQ_UNITS>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__ q_rec, OT* __restrict__ k_new,
                       OT* __restrict__ cq, const LatentCommit c, int* status, int vec4, int cq_vec) {
@@ -97,13 +97,18 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
     __shared__ __align__(16) float ang[LATENT_MAX_ROT];        // cos[rot / 2], sin[rot / 2]
     const int t = blockIdx.x, rot = a.rot, half = rot / 2, D = a.D, r = a.r;
     pdl_sync();
-    if (rot > 0) {
-        const float p = (float)a.pos[t];
-        for (int i = threadIdx.x; i < half; i += blockDim.x) {
-            float sn, cs;
-            sincosf(p * a.freq[i], &sn, &cs);
-            ang[i] = cs * a.mscale, ang[half + i] = sn * a.mscale;
+    auto angles = [&]() {      // (read after the next barrier)
+        if (rot > 0) {
+            const float p = (float)a.pos[t];
+            for (int i = threadIdx.x; i < half; i += blockDim.x) {
+                float sn, cs;
+                sincosf(p * a.freq[i], &sn, &cs);
+                ang[i] = cs * a.mscale, ang[half + i] = sn * a.mscale;
+            }
         }
+    };
+    if (!k_new) {
+        angles();
         __syncthreads();
     }
     // element j of the rotated vector whose rotated part starts at v
@@ -118,18 +123,21 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
         // registers (four elements a unit) where it fits, and both sums share their barriers.
         const float* row = a.proj + (size_t)t * a.ld;
         const float* lat = row + a.lat_at;
-        float4 cu[CQ_UNITS];
+        const float lat0 = (int)threadIdx.x < r ? lat[threadIdx.x] : 0.f;
+        float4 cu[CQ_UNITS > 0 ? CQ_UNITS : 1];
         const bool cq_regs = cq_vec && a.q_rank <= 4 * CQ_UNITS * (int)blockDim.x;
         float ss = 0.f, sq = 0.f;
-        if (a.cq_w && cq_regs) {
+        if (CQ_UNITS > 0 && a.cq_w && cq_regs) {
 #pragma unroll
             for (int u = 0; u < CQ_UNITS; u++) {
                 const int i = (threadIdx.x + u * blockDim.x) * 4;
                 cu[u] = i < a.q_rank ? *reinterpret_cast<const float4*>(row + i) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
         }
-        for (int i = threadIdx.x; i < r; i += blockDim.x) ss += lat[i] * lat[i];
-        if (a.cq_w) {
+        angles();
+        ss = lat0 * lat0;
+        for (int i = threadIdx.x + blockDim.x; i < r; i += blockDim.x) ss += lat[i] * lat[i];
+        if (CQ_UNITS > 0 && a.cq_w) {
             if (cq_regs) {
 #pragma unroll
                 for (int u = 0; u < CQ_UNITS; u++)
@@ -164,7 +172,7 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
             if (cd) st_f(cd + i, x);
             if (cv) st_f(cv + i, x);
         }
-        if (a.cq_w) {
+        if (CQ_UNITS > 0 && a.cq_w) {
             const float qi = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps);
             OT* cr = cq + (size_t)t * a.q_rank;
             if (cq_regs) {
@@ -383,11 +391,16 @@ MOE_API int moe_latent_prepare(const float* proj, int ld, int lat_at, int r, con
     const int cq_vec = cq_w && q_rank % 4 == 0 && ld % 4 == 0 && ((uintptr_t)proj | (uintptr_t)cq_w) % 16 == 0 && (uintptr_t)cq % al == 0;
     // keys alone are little work a token: smaller blocks, more of them on an SM
     const int threads = q32 || num_tokens < 512 ? 256 : 128;
-    if (out_dt == DT_F32)
-        return launch_pdl(latent_prepare_kernel<float>, num_tokens, threads, 0, stream, a, (float*)q_t, (float*)q_rec,
-                          (float*)k_new, (float*)cq, c, status, vec4, cq_vec);
-    return launch_pdl(latent_prepare_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, a, (__nv_bfloat16*)q_t,
-                      (__nv_bfloat16*)q_rec, (__nv_bfloat16*)k_new, (__nv_bfloat16*)cq, c, status, vec4, cq_vec);
+#define PREP(OT_, U_)                                                                                                  \
+    return launch_pdl(latent_prepare_kernel<OT_, U_>, num_tokens, threads, 0, stream, a, (OT_*)q_t, (OT_*)q_rec,       \
+                      (OT_*)k_new, (OT_*)cq, c, status, vec4, cq_vec)
+    if (out_dt == DT_F32) {
+        if (cq_w) PREP(float, 4);
+        PREP(float, 0);
+    }
+    if (cq_w) PREP(__nv_bfloat16, 4);
+    PREP(__nv_bfloat16, 0);
+#undef PREP
 }
 
 // src: element (a, b, j) at a * s_outer + b * s_inner + j, j < n; dst: [B, A, wd] with rows of ldd elements (dense

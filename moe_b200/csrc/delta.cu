@@ -249,8 +249,9 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
 // one token at a time the products with S are eight independent sums instead of two with an update between
 // them, their sums over the threads are formed together, and the state is multiplied by a decay once.
 //
-// grid (ceil(dv / 32), heads, sequences), 128 threads: thread (kp = tid % 16, cg = tid / 16) holds rows kp * RPT ...
-// of four neighbouring columns of S in registers (rows beyond d stay zero).  A run of sixteen tokens is staged
+// grid (ceil(dv / 32), heads, sequences), 128 threads: thread (kp = tid % 16, cg = tid / 16) holds four neighbouring
+// columns of rows 4 kp ... 4 kp + 3 of every 64 rows of S in registers (rows beyond d stay zero; the sixteen
+// threads' reads of a token's k and q are then neighbours in shared memory).  A run of sixteen tokens is staged
 // in shared memory as [k | q | the block's columns of v] a token (cp.async, two buffers; rows beyond the
 // sequence's last token are zeros with beta 0 and decay 1: they change nothing); warp w forms the scalars of the
 // run's group w.  Within a run the groups follow one another without a block barrier.
@@ -267,7 +268,7 @@ __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes
 
 // VEC: rows of q, k and v start on 16-byte boundaries and hold whole 16-byte units.
 template <int RPT, bool VEC>
-__global__ void __launch_bounds__(DTHREADS)
+__global__ void __launch_bounds__(DTHREADS, RPT <= 8 ? 4 : 2)
 delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     constexpr int NP = RPT * DKP;
     constexpr int ROWLEN = 2 * NP + DCOLS;
@@ -288,7 +289,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     float sreg[RPT][4];
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
-        const int n = kp * RPT + m;
+        const int n = (m / 4) * 64 + kp * 4 + m % 4;
         if (vec_state && n < d && col < dv) {
             const float4 t4 = *reinterpret_cast<const float4*>(S + (size_t)n * dv + col);
             sreg[m][0] = t4.x, sreg[m][1] = t4.y, sreg[m][2] = t4.z, sreg[m][3] = t4.w;
@@ -304,13 +305,14 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
         float* dst = sm + buf * DRUN * ROWLEN;
         constexpr int W = VEC ? 4 : 1;
         const int kw = d / W, vw = ncols / W, per = 2 * kw + vw;
-        for (int i = tid; i < DRUN * per; i += DTHREADS) {
-            const int tt = i / per, e = i - tt * per;
+        for (int tt = warp; tt < DRUN; tt += DTHREADS / 32) {           // a warp a token
             const bool on = t0 + tt < cnt;
             const float* row = base + (size_t)min(t0 + tt, cnt - 1) * channels;
-            if (e < kw) cp_zfill(dst + tt * ROWLEN + e * W, row + k_at + e * W, 4 * W, on);
-            else if (e < 2 * kw) cp_zfill(dst + tt * ROWLEN + NP + (e - kw) * W, row + q_at + (e - kw) * W, 4 * W, on);
-            else cp_zfill(dst + tt * ROWLEN + 2 * NP + (e - 2 * kw) * W, row + v_at + (e - 2 * kw) * W, 4 * W, on);
+            float* to = dst + tt * ROWLEN;
+            for (int e = lane; e < per; e += 32) {
+                const int x = e < kw ? e : e < 2 * kw ? e - kw : e - 2 * kw;
+                cp_zfill(to + (e < kw ? 0 : e < 2 * kw ? NP : 2 * NP) + x * W, row + (e < kw ? k_at : e < 2 * kw ? q_at : v_at) + x * W, 4 * W, on);
+            }
         }
         if (tid < 2 * DRUN) {
             const int tt = tid % DRUN, which = tid / DRUN;
@@ -396,7 +398,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
         __syncthreads();
         const int groups = (min(DRUN, cnt - t0) + DG - 1) / DG;
         for (int gr = 0; gr < groups; gr++) {
-            const float* row = run + gr * DG * ROWLEN + kp * RPT;
+            const float* row = run + gr * DG * ROWLEN + kp * 4;
             float kr[DG][RPT];
             float hk[DG][4], hq[DG][4];
 #pragma unroll
@@ -407,8 +409,8 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             for (int m0 = 0; m0 < RPT; m0 += 4) {
 #pragma unroll
                 for (int i = 0; i < DG; i++) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + m0);
-                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0);
+                    const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + m0 * DKP);
+                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0 * DKP);
                     kr[i][m0] = k4.x, kr[i][m0 + 1] = k4.y, kr[i][m0 + 2] = k4.z, kr[i][m0 + 3] = k4.w;
                     const float qi[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
@@ -487,7 +489,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     }
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
-        const int n = kp * RPT + m;
+        const int n = (m / 4) * 64 + kp * 4 + m % 4;
         if (n >= d) continue;
         if (vec_state && col < dv) {
             *reinterpret_cast<float4*>(S + (size_t)n * dv + col) = make_float4(sreg[m][0], sreg[m][1], sreg[m][2], sreg[m][3]);
