@@ -258,6 +258,78 @@ latent_prepare_kernel(const LatentArgs a, OT* __restrict__ q_t, OT* __restrict__
     }
 }
 
+// Keys and the queries' latent of many tokens: a warp a token, no barrier between loads, sums and stores.  CU: 16-byte
+// units of the queries' latent a lane holds (q_rank <= 128 CU); latents of up to 256, rotated parts of up to 64.
+constexpr int LK_WARPS = 4;
+template <typename OT, int CU>
+__global__ void __launch_bounds__(LK_WARPS * 32)
+latent_keys_kernel(const LatentArgs a, OT* __restrict__ k_new, OT* __restrict__ cq, const LatentCommit c, int* status) {
+    const int lane = threadIdx.x & 31;
+    const int t = blockIdx.x * LK_WARPS + (threadIdx.x >> 5);
+    pdl_sync();
+    if (t >= a.num_tokens) return;                   // (the whole warp)
+    const int r = a.r, rot = a.rot, half = rot / 2, D = a.D;
+    const float* row = a.proj + (size_t)t * a.ld;
+    const float* lat = row + a.lat_at;
+    float4 cu[CU];
+    float lx[8];
+#pragma unroll
+    for (int u = 0; u < CU; u++) {
+        const int i = (u * 32 + lane) * 4;
+        cu[u] = i < a.q_rank ? *reinterpret_cast<const float4*>(row + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int u = 0; u < 8; u++) lx[u] = u * 32 + lane < r ? lat[u * 32 + lane] : 0.f;
+    // lane i < rot / 2 turns pair i
+    float lo = 0.f, hi = 0.f, sn = 0.f, cs = 1.f;
+    const int at_lo = a.interleaved ? 2 * lane : lane, at_hi = a.interleaved ? 2 * lane + 1 : lane + half;
+    if (lane < half) {
+        lo = lat[r + at_lo], hi = lat[r + at_hi];
+        sincosf((float)a.pos[t] * a.freq[lane], &sn, &cs);
+        sn *= a.mscale, cs *= a.mscale;
+    }
+    OT* cd = nullptr;
+    OT* cv = nullptr;
+    if (c.k_cache) {
+        const int s = a.seq_of_token[t], p = a.pos[t];
+        if (s >= 0 && !(c.ring > 0 && p < c.seq_end[s] - c.ring)) {
+            const CachePos cp = cache_pos(p, c.ring, c.tables + (size_t)c.slots[s] * c.table_stride, c.page_size, c.num_pages, status);
+            const size_t at = cache_index(cp, 0, 1, c.page_size, D);
+            cd = (OT*)c.k_cache + at;
+            if (c.v_cache && c.v_cache != c.k_cache) cv = (OT*)c.v_cache + at;
+        }
+    }
+    float ss = 0.f, sq = 0.f;
+#pragma unroll
+    for (int u = 0; u < 8; u++) ss = fmaf(lx[u], lx[u], ss);
+#pragma unroll
+    for (int u = 0; u < CU; u++)
+        sq = fmaf(cu[u].x, cu[u].x, fmaf(cu[u].y, cu[u].y, fmaf(cu[u].z, cu[u].z, fmaf(cu[u].w, cu[u].w, sq))));
+    ss = warp_sum(ss), sq = warp_sum(sq);
+    const float inv = 1.0f / sqrtf(ss / (float)r + a.eps), qi = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps);
+    OT* kd = k_new + (size_t)t * D;
+    auto put = [&](int i, float x) {
+        st_f(kd + i, x);
+        if (cd) st_f(cd + i, x);
+        if (cv) st_f(cv + i, x);
+    };
+#pragma unroll
+    for (int u = 0; u < 8; u++)
+        if (u * 32 + lane < r) put(u * 32 + lane, lx[u] * inv * a.w[u * 32 + lane]);
+    if (lane < half) put(r + at_lo, rot_lo(lo, hi, cs, sn)), put(r + at_hi, rot_hi(lo, hi, cs, sn));
+    for (int i = r + rot + lane; i < D; i += 32) put(i, 0.f);
+    OT* cr = cq + (size_t)t * a.q_rank;
+#pragma unroll
+    for (int u = 0; u < CU; u++) {
+        const int i = (u * 32 + lane) * 4;
+        if (i < a.q_rank) {
+            const float4 w = *reinterpret_cast<const float4*>(a.cq_w + i);
+            const float v[4] = {cu[u].x * qi * w.x, cu[u].y * qi * w.y, cu[u].z * qi * w.z, cu[u].w * qi * w.w};
+            st4(cr + i, v);
+        }
+    }
+}
+
 __device__ __forceinline__ void ld2(const float* p, float* v) {
     const float2 x = *reinterpret_cast<const float2*>(p);
     v[0] = x.x, v[1] = x.y;
@@ -389,6 +461,18 @@ MOE_API int moe_latent_prepare(const float* proj, int ld, int lat_at, int r, con
                      (!q_major || D % 4 == 0) && (uintptr_t)q_t % (out_dt == DT_F32 ? 16 : 8) == 0;
     const int al = out_dt == DT_F32 ? 16 : 8;
     const int cq_vec = cq_w && q_rank % 4 == 0 && ld % 4 == 0 && ((uintptr_t)proj | (uintptr_t)cq_w) % 16 == 0 && (uintptr_t)cq % al == 0;
+    if (cq_vec && !q32 && num_tokens >= 512 && q_rank <= 2048 && r <= 256 && rot <= 64) {
+#define KEYS(OT_, CU_)                                                                                                 \
+    return launch_pdl(latent_keys_kernel<OT_, CU_>, (num_tokens + LK_WARPS - 1) / LK_WARPS, LK_WARPS * 32, 0, stream, a, \
+                      (OT_*)k_new, (OT_*)cq, c, status)
+        if (out_dt == DT_F32) {
+            if (q_rank <= 1024) KEYS(float, 8);
+            KEYS(float, 16);
+        }
+        if (q_rank <= 1024) KEYS(__nv_bfloat16, 8);
+        KEYS(__nv_bfloat16, 16);
+#undef KEYS
+    }
     // keys alone are little work a token: smaller blocks, more of them on an SM
     const int threads = q32 || num_tokens < 512 ? 256 : 128;
 #define PREP(OT_, U_)                                                                                                  \

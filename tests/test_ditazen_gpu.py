@@ -175,18 +175,18 @@ def test_exact_gelu_alone_and_in_the_tensor_core_product(M, N, K):
 @pytest.mark.parametrize("neighbours", [False, True])
 @pytest.mark.parametrize("H,d,rot,r,D", [(3, 24, 8, 40, 48), (1, 8, 2, 5, 16), (5, 64, 64, 64, 128), (2, 10, 6, 20, 32), (4, 32, 16, 112, 128),
                                          (16, 96, 32, 96, 128)])
-def test_latent_records_and_queries_are_normed_rotated_and_laid_out(bf16, neighbours, H, d, rot, r, D):
-    """Both layouts of the queries, both pairings of the rotation, positions into the thousands, a factor on
+@pytest.mark.parametrize("starts,counts,qr", [([0, 3990], [9, 4], 20), ([0, 3400], [9, 600], 52), ([3, 64], [1, 520], 1100)])
+def test_latent_records_and_queries_are_normed_rotated_and_laid_out(bf16, neighbours, H, d, rot, r, D, starts, counts, qr):
+    """Few and many tokens, both layouts of the queries, both pairings of the rotation, positions into the thousands, a factor on
     cos and sin, the queries' own latent, and the append to the paged cache."""
     from moe_b200.cache import KVCache, KVRequest
     from moe_b200.ops import core
 
     g = torch.Generator().manual_seed(H * 100 + r)
-    eps, qr = 1e-5, 20
+    eps = 1e-5
     dt = torch.bfloat16 if bf16 else torch.float32
     scaling = {"factor": 4.0, "original": 512, "fast": 16.0, "slow": 1.0}
     freq, mscale = plain.frequencies({"dims": rot, "base": 5000.0, "scaling": scaling})
-    starts, counts = [0, 3990], [9, 4]
     T = sum(counts)
     pos = torch.cat([torch.arange(a, a + n) for a, n in zip(starts, counts)])
     proj = 3 * torch.randn(T, qr + r + rot + 3, generator=g)
@@ -212,10 +212,8 @@ def test_latent_records_and_queries_are_normed_rotated_and_laid_out(bf16, neighb
     assert D == r + rot or float(k_new[:, 0, r + rot:].abs().max()) == 0.0
     close(cq, plain.unit_rms(proj[:, :qr].double(), eps) * cw.double(), tol)
     table = cache.groups[0].table.cpu()
-    for t in range(T):
-        s = slots[0] if t < counts[0] else slots[1]
-        page, off = int(table[s, int(pos[t]) // 64]), int(pos[t]) % 64
-        assert torch.equal(cache.view(0).k[page, 0, off].cpu(), k_new[t, 0].cpu())
+    slot = torch.tensor([slots[0]] * counts[0] + [slots[1]] * counts[1])
+    assert torch.equal(cache.view(0).k.cpu()[table[slot, pos // 64].long(), 0, pos % 64], k_new[:, 0].cpu())
     # queries: records token by token from rows of r + rot, and head by head with the rotated part in the records
     q = torch.full((T, H, D), 7.0, dtype=dt, device=DEV)
     core.latent_prepare(None, batch, q32=dev(rec32), nh=H, d=r, r=r, width=D, q_t=q, token_major=True, status=st, **turn)
