@@ -186,7 +186,7 @@ conv_heads_prepare_kernel(const float* __restrict__ proj, int ld, const float* _
     }
 }
 
-// One block per sequence of the step.
+// grid (sequence of the step, run of channels): channels have nothing to do with one another.
 __global__ void __launch_bounds__(256)
 conv_state_update_kernel(const float* __restrict__ proj, int ld, float* __restrict__ state, long long state_pitch,
                          int taps, int channels, const int* __restrict__ cu_seqlens, const int* __restrict__ slots) {
@@ -195,7 +195,7 @@ conv_state_update_kernel(const float* __restrict__ proj, int ld, float* __restri
     const int tok0 = cu_seqlens[s], cnt = cu_seqlens[s + 1] - tok0;
     if (cnt <= 0) return;                                      // a sequence of a padded step that brings nothing
     float* st = state + (size_t)slots[s] * state_pitch;
-    for (int ch = threadIdx.x; ch < channels; ch += blockDim.x)
+    for (int ch = blockIdx.y * blockDim.x + threadIdx.x; ch < channels; ch += gridDim.y * blockDim.x)
         for (int i = 0; i < taps - 1; i++) {                   // ascending: an entry is read before it is written
             const int r = cnt - (taps - 1) + i;
             st[(size_t)i * channels + ch] = r >= 0 ? proj[(size_t)(tok0 + r) * ld + ch]
@@ -255,6 +255,7 @@ MOE_API int moe_conv_state_update(const float* proj, int ld, float* state, long 
     if (num_seqs <= 0 || taps <= 1) return 0;
     if (!proj || !state || ld < channels || state_pitch < (long long)(taps - 1) * channels || taps > MAX_TAPS)
         return (int)cudaErrorInvalidValue;
-    return launch_pdl(conv_state_update_kernel, dim3(num_seqs), 256, 0, stream, proj, ld, state, state_pitch, taps,
+    const int runs = (channels + 255) / 256;
+    return launch_pdl(conv_state_update_kernel, dim3(num_seqs, runs < 65535 ? runs : 65535), 256, 0, stream, proj, ld, state, state_pitch, taps,
                       channels, cu_seqlens, slots);
 }
