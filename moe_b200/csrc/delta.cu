@@ -582,6 +582,8 @@ MOE_API int moe_delta_scan(const float* qkv, const float* step, float* state, lo
     const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv};
     const dim3 grid((dv + DCOLS - 1) / DCOLS, H, num_seqs);
     const bool vec = d % 4 == 0 && dv % 4 == 0 && aligned16(qkv);
+    // An ordinary launch: blocks that are placed while the kernel before still occupies some SMs end up several to
+    // an SM beside empty ones, and a scan is as slow as its most crowded SM.
 #define SCAN_V(RPT_, V_)                                                                                               \
     do {                                                                                                               \
         constexpr size_t smem = (size_t)(2 * DRUN * (2 * RPT_ * DKP + DCOLS) + 4 * DRUN + 4 * 32 + DG * DCOLS) * sizeof(float); \
@@ -589,7 +591,8 @@ MOE_API int moe_delta_scan(const float* qkv, const float* step, float* state, lo
             cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                       \
         }                                                                                                              \
-        return launch_pdl(delta_scan_kernel<RPT_, V_>, grid, dim3(DTHREADS), smem, stream, p, o);                      \
+        delta_scan_kernel<RPT_, V_><<<grid, DTHREADS, smem, stream>>>(p, o);                                           \
+        return launch_status();                                                                                        \
     } while (0)
 #define SCAN(RPT_)                                                                                                     \
     do {                                                                                                               \
