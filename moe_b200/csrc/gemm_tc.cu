@@ -14,7 +14,8 @@
 //   warps 2-5   epilogue: tensor memory -> registers -> global memory
 //
 // Modes
-//   PLAIN    out[t, n] = f(acc (+ bias[n])); out is float32 or bfloat16; f is the identity, or plain_act (ACT_RELU2, ACT_GELU)
+//   PLAIN    out[t, n] = acc (+ bias[n]); out is float32 or bfloat16
+//   ACT      the same passed through plain_act (ACT_RELU2, ACT_GELU)
 //   SWIGLU   W holds gate rows [0, I) and up rows [I, 2I) per group; two accumulators;
 //            out[t, j] = silu(gate) * up  (reference: src/model.rs:26-35)
 // Groups (routed experts): rows of X are partitioned by group_offsets[G + 1]; group g
@@ -45,7 +46,14 @@ constexpr int MAX_SPLITS = 16;
 
 // MODE_SWIGLU_IL (persistent form only): gate and up rows of the same 16 features alternate within a
 // 128-row weight tile (see gemm_tc_persistent_kernel), so that SwiGLU needs ONE accumulator.
-enum { MODE_PLAIN = 0, MODE_SWIGLU = 1, MODE_SWIGLU_IL = 2 };
+// MODE_ACT is MODE_PLAIN whose output passes plain_act: a mode of its own, so that the products without one carry
+// nothing of it (the exact GELU in every epilogue cost decode steps of other models 1 - 2 %).
+enum { MODE_PLAIN = 0, MODE_SWIGLU = 1, MODE_SWIGLU_IL = 2, MODE_ACT = 3 };
+__host__ __device__ constexpr bool plain_mode(int mode) { return mode == MODE_PLAIN || mode == MODE_ACT; }
+template <int MODE>
+__device__ __forceinline__ float plain_out(const int act, float v) {
+    return MODE == MODE_ACT ? plain_act(act, v) : v;
+}
 
 struct Params {
     void* out;
@@ -251,7 +259,7 @@ struct Cfg {
     static constexpr int STAGE_BYTES = NW * W_BYTES + X_BYTES;
     // few tokens: the weight stream bounds the time, and two CTAs per SM (each with fewer stages)
     // hide one CTA's set-up and epilogue behind the other's loads
-    static constexpr int BUDGET = BN <= 64 ? (MODE == MODE_PLAIN ? 100 : 110) * 1024 : 196 * 1024;
+    static constexpr int BUDGET = BN <= 64 ? (plain_mode(MODE) ? 100 : 110) * 1024 : 196 * 1024;
     static constexpr int STAGES_RAW = BUDGET / STAGE_BYTES;
     static constexpr int STAGES = STAGES_RAW > 8 ? 8 : (STAGES_RAW < 2 ? 2 : STAGES_RAW);
     static constexpr int TMEM_COLS_RAW = NW * BN;
@@ -444,7 +452,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             tc_fence_after();
             const uint32_t taddr = tmem + ((uint32_t)(q * 32) << 16);
             const int cols = MODE == MODE_SWIGLU ? 2 * p.N : p.N;
-            const float bias = (MODE == MODE_PLAIN && p.bias && n_ok) ? p.bias[n] : 0.f;
+            const float bias = (plain_mode(MODE) && p.bias && n_ok) ? p.bias[n] : 0.f;
             const int rows_here = min(BN, row_end - row0);
             if (p.cluster) {
                 // the K splits of a tile are the CTAs of one cluster: each leaves its partial tile in
@@ -474,7 +482,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                     for (int j = 0; j < 16; j++) {
                         const int t = row0 + c0 + j;
                         if (n_ok && t < row_end) {
-                            const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], b[j]) : plain_act(p.act, a[j] + bias);
+                            const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], b[j]) : plain_out<MODE>(p.act, a[j] + bias);
                             if (p.out_bf16)
                                 ((__nv_bfloat16*)p.out)[(size_t)t * p.ldo + n] = __float2bfloat16_rn(v);
                             else
@@ -541,7 +549,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                                     sa += va[r][s];
                                     if (MODE == MODE_SWIGLU) sb += vb[r][s];
                                 }
-                                const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, sa, sb) : plain_act(p.act, sa + bias);
+                                const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, sa, sb) : plain_out<MODE>(p.act, sa + bias);
                                 if (p.out_bf16)
                                     ((__nv_bfloat16*)p.out)[(size_t)t * p.ldo + n] = __float2bfloat16_rn(v);
                                 else
@@ -565,7 +573,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
             const uint32_t S = (uint32_t)p.splits, rank = cluster_ctarank();
             const int f = (warp & 3) * 32 + lane, n = n0 + f;
             const int rows_here = min(BN, row_end - row0);
-            const float bias = (MODE == MODE_PLAIN && p.bias && n < p.N) ? p.bias[n] : 0.f;
+            const float bias = (plain_mode(MODE) && p.bias && n < p.N) ? p.bias[n] : 0.f;
             uint32_t peer[8];
 #pragma unroll
             for (uint32_t s = 0; s < 8; s++) peer[s] = mapa_cluster(base, s < S ? s : 0);
@@ -592,7 +600,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
                         sa += va[r][s];
                         if (MODE == MODE_SWIGLU) sb += vb[r][s];
                     }
-                    const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, sa, sb) : plain_act(p.act, sa + bias);
+                    const float v = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, sa, sb) : plain_out<MODE>(p.act, sa + bias);
                     if (p.out_bf16)
                         ((__nv_bfloat16*)p.out)[(size_t)(row0 + t) * p.ldo + n] = __float2bfloat16_rn(v);
                     else
@@ -620,7 +628,7 @@ template <int BN, int MODE>
 __device__ __forceinline__ void epilogue_part(const Params& p, uint32_t taddr, int n, int row0, int row_end, int c_lo,
                                               int c_hi) {
     const bool n_ok = n < p.N;
-    const float bias = (MODE == MODE_PLAIN && p.bias && n_ok) ? p.bias[n] : 0.f;
+    const float bias = (plain_mode(MODE) && p.bias && n_ok) ? p.bias[n] : 0.f;
     for (int c0 = c_lo; c0 < c_hi; c0 += 32) {
         float a[32], bb[32];
         __syncwarp();
@@ -631,13 +639,13 @@ __device__ __forceinline__ void epilogue_part(const Params& p, uint32_t taddr, i
 #pragma unroll
             for (int j = 0; j < 32; j++)
                 if (n_ok && row0 + c0 + j < row_end)
-                    o[(size_t)j * p.ldo] = __float2bfloat16_rn(MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], bb[j]) : plain_act(p.act, a[j] + bias));
+                    o[(size_t)j * p.ldo] = __float2bfloat16_rn(MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], bb[j]) : plain_out<MODE>(p.act, a[j] + bias));
         } else {
             float* o = (float*)p.out + (size_t)(row0 + c0) * p.ldo + n;
 #pragma unroll
             for (int j = 0; j < 32; j++)
                 if (n_ok && row0 + c0 + j < row_end)
-                    o[(size_t)j * p.ldo] = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], bb[j]) : plain_act(p.act, a[j] + bias);
+                    o[(size_t)j * p.ldo] = MODE == MODE_SWIGLU ? glu_mul(p.act, p.act_param, a[j], bb[j]) : plain_out<MODE>(p.act, a[j] + bias);
         }
     }
 }
@@ -1241,6 +1249,7 @@ MOE_API int moe_gemm_tc(const void* X, int ldx, const void* W, int num_groups, i
             const long long pair_items = (long long)mt * ((N + 2 * TILE_W - 1) / (2 * TILE_W));
             const int pcap = pair_items > (1 << 30) ? (1 << 30) : (int)pair_items;
             if (mode == MODE_SWIGLU) return launch_pair<128, MODE_SWIGLU>(tmW, tmX, p, pcap, stream);
+            if (act) return pbn == 128 ? launch_pair<128, MODE_ACT>(tmW, tmX, p, pcap, stream) : launch_pair<256, MODE_ACT>(tmW, tmX, p, pcap, stream);
             if (pbn == 128) return launch_pair<128, MODE_PLAIN>(tmW, tmX, p, pcap, stream);
             return launch_pair<256, MODE_PLAIN>(tmW, tmX, p, pcap, stream);
         }
@@ -1261,6 +1270,7 @@ MOE_API int moe_gemm_tc(const void* X, int ldx, const void* W, int num_groups, i
             }
         }
         if (mode == MODE_SWIGLU) return launch_persistent<128, MODE_SWIGLU>(tmW, tmX, p, cap, stream);
+        if (act) return pbn == 128 ? launch_persistent<128, MODE_ACT>(tmW, tmX, p, cap, stream) : launch_persistent<256, MODE_ACT>(tmW, tmX, p, cap, stream);
         if (pbn == 128) return launch_persistent<128, MODE_PLAIN>(tmW, tmX, p, cap, stream);
         return launch_persistent<256, MODE_PLAIN>(tmW, tmX, p, cap, stream);
     }
@@ -1270,6 +1280,7 @@ MOE_API int moe_gemm_tc(const void* X, int ldx, const void* W, int num_groups, i
 #define GO(BN_)                                                                              \
     if (bn == BN_)                                                                           \
         return mode == MODE_SWIGLU ? launch<BN_, MODE_SWIGLU>(tmW, tmX, p, grid, stream)     \
+               : act               ? launch<BN_, MODE_ACT>(tmW, tmX, p, grid, stream)        \
                                    : launch<BN_, MODE_PLAIN>(tmW, tmX, p, grid, stream);
     GO(16) GO(32) GO(64) GO(128) GO(256)
 #undef GO
