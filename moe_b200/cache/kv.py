@@ -3,7 +3,9 @@
 Layers whose mixers ask for the same record (kv heads, head size, window) form a
 *group* with storage and a page table of its own.  A group without a window
 keeps every position; a windowed group is a ring of ``ceil(window / 64)`` pages
-per sequence, position p living at ``p mod ring``.
+per sequence, position p living at ``p mod ring``.  Where a window keeps a sequence's first
+positions in sight (``KVRequest.keep``), the whole pages that cover them lie in front of the ring and are
+never written over: positions below ``pinned`` live where they are, p beyond at ``pinned + (p - pinned) mod ring``.
 
 One layer of a group is laid out ``[page][kv_head][64][head_dim]`` for keys and
 the same for values, so that the 64 positions of a page are contiguous per head.
@@ -32,6 +34,17 @@ class KVRequest:
     # the values are the keys (attention over one latent record per position): one plane is stored,
     # and a layer's view hands it out as both
     values_are_keys: bool = False
+    # with a window: the first ``keep`` positions of a sequence stay in sight of every later one
+    keep: int = 0
+
+    @property
+    def pinned_pages(self) -> int:
+        return -(-self.keep // PAGE_TOKENS) if self.window is not None else 0
+
+    @property
+    def ring_pages(self) -> int:
+        """Most pages a sequence holds (0: it grows without bound): the pinned ones and the window's ring."""
+        return 0 if self.window is None else self.pinned_pages + -(-self.window // PAGE_TOKENS)
 
 
 @dataclass(frozen=True)
@@ -49,8 +62,9 @@ class CacheGroup:
         self.num_kv_heads, self.head_dim, self.window = req.num_kv_heads, req.head_dim, req.window
         self.cache_ids = list(cache_ids)
         self.page_size = PAGE_TOKENS
-        self.ring_pages = 0 if req.window is None else -(-req.window // PAGE_TOKENS)
-        self.ring = self.ring_pages * PAGE_TOKENS
+        self.ring_pages = req.ring_pages                  # pinned ones included
+        self.pinned = req.pinned_pages * PAGE_TOKENS
+        self.ring = self.ring_pages * PAGE_TOKENS - self.pinned
         self.num_pages = num_pages
         self.dtype = dtype
         self.max_pages_per_seq = max_pages_per_seq
@@ -99,7 +113,7 @@ class KVCache:
         self.groups: List[CacheGroup] = []
         self._views: Dict[int, CacheView] = {}
         for gi, (req, cids) in enumerate(by_key.items()):
-            ring_pages = 0 if req.window is None else -(-req.window // PAGE_TOKENS)
+            ring_pages = req.ring_pages
             if ring_pages:
                 per_seq = min(ring_pages, budget_pages)
                 pages = min(budget_pages, max_slots * ring_pages) + 1
@@ -151,4 +165,5 @@ class KVCache:
         refuses a rewind (a mixer that wants it has to keep snapshots of its own)."""
         if self._states and new_length < self.length(slot):
             raise CacheError("this model keeps per-sequence state of fixed size, which cannot be rewound")
-        self.ledger.truncate(slot, new_length, [g.window or 0 for g in self.groups])
+        # (a ring behind pinned pages holds that many positions fewer than the ledger's count of its pages says)
+        self.ledger.truncate(slot, new_length, [g.window + g.pinned if g.window else 0 for g in self.groups])

@@ -15,3 +15,4 @@ from .fogapel import FogapelConfig  # noqa: F401  (registers the architecture)
 from .zosipel import ZosipelConfig  # noqa: F401  (registers the architecture)
 from .divadra import DivadraConfig  # noqa: F401  (registers the architecture)
 from .ditazen import DitazenConfig  # noqa: F401  (registers the architecture)
+from .kulanex import KulanexConfig  # noqa: F401  (registers the architecture)

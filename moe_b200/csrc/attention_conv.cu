@@ -26,7 +26,7 @@ struct ConvCommit {
     void* v_cache;
     const int* seq_end;
     const int* tables;
-    int table_stride, ring, page_size, num_pages;
+    int table_stride, ring, page_size, num_pages, pinned;
 };
 
 constexpr int CONV_WARPS = 8;
@@ -78,8 +78,8 @@ conv_heads_prepare_kernel(const float* __restrict__ proj, int ld, const float* _
     bool append = false;
     CachePos cp;
     cp.page = 0, cp.off = 0;
-    if (c.k_cache && s >= 0 && !(c.ring > 0 && p_int < c.seq_end[s] - c.ring)) {
-        cp = cache_pos(p_int, c.ring, c.tables + (size_t)slots[s] * c.table_stride, c.page_size, c.num_pages, status);
+    if (c.k_cache && s >= 0 && cache_holds(p_int, c.seq_end[s], c.ring, c.pinned)) {
+        cp = cache_pos(p_int, c.ring, c.tables + (size_t)slots[s] * c.table_stride, c.page_size, c.num_pages, status, c.pinned);
         append = true;
     }
     const int hs_count = nh + 2 * nkv;
@@ -215,7 +215,7 @@ MOE_API int moe_conv_heads_prepare(const float* proj, int ld, const float* taps_
                                    int rot, int num_tokens, int nh, int nkv, int d, int dv, int D, void* q, void* k,
                                    void* v, long long ldq, long long ldkv, int out_dt, void* k_cache, void* v_cache,
                                    const int* seq_end, const int* tables, int table_stride, int ring, int page_size,
-                                   int num_pages, int* status, cudaStream_t stream) {
+                                   int num_pages, int pinned, int* status, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     const int channels = (nh + nkv) * d + nkv * dv;
     if (rot < 0 || rot > d || (rot & 1) || (rot > 0 && !freq) || d <= 0 || dv <= 0 || D < d || D < dv || !q || !k || !v ||
@@ -225,7 +225,7 @@ MOE_API int moe_conv_heads_prepare(const float* proj, int ld, const float* taps_
     if (taps_w && (taps < 1 || taps > MAX_TAPS || (taps > 1 && (!state || state_pitch < (long long)(taps - 1) * channels))))
         return (int)cudaErrorInvalidValue;
     if (k_cache && (!v_cache || !seq_end || !tables)) return (int)cudaErrorInvalidValue;
-    const ConvCommit c{k_cache, v_cache, seq_end, tables, table_stride, ring, page_size, num_pages};
+    const ConvCommit c{k_cache, v_cache, seq_end, tables, table_stride, ring, page_size, num_pages, pinned};
     const int dmax = d > dv ? d : dv;
     const size_t smem = ((size_t)rot + (size_t)CONV_WARPS * dmax) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;

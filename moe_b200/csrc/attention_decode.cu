@@ -183,9 +183,12 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     const int width = (nh + 2 * nkv) * HD;
     const bool owner = FUSED && split == nsplit - 1 && warp == 0;   // takes the new key (and, for h0 == 0, appends it)
     // tiles of 32 positions, aligned to 32: the keys of a tile are contiguous in one page
-    const int tile_lo = lo / 32, tile_hi = p / 32 + 1;
-    const int tps = (tile_hi - tile_lo + nsplit - 1) / nsplit;
-    const int tb = tile_lo + split * tps, te = min(tile_hi, tb + tps);
+    // (kept first positions: their tiles come first, then those of the window; attn_seen turns a tile's number
+    // in that order into its place)
+    const int tile_lo = lo / 32, kept_tiles = min((av.keep + 31) / 32, tile_lo), pinned = attn_pinned(av);
+    const int n_tiles = kept_tiles + p / 32 + 1 - tile_lo;
+    const int tps = (n_tiles + nsplit - 1) / nsplit;
+    const int tb = split * tps, te = min(n_tiles, tb + tps);
     const int* table = tables + (size_t)(s < 0 ? 0 : slots[s]) * table_stride;
     if (s >= 0 && h0 == 0) {
         constexpr int LINES = 32 * HD * (int)sizeof(T) / 128;     // 128-byte lines of a tile of keys
@@ -198,7 +201,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
         const int ahead = (int)max(1ll, min((long long)(te - tb), share));
         for (int i = threadIdx.x; i < ahead * 2 * LINES; i += blockDim.x) {
             const int tile = tb + i / (2 * LINES), r = i % (2 * LINES);
-            const CachePos cp = cache_pos(tile * 32, ring, table, page_size, num_pages, nullptr);
+            const CachePos cp = cache_pos(attn_seen(tile, kept_tiles, tile_lo) * 32, ring, table, page_size, num_pages, nullptr, pinned);
             const size_t at = cache_index(cp, kvh, nkv, page_size, HD) + (size_t)(r % LINES) * (128 / sizeof(T));
             prefetch_l2((r < LINES ? k_cache : v_cache) + at);
         }
@@ -237,8 +240,8 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             for (int e = 0; e < EPC; e++) acc[g][e] = 0.f;
         }
         for (int tile = tb + warp; tile < te; tile += WARPS) {
-            const int j0 = tile * 32;
-            const CachePos cp = cache_pos(j0, ring, table, page_size, num_pages, status);
+            const int j0 = attn_seen(tile, kept_tiles, tile_lo) * 32;
+            const CachePos cp = cache_pos(j0, ring, table, page_size, num_pages, status, pinned);
             const size_t base = cache_index(cp, kvh, nkv, page_size, HD);
             const T* kt = k_cache + base + (size_t)rgrp * HD + sub * EPC;
             const T* vt = v_cache + base + (size_t)rgrp * HD + sub * EPC;
@@ -248,7 +251,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             for (int i = 0; i < NI; i++) raw[i] = *reinterpret_cast<const uint4*>(kt + (size_t)i * RPI * HD);
             const int my_row = sub * RPI + rgrp;          // the row whose score this lane ends up with
             const int my_j = j0 + my_row;
-            const bool valid = my_j >= lo && my_j <= hi;
+            const bool valid = (my_j >= lo || my_j < av.keep) && my_j <= hi;
             float sc[GH];
 #pragma unroll
             for (int g = 0; g < GH; g++) {
@@ -295,10 +298,10 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                 for (int e = 0; e < EPC; e++) acc[g][e] *= alpha;
 #pragma unroll
                 for (int i = 0; i < NI; i++) {
-                    // rows outside [lo, p] may hold anything: they are skipped, not multiplied by zero
+                    // rows out of sight may hold anything: they are skipped, not multiplied by zero
                     const int j = j0 + i * RPI + rgrp;
                     const float pi = __shfl_sync(0xffffffffu, pr, lane - sub + i);   // holder of row (i, rgrp)
-                    if (j >= lo && j <= hi) {
+                    if ((j >= lo || j < av.keep) && j <= hi) {
                         float vc[EPC];
                         Chunk<T>::unpack(raw[i], vc);
 #pragma unroll
@@ -315,7 +318,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             rotated_chunk<T, EPC>(row + (size_t)(nh + kvh) * HD, sub * EPC, half, fa.rot, ang, kn);
             rotated_chunk<T, EPC>(row + (size_t)(nh + nkv + kvh) * HD, sub * EPC, 0, 0, ang, vn);
             if (rgrp == 0 && h0 == 0) {
-                const CachePos cp = cache_pos(p, ring, table, page_size, num_pages, status);
+                const CachePos cp = cache_pos(p, ring, table, page_size, num_pages, status, pinned);
                 const size_t at = cache_index(cp, kvh, nkv, page_size, HD) + sub * EPC;
                 store_chunk((T*)fa.k_append + at, kn);
                 store_chunk((T*)fa.v_append + at, vn);
@@ -431,11 +434,12 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     if (s < 0) return;
     const int p = pos[t];
     const int lo = attn_lo(p, window, av.chunk);
-    const int n_keys = p + 1 - lo;
+    const int kept = attn_kept(av, lo), pinned = attn_pinned(av);
+    const int n_keys = kept + p + 1 - lo;                 // numbered kept ones first (attn_seen)
     int per = (n_keys + nsplit - 1) / nsplit;
     per = (per + 31) & ~31;
-    const int k_begin = lo + split * per;
-    const int k_end = min(p + 1, k_begin + per);
+    const int k_begin = split * per;
+    const int k_end = min(n_keys, k_begin + per);
     const int* table = tables + (size_t)slots[s] * table_stride;
     constexpr int EPC = Chunk<T>::N;
 
@@ -457,14 +461,14 @@ attn_decode_rows_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             for (int i = 0; i < MD / 32; i++) acc[g][i] = 0.f;
         }
         for (int j0 = k_begin + warp * 32; j0 < k_end; j0 += WARPS * 32) {
-            const int j = j0 + lane;
-            const bool valid = j < k_end;
+            const int j = attn_seen(j0 + lane, kept, lo);
+            const bool valid = j0 + lane < k_end;
             const T* vp = nullptr;
             float sc[GHS];
 #pragma unroll
             for (int g = 0; g < GHS; g++) sc[g] = 0.f;
             if (valid) {
-                const CachePos cp = cache_pos(j, ring, table, page_size, num_pages, status);
+                const CachePos cp = cache_pos(j, ring, table, page_size, num_pages, status, pinned);
                 const size_t r = cache_index(cp, kvh, nkv, page_size, hd);
                 const T* kp = k_cache + r;
                 vp = v_cache + r;
@@ -650,9 +654,10 @@ attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
     if (s < 0) return;                                   // a row of no sequence: the merge writes zeros
     const int p = pos[t];
     const int lo = attn_lo(p, window, av.chunk);
-    const int tile_lo = lo / GT_KEYS, tile_hi = p / GT_KEYS + 1;
-    const int tps = (tile_hi - tile_lo + nsplit - 1) / nsplit;
-    const int tb = tile_lo + split * tps, te = min(tile_hi, tb + tps);
+    const int tile_lo = lo / GT_KEYS, kept_tiles = min((av.keep + GT_KEYS - 1) / GT_KEYS, tile_lo), pinned = attn_pinned(av);
+    const int n_tiles = kept_tiles + p / GT_KEYS + 1 - tile_lo;      // kept positions' tiles first (attn_seen)
+    const int tps = (n_tiles + nsplit - 1) / nsplit;
+    const int tb = split * tps, te = min(n_tiles, tb + tps);
     const int* table = tables + (size_t)slots[s] * table_stride;
 
     // the group's queries: 16 rows, zeros beyond the group
@@ -663,7 +668,7 @@ attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
         *reinterpret_cast<uint4*>(gsm + r * ROW + ch * 16) = v;
     }
     auto load_tile = [&](int tile, int buf) {
-        const CachePos cp = cache_pos(tile * GT_KEYS, ring, table, GT_KEYS, num_pages, status);
+        const CachePos cp = cache_pos(attn_seen(tile, kept_tiles, tile_lo) * GT_KEYS, ring, table, GT_KEYS, num_pages, status, pinned);
         const size_t at = cache_index(cp, kvh, nkv, GT_KEYS, HD);
         for (int c = threadIdx.x; c < GT_KEYS * CPR; c += WARPS * 32) {
             const int r = c / CPR, ch = c % CPR;
@@ -692,8 +697,8 @@ attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
         }
         __syncthreads();
         const uint32_t kb = sK + buf * GT_KEYS * ROW, vb = sV + buf * GT_KEYS * ROW;
-        const int j0 = tile * GT_KEYS + warp * 16;       // this warp's 16 keys
-        if (j0 <= p && j0 + 15 >= lo) {                   // (warp-uniform) some of them are seen
+        const int j0 = attn_seen(tile, kept_tiles, tile_lo) * GT_KEYS + warp * 16;       // this warp's 16 keys
+        if (j0 <= p && (j0 + 15 >= lo || j0 < av.keep)) {                   // (warp-uniform) some of them are seen
             float sc[2][4], sd[2][4];                     // two chains a tile of eight keys, summed below
 #pragma unroll
             for (int i = 0; i < 2; i++) {
@@ -719,7 +724,7 @@ attn_decode_grouped_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloa
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
                     const int j = j0 + i * 8 + (lane & 3) * 2 + (e & 1);
-                    const float x = (j >= lo && j <= p)
+                    const float x = ((j >= lo || j < av.keep) && j <= p)
                                         ? attn_logit(av, min(kvh * group + h0 + (lane >> 2) + 8 * (e >> 1), nh - 1), sc[i][e], scale)
                                         : -INFINITY;
                     sc[i][e] = x;
@@ -863,7 +868,7 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, f
            const int* seq_of_token, const int* pos, const int* slots, const int* tables, int table_stride, int ring,
            int page_size, int num_pages, int num_tokens, int nh, int nkv, int hd, int window, float scale, int nsplit,
            int* status, cudaStream_t stream, const FusedArgs* fused = nullptr, const GateOut go = GateOut{nullptr, 0, 0, 0},
-           const AttnVariant av = AttnVariant{0, 0.f, 0, nullptr}) {
+           const AttnVariant av = AttnVariant{0, 0.f, 0, nullptr, 0}) {
     const int group = nh / nkv;
     dim3 grid(nsplit, nkv, num_tokens);
     const int row_bytes = hd * (int)sizeof(T);
@@ -980,11 +985,11 @@ MOE_API int moe_attention_decode(const void* q, const void* k_cache, const void*
                                  const int* tables, int table_stride, int ring, int page_size, int num_pages,
                                  int num_tokens, int nh, int nkv, int hd, int window, float scale, int nsplit,
                                  const float* gate, int gate_ld, int dv, int* status, int chunk, float softcap,
-                                 int sink, const float* sink_vals, cudaStream_t stream) {
+                                 int sink, const float* sink_vals, int keep, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (dv < 0 || dv > hd || (gate && dv == 0)) return (int)cudaErrorInvalidValue;
     const GateOut go{gate, gate_ld < 0 ? -gate_ld : gate_ld, dv, gate_ld < 0};
-    const AttnVariant av{chunk, softcap, sink, sink_vals};
+    const AttnVariant av{chunk, softcap, sink, sink_vals, keep};
     if (hd % 16 != 0 || hd > WIDE_HD || hd <= 0 || nkv <= 0 || nh <= 0 || nh > 65535 || nh % nkv != 0 || nsplit < 1 ||
         nsplit > 65535 || nkv > 65535 || num_tokens > 65535 || !q || !k_cache || !v_cache || !out || !partial)
         return (int)cudaErrorInvalidValue;

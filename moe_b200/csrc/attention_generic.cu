@@ -78,9 +78,11 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const 
     for (int i = 0; i < MAX_HD / 32; i++) acc[i] = 0.f;
     float m = -INFINITY, l = 0.f;
 
-    for (int j0 = lo; j0 <= p; j0 += 32) {
-        const int j = j0 + lane;
-        const bool valid = j <= p;
+    const int kept = attn_kept(av, lo), pinned = attn_pinned(av);
+    const int n_keys = kept + p + 1 - lo;
+    for (int v0 = 0; v0 < n_keys; v0 += 32) {
+        const int j = attn_seen(v0 + lane, kept, lo);
+        const bool valid = v0 + lane < n_keys;
         const T* kp = nullptr;
         const T* vp = nullptr;
         if (valid) {
@@ -88,7 +90,7 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const 
                 const size_t r = ((size_t)(tok0 + (j - p0)) * nkv + kvh) * hd;
                 kp = k_new + r, vp = v_new + r;
             } else {
-                const CachePos cp = cache_pos(j, ring, table, page_size, num_pages, status);
+                const CachePos cp = cache_pos(j, ring, table, page_size, num_pages, status, pinned);
                 const size_t r = cache_index(cp, kvh, nkv, page_size, hd);
                 kp = k_cache + r, vp = v_cache + r;
             }
@@ -101,7 +103,7 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const 
         m = m_new;
 #pragma unroll
         for (int i = 0; i < MAX_HD / 32; i++) acc[i] *= alpha;
-        const int n_valid = min(32, p - j0 + 1);
+        const int n_valid = min(32, n_keys - v0);
         for (int jj = 0; jj < n_valid; jj++) {
             const float pj = __shfl_sync(0xffffffffu, pr, jj);
             const T* vj = (const T*)__shfl_sync(0xffffffffu, (unsigned long long)vp, jj);
@@ -127,8 +129,8 @@ MOE_API int moe_attention_generic(const void* q, const void* k_new, const void* 
                                   const int* seq_start, const int* cu_seqlens, const int* slots, const int* tables,
                                   int table_stride, int ring, int page_size, int num_pages, int num_tokens, int nh,
                                   int nkv, int hd, int window, float scale, int use_local, int* status,
-                                  int chunk, float softcap, int sink, const float* sink_vals, cudaStream_t stream) {
-    const AttnVariant av{chunk, softcap, sink, sink_vals};
+                                  int chunk, float softcap, int sink, const float* sink_vals, int keep, cudaStream_t stream) {
+    const AttnVariant av{chunk, softcap, sink, sink_vals, keep};
     if (num_tokens <= 0) return 0;
     if (hd % 16 != 0 || hd > WIDE_HD || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535)
         return (int)cudaErrorInvalidValue;

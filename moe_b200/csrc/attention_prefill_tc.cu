@@ -42,6 +42,7 @@
 // The output is [T, nh, HD], or with dv > 0 packed to [T, nh * dv], the first dv columns of every head (only
 // those are computed), times the sigmoid of one gate logit a head: rounded to bfloat16 before the gate is
 // multiplied in, as the merge of a single-token step rounds it.
+#include <climits>
 #include <cuda.h>
 
 #include <mutex>
@@ -252,7 +253,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int kt_lo = lo_pos / KT;
     const int nc = lo_pos < start ? (start - 1) / KT - kt_lo + 1 : 0;
     const int t_lo = max(0, lo_pos - start) / KT;
-    const int n_tiles = nc + q_last / KT - t_lo + 1;
+    // Kept first positions (AttnVariant::keep) that lie in front of the window: `kc` tiles of the cache and `kl` of
+    // the step's own tokens.  The tiles' order: kept cached, cached, kept own, own; a kept tile is never one
+    // of the window's.
+    const int kc = min((min(av.keep, start) + KT - 1) / KT, nc > 0 ? kt_lo : INT_MAX);
+    const int kl = min((max(0, av.keep - start) + KT - 1) / KT, t_lo);
+    const int n_cached = kc + nc;
+    const int n_tiles = n_cached + kl + q_last / KT - t_lo + 1;
+    // where tile `it` starts: a multiple of KT, an absolute position for a cached tile, a token of the step else
+    auto tile_at = [&](int it) {
+        return it < n_cached ? (it < kc ? it : kt_lo + it - kc) * KT : (it - n_cached < kl ? it - n_cached : t_lo + it - n_cached - kl) * KT;
+    };
 
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t sQ = base;
@@ -303,17 +314,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             // the values, as the MMA issuer asks for them (scores of tile j + 1 before P V of tile j).
             bool ok = true;
             int nk = 0, nv = 0;                         // tiles whose keys / values have been requested
-            const int* table = nc > 0 ? tables + (size_t)slots[seq] * table_stride : nullptr;
+            const int* table = n_cached > 0 ? tables + (size_t)slots[seq] * table_stride : nullptr;
+            const int pinned = attn_pinned(av);
             int page_row[2][2];                         // of a cache tile's two pages: first row in the cache seen
                                                         // as rows of one head's keys, [page][kv head][64] of them
             auto find_pages = [&](int it) {
                 for (int h = 0; h < 2; h++) {
-                    const int a = (kt_lo + it) * KT + h * 64;         // first position of the page
-                    int page = table[(ring > 0 ? a % ring : a) >> 6];
+                    const int a = tile_at(it) + h * 64;               // first position of the page
+                    int page = table[((ring > 0 && a >= pinned) ? pinned + (a - pinned) % ring : a) >> 6];
                     if (page < 0 || page >= num_pages) {
                         // only a page that holds a key some row needs is an error; the half of a tile
                         // beyond the sequence's cached tokens just has to be finite, and every page is
-                        if (a < start && a + 63 >= lo_pos) atomicOr(status, ST_BAD_PAGE);
+                        if (a < start && (a + 63 >= lo_pos || a < av.keep)) atomicOr(status, ST_BAD_PAGE);
                         page = 0;
                     }
                     page_row[it & 1][h] = (page * nkv + kvh) * 64;
@@ -322,14 +334,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             auto load_k = [&](int it) {
                 const int st = it % NST, pb = it & 1;
                 if (!mbar_wait(k_empty(st), ((it / NST) & 1) ^ 1, &s_abort, status, 0x41)) return false;
-                if (it < nc) find_pages(it);
+                if (it < n_cached) find_pages(it);
                 mbar_expect_tx(k_full(st), TILE_BYTES);
                 for (int c = 0; c < CH; c++) {
-                    if (it < nc) {
+                    if (it < n_cached) {
                         tma_load_2d(sK(st) + c * 16384, &tmKc, c * 64, page_row[pb][0], k_full(st));
                         tma_load_2d(sK(st) + c * 16384 + 8192, &tmKc, c * 64, page_row[pb][1], k_full(st));
                     } else {
-                        tma_load_3d(sK(st) + c * 16384, &tmK, c * 64, kvh, tok0 + (t_lo + it - nc) * KT, k_full(st));
+                        tma_load_3d(sK(st) + c * 16384, &tmK, c * 64, kvh, tok0 + tile_at(it), k_full(st));
                     }
                 }
                 nk = it + 1;
@@ -340,11 +352,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                 if (!mbar_wait(v_empty(st), ((it >> 1) & 1) ^ 1, &s_abort, status, 0x42)) return false;
                 mbar_expect_tx(v_full(st), TILE_BYTES);
                 for (int c = 0; c < CH; c++) {
-                    if (it < nc) {
+                    if (it < n_cached) {
                         tma_load_2d(sV(st) + c * 16384, &tmVc, c * 64, page_row[st][0], v_full(st));
                         tma_load_2d(sV(st) + c * 16384 + 8192, &tmVc, c * 64, page_row[st][1], v_full(st));
                     } else {
-                        tma_load_3d(sV(st) + c * 16384, &tmV, c * 64, kvh, tok0 + (t_lo + it - nc) * KT, v_full(st));
+                        tma_load_3d(sV(st) + c * 16384, &tmV, c * 64, kvh, tok0 + tile_at(it), v_full(st));
                     }
                 }
                 nv = it + 1;
@@ -450,16 +462,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             tc_fence_after();
             const uint32_t ts = tmem + COL_S + b * KT + lane_base + half * (KT / 2);
             // the tile's first position, and the end of what its source holds of the sequence
-            const int j0 = it < nc ? (kt_lo + it) * KT : start + (t_lo + it - nc) * KT;
-            const int jmax = it < nc ? start : start + len;
+            const int j0 = it < n_cached ? tile_at(it) : start + tile_at(it);
+            const int jmax = it < n_cached ? start : start + len;
             const int jh = j0 + half * (KT / 2);
             // a tile strictly below the diagonal, inside the window and inside the sequence needs no mask
             const bool full = j0 + KT - 1 <= start + q0 && j0 + KT <= jmax &&
                               (av.chunk > 0 ? j0 >= attn_lo(start + q0 + QT - 1, 0, av.chunk)
-                                            : (window <= 0 || j0 >= start + q0 + QT - window));
+                                            : (window <= 0 || j0 >= start + q0 + QT - window || j0 + KT <= av.keep));
             auto tile_softmax = [&](auto masked_tag) -> bool {
                 constexpr bool MASKED = decltype(masked_tag)::value;
-                auto visible = [&](int j) { return j <= prow && j < jmax && j >= lo_row; };
+                auto visible = [&](int j) { return j <= prow && j < jmax && (j >= lo_row || j < av.keep); };
                 float m_new = m, alpha = 1.f;
                 if (!sigmoid_w) {
                 // pass 1: the maximum of the half row (of the raw scores: the scale is positive)
@@ -715,7 +727,7 @@ bool takes(int hd, bool shared, int dv, const float* gate) {
 // does not take: the caller then uses moe_attention_prefill_bf16.
 MOE_API int moe_attention_prefill_tc(const void* q, const void* k, const void* v, void* out, const int* cu_seqlens,
                                      int num_seqs, int num_tokens, int nh, int nkv, int hd, int window, float scale,
-                                     int* status, int chunk, float softcap, int sink, const float* sink_vals, int dv,
+                                     int* status, int chunk, float softcap, int sink, const float* sink_vals, int keep, int dv,
                                      const float* gate, int gate_ld, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (nkv <= 0 || nh % nkv != 0 || nh > 65535 || dv < 0 || dv > hd) return (int)cudaErrorInvalidValue;
@@ -724,7 +736,7 @@ MOE_API int moe_attention_prefill_tc(const void* q, const void* k, const void* v
     if ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)out) & 15) != 0) return -1;
     CacheArgs c{};
     return run(q, k, v, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, hd, window, scale, status,
-               AttnVariant{chunk, softcap, sink, sink_vals}, PackedOut{dv, gate, gate_ld}, shared, stream);
+               AttnVariant{chunk, softcap, sink, sink_vals, keep}, PackedOut{dv, gate, gate_ld}, shared, stream);
 }
 
 // The same for sequences that go on from the cache: sequence i held seq_start[i] tokens before the
@@ -738,7 +750,7 @@ MOE_API int moe_attention_cached_tc(const void* q, const void* k, const void* v,
                                     const int* slots, const int* tables, int table_stride, int ring, int page_size,
                                     int num_pages, int num_seqs, int num_tokens, int nh, int nkv, int hd, int window,
                                     float scale, int* status, int chunk, float softcap, int sink, const float* sink_vals,
-                                    int dv, const float* gate, int gate_ld, cudaStream_t stream) {
+                                    int keep, int dv, const float* gate, int gate_ld, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (nkv <= 0 || nh % nkv != 0 || nh > 65535 || num_pages <= 0 || dv < 0 || dv > hd) return (int)cudaErrorInvalidValue;
     if (!seq_start || !slots || !tables || !k_cache || !v_cache) return (int)cudaErrorInvalidValue;
@@ -754,5 +766,5 @@ MOE_API int moe_attention_cached_tc(const void* q, const void* k, const void* v,
         !make_cache_map(&c.tmV, v_cache, (long long)num_pages * nkv * 64, hd))
         return -1;
     return run(q, k, v, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, hd, window, scale, status,
-               AttnVariant{chunk, softcap, sink, sink_vals}, PackedOut{dv, gate, gate_ld}, shared, stream);
+               AttnVariant{chunk, softcap, sink, sink_vals, keep}, PackedOut{dv, gate, gate_ld}, shared, stream);
 }

@@ -23,7 +23,7 @@ struct PrepCommit {
     const int* seq_end;
     const int* slots;
     const int* tables;
-    int table_stride, ring, page_size, num_pages;
+    int table_stride, ring, page_size, num_pages, pinned;
 };
 
 constexpr int PREP_WARPS = 8;
@@ -75,9 +75,9 @@ heads_prepare_kernel(const float* __restrict__ proj, int ld, const int* __restri
     cp.page = 0, cp.off = 0;
     if (c.k_cache) {
         const int s = seq_of_token[t];
-        if (s >= 0 && !(c.ring > 0 && p_int < c.seq_end[s] - c.ring)) {
+        if (s >= 0 && cache_holds(p_int, c.seq_end[s], c.ring, c.pinned)) {
             cp = cache_pos(p_int, c.ring, c.tables + (size_t)c.slots[s] * c.table_stride, c.page_size, c.num_pages,
-                           status);
+                           status, c.pinned);
             append = true;
         }
     }
@@ -216,14 +216,14 @@ MOE_API int moe_heads_prepare(const float* proj, int ld, const int* pos, const i
                               const float* k_norm, float eps, const float* freq, int rot, float mscale,
                               int num_tokens, int nh, int nkv, int d, int dv, int D, void* q, void* k, void* v,
                               long long ldq, long long ldkv, int out_dt, void* k_cache, void* v_cache, const int* seq_end, const int* slots,
-                              const int* tables, int table_stride, int ring, int page_size, int num_pages,
+                              const int* tables, int table_stride, int ring, int page_size, int num_pages, int pinned,
                               int* status, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (rot < 0 || rot > d || (rot & 1) || (rot > 0 && !freq) || d <= 0 || dv <= 0 || D < d || D < dv || !q ||
         !k || !v || ld < (nh + nkv) * d + nkv * dv || ldq < (long long)nh * D || ldkv < (long long)nkv * D)
         return (int)cudaErrorInvalidValue;
     if (k_cache && (!v_cache || !seq_end || !slots || !tables || !seq_of_token)) return (int)cudaErrorInvalidValue;
-    PrepCommit c{k_cache, v_cache, seq_end, slots, tables, table_stride, ring, page_size, num_pages};
+    PrepCommit c{k_cache, v_cache, seq_end, slots, tables, table_stride, ring, page_size, num_pages, pinned};
     const int dmax = ((d > dv ? d : dv) + 3) & ~3;
     const size_t smem = ((size_t)((rot + 3) & ~3) + (size_t)PREP_WARPS * dmax) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;

@@ -100,20 +100,23 @@ attn_tiled_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const T*
     }
     const int ncol = hd / 64 + (hd % 64 ? 1 : 0);      // float4 column groups of the output per thread: d = 4 tx + 64 i
 
-    for (int j0 = (lo_min / BK) * BK; j0 <= p_last; j0 += BK) {
+    // (kept first positions: their tiles come first, then those of the window)
+    const int tile_lo = lo_min / BK, kept_tiles = min((var.keep + BK - 1) / BK, tile_lo), pinned = attn_pinned(var);
+    for (int tile = 0; attn_seen(tile, kept_tiles, tile_lo) * BK <= p_last; tile++) {
+        const int j0 = attn_seen(tile, kept_tiles, tile_lo) * BK;
         __syncthreads();                 // the previous tile's K, V and P are no longer read
         // ---- a tile of keys (transposed) and values -------------------------------------------
         for (int idx = tid; idx < BK * (hd / 4); idx += THREADS) {
             const int c = idx / (hd / 4), d = (idx % (hd / 4)) * 4;
             const int j = j0 + c;
             float kv[4] = {0.f, 0.f, 0.f, 0.f}, vv[4] = {0.f, 0.f, 0.f, 0.f};
-            if (j <= p_last && j >= lo_min) {
+            if (j <= p_last && (j >= lo_min || j < var.keep)) {
                 if (j >= local_from) {
                     const size_t at = ((size_t)(tok0 + (j - start)) * nkv + kvh) * hd + d;
                     load_chunk<T>(k_new + at, kv);
                     load_chunk<T>(v_new + at, vv);
                 } else {
-                    const CachePos cp = cache_pos(j, ring, table, BK, num_pages, status);
+                    const CachePos cp = cache_pos(j, ring, table, BK, num_pages, status, pinned);
                     const size_t at = cache_index(cp, kvh, nkv, BK, hd) + d;
                     load_chunk<T>(k_cache + at, kv);
                     load_chunk<T>(v_cache + at, vv);
@@ -150,7 +153,7 @@ attn_tiled_kernel(const T* __restrict__ q, const T* __restrict__ k_new, const T*
 #pragma unroll
             for (int c = 0; c < 4; c++) {
                 const int j = j0 + tx * 4 + c;
-                const bool seen = row < rows && j <= p && j >= lo;
+                const bool seen = row < rows && j <= p && (j >= lo || j < var.keep);
                 s[r][c] = seen ? attn_logit(var, h, s[r][c], scale) : -INFINITY;
                 mx = fmaxf(mx, s[r][c]);
             }
@@ -235,9 +238,9 @@ MOE_API int moe_attention_tiled(const void* q, const void* k_new, const void* v_
                                 const int* slots, const int* tables, int table_stride, int ring, int page_size,
                                 int num_pages, int num_seqs, int num_tokens, int nh, int nkv, int hd, int window,
                                 float scale, int use_local, int* status, int chunk, float softcap, int sink,
-                                const float* sink_vals, cudaStream_t stream) {
+                                const float* sink_vals, int keep, cudaStream_t stream) {
     if (num_tokens <= 0 || num_seqs <= 0) return 0;
-    const AttnVariant av{chunk, softcap, sink, sink_vals};
+    const AttnVariant av{chunk, softcap, sink, sink_vals, keep};
     if (hd > 256) return -1;
     if (hd % 16 != 0 || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return (int)cudaErrorInvalidValue;
     if (page_size != BK || (ring % BK) != 0) return -1;

@@ -101,6 +101,12 @@ __device__ __forceinline__ float glu_mul(int act, float param, float g, float u)
     return (g / (1.0f + expf(-g))) * u;
 }
 
+// A recurrent mixer's output gate: what multiplies the normed output, from the gate's logit.
+enum : int { GATE_SILU = 0, GATE_SIGMOID = 1 };
+__device__ __forceinline__ float gate_value(int fn, float g) {
+    return (fn == GATE_SIGMOID ? 1.0f : g) / (1.0f + expf(-g));
+}
+
 // ---- variants of the attention score and mask, shared by every attention kernel ----------------
 //   chunk > 0   position p sees the keys of its own chunk only: lo = (p / chunk) * chunk (chunks are
 //               counted from position 0 of the sequence); else window > 0: lo = max(0, p + 1 - window)
@@ -116,13 +122,26 @@ __device__ __forceinline__ float glu_mul(int act, float param, float g, float u)
 //                             their running maximum and rescaling: the "score" they see is
 //                             log sigmoid(s_j + b_h) <= 0, so exp(score - m) is the weight over exp(m),
 //                             and the denominator at the end is exp(-m) in place of the sum.
+//   keep > 0    (with a window) the first `keep` positions of the sequence stay in sight of every later
+//               one: p sees [0, min(keep, lo)) beside [lo, p].  The kernels walk the kept keys first, then the
+//               window's; in a ring-shaped cache the kept positions' pages do not take part in the ring
+//               (`pinned` in cache_pos).
 enum : int { ATTN_SOFTMAX = 0, ATTN_SINK = 1, ATTN_SIGMOID = 2 };
 struct AttnVariant {
     int chunk;
     float softcap;
     int sink;
     const float* sink_vals;
+    int keep;
 };
+// positions at the front of a ring-shaped cache that are never written over: whole pages that cover the
+// kept ones
+constexpr int PIN_PAGE = 64;
+__device__ __forceinline__ int attn_pinned(const AttnVariant& av) { return (av.keep + PIN_PAGE - 1) / PIN_PAGE * PIN_PAGE; }
+// kept keys that a query whose window starts at lo sees in front of it
+__device__ __forceinline__ int attn_kept(const AttnVariant& av, int lo) { return min(av.keep, lo); }
+// the v-th key a query sees, `kept` of them in front of its window [lo, ...]
+__device__ __forceinline__ int attn_seen(int v, int kept, int lo) { return v < kept ? v : v - kept + lo; }
 __device__ __forceinline__ float attn_sink_value(const AttnVariant& av, int h) {
     return (av.sink && av.sink_vals) ? av.sink_vals[h] : 0.f;
 }
@@ -251,14 +270,15 @@ __device__ __forceinline__ float rot_hi(float a, float b, float cs, float sn) {
 
 // Logical position -> (page, offset) of a paged, optionally ring-shaped, cache.
 //   ring:  positions wrap at `ring` (a multiple of the page size); 0 = no wrap
+//   pinned: the first `pinned` positions (a multiple of the page size) lie in front of the ring and stay
 //   table: the sequence's page list; page p holds `page_size` consecutive positions
 // One layer's keys (or values) are laid out [page][kv_head][offset][head_dim].
 struct CachePos {
     int page, off;
 };
 __device__ __forceinline__ CachePos cache_pos(int pos, int ring, const int* table, int page_size, int num_pages,
-                                              int* status) {
-    int r = ring > 0 ? pos % ring : pos;
+                                              int* status, int pinned = 0) {
+    int r = (ring > 0 && pos >= pinned) ? pinned + (pos - pinned) % ring : pos;
     int page = table[r / page_size];
     if (page < 0 || page >= num_pages) {
         if (status) atomicOr(status, ST_BAD_PAGE);
@@ -268,6 +288,10 @@ __device__ __forceinline__ CachePos cache_pos(int pos, int ring, const int* tabl
     c.page = page;
     c.off = r % page_size;
     return c;
+}
+// whether position `pos` of a sequence of `end` tokens (after the step) is to be found in the cache
+__device__ __forceinline__ bool cache_holds(int pos, int end, int ring, int pinned) {
+    return ring <= 0 || pos < pinned || pos >= end - ring;
 }
 __device__ __forceinline__ size_t cache_index(CachePos c, int kv_head, int num_kv_heads, int page_size, int head_dim) {
     return (((size_t)c.page * num_kv_heads + kv_head) * page_size + c.off) * head_dim;

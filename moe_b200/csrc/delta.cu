@@ -12,6 +12,8 @@
 //   delta_step      one token a sequence: the recurrence with the state read once and written once, and
 //                   the output's norm and gate behind it, a block a (head, sequence).
 //   delta_scan      several tokens a sequence, four at a time, the state in registers.
+// The decay g is one number a value head, or one a value head and key channel (the rows of S then shrink each by their
+// own): delta_prepare forms those from a product's rows of their own, g = exp(-exp(A_log_h) softplus(a + dt_bias)).
 // Everything here is 32-bit arithmetic; only the normed, gated output of delta_step is rounded.
 #include "common.cuh"
 
@@ -39,6 +41,10 @@ struct DeltaPrep {
     float eps, q_scale;
     float* out;                // [T, channels]: q, k, v
     float* step;               // [T, 2 H]: beta, logarithm of the decay
+    // decays of a channel (decay not null): a's rows, [T, lda] with H * d columns; dt_bias is [H * d]
+    const float* a_rows;
+    long long lda;
+    float* decay;              // [T, H * d]: the decays themselves
 };
 
 // W neighbouring channels of row t convolved and passed through silu; `st`: the sequence's state, li: the row's place
@@ -75,7 +81,8 @@ delta_prepare_kernel(const DeltaPrep p) {
     const int t = blockIdx.x;
     const int qk = 2 * p.G * p.d, channels = qk + p.H * p.dv;
     const int vruns = (p.H * p.dv + 32 * W - 1) / (32 * W);
-    const int items = 2 * p.G + vruns + 1;
+    const int druns = p.decay ? (p.H * p.d + 32 * W - 1) / (32 * W) : 0;
+    const int items = 2 * p.G + vruns + 1 + druns;
     pdl_sync();
     const int s = p.seq_of_token[t];
     float* out = p.out + (size_t)t * channels;
@@ -89,8 +96,11 @@ delta_prepare_kernel(const DeltaPrep p) {
             } else if (item < 2 * p.G + vruns) {
                 for (int e = (item - 2 * p.G) * 32 * W + lane; e < min(p.H * p.dv, (item - 2 * p.G + 1) * 32 * W); e += 32)
                     out[qk + e] = 0.f;
-            } else {
+            } else if (item == 2 * p.G + vruns) {
                 for (int h = lane; h < 2 * p.H; h += 32) stp[h] = 0.f;
+            } else {
+                const int r0 = (item - 2 * p.G - vruns - 1) * 32 * W;
+                for (int e = r0 + lane; e < min(p.H * p.d, r0 + 32 * W); e += 32) p.decay[(size_t)t * p.H * p.d + e] = 1.f;
             }
             continue;
         }
@@ -132,11 +142,25 @@ delta_prepare_kernel(const DeltaPrep p) {
                 else
                     out[qk + e] = y[0];
             }
-        } else {
+        } else if (item == 2 * p.G + vruns) {
             const float* row = p.proj + (size_t)t * p.ld;
             for (int h = lane; h < p.H; h += 32) {
                 stp[h] = 1.0f / (1.0f + expf(-row[p.b_at + h]));
-                stp[p.H + h] = -expf(p.a_log[h]) * softplus_dt(row[p.a_at + h] + p.dt_bias[h]);
+                stp[p.H + h] = p.decay ? 0.f : -expf(p.a_log[h]) * softplus_dt(row[p.a_at + h] + p.dt_bias[h]);
+            }
+        } else {
+            const int e = ((item - 2 * p.G - vruns - 1) * 32 + lane) * W;
+            if (e < p.H * p.d) {
+                const float* a = p.a_rows + (size_t)t * p.lda + e;
+                const float rate = expf(p.a_log[e / p.d]);            // (W neighbours lie in one head)
+                float* dst = p.decay + (size_t)t * p.H * p.d + e;
+                if (W == 4) {
+                    const float4 x = *reinterpret_cast<const float4*>(a), b = *reinterpret_cast<const float4*>(p.dt_bias + e);
+                    *reinterpret_cast<float4*>(dst) = make_float4(expf(-rate * softplus_dt(x.x + b.x)), expf(-rate * softplus_dt(x.y + b.y)),
+                                                                  expf(-rate * softplus_dt(x.z + b.z)), expf(-rate * softplus_dt(x.w + b.w)));
+                } else {
+                    *dst = expf(-rate * softplus_dt(*a + p.dt_bias[e]));
+                }
             }
         }
     }
@@ -150,16 +174,17 @@ struct DeltaSeq {
     const int* cu_seqlens;
     const int* slots;
     int H, G, d, dv;
+    const float* decay;        // [T, H d]: a decay a channel; null: one a head (step)
 };
 
 // ---- one token a sequence --------------------------------------------------------------------------
 // A block a (head, sequence): thread (cg, kp) holds four neighbouring columns of every KP-th row of S.  The
 // state is asked for before the wait for the predecessor: nothing since the step before has written it.
-template <typename OT, int UNITS>
+template <typename OT, int UNITS, bool CH>
 __global__ void __launch_bounds__(256)
 delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ldg, const float* __restrict__ norm_w,
-                  float norm_eps, const int* __restrict__ seq_of_token, int num_tokens, OT* __restrict__ out) {
-    extern __shared__ __align__(16) float ds_smem[];         // k [d] | q [d] | u [dv] | parts [KP][dv]
+                  float norm_eps, const int* __restrict__ seq_of_token, int num_tokens, int gate_fn, OT* __restrict__ out) {
+    extern __shared__ __align__(16) float ds_smem[];         // k [d] | q [d] | u [dv] | parts [KP][dv] | CH: decays [d]
     __shared__ float red[32];
     const int h = blockIdx.x, s = blockIdx.y, d = p.d, dv = p.dv;
     const int CG = dv / 4, KP = blockDim.x / CG, cg = threadIdx.x % CG, kp = threadIdx.x / CG;
@@ -168,6 +193,7 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
     float* sq = sk + d;
     float* su = sq + d;
     float* parts = su + dv;
+    float* sg = parts + KP * dv;
     const int t = p.cu_seqlens[s];
     const bool live = p.cu_seqlens[s + 1] > t && t < num_tokens && seq_of_token[t] >= 0;
     float* S = p.state + (size_t)p.slots[s] * p.state_pitch + (size_t)h * d * dv;
@@ -187,12 +213,16 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
     const int g = h / (p.H / p.G), channels = 2 * p.G * d + p.H * dv;
     const float* row = p.qkv + (size_t)t * channels;
     for (int i = threadIdx.x; i < d; i += blockDim.x) sq[i] = row[(size_t)g * d + i], sk[i] = row[(size_t)(p.G + g) * d + i];
-    const float beta = p.step[(size_t)t * 2 * p.H + h], decay = expf(p.step[(size_t)t * 2 * p.H + p.H + h]);
+    if (CH)
+        for (int i = threadIdx.x; i < d; i += blockDim.x) sg[i] = p.decay[((size_t)t * p.H + h) * d + i];
+    const float beta = p.step[(size_t)t * 2 * p.H + h];
+    float decay = CH ? 1.f : expf(p.step[(size_t)t * 2 * p.H + p.H + h]);
     __syncthreads();
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < UNITS; i++) {
         const int rr = kp + i * KP;
+        if (CH) decay = (worker && rr < d) ? sg[rr] : 0.f;
         r[i].x *= decay, r[i].y *= decay, r[i].z *= decay, r[i].w *= decay;
         if (worker && rr < d) {
             const float k = sk[rr];
@@ -236,7 +266,7 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
     const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)dv + norm_eps);
     for (int c = threadIdx.x; c < dv; c += blockDim.x)
         st_f(out + ((size_t)t * p.H + h) * dv + c,
-             su[c] * inv * norm_w[(size_t)h * dv + c] * silu32(gate[(size_t)t * ldg + (size_t)h * dv + c]));
+             su[c] * inv * norm_w[(size_t)h * dv + c] * gate_value(gate_fn, gate[(size_t)t * ldg + (size_t)h * dv + c]));
 }
 
 // ---- several tokens a sequence: four at a time ------------------------------------------------------------
@@ -245,6 +275,10 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
 //     u_i = beta_i v_i - beta_i e^(b_i) S^T k_i - sum_(j<i) beta_i e^(b_i - b_j) (k_i . k_j) u_j
 //     o_i = e^(b_i) S^T q_i + sum_(j<=i) e^(b_i - b_j) (q_i . k_j) u_j
 //     S   <- e^(b_4) S + sum_j k_j (e^(b_4 - b_j) u_j)^T
+// (CH, a decay a channel: with G_i the product of the channel's decays from the group's first token to its i-th and
+// D_ij that from the one after j to i, e^(b_i) S^T k_i becomes S^T (G_i k_i), e^(b_i - b_j) (k_i . k_j) the sum over the
+// channels of D_ij k_i k_j, and S <- G_4 S + sum_j (D_4j k_j) u_j^T; every factor is a product of decays, none a
+// quotient.  The warp that forms a group's scalars puts G_i k_i, G_i q_i and D_4j k_j in the place of k, q and the decays.)
 // which is the recurrence written out: every exponent is <= 0, only the order of additions differs.  Against
 // one token at a time the products with S are eight independent sums instead of two with an update between
 // them, their sums over the threads are formed together, and the state is multiplied by a decay once.
@@ -267,15 +301,21 @@ __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes
 }
 
 // VEC: rows of q, k and v start on 16-byte boundaries and hold whole 16-byte units.
-template <int RPT, bool VEC>
-__global__ void __launch_bounds__(DTHREADS, RPT <= 8 ? 4 : 2)
+template <int RPT, bool CH>
+__host__ __device__ constexpr size_t delta_scan_floats() {
+    return (size_t)2 * DRUN * ((CH ? 3 : 2) * RPT * DKP + DCOLS) + 4 * DRUN + 4 * 32 + DG * DCOLS + (CH ? 4 * RPT * DKP : 0);
+}
+template <int RPT, bool VEC, bool CH>
+__global__ void __launch_bounds__(DTHREADS, RPT <= 8 ? (CH && RPT == 8 ? 3 : 4) : 2)
 delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     constexpr int NP = RPT * DKP;
-    constexpr int ROWLEN = 2 * NP + DCOLS;
+    constexpr int V_AT = (CH ? 3 : 2) * NP;                   // a token's row: k, q, CH: its decays, then v
+    constexpr int ROWLEN = V_AT + DCOLS;
     extern __shared__ __align__(16) float sm[];               // [2][DRUN][ROWLEN] | steps [2][2][DRUN] | scalars [4][32] | u [DG][DCOLS]
-    float* s_step = sm + 2 * DRUN * ROWLEN;
+    float* s_step = sm + 2 * DRUN * ROWLEN;                   // | CH: a group's decay of a channel [4][NP]
     float* s_coef = s_step + 4 * DRUN;
     float* s_u = s_coef + 4 * 32;
+    float* s_g4 = s_u + DG * DCOLS;
     const int tid = threadIdx.x, kp = tid % DKP, cg = tid / DKP, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, s = blockIdx.z, g = h / (p.H / p.G), d = p.d, dv = p.dv;
     const int c0 = blockIdx.x * DCOLS, col = c0 + cg * 4;
@@ -300,18 +340,24 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     }
     const float* base = p.qkv + (size_t)tok0 * channels;
     const float* sbase = p.step + (size_t)tok0 * 2 * p.H + h;
+    const float* gbase = CH ? p.decay + ((size_t)tok0 * p.H + h) * d : nullptr;
     const int k_at = (p.G + g) * d, q_at = g * d, v_at = 2 * p.G * d + h * dv + c0;
     auto stage = [&](int t0, int buf) {
         float* dst = sm + buf * DRUN * ROWLEN;
         constexpr int W = VEC ? 4 : 1;
-        const int kw = d / W, vw = ncols / W, per = 2 * kw + vw;
+        const int kw = d / W, vw = ncols / W, per = 2 * kw + vw + (CH ? kw : 0);
         for (int tt = warp; tt < DRUN; tt += DTHREADS / 32) {           // a warp a token
             const bool on = t0 + tt < cnt;
             const float* row = base + (size_t)min(t0 + tt, cnt - 1) * channels;
             float* to = dst + tt * ROWLEN;
             for (int e = lane; e < per; e += 32) {
+                if (CH && e >= 2 * kw + vw) {
+                    const int x = e - 2 * kw - vw;
+                    cp_zfill(to + 2 * NP + x * W, gbase + (size_t)min(t0 + tt, cnt - 1) * p.H * d + x * W, 4 * W, on);
+                    continue;
+                }
                 const int x = e < kw ? e : e < 2 * kw ? e - kw : e - 2 * kw;
-                cp_zfill(to + (e < kw ? 0 : e < 2 * kw ? NP : 2 * NP) + x * W, row + (e < kw ? k_at : e < 2 * kw ? q_at : v_at) + x * W, 4 * W, on);
+                cp_zfill(to + (e < kw ? 0 : e < 2 * kw ? NP : V_AT) + x * W, row + (e < kw ? k_at : e < 2 * kw ? q_at : v_at) + x * W, 4 * W, on);
             }
         }
         if (tid < 2 * DRUN) {
@@ -328,10 +374,10 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();                              // this run is there, and the one before is no longer read
         if (t0 + DRUN < cnt) stage(t0 + DRUN, buf ^ 1);
-        const float* run = sm + buf * DRUN * ROWLEN;
+        float* run = sm + buf * DRUN * ROWLEN;
         {
             // the scalars of group `warp`: products of its keys and queries, then everything made of them
-            const float* row = run + warp * DG * ROWLEN;
+            float* row = run + warp * DG * ROWLEN;
             float dots[16];                           // [0 ... 5] k_i . k_j, j < i;  [6 ... 15] q_i . k_j, j <= i
 #pragma unroll
             for (int i = 0; i < 16; i++) dots[i] = 0.f;
@@ -341,6 +387,33 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
                 for (int i = 0; i < DG; i++) {
                     k4[i] = *reinterpret_cast<const float4*>(row + i * ROWLEN + e);
                     q4[i] = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + e);
+                }
+                if (CH) {
+                    const int left = cnt - t0 - warp * DG;        // tokens of the group; places beyond keep what there is
+                    float4 g4[DG];
+#pragma unroll
+                    for (int i = 0; i < DG; i++)
+                        g4[i] = i < left ? *reinterpret_cast<const float4*>(row + i * ROWLEN + 2 * NP + e) : make_float4(1.f, 1.f, 1.f, 1.f);
+                    auto mul = [](float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); };
+                    auto dot3 = [](float4 a, float4 b, float4 c, float s) {
+                        return fmaf(a.x * c.x, b.x, fmaf(a.y * c.y, b.y, fmaf(a.z * c.z, b.z, fmaf(a.w * c.w, b.w, s))));
+                    };
+                    float4 all = make_float4(1.f, 1.f, 1.f, 1.f);
+#pragma unroll
+                    for (int j = 0; j < DG; j++) {
+                        float4 since = make_float4(1.f, 1.f, 1.f, 1.f);        // from the token after j to i
+#pragma unroll
+                        for (int i = j; i < DG; i++) {
+                            if (i > j) since = mul(since, g4[i]), dots[i * (i - 1) / 2 + j] = dot3(k4[i], k4[j], since, dots[i * (i - 1) / 2 + j]);
+                            dots[6 + i * (i + 1) / 2 + j] = dot3(q4[i], k4[j], since, dots[6 + i * (i + 1) / 2 + j]);
+                        }
+                        all = mul(all, g4[j]);
+                        *reinterpret_cast<float4*>(row + j * ROWLEN + e) = mul(k4[j], all);
+                        *reinterpret_cast<float4*>(row + j * ROWLEN + NP + e) = mul(q4[j], all);
+                        *reinterpret_cast<float4*>(row + j * ROWLEN + 2 * NP + e) = mul(k4[j], since);
+                    }
+                    *reinterpret_cast<float4*>(s_g4 + warp * NP + e) = all;
+                    continue;
                 }
                 int x = 0;
 #pragma unroll
@@ -382,17 +455,17 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             const int n = lane & 15;
             if (lane < 16) {
                 const int i = n & 3;
-                const float ei = expf(i == 0 ? bs[0] : i == 1 ? bs[1] : i == 2 ? bs[2] : bs[3]);
+                const float ei = CH ? 1.f : expf(i == 0 ? bs[0] : i == 1 ? bs[1] : i == 2 ? bs[2] : bs[3]);
                 float rest = 0.f;                     // b_4 - b_i, added up and not subtracted
                 for (int e = i + 1; e < DG; e++) rest += lg[e];
-                s_coef[warp * 32 + n] = n < 4 ? be[i] : n < 8 ? be[i] * ei : n < 12 ? ei : expf(rest);
+                s_coef[warp * 32 + n] = n < 4 ? be[i] : n < 8 ? be[i] * ei : n < 12 ? ei : CH ? 1.f : expf(rest);
             } else {
                 // pair number n: j < i of the keys, then j <= i of queries and keys
                 const int i = n < 6 ? (n < 1 ? 1 : n < 3 ? 2 : 3) : (n < 7 ? 0 : n < 9 ? 1 : n < 12 ? 2 : 3);
                 const int j = n < 6 ? n - i * (i - 1) / 2 : n - 6 - i * (i + 1) / 2;
                 float decay = 0.f;                    // b_i - b_j, the same
                 for (int e = j + 1; e <= i; e++) decay += lg[e];
-                s_coef[warp * 32 + 16 + n] = dot * expf(decay) * (n < 6 ? be[i] : 1.f);
+                s_coef[warp * 32 + 16 + n] = dot * (CH ? 1.f : expf(decay)) * (n < 6 ? be[i] : 1.f);
             }
         }
         __syncthreads();
@@ -448,7 +521,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             }
             // (threads of the queries' half go through the same motions with their own sums; their u is not used)
             float u[DG];
-            const float* vrow = run + gr * DG * ROWLEN + 2 * NP + cg * 4 + my_col;
+            const float* vrow = run + gr * DG * ROWLEN + V_AT + cg * 4 + my_col;
             u[0] = cf[0] * vrow[0] - cf[4] * rr[0];
             u[1] = cf[1] * vrow[ROWLEN] - cf[5] * rr[1] - cf[16] * u[0];
             u[2] = cf[2] * vrow[2 * ROWLEN] - cf[6] * rr[2] - cf[17] * u[0] - cf[18] * u[1];
@@ -476,8 +549,28 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
                 uw[i][0] = u4.x, uw[i][1] = u4.y, uw[i][2] = u4.z, uw[i][3] = u4.w;
             }
             __syncwarp();                             // read by all before the next group's are written
+            if (CH) {                                 // the decays and the keys of the update, row by row
 #pragma unroll
-            for (int m = 0; m < RPT; m++)
+                for (int m0 = 0; m0 < RPT; m0 += 4) {
+                    const float4 g4 = *reinterpret_cast<const float4*>(s_g4 + gr * NP + kp * 4 + m0 * DKP);
+                    const float gm[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                    for (int z = 0; z < 4; z++)
+#pragma unroll
+                        for (int c = 0; c < 4; c++) sreg[m0 + z][c] *= gm[z];
+#pragma unroll
+                    for (int i = 0; i < DG; i++) {
+                        const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + 2 * NP + m0 * DKP);
+                        const float km[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+                        for (int z = 0; z < 4; z++)
+#pragma unroll
+                            for (int c = 0; c < 4; c++) sreg[m0 + z][c] = fmaf(km[z], uw[i][c], sreg[m0 + z][c]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < (CH ? 0 : RPT); m++)
 #pragma unroll
                 for (int c = 0; c < 4; c++) {
                     float x = cf[11] * sreg[m][c];
@@ -508,23 +601,26 @@ bool aligned16(const void* p) { return (uintptr_t)p % 16 == 0; }
 // proj: [T, ld] 32-bit: q (G * d columns), k (G * d), v (H * dv), b and a (a column a value head) from b_at and
 // a_at; taps_w: [taps, channels]; state: (taps - 1) * channels floats a slot from the pointer given; out: [T, channels]
 // 32-bit; step: [T, 2 H] 32-bit (beta, then the decay's logarithm).  `shift`: the step brings one token a sequence and the state moves on here.
+// With `decay` not null there is a decay a channel: a_rows [T, lda] holds a (H * d columns), dt_bias [H * d], and decay
+// [T, H * d] receives the decays (a_at is not read then).
 MOE_API int moe_delta_prepare(const float* proj, long long ld, int b_at, int a_at, const float* taps_w, int taps,
                               float* state, long long state_pitch, const float* a_log, const float* dt_bias,
                               const int* seq_of_token, const int* cu_seqlens, const int* slots, int num_tokens, int H,
                               int G, int d, int dv, float eps, float q_scale, int shift, float* out, float* step,
-                              cudaStream_t stream) {
+                              const float* a_rows, long long lda, float* decay, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     const long long channels = 2LL * G * d + (long long)H * dv;
     if (!proj || !taps_w || !a_log || !dt_bias || !seq_of_token || !cu_seqlens || !slots || !out || !step || H <= 0 || G <= 0 ||
         H % G || d <= 0 || d > DP_MAX_D || dv <= 0 || taps < 1 || taps > 16 || (taps > 1 && !state) || ld < channels ||
-        b_at < 0 || a_at < 0 || b_at + H > ld || a_at + H > ld || (taps > 1 && state_pitch < (taps - 1) * channels))
+        b_at < 0 || b_at + H > ld || (decay ? !a_rows || lda < (long long)H * d : a_at < 0 || a_at + H > ld) || (taps > 1 && state_pitch < (taps - 1) * channels))
         return (int)cudaErrorInvalidValue;
     const DeltaPrep p{proj, ld, b_at, a_at, taps_w, state, state_pitch, a_log, dt_bias, seq_of_token, cu_seqlens, slots,
-                      num_tokens, taps, H, G, d, dv, shift, eps, q_scale, out, step};
+                      num_tokens, taps, H, G, d, dv, shift, eps, q_scale, out, step, a_rows, lda, decay};
     const bool vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && state_pitch % 4 == 0 && aligned16(proj) && aligned16(taps_w) &&
-                     aligned16(state) && aligned16(out);
+                     aligned16(state) && aligned16(out) &&
+                     (!decay || (lda % 4 == 0 && aligned16(a_rows) && aligned16(decay) && aligned16(dt_bias)));
     const int per = vec ? 128 : 32;
-    const int items = 2 * G + (H * dv + per - 1) / per + 1;
+    const int items = 2 * G + (H * dv + per - 1) / per + 1 + (decay ? (H * d + per - 1) / per : 0);
     // few tokens: a warp an item; many: a block a token
     const dim3 grid(num_tokens, num_tokens >= 128 ? 1 : (items + DP_WARPS - 1) / DP_WARPS);
     if (grid.y > 65535) return (int)cudaErrorInvalidValue;
@@ -541,24 +637,29 @@ MOE_API int moe_delta_prepare(const float* proj, long long ld, int b_at, int a_a
 }
 
 // One token a sequence.  qkv, step: as moe_delta_prepare leaves them; state: H * d * dv floats a slot from the pointer
-// given; gate: [T, H * dv] 32-bit logits, rows of ldg; norm_w: [H * dv]; out: [T, H * dv] in out_dt (rows of no
+// given; decay: [T, H * d] or null; gate: [T, H * dv] 32-bit logits, rows of ldg, through gate_fn (GATE_*); norm_w: [H * dv]; out: [T, H * dv] in out_dt (rows of no
 // sequence become zeros).  Returns -1, with nothing launched, for sizes it does not take.
 MOE_API int moe_delta_step(const float* qkv, const float* step, float* state, long long state_pitch, const float* gate,
                            long long ldg, const float* norm_w, float norm_eps, const int* seq_of_token,
                            const int* cu_seqlens, const int* slots, int num_tokens, int num_seqs, int H, int G, int d,
-                           int dv, void* out, int out_dt, cudaStream_t stream) {
+                           int dv, const float* decay, int gate_fn, void* out, int out_dt, cudaStream_t stream) {
     if (num_seqs <= 0 || num_tokens <= 0) return 0;
     if (!qkv || !step || !state || !gate || !norm_w || !seq_of_token || !cu_seqlens || !slots || !out || H <= 0 || G <= 0 ||
         H % G || d <= 0 || dv <= 0 || ldg < (long long)H * dv || state_pitch < (long long)H * d * dv || num_seqs > 65535)
         return (int)cudaErrorInvalidValue;
     if (dv % 4 || dv > 512 || d > 256 || state_pitch % 4 || !aligned16(state)) return -1;
     const int cg = dv / 4, kp = 256 / cg, units = (d + kp - 1) / kp;
-    const size_t smem = ((size_t)2 * ((d + 1) / 2 * 2) + dv + (size_t)kp * dv) * sizeof(float);
+    const size_t smem = ((size_t)2 * ((d + 1) / 2 * 2) + dv + (size_t)kp * dv + (decay ? d : 0)) * sizeof(float);
     if (units > 32 || smem > 48 * 1024 || d % 2) return -1;
-    const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv};
+    const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv, decay};
+#define STEP_C(OT_, U_, C_)                                                                                            \
+    return launch_pdl(delta_step_kernel<OT_, U_, C_>, dim3(H, num_seqs), dim3(256), smem, stream, p, gate, ldg, norm_w, norm_eps, \
+                      seq_of_token, num_tokens, gate_fn, (OT_*)out)
 #define STEP(OT_, U_)                                                                                                  \
-    return launch_pdl(delta_step_kernel<OT_, U_>, dim3(H, num_seqs), dim3(256), smem, stream, p, gate, ldg, norm_w, norm_eps, \
-                      seq_of_token, num_tokens, (OT_*)out)
+    do {                                                                                                               \
+        if (decay) STEP_C(OT_, U_, true);                                                                              \
+        STEP_C(OT_, U_, false);                                                                                        \
+    } while (0)
 #define STEP_U(OT_)                                                                                                    \
     do {                                                                                                               \
         if (units <= 4) STEP(OT_, 4);                                                                                  \
@@ -570,34 +671,40 @@ MOE_API int moe_delta_step(const float* qkv, const float* step, float* state, lo
     STEP_U(__nv_bfloat16);
 #undef STEP_U
 #undef STEP
+#undef STEP_C
 }
 
 // Several tokens a sequence; o: [T, H * dv] 32-bit (rows of no sequence are left alone).
 MOE_API int moe_delta_scan(const float* qkv, const float* step, float* state, long long state_pitch, const int* cu_seqlens,
-                           const int* slots, int num_seqs, int H, int G, int d, int dv, float* o, cudaStream_t stream) {
+                           const int* slots, int num_seqs, int H, int G, int d, int dv, const float* decay, float* o,
+                           cudaStream_t stream) {
     if (num_seqs <= 0) return 0;
     if (!qkv || !step || !state || !cu_seqlens || !slots || !o || H <= 0 || G <= 0 || H % G || d <= 0 || d > 256 || dv <= 0 ||
         state_pitch < (long long)H * d * dv || H > 65535 || num_seqs > 65535)
         return (int)cudaErrorInvalidValue;
-    const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv};
+    const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv, decay};
     const dim3 grid((dv + DCOLS - 1) / DCOLS, H, num_seqs);
-    const bool vec = d % 4 == 0 && dv % 4 == 0 && aligned16(qkv);
+    const bool vec = d % 4 == 0 && dv % 4 == 0 && aligned16(qkv) && aligned16(decay);
     // An ordinary launch: blocks that are placed while the kernel before still occupies some SMs end up several to
     // an SM beside empty ones, and a scan is as slow as its most crowded SM.
-#define SCAN_V(RPT_, V_)                                                                                               \
+#define SCAN_V(RPT_, V_, C_)                                                                                           \
     do {                                                                                                               \
-        constexpr size_t smem = (size_t)(2 * DRUN * (2 * RPT_ * DKP + DCOLS) + 4 * DRUN + 4 * 32 + DG * DCOLS) * sizeof(float); \
+        constexpr size_t smem = delta_scan_floats<RPT_, C_>() * sizeof(float);                                         \
         if (smem > 48 * 1024) {                                                                                        \
-            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, V_, C_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                       \
         }                                                                                                              \
-        delta_scan_kernel<RPT_, V_><<<grid, DTHREADS, smem, stream>>>(p, o);                                           \
+        delta_scan_kernel<RPT_, V_, C_><<<grid, DTHREADS, smem, stream>>>(p, o);                                       \
         return launch_status();                                                                                        \
     } while (0)
 #define SCAN(RPT_)                                                                                                     \
     do {                                                                                                               \
-        if (vec) SCAN_V(RPT_, true);                                                                                   \
-        SCAN_V(RPT_, false);                                                                                           \
+        if (decay) {                                                                                                   \
+            if (vec) SCAN_V(RPT_, true, true);                                                                         \
+            SCAN_V(RPT_, false, true);                                                                                 \
+        }                                                                                                              \
+        if (vec) SCAN_V(RPT_, true, false);                                                                            \
+        SCAN_V(RPT_, false, false);                                                                                    \
     } while (0)
     if (d <= 64) SCAN(4);
     if (d <= 128) SCAN(8);

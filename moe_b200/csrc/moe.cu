@@ -225,8 +225,9 @@ __global__ void sum_slices_kernel(const float* __restrict__ part, float* __restr
     out[i] = s;
 }
 
-// Softmax over all experts, top-k and weights of ONE token, by one warp.  `sc` is shared memory
-// of num_experts floats owned by the warp.
+// Scores of all experts (their softmax, or each logit's sigmoid), top-k and weights of ONE token, by one
+// warp.  `sc` is shared memory of num_experts floats owned by the warp.  norm_topk: ROUTE_* flags.
+enum : int { ROUTE_NORM = 1, ROUTE_SIGMOID = 2 };
 __device__ __forceinline__ void route_token(const float* __restrict__ lg, float* sc, int lane, bool padding,
                                             int num_experts, int rows, int top_k, int norm_topk, float scale,
                                             int* __restrict__ idx_out, float* __restrict__ w_out,
@@ -242,17 +243,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ lg, float*
     }
     if (gate_out && rows > num_experts && lane == 0) *gate_out = 1.0f / (1.0f + expf(-lg[num_experts]));
     // (bias: one constant per expert, added to its logit before anything else looks at it)
-    float m = -INFINITY;
-    for (int e = lane; e < num_experts; e += 32) m = fmaxf(m, lg[e] + (bias ? bias[e] : 0.f));
-    m = warp_max(m);
-    float z = 0.f;
-    for (int e = lane; e < num_experts; e += 32) {
-        const float v = expf(lg[e] + (bias ? bias[e] : 0.f) - m);
-        sc[e] = v;
-        z += v;
+    if (norm_topk & ROUTE_SIGMOID) {
+        for (int e = lane; e < num_experts; e += 32) sc[e] = 1.0f / (1.0f + expf(-(lg[e] + (bias ? bias[e] : 0.f))));
+    } else {
+        float m = -INFINITY;
+        for (int e = lane; e < num_experts; e += 32) m = fmaxf(m, lg[e] + (bias ? bias[e] : 0.f));
+        m = warp_max(m);
+        float z = 0.f;
+        for (int e = lane; e < num_experts; e += 32) {
+            const float v = expf(lg[e] + (bias ? bias[e] : 0.f) - m);
+            sc[e] = v;
+            z += v;
+        }
+        z = warp_sum(z);
+        for (int e = lane; e < num_experts; e += 32) sc[e] = sc[e] / z;
     }
-    z = warp_sum(z);
-    for (int e = lane; e < num_experts; e += 32) sc[e] = sc[e] / z;
+    norm_topk &= ROUTE_NORM;
     __syncwarp();
     if (groups > 1 && keep > 0 && keep < groups) {
         // Experts form `groups` equal groups of neighbours; a group's score is its best expert's, and
@@ -444,6 +450,42 @@ route_dispatch_kernel(const float* __restrict__ logits, const int* __restrict__ 
     }
 }
 
+// What the experts read where a pick's weight multiplies an expert's INPUT: for every (token t, pick j) that has a place,
+// xs[pos[t, j]] = w[t, j] * x[t], from the 32-bit row, rounded once.  A block a token.
+template <typename OT, bool VEC>
+__global__ void __launch_bounds__(256)
+weighted_rows_kernel(const float* __restrict__ x, const int* __restrict__ pos_of_pair, const float* __restrict__ w,
+                     int top_k, int hidden, int num_rows, OT* __restrict__ xs, int* status) {
+    pdl_sync();
+    const int t = blockIdx.x;
+    const float* row = x + (size_t)t * hidden;
+    for (int j = 0; j < top_k; j++) {
+        const int at = pos_of_pair[(size_t)t * top_k + j];
+        if (at < 0) continue;
+        if (at >= num_rows) {
+            if (threadIdx.x == 0) atomicOr(status, ST_BAD_ROW);
+            continue;
+        }
+        const float wj = w[(size_t)t * top_k + j];
+        OT* dst = xs + (size_t)at * hidden;
+        if (VEC) {
+            for (int c = threadIdx.x + blockIdx.y * blockDim.x; c < hidden / 4; c += blockDim.x * gridDim.y) {
+                const float4 v = *reinterpret_cast<const float4*>(row + 4 * c);
+                if constexpr (sizeof(OT) == 4) {
+                    *reinterpret_cast<float4*>(dst + 4 * c) = make_float4(wj * v.x, wj * v.y, wj * v.z, wj * v.w);
+                } else {
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(wj * v.x, wj * v.y), hi = __floats2bfloat162_rn(wj * v.z, wj * v.w);
+                    uint2 u;
+                    u.x = *reinterpret_cast<const unsigned*>(&lo), u.y = *reinterpret_cast<const unsigned*>(&hi);
+                    *reinterpret_cast<uint2*>(dst + 4 * c) = u;
+                }
+            }
+        } else {
+            for (int c = threadIdx.x + blockIdx.y * blockDim.x; c < hidden; c += blockDim.x * gridDim.y) st_f(dst + c, wj * row[c]);
+        }
+    }
+}
+
 // act[m, j] = f(gu[m, j]) * gu[m, inter + j], f = silu, silu(a) = a / (1 + exp(-a))
 // (reference: src/model.rs:31-33), or another gate activation (glu_mul in common.cuh).
 template <typename OT>
@@ -457,7 +499,7 @@ __global__ void swiglu_kernel(const float* __restrict__ gu, OT* __restrict__ act
     st_f(act + i, glu_mul(f, f_param, a, b));
 }
 
-// One block per token: out[t] = sum_j w[t, j] * y[pos_of_pair[t k + j]] + g[t] * shared[t]
+// One block per token: out[t] = sum_j w[t, j] * y[pos_of_pair[t k + j]] + g[t] * shared[t]  (topk_w null: weights of 1)
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of_pair,
                                    const float* __restrict__ topk_w, int top_k, const float* __restrict__ shared,
                                    const float* __restrict__ shared_gate, float* __restrict__ out, int hidden,
@@ -469,7 +511,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     float* sw = reinterpret_cast<float*>(pick + top_k);
     for (int j = threadIdx.x; j < top_k; j += blockDim.x) {
         sp[j] = pos_of_pair[(size_t)t * top_k + j];
-        sw[j] = topk_w[(size_t)t * top_k + j];
+        sw[j] = topk_w ? topk_w[(size_t)t * top_k + j] : 1.f;
     }
     const float g = shared_gate ? shared_gate[t] : 1.0f;
     __syncthreads();
@@ -1021,6 +1063,26 @@ MOE_API int moe_route_dispatch(const float* logits, const int* seq_of_token, int
                       num_experts + (has_gate_row ? 1 : 0), top_k, norm_topk, scale, topk_idx, topk_w, shared_gate,
                       offsets, sorted_token, pos_of_pair, (const uint4*)x, (uint4*)xs, row_bytes / 16, status, bias, groups,
                       keep);
+}
+
+// x: [T, hidden] 32-bit; pos_of_pair, w: [T, top_k]; xs: [num_rows, hidden] in out_dt (rows without a pick are left alone).
+MOE_API int moe_weighted_rows(const float* x, const int* pos_of_pair, const float* w, int num_tokens, int top_k, int hidden,
+                              int num_rows, void* xs, int out_dt, int* status, cudaStream_t stream) {
+    if (num_tokens <= 0) return 0;
+    if (!x || !pos_of_pair || !w || !xs || !status || top_k <= 0 || hidden <= 0) return (int)cudaErrorInvalidValue;
+    const bool vec = hidden % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)xs % (out_dt == DT_F32 ? 16 : 8) == 0;
+    const int units = vec ? hidden / 4 : hidden;
+    const dim3 grid(num_tokens, num_tokens >= 256 ? 1 : max(1, min(8, units / 256)));
+#define WROWS(OT_, V_)                                                                                                 \
+    return launch_pdl(weighted_rows_kernel<OT_, V_>, grid, dim3(256), 0, stream, x, pos_of_pair, w, top_k, hidden,     \
+                      num_rows, (OT_*)xs, status)
+    if (out_dt == DT_F32) {
+        if (vec) WROWS(float, true);
+        WROWS(float, false);
+    }
+    if (vec) WROWS(__nv_bfloat16, true);
+    WROWS(__nv_bfloat16, false);
+#undef WROWS
 }
 
 MOE_API int moe_swiglu(const float* gu, void* act, int out_dt, long long rows, int inter, int f, float f_param,

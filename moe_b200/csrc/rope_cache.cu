@@ -189,14 +189,14 @@ __global__ void kv_commit_kernel(const T* __restrict__ k_new, const T* __restric
                                  T* __restrict__ v_cache, const int* __restrict__ seq_of_token,
                                  const int* __restrict__ pos, const int* __restrict__ seq_end,
                                  const int* __restrict__ slots, const int* __restrict__ tables, int table_stride,
-                                 int ring, int page_size, int num_pages, int nkv, int hd, int* status) {
+                                 int ring, int page_size, int num_pages, int pinned, int nkv, int hd, int* status) {
     const int t = blockIdx.x;
     const int s = seq_of_token[t];
     if (s < 0) return;
     const int p = pos[t];
-    if (ring > 0 && p < seq_end[s] - ring) return;
+    if (!cache_holds(p, seq_end[s], ring, pinned)) return;
     const int* table = tables + (size_t)slots[s] * table_stride;
-    const CachePos cp = cache_pos(p, ring, table, page_size, num_pages, status);
+    const CachePos cp = cache_pos(p, ring, table, page_size, num_pages, status, pinned);
     for (int i = threadIdx.x; i < nkv * hd; i += blockDim.x) {
         const int h = i / hd, d = i % hd;
         const size_t dst = cache_index(cp, h, nkv, page_size, hd) + d;
@@ -207,19 +207,19 @@ __global__ void kv_commit_kernel(const T* __restrict__ k_new, const T* __restric
 
 MOE_API int moe_kv_commit(const void* k_new, const void* v_new, void* k_cache, void* v_cache, int dt,
                           const int* seq_of_token, const int* pos, const int* seq_end, const int* slots,
-                          const int* tables, int table_stride, int ring, int page_size, int num_pages, int num_tokens,
+                          const int* tables, int table_stride, int ring, int page_size, int num_pages, int pinned, int num_tokens,
                           int nkv, int hd, int* status, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     const int threads = 128;
     if (dt == DT_F32)
         kv_commit_kernel<float><<<num_tokens, threads, 0, stream>>>(
             (const float*)k_new, (const float*)v_new, (float*)k_cache, (float*)v_cache, seq_of_token, pos, seq_end,
-            slots, tables, table_stride, ring, page_size, num_pages, nkv, hd, status);
+            slots, tables, table_stride, ring, page_size, num_pages, pinned, nkv, hd, status);
     else
         kv_commit_kernel<__nv_bfloat16><<<num_tokens, threads, 0, stream>>>(
             (const __nv_bfloat16*)k_new, (const __nv_bfloat16*)v_new, (__nv_bfloat16*)k_cache,
             (__nv_bfloat16*)v_cache, seq_of_token, pos, seq_end, slots, tables, table_stride, ring, page_size,
-            num_pages, nkv, hd, status);
+            num_pages, pinned, nkv, hd, status);
     return launch_status();
 }
 

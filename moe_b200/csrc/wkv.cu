@@ -21,7 +21,7 @@
 //                   the decay and the block's columns of v pass through shared memory a few tokens
 //                   at a time, the next run's loads in flight while a run is worked on.
 //   wkv_finish      each head's o_t is divided by its root mean square (x / sqrt(mean(x^2) + eps)),
-//                   multiplied by a weight per channel and by silu(gate projection), and rounded to
+//                   multiplied by a weight per channel and by silu(gate projection) or its sigmoid, and rounded to
 //                   the activation dtype for the output projection.
 // Everything here is 32-bit arithmetic; only wkv_shift_mix and wkv_finish round their stores.
 #include "common.cuh"
@@ -353,7 +353,7 @@ template <typename OT>
 __global__ void __launch_bounds__(256)
 wkv_finish_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ldg,
                   const float* __restrict__ norm_w, float eps, const int* __restrict__ seq_of_token, int num_tokens,
-                  int heads, int d, OT* __restrict__ out) {
+                  int heads, int d, int gate_fn, OT* __restrict__ out) {
     pdl_sync();
     const int lane = threadIdx.x & 31;
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -373,7 +373,7 @@ wkv_finish_kernel(const float* __restrict__ o, const float* __restrict__ gate, l
     const float inv = 1.0f / sqrtf(ss / (float)d + eps);
     for (int e = lane; e < d; e += 32) {
         const float g = gate[(size_t)t * ldg + (size_t)head * d + e];
-        st_f(out + base + e, o[base + e] * inv * norm_w[(size_t)head * d + e] * (g / (1.0f + expf(-g))));
+        st_f(out + base + e, o[base + e] * inv * norm_w[(size_t)head * d + e] * gate_value(gate_fn, g));
     }
 }
 
@@ -383,7 +383,7 @@ template <typename OT, int LPH, int UNITS>
 __global__ void __launch_bounds__(256)
 wkv_finish_vec_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long ldg,
                       const float* __restrict__ norm_w, float eps, const int* __restrict__ seq_of_token, int num_tokens,
-                      int heads, int d, OT* __restrict__ out) {
+                      int heads, int d, int gate_fn, OT* __restrict__ out) {
     pdl_sync();
     const int lane = threadIdx.x % LPH;
     const long long item = (long long)blockIdx.x * (256 / LPH) + threadIdx.x / LPH;
@@ -411,8 +411,8 @@ wkv_finish_vec_kernel(const float* __restrict__ o, const float* __restrict__ gat
         const int e = (u * LPH + lane) * 4;
         if (!there || e >= d) continue;
         const float4 w = *reinterpret_cast<const float4*>(norm_w + (size_t)head * d + e);
-        const float y[4] = {x[u].x * inv * w.x * (g[u].x / (1.0f + expf(-g[u].x))), x[u].y * inv * w.y * (g[u].y / (1.0f + expf(-g[u].y))),
-                            x[u].z * inv * w.z * (g[u].z / (1.0f + expf(-g[u].z))), x[u].w * inv * w.w * (g[u].w / (1.0f + expf(-g[u].w)))};
+        const float y[4] = {x[u].x * inv * w.x * gate_value(gate_fn, g[u].x), x[u].y * inv * w.y * gate_value(gate_fn, g[u].y),
+                            x[u].z * inv * w.z * gate_value(gate_fn, g[u].z), x[u].w * inv * w.w * gate_value(gate_fn, g[u].w)};
         if constexpr (sizeof(OT) == 4) {
             *reinterpret_cast<float4*>(out + base + e) = make_float4(y[0], y[1], y[2], y[3]);
         } else {
@@ -498,9 +498,9 @@ MOE_API int moe_wkv_scan(const float* r, const float* k, const float* v, const f
 }
 
 // o: [T, heads * d] 32-bit; gate: the gate projection's output, 32-bit, row pitch ldg; norm_w: [heads * d];
-// out: [T, heads * d] in out_dt.
+// out: [T, heads * d] in out_dt.  gate_fn: GATE_SILU or GATE_SIGMOID.
 MOE_API int moe_wkv_finish(const float* o, const float* gate, long long ldg, const float* norm_w, float eps,
-                           const int* seq_of_token, int num_tokens, int heads, int d, void* out, int out_dt,
+                           const int* seq_of_token, int num_tokens, int heads, int d, int gate_fn, void* out, int out_dt,
                            cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
     if (!o || !gate || !norm_w || !out || heads <= 0 || d <= 0 || ldg < (long long)heads * d)
@@ -511,7 +511,7 @@ MOE_API int moe_wkv_finish(const float* o, const float* gate, long long ldg, con
         (uintptr_t)out % (out_dt == DT_F32 ? 16 : 8) == 0) {
 #define FIN(OT_, LPH_, U_)                                                                                             \
     return launch_pdl(wkv_finish_vec_kernel<OT_, LPH_, U_>, dim3((unsigned)((items + 256 / LPH_ - 1) / (256 / LPH_))), 256, 0, \
-                      stream, o, gate, ldg, norm_w, eps, seq_of_token, num_tokens, heads, d, (OT_*)out)
+                      stream, o, gate, ldg, norm_w, eps, seq_of_token, num_tokens, heads, d, gate_fn, (OT_*)out)
 #define FIN_D(OT_)                                                                                                     \
     do {                                                                                                               \
         if (d <= 32) FIN(OT_, 8, 1);                                                                                   \
@@ -526,7 +526,7 @@ MOE_API int moe_wkv_finish(const float* o, const float* gate, long long ldg, con
     }
     if (out_dt == DT_F32)
         return launch_pdl(wkv_finish_kernel<float>, dim3(blocks), 256, 0, stream, o, gate, ldg, norm_w, eps,
-                          seq_of_token, num_tokens, heads, d, (float*)out);
+                          seq_of_token, num_tokens, heads, d, gate_fn, (float*)out);
     return launch_pdl(wkv_finish_kernel<__nv_bfloat16>, dim3(blocks), 256, 0, stream, o, gate, ldg, norm_w, eps,
-                      seq_of_token, num_tokens, heads, d, (__nv_bfloat16*)out);
+                      seq_of_token, num_tokens, heads, d, gate_fn, (__nv_bfloat16*)out);
 }

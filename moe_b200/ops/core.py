@@ -36,7 +36,8 @@ def lib():
         sig = {
             "moe_embed": [P, I, P, P, I, I, I, P, P, P, P, F, P],
             "moe_dyt": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P, P],
-            "moe_heads_prepare": [P, I, P, P, P, P, F, P, I, F, I, I, I, I, I, I, P, P, P, LL, LL, I, P, P, P, P, P, I, I, I, I, P, P],
+            "moe_heads_prepare": [P, I, P, P, P, P, F, P, I, F, I, I, I, I, I, I, P, P, P, LL, LL, I, P, P, P, P, P, I, I, I, I, I, P,
+                                  P],
             "moe_gate_pack": [P, P, I, I, I, I, I, P, I, I, P],
             "moe_latent_prepare": [P, I, I, I, P, F, P, I, P, P, I, I, I, I, P, I, I, F, P, P, I, I, P, P, P, I, P, P, P, P,
                                    P, I, I, I, I, P, P],
@@ -49,23 +50,23 @@ def lib():
             "moe_add_inplace": [P, P, LL, P],
             "moe_gemm_generic": [P, I, I, P, I, P, I, LL, P, I, I, P, P, I, I, I, I, P, P],
             "moe_rope_split": [P, P, P, I, I, I, I, I, P, P, P, I, P, P, P, P, P, P, I, I, I, I, P, P],
-            "moe_kv_commit": [P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, P, P],
-            "moe_attention_generic": [P, P, P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, F, I, P, P],
+            "moe_kv_commit": [P, P, P, P, I, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P],
+            "moe_attention_generic": [P, P, P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, F, I, P, I, P],
             "moe_router": [P, P, P, I, P, I, I, I, I, I, F, P, P, P, P, P, LL, P, I, I, P],
             "moe_router_logits": [P, P, P, I, I, I, I, P, P, LL, P],
             "moe_router_topk": [P, P, I, I, I, I, I, F, P, P, P, P, I, I, P],
             "moe_split3": [P, P, LL, I, P],
             "moe_route_dispatch": [P, P, I, I, I, I, I, F, P, P, P, P, P, P, P, P, I, P, P, I, I, P],
             "moe_rope_commit": [P, P, P, I, I, I, I, I, P, P, P, I, P, P, P, I, I, I, I, P, P],
-            "moe_attention_decode": [P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, I, P, I, F, I, P, P],
-            "moe_attention_tiled": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, I, F, I, P, P],
+            "moe_attention_decode": [P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, I, P, I, F, I, P, I, P],
+            "moe_attention_tiled": [P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, I, P, I, F, I, P, I, P],
             "moe_conv_heads_prepare": [P, I, P, I, P, LL, P, P, P, P, F, I, P, I, I, I, I, I, I, I, P, P, P, LL, LL, I, P, P,
-                                       P, P, I, I, I, I, P, P],
+                                       P, P, I, I, I, I, I, P, P],
             "moe_conv_state_update": [P, I, P, LL, I, I, P, P, I, P],
             "moe_wkv_shift_mix": [P, P, I, P, LL, P, P, P, P, I, I, P, I, P, P, P, P, I, I, P, P],
             "moe_wkv_decay": [P, P, P, I, I, I, P, P],
             "moe_wkv_scan": [P, P, P, P, LL, P, P, LL, P, P, I, I, I, P, I, I, P, P, P],
-            "moe_wkv_finish": [P, P, LL, P, F, P, I, I, I, P, I, P],
+            "moe_wkv_finish": [P, P, LL, P, F, P, I, I, I, I, P, I, P],
             "moe_rmsnorm_scaled": [P, P, P, P, P, P, P, P, P, I, I, I, F, I, P, P, P, P, I, P, P, P, P],
             "moe_attention_decode_fused": [P, P, I, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, I, P, P],
             "moe_norm_route": [P, P, P, F, I, I, P, P, P, P, I, I, I, I, F, P, P, P, P, P, P, P, P, P, P, I, I, P],
@@ -77,7 +78,9 @@ def lib():
             "moe_seed_rng": [P, P, P, I, P],
             "moe_table_update": [P, I, P, I, P],
             "moe_whole_prepare": [P, I, P, P, P, P, F, P, I, P, I, I, I, I, I, I, P, P, P, LL, LL, I, P, P, P, P, P, I, I, I, I,
-                                  P, P],
+                                  I, P, P],
+            "moe_whole_conv_prepare": [P, I, P, I, P, LL, I, P, P, P, P, P, P, F, P, I, I, I, I, I, I, I, I, I, P, P, P, LL, LL,
+                                       I, P, P, P, P, I, I, I, I, I, P, P],
             "moe_unrotate_pack": [P, P, P, I, I, I, I, P, I, P],
             "moe_seq_conv": [I, P, LL, P, P, P, P, P, P, LL, P, P, P, P, P, I, I, LL, P, P, P, P, I, I, I, I, P],
             "moe_embed_pair": [P, P, I, P, F, P, P, I, I, I, I, I, I, P, P, P, P, P, P, P, P],
@@ -86,14 +89,19 @@ def lib():
             "moe_table_route": [P, I, P, P, P, P, I, I, I, I, P, P, P, P],
             "moe_ssd_scan": [P, LL, P, LL, P, P, P, P, LL, P, P, I, I, I, I, I, P, I, I, P, P, P],
             "moe_ssd_finish": [P, P, LL, P, F, P, I, I, I, P, I, P],
-            "moe_delta_prepare": [P, LL, I, I, P, I, P, LL, P, P, P, P, P, I, I, I, I, I, F, F, I, P, P, P],
-            "moe_delta_step": [P, P, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P],
-            "moe_delta_scan": [P, P, P, LL, P, P, I, I, I, I, I, P, P],
+            "moe_delta_prepare": [P, LL, I, I, P, I, P, LL, P, P, P, P, P, I, I, I, I, I, F, F, I, P, P, P, LL, P, P],
+            "moe_delta_step": [P, P, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P, I, P],
+            "moe_delta_scan": [P, P, P, LL, P, P, I, I, I, I, I, P, P, P],
+            "moe_mlstm_scan": [P, LL, I, I, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, P, P, P],
+            "moe_mlstm_step": [P, LL, I, I, I, I, I, P, P, F, F, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P],
+            "moe_post_norm": [P, P, F, P, F, P, P, P, I, P, P, F, P, F, P, P, P, I, I, I, I, P, P],
+            "moe_weighted_rows": [P, P, P, I, I, I, I, P, I, P, P],
         }
         for name, argtypes in sig.items():
             fn = getattr(L, name)
             fn.argtypes = argtypes
             fn.restype = c_int
+        L.moe_mlstm_state_floats.argtypes, L.moe_mlstm_state_floats.restype = [I, I, I], LL
         L.moe_router_scratch_floats.argtypes = [I, I, I, I]
         L.moe_router_scratch_floats.restype = LL
         L.moe_set_pdl.argtypes = [c_int]
@@ -364,17 +372,17 @@ def heads_prepare(proj, pos, seq_of_token, *, nh, nkv, d, dv, width, q, k, v, q_
         if freq.numel() < rot // 2:
             raise KernelError("heads_prepare: frequency table too short")
     kc = vc = se = sl = tb = None
-    ts = ring = ps = npg = 0
+    ts = ring = ps = npg = pin = 0
     if commit is not None:
         view, batch = commit
         g = view.group
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("heads_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, sl, tb = view.k, view.v, batch.seq_end, batch.slots, g.table
-        ts, ring, ps, npg = g.table.stride(0), g.ring, g.page_size, g.num_pages
+        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_heads_prepare(_p(proj), proj.stride(0), _p(pos), _p(seq_of_token), _p(q_norm), _p(k_norm), float(eps),
                                 _p(freq) if rot else None, int(rot), float(mscale), T, nh, nkv, d, dv, width, _p(q),
-                                _p(k), _p(v), q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(sl), _p(tb), ts, ring, ps, npg,
+                                _p(k), _p(v), q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(sl), _p(tb), ts, ring, ps, npg, pin,
                                 _p(status), _stream()), "heads_prepare")
 
 
@@ -539,18 +547,18 @@ def conv_heads_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, taps_w=No
         if freq.numel() < rot // 2:
             raise KernelError("conv_heads_prepare: frequency table too short")
     kc = vc = se = tb = None
-    ts = ring = ps = npg = 0
+    ts = ring = ps = npg = pin = 0
     if commit is not None:
         g = commit.group
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("conv_heads_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, tb = commit.k, commit.v, batch.seq_end, g.table
-        ts, ring, ps, npg = g.table.stride(0), g.ring, g.page_size, g.num_pages
+        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_conv_heads_prepare(_p(proj), proj.stride(0), _p(taps_w), taps, _p(state),
                                      state.stride(0) if state is not None else 0, _p(batch.pos), _p(batch.seq_of_token),
                                      _p(batch.cu_seqlens), _p(batch.slots), float(eps), 1 if unit_norm else 0,
                                      _p(freq) if rot else None, int(rot), T, nh, nkv, d, dv, width, _p(q), _p(k), _p(v),
-                                     q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(tb), ts, ring, ps, npg,
+                                     q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(tb), ts, ring, ps, npg, pin,
                                      _p(status), _stream()), "conv_heads_prepare")
 
 
@@ -558,11 +566,10 @@ def conv_state_update(proj, state, batch, *, taps, channels, offset=0):
     """state[slot] <- the last ``taps - 1`` rows of ``proj`` that each sequence of the step holds by now.
     ``proj``: float32 [T, >= channels] (a column slice is fine); the rows live from float ``offset`` on
     in a slot's row of ``state``."""
-    _chk(state, "state", torch.float32, 2)
     if (proj.dtype != torch.float32 or not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1
-            or proj.shape[1] < channels or offset + (taps - 1) * channels > state.shape[1]):
-        raise KernelError("conv_state_update: the rows must be float32 [T, >= channels] and fit the state")
-    _ok(lib().moe_conv_state_update(_p(proj), proj.stride(0), state.data_ptr() + 4 * int(offset), state.stride(0),
+            or proj.shape[1] < channels):
+        raise KernelError("conv_state_update: the rows must be float32 [T, >= channels]")
+    _ok(lib().moe_conv_state_update(_p(proj), proj.stride(0), _state_at(state, offset, (taps - 1) * channels), state.stride(0),
                                     int(taps), int(channels), _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs,
                                     _stream()), "conv_state_update")
 
@@ -642,14 +649,18 @@ def wkv_scan(r, k, v, w, u, state, batch, out, *, heads, d, segments=None):
                            _p(decays), _stream()), "wkv_scan")
 
 
-def wkv_finish(o, gate, norm_w, eps, batch, out, *, heads, d):
-    """out = o / rms(o over each head) * norm_w * silu(gate), rounded to ``out``'s dtype."""
+GATES = {"silu": 0, "sigmoid": 1}      # GATE_* in csrc/common.cuh
+
+
+def wkv_finish(o, gate, norm_w, eps, batch, out, *, heads, d, gate_fn="silu"):
+    """out = o / rms(o over each head) * norm_w * silu(gate) (``gate_fn`` "sigmoid": * sigmoid(gate)), rounded to
+    ``out``'s dtype."""
     _chk(o, "o", torch.float32, 2), _chk(norm_w, "norm weight", torch.float32, 1), _chk(out, "out", dims=2)
     T = o.shape[0]
     if gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * d) or out.shape != o.shape:
         raise KernelError("wkv_finish: shapes")
     _ok(lib().moe_wkv_finish(_p(o), _p(gate), gate.stride(0), _p(norm_w), float(eps), _p(batch.seq_of_token), T, heads, d,
-                             _p(out), _dt(out), _stream()), "wkv_finish")
+                             GATES[gate_fn], _p(out), _dt(out), _stream()), "wkv_finish")
 
 
 def rmsnorm_scaled(x, a, sa, b, sb, weight, eps, *, rows=None, out32=None, out16=None, write_back=True, status=None,
@@ -789,7 +800,7 @@ def kv_commit(k_new, v_new, view, batch, status):
         raise KernelError("kv_commit: cache dtype differs from the keys'")
     _ok(lib().moe_kv_commit(_p(k_new), _p(v_new), _p(view.k), _p(view.v), _dt(k_new), _p(batch.seq_of_token),
                             _p(batch.pos), _p(batch.seq_end), _p(batch.slots), _p(g.table), g.table.stride(0),
-                            g.ring, g.page_size, g.num_pages, T, g.num_kv_heads, g.head_dim, _p(status), _stream()),
+                            g.ring, g.page_size, g.num_pages, g.pinned, T, g.num_kv_heads, g.head_dim, _p(status), _stream()),
         "kv_commit")
 
 
@@ -804,25 +815,29 @@ class SigmoidWeights:
 ATTN_SIGMOID = 2     # AttnVariant.sink in csrc/common.cuh
 
 
-def _variant(chunk, softcap, sink):
-    """(chunk, softcap, sink, the sink's values per head) as the kernels take them: see AttnVariant in
+def _variant(chunk, softcap, sink, keep=0):
+    """(chunk, softcap, sink, the sink's values per head, keep) as the kernels take them: see AttnVariant in
     csrc/common.cuh.  ``sink``: False, True (a term of score 0), a float32 tensor with one number
-    per query head (the term's own score), or ``SigmoidWeights``."""
+    per query head (the term's own score), or ``SigmoidWeights``.  ``keep``: first positions that stay in
+    sight beside the window."""
+    if keep and chunk:
+        raise KernelError("attention: kept first positions go with a window, not with chunks")
     if isinstance(sink, SigmoidWeights):
         if sink.bias is not None:
             _chk(sink.bias, "head bias", torch.float32, 1)
-        return int(chunk or 0), float(softcap or 0.0), ATTN_SIGMOID, _p(sink.bias)
+        return int(chunk or 0), float(softcap or 0.0), ATTN_SIGMOID, _p(sink.bias), int(keep)
     if isinstance(sink, torch.Tensor):
         _chk(sink, "sink", torch.float32, 1)
-        return int(chunk or 0), float(softcap or 0.0), 1, sink.data_ptr()
-    return int(chunk or 0), float(softcap or 0.0), 1 if sink else 0, None
+        return int(chunk or 0), float(softcap or 0.0), 1, sink.data_ptr(), int(keep)
+    return int(chunk or 0), float(softcap or 0.0), 1 if sink else 0, None, int(keep)
 
 
 def attention_generic(q, k_new, v_new, view, batch, out, *, nh, window, scale, use_local, status, chunk=0,
-                      softcap=0.0, sink=False):
+                      softcap=0.0, sink=False, keep=0):
     """``chunk``: a position sees the keys of its own chunk of that many positions only (instead of a
     window); ``softcap``: scores pass cap * tanh(s / cap); ``sink``: the softmax's denominator has one
-    more term exp(0).  The same three options in every attention kernel."""
+    more term exp(0); ``keep``: with a window, that many first positions of the sequence stay in sight.
+    The same options in every attention kernel."""
     g = view.group
     T = batch.num_tokens
     if q.dtype != g.dtype or out.dtype != q.dtype:
@@ -831,12 +846,12 @@ def attention_generic(q, k_new, v_new, view, batch, out, *, nh, window, scale, u
                                     _p(batch.seq_of_token), _p(batch.pos), _p(batch.seq_start), _p(batch.cu_seqlens),
                                     _p(batch.slots), _p(g.table), g.table.stride(0), g.ring, g.page_size,
                                     g.num_pages, T, nh, g.num_kv_heads, g.head_dim, int(window or 0), float(scale),
-                                    1 if use_local else 0, _p(status), *_variant(chunk, softcap, sink), _stream()),
+                                    1 if use_local else 0, _p(status), *_variant(chunk, softcap, sink, keep), _stream()),
         "attention_generic")
 
 
 def attention_tiled(q, k_new, v_new, view, batch, out, *, nh, window, scale, use_local, status, chunk=0, softcap=0.0,
-                    sink=False) -> bool:
+                    sink=False, keep=0) -> bool:
     """The same as ``attention_generic`` with 64 queries of a (sequence, head) to a block and the
     keys staged through shared memory (32-bit arithmetic on the CUDA cores).  False, with nothing
     launched, for a layout it does not take (a page size other than 64, unaligned rows)."""
@@ -847,7 +862,7 @@ def attention_tiled(q, k_new, v_new, view, batch, out, *, nh, window, scale, use
                                      _p(batch.cu_seqlens), _p(batch.seq_start), _p(batch.slots), _p(g.table),
                                      g.table.stride(0), g.ring, g.page_size, g.num_pages, batch.num_seqs,
                                      batch.num_tokens, nh, g.num_kv_heads, g.head_dim, int(window or 0), float(scale),
-                                     1 if use_local else 0, _p(status), *_variant(chunk, softcap, sink), _stream())
+                                     1 if use_local else 0, _p(status), *_variant(chunk, softcap, sink, keep), _stream())
     if code == -1:
         return False
     _ok(code, "attention_tiled")
@@ -862,9 +877,17 @@ def _router_bias(bias, E):
     return bias
 
 
+def _route_flags(norm_topk, score):
+    """What the routing kernels take: whether the picked weights are renormalised, and how a logit becomes a
+    score ("softmax" over all experts, or each one's own "sigmoid")."""
+    if score not in ("softmax", "sigmoid"):
+        raise KernelError(f"router: score '{score}' is neither softmax nor sigmoid")
+    return (1 if norm_topk else 0) | (2 if score == "sigmoid" else 0)
+
+
 def router(h32, w_router, top_k, norm_topk, scale, topk_idx, topk_w, *, shared_gate_w=None, shared_gate=None,
-           seq_of_token=None, bias=None, groups=0, keep=0):
-    """``bias``: float32 [E], added to the logits before the softmax and the pick.  ``groups``, ``keep``:
+           seq_of_token=None, bias=None, groups=0, keep=0, score="softmax"):
+    """``score``: see ``_route_flags``.  ``bias``: float32 [E], added to the logits before the softmax and the pick.  ``groups``, ``keep``:
     the experts form ``groups`` equal groups of neighbours, and only experts of the ``keep`` groups
     whose best score is largest may be picked (0: no groups)."""
     _chk(h32, "h", torch.float32, 2), _chk(w_router, "router weight", dims=2)
@@ -884,7 +907,7 @@ def router(h32, w_router, top_k, norm_topk, scale, topk_idx, topk_w, *, shared_g
     need = lib().moe_router_scratch_floats(T, H, E, 1 if shared_gate_w is not None else 0)
     scratch = torch.empty((need,), dtype=torch.float32, device=h32.device) if need else None
     _ok(lib().moe_router(_p(h32), _p(w_router), _p(shared_gate_w), _dt(w_router), _p(seq_of_token), T, H, E, top_k,
-                         1 if norm_topk else 0, float(scale), _p(logits), _p(topk_idx), _p(topk_w), _p(shared_gate),
+                         _route_flags(norm_topk, score), float(scale), _p(logits), _p(topk_idx), _p(topk_w), _p(shared_gate),
                          _p(scratch), need, _p(_router_bias(bias, E)), int(groups), int(keep), _stream()), "router")
 
 
@@ -898,7 +921,7 @@ def split3(x32: torch.Tensor) -> torch.Tensor:
 
 
 def router_topk(logits, top_k, norm_topk, scale, topk_idx, topk_w, *, num_experts, shared_gate=None, seq_of_token=None,
-                bias=None, groups=0, keep=0):
+                bias=None, groups=0, keep=0, score="softmax"):
     """Picks and weights from logits [T, E (+ 1 row for the shared gate)] that are already there."""
     _chk(logits, "logits", torch.float32, 2)
     T = logits.shape[0]
@@ -906,7 +929,7 @@ def router_topk(logits, top_k, norm_topk, scale, topk_idx, topk_w, *, num_expert
     if logits.shape[1] not in (num_experts, num_experts + 1) or (gate_row and shared_gate is None):
         raise KernelError("router_topk: logits must have one column per expert (and one for the shared gate)")
     _ok(lib().moe_router_topk(_p(logits), _p(seq_of_token), T, num_experts, 1 if gate_row else 0, top_k,
-                              1 if norm_topk else 0, float(scale), _p(topk_idx), _p(topk_w), _p(shared_gate),
+                              _route_flags(norm_topk, score), float(scale), _p(topk_idx), _p(topk_w), _p(shared_gate),
                               _p(_router_bias(bias, num_experts)), int(groups), int(keep), _stream()),
         "router_topk")
 
@@ -967,7 +990,7 @@ def _gate_args(out, T, nh, hd, gate, dv, per_head=False):
 
 
 def attention_decode(q, view, batch, out, *, nh, window, scale, status, gate=None, dv=0, chunk=0, softcap=0.0,
-                     sink=False):
+                     sink=False, keep=0):
     """Attention of one new token per sequence over the cache alone (its own key already
     appended); split along the keys and merged.  With ``dv`` the merge writes [T, nh * dv], the
     first dv columns of every head, times sigmoid(``gate``) (a float32 column slice [T, nh * dv], or
@@ -983,7 +1006,7 @@ def attention_decode(q, view, batch, out, *, nh, window, scale, status, gate=Non
                                    _p(batch.seq_of_token), _p(batch.pos), _p(batch.slots), _p(g.table),
                                    g.table.stride(0), g.ring, g.page_size, g.num_pages, T, nh, g.num_kv_heads,
                                    g.head_dim, int(window or 0), float(scale), nsplit, gp, gld, gdv, _p(status),
-                                   *_variant(chunk, softcap, sink), _stream()),
+                                   *_variant(chunk, softcap, sink, keep), _stream()),
         "attention_decode")
 
 
@@ -1131,7 +1154,7 @@ def rope_commit(qkv, pos, inv_freq, nh, nkv, hd, rot, q, view, batch, status):
 
 
 def norm_route(x, delta, norm_w, eps, w_router, top_k, norm_topk, scale, *, bf16, shared_gate_w=None,
-               seq_of_token=None, status=None, groups=0, keep=0):
+               seq_of_token=None, status=None, groups=0, keep=0, score="softmax"):
     """Few tokens: ``x += delta``, RMS norm, router logits, pick, table inversion and gather of the
     normalised bfloat16 rows in ONE launch.  Returns None (nothing launched) for sizes the kernel
     does not take, else (out32 or None, out16 or None, topk_idx, topk_w, shared_gate, offsets,
@@ -1154,7 +1177,7 @@ def norm_route(x, delta, norm_w, eps, w_router, top_k, norm_topk, scale, *, bf16
     xs = torch.empty((P_, H), dtype=torch.bfloat16, device=dev) if bf16 and (H * 2) % 16 == 0 else None
     ticket = _tickets(dev, 1)
     code = lib().moe_norm_route(_p(x), _p(delta), _p(norm_w), float(eps), H, T, _p(out32), _p(out16), _p(w_router),
-                                _p(shared_gate_w), _dt(w_router), E, top_k, 1 if norm_topk else 0, float(scale),
+                                _p(shared_gate_w), _dt(w_router), E, top_k, _route_flags(norm_topk, score), float(scale),
                                 _p(seq_of_token), _p(topk_idx), _p(topk_w), _p(sg), _p(offsets), _p(sorted_token),
                                 _p(pos_of_pair), _p(xs), _p(ticket), _p(status), int(groups), int(keep), _stream())
     if code == -1:
@@ -1164,7 +1187,7 @@ def norm_route(x, delta, norm_w, eps, w_router, top_k, norm_topk, scale, *, bf16
 
 
 def route_dispatch(h32, w_router, top_k, norm_topk, scale, *, shared_gate_w=None, seq_of_token=None, gather=None,
-                   status=None, bias=None, groups=0, keep=0):
+                   status=None, bias=None, groups=0, keep=0, score="softmax"):
     """Few tokens (<= 64) and <= 256 experts: router logits, then pick + table inversion + gather in
     ONE more launch.  Returns (topk_idx, topk_w, shared_gate, offsets, sorted_token, pos_of_pair,
     gathered) where ``gathered[p] = gather[sorted_token[p]]`` (or None)."""
@@ -1192,7 +1215,7 @@ def route_dispatch(h32, w_router, top_k, norm_topk, scale, *, shared_gate_w=None
         else:
             xs = torch.empty((P_, gather.shape[1]), dtype=gather.dtype, device=dev)
     _ok(lib().moe_route_dispatch(_p(logits), _p(seq_of_token), T, E, 1 if shared_gate_w is not None else 0, top_k,
-                                 1 if norm_topk else 0, float(scale), _p(topk_idx), _p(topk_w), _p(sg), _p(offsets),
+                                 _route_flags(norm_topk, score), float(scale), _p(topk_idx), _p(topk_w), _p(sg), _p(offsets),
                                  _p(sorted_token), _p(pos_of_pair), _p(gather), _p(xs), row_bytes, _p(status),
                                  _p(_router_bias(bias, E)), int(groups), int(keep), _stream()), "route_dispatch")
     return topk_idx, topk_w, sg, offsets, sorted_token, pos_of_pair, xs
@@ -1228,17 +1251,70 @@ def whole_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, q_norm=None, k
         if dv % 2 or vfreq.numel() < dv // 2:
             raise KernelError("whole_prepare: rotated values need an even width and dv / 2 frequencies")
     kc = vc = se = sl = tb = None
-    ts = ring = ps = npg = 0
+    ts = ring = ps = npg = pin = 0
     if commit is not None:
         g = commit.group
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("whole_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, sl, tb = commit.k, commit.v, batch.seq_end, batch.slots, g.table
-        ts, ring, ps, npg = g.table.stride(0), g.ring, g.page_size, g.num_pages
+        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_whole_prepare(_p(proj), proj.stride(0), _p(batch.pos), _p(batch.seq_of_token), _p(q_norm), _p(k_norm),
                                 float(eps), _p(freq) if rot else None, int(rot), _p(vfreq), T, nh, nkv, d, dv, width,
                                 _p(q), _p(k), _p(v), q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(sl),
-                                _p(tb), ts, ring, ps, npg, _p(status), _stream()), "whole_prepare")
+                                _p(tb), ts, ring, ps, npg, pin, _p(status), _stream()), "whole_prepare")
+
+
+def whole_conv_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, taps_w=None, state=None, q_norm=None, k_norm=None,
+                       eps=0.0, freq=None, rot=0, neighbours=False, values_are_keys=False, commit=None, status=None) -> bool:
+    """``whole_prepare`` behind a short causal convolution: per channel of the 32-bit projection rows [q heads | k heads
+    (| v heads)] the sum of ``taps_w`` (float32 [taps, channels]; None: no convolution) times the last rows of the
+    sequence, which come from the step or from ``state`` ([slots + 1, >= (taps - 1) * channels]); then the norms over the
+    whole of q and of k, the rotation of the first ``rot`` dimensions of every query and key head (``neighbours``: of
+    pairs (2i, 2i + 1)), the split and optionally the append to the cache layer ``commit``.  ``values_are_keys``: the values
+    are the keys as they leave the convolution, and the projection has no rows for them.  Returns True if it has also
+    moved the convolution's state on (a step of one token a sequence); else the caller runs ``conv_state_update``."""
+    _chk(proj, "proj", torch.float32, 2)
+    T = proj.shape[0]
+    channels = (nh + nkv) * d + (0 if values_are_keys else nkv * dv)
+    for t, n in ((q, nh), (k, nkv), (v, nkv)):
+        if (not t.is_cuda or t.dtype != q.dtype or tuple(t.shape) != (T, n, width) or t.stride(2) != 1
+                or t.stride(1) != width or t.stride(0) < n * width):
+            raise KernelError("whole_conv_prepare: q, k, v must be [T, heads, width] with dense heads, of one dtype")
+    if k.stride(0) != v.stride(0) or proj.shape[1] < channels or (values_are_keys and dv != d):
+        raise KernelError("whole_conv_prepare: token pitch of keys and values, or projection width")
+    for w, n in ((q_norm, nh * d), (k_norm, nkv * d)):
+        if w is not None:
+            _chk(w, "norm weight", torch.float32, 1)
+            if w.numel() != n:
+                raise KernelError("whole_conv_prepare: a norm weight has one factor per channel of the projection")
+    taps, st, pitch = 1, None, 0
+    if taps_w is not None:
+        _chk(taps_w, "taps", torch.float32, 2)
+        taps = taps_w.shape[0]
+        if taps_w.shape[1] != channels:
+            raise KernelError("whole_conv_prepare: a tap has one factor per channel")
+        if taps > 1:
+            st, pitch = _state_at(state, 0, (taps - 1) * channels), state.stride(0)
+    if rot:
+        _chk(freq, "freq", torch.float32, 1)
+        if freq.numel() < rot // 2:
+            raise KernelError("whole_conv_prepare: frequency table too short")
+    kc = vc = se = tb = None
+    ts = ring = ps = npg = pin = 0
+    if commit is not None:
+        g = commit.group
+        if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
+            raise KernelError("whole_conv_prepare: the cache layer differs from the keys in dtype or shape")
+        kc, vc, se, tb = commit.k, commit.v, batch.seq_end, g.table
+        ts, ring, ps, npg, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
+    shift = bool(batch.all_decode and taps > 1)
+    _ok(lib().moe_whole_conv_prepare(_p(proj), proj.stride(0), _p(taps_w), taps, st, pitch, 1 if shift else 0, _p(batch.pos),
+                                     _p(batch.seq_of_token), _p(batch.cu_seqlens), _p(batch.slots), _p(q_norm), _p(k_norm),
+                                     float(eps), _p(freq) if rot else None, int(rot), 1 if neighbours else 0,
+                                     1 if values_are_keys else 0, T, nh, nkv, d, dv, width, _p(q), _p(k), _p(v), q.stride(0),
+                                     k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(tb), ts, ring, ps, npg, pin, _p(status),
+                                     _stream()), "whole_conv_prepare")
+    return shift or taps == 1
 
 
 def unrotate_pack(ctx, pos, vfreq, out, *, nh, dv, width):
@@ -1410,68 +1486,195 @@ def ssd_finish(y, z, norm_w, eps, batch, out, *, norm_groups):
                              int(norm_groups), _p(out), _dt(out), _stream()), "ssd_finish")
 
 
-def _delta_state(state, offset, floats):
+def _state_at(state, offset, floats):
     if not state.is_cuda or state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1:
-        raise KernelError("delta: the state must be float32 rows (a column slice is fine)")
+        raise KernelError("state: must be float32 rows (a column slice is fine)")
     if offset + floats > state.shape[1]:
-        raise KernelError("delta: the state's row is too short")
+        raise KernelError("state: its rows are too short")
     return state.data_ptr() + 4 * int(offset)
 
 
 def delta_prepare(proj, taps_w, a_log, dt_bias, state, batch, out, step, *, heads, kv_heads, d, dv, b_at, a_at, eps, q_scale,
-                  offset=0):
+                  offset=0, a_rows=None, decay=None):
     """From 32-bit projection rows [q (kv_heads x d) | k (kv_heads x d) | v (heads x dv) | ...] with the columns of b
     and a (one a value head) from ``b_at`` and ``a_at``: the causal convolution of q, k and v (``taps_w`` float32 [taps,
     channels]; earlier rows come from the step or from ``state``, whose rows hold (taps - 1) * channels floats from
     ``offset``) and silu; query and key heads divided by sqrt(sum(x^2) + eps), queries also times ``q_scale``, into ``out``
     float32 [T, channels]; sigmoid(b) and -exp(a_log) softplus(a + dt_bias) into ``step`` float32 [T, 2 heads].  In a step
-    of one token a sequence the convolution's state is moved on here; else the caller runs ``conv_state_update``."""
+    of one token a sequence the convolution's state is moved on here; else the caller runs ``conv_state_update``.
+
+    With ``decay`` (float32 [T, heads * d]) there is a decay a key channel: ``a_rows`` float32 [T, heads * d] (a column slice is
+    fine) holds a, ``dt_bias`` has an entry a channel, and exp(-exp(a_log) softplus(a + dt_bias)) goes into ``decay``."""
     _chk(proj, "proj", torch.float32, 2), _chk(taps_w, "taps", torch.float32, 2), _chk(out, "out", torch.float32, 2)
     _chk(a_log, "A_log", torch.float32, 1), _chk(dt_bias, "dt_bias", torch.float32, 1), _chk(step, "step", torch.float32, 2)
     T, channels, taps = proj.shape[0], 2 * kv_heads * d + heads * dv, taps_w.shape[0]
     if (taps_w.shape[1] != channels or tuple(out.shape) != (T, channels) or tuple(step.shape) != (T, 2 * heads)
-            or a_log.numel() != heads or dt_bias.numel() != heads or proj.shape[1] < max(channels, b_at + heads, a_at + heads)):
+            or a_log.numel() != heads or dt_bias.numel() != (heads if decay is None else heads * d)
+            or proj.shape[1] < max(channels, b_at + heads, a_at + heads if decay is None else 0)):
         raise KernelError("delta_prepare: shapes")
-    st = _delta_state(state, offset, (taps - 1) * channels) if taps > 1 else None
+    if decay is not None:
+        _chk(decay, "decay", torch.float32, 2)
+        if (tuple(decay.shape) != (T, heads * d) or a_rows is None or a_rows.dtype != torch.float32 or not a_rows.is_cuda
+                or a_rows.stride(1) != 1 or tuple(a_rows.shape) != (T, heads * d)):
+            raise KernelError("delta_prepare: the channels' decays")
+    st = _state_at(state, offset, (taps - 1) * channels) if taps > 1 else None
     _ok(lib().moe_delta_prepare(_p(proj), proj.stride(0), int(b_at), int(a_at), _p(taps_w), taps, st,
                                 state.stride(0) if taps > 1 else 0, _p(a_log), _p(dt_bias), _p(batch.seq_of_token),
                                 _p(batch.cu_seqlens), _p(batch.slots), T, heads, kv_heads, d, dv, float(eps), float(q_scale),
-                                1 if (batch.all_decode and taps > 1) else 0, _p(out), _p(step), _stream()), "delta_prepare")
+                                1 if (batch.all_decode and taps > 1) else 0, _p(out), _p(step),
+                                _p(a_rows) if decay is not None else None, a_rows.stride(0) if decay is not None else 0,
+                                _p(decay), _stream()), "delta_prepare")
 
 
-def _delta_chk(qkv, step, heads, kv_heads, d, dv):
+def _delta_chk(qkv, step, heads, kv_heads, d, dv, decay=None):
     _chk(qkv, "qkv", torch.float32, 2), _chk(step, "step", torch.float32, 2)
     T = qkv.shape[0]
+    if decay is not None:
+        _chk(decay, "decay", torch.float32, 2)
+        if tuple(decay.shape) != (T, heads * d):
+            raise KernelError("delta: the channels' decays")
     if qkv.shape[1] != 2 * kv_heads * d + heads * dv or tuple(step.shape) != (T, 2 * heads) or heads % kv_heads:
         raise KernelError("delta: shapes")
     return T
 
 
-def delta_step(qkv, step, state, gate, norm_w, norm_eps, batch, out, *, heads, kv_heads, d, dv, offset=0) -> bool:
-    """One token a sequence of the gated delta rule on what ``delta_prepare`` left, with the head norm (RMS, times
-    ``norm_w`` [heads * dv]) and silu(``gate``) behind it, into ``out`` [T, heads * dv]; ``state`` rows hold heads * d * dv
+def delta_step(qkv, step, state, gate, norm_w, norm_eps, batch, out, *, heads, kv_heads, d, dv, offset=0, decay=None,
+               gate_fn="silu") -> bool:
+    """One token a sequence of the gated delta rule on what ``delta_prepare`` left (``decay``: a decay a channel), with the
+    head norm (RMS, times ``norm_w`` [heads * dv]) and silu(``gate``), or its sigmoid, behind it, into ``out`` [T, heads * dv]; ``state`` rows hold heads * d * dv
     floats from ``offset``.  False, with nothing launched, for sizes the kernel does not take."""
-    T = _delta_chk(qkv, step, heads, kv_heads, d, dv)
+    T = _delta_chk(qkv, step, heads, kv_heads, d, dv, decay)
     _chk(norm_w, "norm weight", torch.float32, 1), _chk(out, "out", dims=2)
     if (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * dv)
             or tuple(out.shape) != (T, heads * dv) or norm_w.numel() != heads * dv):
         raise KernelError("delta_step: shapes")
-    code = lib().moe_delta_step(_p(qkv), _p(step), _delta_state(state, offset, heads * d * dv), state.stride(0), _p(gate),
+    code = lib().moe_delta_step(_p(qkv), _p(step), _state_at(state, offset, heads * d * dv), state.stride(0), _p(gate),
                                 gate.stride(0), _p(norm_w), float(norm_eps), _p(batch.seq_of_token), _p(batch.cu_seqlens),
-                                _p(batch.slots), T, batch.num_seqs, heads, kv_heads, d, dv, _p(out), _dt(out), _stream())
+                                _p(batch.slots), T, batch.num_seqs, heads, kv_heads, d, dv, _p(decay), GATES[gate_fn], _p(out), _dt(out),
+                                _stream())
     if code == -1:
         return False
     _ok(code, "delta_step")
     return True
 
 
-def delta_scan(qkv, step, state, batch, o, *, heads, kv_heads, d, dv, offset=0):
+def delta_scan(qkv, step, state, batch, o, *, heads, kv_heads, d, dv, offset=0, decay=None):
     """Per sequence and value head, tokens in order: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q, on
-    what ``delta_prepare`` left; o: float32 [T, heads * dv]."""
-    T = _delta_chk(qkv, step, heads, kv_heads, d, dv)
+    what ``delta_prepare`` left (``decay``: a decay a channel, each for its row of S); o: float32 [T, heads * dv]."""
+    T = _delta_chk(qkv, step, heads, kv_heads, d, dv, decay)
     _chk(o, "o", torch.float32, 2)
     if tuple(o.shape) != (T, heads * dv):
         raise KernelError("delta_scan: shapes")
-    _ok(lib().moe_delta_scan(_p(qkv), _p(step), _delta_state(state, offset, heads * d * dv), state.stride(0),
-                             _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs, heads, kv_heads, d, dv, _p(o), _stream()),
-        "delta_scan")
+    _ok(lib().moe_delta_scan(_p(qkv), _p(step), _state_at(state, offset, heads * d * dv), state.stride(0),
+                             _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs, heads, kv_heads, d, dv, _p(decay), _p(o),
+                             _stream()), "delta_scan")
+
+
+def mlstm_state_floats(heads, d, dv) -> int:
+    """Floats of a sequence's state (csrc/mlstm.cu): the memory, its normaliser (once for every 32 columns of the
+    memory) and the running maximum of every head."""
+    return heads * d * (dv + -(-dv // 32)) + heads
+
+
+def _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, heads, d, dv):
+    _chk(proj, "proj", torch.float32, 2), _chk(i_bias, "input gate bias", torch.float32, 1)
+    _chk(f_bias, "forget gate bias", torch.float32, 1)
+    need = {"q": heads * d, "k": heads * d, "v": heads * dv, "i": heads, "f": heads}
+    if any(at[n] < 0 or at[n] + w > proj.shape[1] for n, w in need.items()) or i_bias.numel() != heads or f_bias.numel() != heads:
+        raise KernelError("mlstm: the projection's columns or the gates' biases")
+    st = _state_at(state, offset, mlstm_state_floats(heads, d, dv))
+    return (_p(proj), proj.stride(0), at["q"], at["k"], at["v"], at["i"], at["f"], _p(i_bias), _p(f_bias), float(cap),
+            float(q_scale), st, state.stride(0))
+
+
+def mlstm_scan(proj, at, i_bias, f_bias, cap, q_scale, state, batch, o, *, heads, d, dv, offset=0):
+    """Several tokens a sequence of the exponentially gated memory (csrc/mlstm.cu) on 32-bit projection rows whose columns
+    of q, k, v and of the gates' logits i and f start at ``at``; queries are multiplied by ``q_scale``; ``state`` rows hold
+    ``mlstm_state_floats`` floats from ``offset``; o: float32 [T, heads * dv]."""
+    _chk(o, "o", torch.float32, 2)
+    T = proj.shape[0]
+    if tuple(o.shape) != (T, heads * dv):
+        raise KernelError("mlstm_scan: shapes")
+    args = _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, heads, d, dv)
+    steps = torch.empty((T, 3 * heads), dtype=torch.float32, device=o.device)
+    _ok(lib().moe_mlstm_scan(*args, _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs, heads, d, dv, _p(steps), _p(o),
+                             _stream()), "mlstm_scan")
+
+
+def mlstm_step(proj, at, i_bias, f_bias, cap, q_scale, state, gate, norm_w, norm_eps, batch, out, *, heads, d, dv, offset=0,
+               gate_fn="sigmoid") -> bool:
+    """The same for one token a sequence, with the head norm (RMS, times ``norm_w`` [heads * dv]) and the gate behind it,
+    into ``out`` [T, heads * dv].  False, with nothing launched, for sizes the kernel does not take."""
+    _chk(norm_w, "norm weight", torch.float32, 1), _chk(out, "out", dims=2)
+    T = proj.shape[0]
+    if (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, heads * dv)
+            or tuple(out.shape) != (T, heads * dv) or norm_w.numel() != heads * dv):
+        raise KernelError("mlstm_step: shapes")
+    args = _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, heads, d, dv)
+    code = lib().moe_mlstm_step(*args, _p(gate), gate.stride(0), _p(norm_w), float(norm_eps), _p(batch.seq_of_token),
+                                _p(batch.cu_seqlens), _p(batch.slots), T, batch.num_seqs, heads, d, dv, GATES[gate_fn], _p(out),
+                                _dt(out), _stream())
+    if code == -1:
+        return False
+    _ok(code, "mlstm_step")
+    return True
+
+
+def post_norm(x, *, a=None, sa=1.0, b=None, sb=1.0, combine=None, post=None, norm=None, rows=None, out32=None, out16=None,
+              write_back=True, status=None):
+    """x[r] += rms(y[r]) * post weight, y = a sa + b sb, or with ``combine`` = (e, pos_of_pair, weights or None, top_k,
+    shared or None) the sum of routed experts' outputs; ``post`` = (weight, eps).  The new row, or with ``norm`` =
+    (weight, eps) its RMS norm, goes to ``out32`` and / or ``out16`` (of the rows in ``rows``, if given: then x is left alone).
+    With neither a nor combine the row is only passed on (or normed)."""
+    _chk(x, "x", torch.float32, 2)
+    S, H = x.shape
+    n_out = S if rows is None else rows.numel()
+    for t in (a, b):
+        if t is not None:
+            _chk(t, "sublayer output", torch.float32, 2)
+            if t.shape != x.shape:
+                raise KernelError("post_norm: shapes")
+    e = pos = ew = shared = None
+    top_k = 0
+    if combine is not None:
+        e, pos, ew, top_k, shared = combine
+        _chk(e, "experts' outputs", torch.float32, 2), _chk(pos, "pos_of_pair", torch.int32)
+        if a is not None or e.shape[1] != H or pos.numel() < S * top_k:
+            raise KernelError("post_norm: the experts' outputs")
+        if ew is not None:
+            _chk(ew, "weights", torch.float32)
+            if ew.numel() < S * top_k:
+                raise KernelError("post_norm: the experts' weights")
+        if shared is not None:
+            _chk(shared, "shared", torch.float32, 2)
+            if shared.shape != x.shape:
+                raise KernelError("post_norm: the shared expert's output")
+    if (a is not None or combine is not None) != (post is not None) or (b is not None and a is None):
+        raise KernelError("post_norm: what is added has a norm of its own")
+    for w in (post, norm):
+        if w is not None:
+            _chk(w[0], "norm weight", torch.float32, 1)
+            if w[0].numel() != H:
+                raise KernelError("post_norm: a norm weight's size")
+    if rows is not None:
+        _chk(rows, "rows", torch.int32, 1)
+    for o, dt in ((out32, torch.float32), (out16, torch.bfloat16)):
+        if o is not None:
+            _chk(o, "out", dt, 2)
+            if o.shape[0] < n_out or o.shape[1] != H:
+                raise KernelError("post_norm: output shape")
+    _ok(lib().moe_post_norm(_p(x), _p(a), float(sa), _p(b), float(sb), _p(e), _p(pos), _p(ew), int(top_k), _p(shared),
+                            _p(post[0]) if post else None, float(post[1]) if post else 0.0, _p(norm[0]) if norm else None,
+                            float(norm[1]) if norm else 0.0, _p(rows), _p(out32), _p(out16), n_out, S, H,
+                            1 if (write_back and rows is None) else 0, _p(status), _stream()), "post_norm")
+
+
+def weighted_rows(x32, pos_of_pair, w, top_k, xs, status):
+    """xs[pos_of_pair[t, j]] = w[t, j] * x32[t] for every pick j of token t that has a place (rounded to ``xs``'s dtype)."""
+    _chk(x32, "x", torch.float32, 2), _chk(pos_of_pair, "pos_of_pair", torch.int32), _chk(w, "weights", torch.float32)
+    _chk(xs, "xs", dims=2)
+    T, H = x32.shape
+    if xs.shape[1] != H or pos_of_pair.numel() < T * top_k or w.numel() < T * top_k:
+        raise KernelError("weighted_rows: shapes")
+    _ok(lib().moe_weighted_rows(_p(x32), _p(pos_of_pair), _p(w), T, int(top_k), H, xs.shape[0], _p(xs), _dt(xs), _p(status),
+                                _stream()), "weighted_rows")

@@ -35,9 +35,9 @@ def lib():
 
         L.moe_attention_prefill_bf16.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P]
         L.moe_attention_prefill_bf16.restype = c_int
-        L.moe_attention_prefill_tc.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P, I, c_float, I, P, I, P, I, P]
+        L.moe_attention_prefill_tc.argtypes = [P, P, P, P, P, I, I, I, I, I, I, c_float, P, I, c_float, I, P, I, I, P, I, P]
         L.moe_attention_prefill_tc.restype = c_int
-        L.moe_attention_cached_tc.argtypes = [P] * 10 + [I] * 10 + [c_float, P, I, c_float, I, P, I, P, I, P]
+        L.moe_attention_cached_tc.argtypes = [P] * 10 + [I] * 10 + [c_float, P, I, c_float, I, P, I, I, P, I, P]
         L.moe_attention_cached_tc.restype = c_int
         L.moe_tc_set_pdl.argtypes = [c_int]
         L.moe_tc_set_pdl.restype = None
@@ -200,20 +200,20 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swiglu: bool
 
 
 def attention_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, batch, out: torch.Tensor, *, nh: int, nkv: int,
-                      hd: int, window, scale: float, status=None, chunk=0, softcap=0.0, sink=False, dv: int = 0,
+                      hd: int, window, scale: float, status=None, chunk=0, softcap=0.0, sink=False, keep=0, dv: int = 0,
                       gate=None) -> bool:
     """Causal (optionally windowed) attention of whole prompts on the tensor cores; every
     sequence of ``batch`` must start at position 0.  False if the head size is not taken.
     Head sizes 64 and 128 (and, where ``v`` is ``k``, 192 and 256) run on tcgen05
     (``attention_prefill_tc.cu``), 16 and 32 on mma.sync.
-    ``chunk``, ``softcap``, ``sink``: as in ``core.attention_generic``; ``dv``, ``gate``: ``out`` is [T, nh * dv],
+    ``chunk``, ``softcap``, ``sink``, ``keep``: as in ``core.attention_generic``; ``dv``, ``gate``: ``out`` is [T, nh * dv],
     the first dv columns (a multiple of 8) of every head, times sigmoid(``gate``) (a float32 column slice [T, nh])
     if given.  Only the tcgen05 kernel takes these."""
     wide = hd in (192, 256) and k.data_ptr() == v.data_ptr()
     if q.dtype != torch.bfloat16 or not (hd in (16, 32, 64, 128) or wide):
         return False
-    variant = core._variant(chunk, softcap, sink)
-    plain = variant == (0, 0.0, 0, None) and not dv and gate is None
+    variant = core._variant(chunk, softcap, sink, keep)
+    plain = variant == (0, 0.0, 0, None, 0) and not dv and gate is None
     on_tc = (hd in (64, 128) or wide) and status is not None and _ATTN_TC
     if not on_tc and (not plain or wide):
         return False
@@ -237,7 +237,7 @@ def attention_prefill(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, batch, 
 
 
 def attention_cached(q: torch.Tensor, k_new: torch.Tensor, v_new: torch.Tensor, view, batch, out: torch.Tensor, *,
-                     nh: int, window, scale: float, status, chunk=0, softcap=0.0, sink=False, dv: int = 0,
+                     nh: int, window, scale: float, status, chunk=0, softcap=0.0, sink=False, keep=0, dv: int = 0,
                      gate=None) -> bool:
     """Causal (optionally windowed) attention of a step whose sequences go on from the cache, on
     tcgen05: the keys before the step from the pages of ``view`` (one layer's cache), the step's own
@@ -253,7 +253,7 @@ def attention_cached(q: torch.Tensor, k_new: torch.Tensor, v_new: torch.Tensor, 
                                          batch.seq_start.data_ptr(), batch.slots.data_ptr(), g.table.data_ptr(),
                                          g.table.stride(0), g.ring, g.page_size, g.num_pages, batch.num_seqs,
                                          batch.num_tokens, nh, g.num_kv_heads, hd, int(window or 0), float(scale),
-                                         status.data_ptr(), *core._variant(chunk, softcap, sink),
+                                         status.data_ptr(), *core._variant(chunk, softcap, sink, keep),
                                          *_packed(out, batch.num_tokens, nh, hd, dv, gate), core._stream())
     if code == -1:
         return False

@@ -48,6 +48,14 @@ A third prepared path, whose kernel ``whole_prepare`` stands in the same place, 
               by its distance to the query;
   sigmoid     the weight of a visible key is sigmoid(score + b_h), b_h a learned number per head
               (tensor role ``head_bias``), and the weights are not normalised over the keys.
+
+With the norm over the whole projection (``qk_norm`` ``whole``), the convolution, a rotation of pairs (2i, 2i + 1) and
+  values_are_keys  the value of a position is its key as it leaves the convolution, before norm and rotation;
+              there is no value projection
+go together; the kernel is then ``whole_conv_prepare``.
+
+  keep_first  (with a window) the first n positions of the sequence stay in sight of every later one, at their
+              true positions; the cache pins their pages in front of the window's ring.
 """
 from __future__ import annotations
 
@@ -104,22 +112,33 @@ class GQAttention(Part):
         self.whole_norm = bool((self.qk_norm or {}).get("whole", False))
         self.rotate_values = bool(p.get("rotate_values", False))
         self.sigmoid = bool(p.get("sigmoid", False))
-        self.whole_path = self.whole_norm or self.rotate_values or self.sigmoid
+        self.values_are_keys = bool(p.get("values_are_keys", False))
+        self.keep_first = int(p.get("keep_first") or 0) if self.window is not None else 0
+        self.whole_path = self.whole_norm or self.rotate_values or self.sigmoid or self.values_are_keys
         pos = dict(p.get("position") or {"kind": "none"})
         self.position = make_part("position", PartSpec(pos.pop("kind"), pos, spec.prefix))
         # the prepared path: a kernel of its own between projection and attention, records of width D
         self.cos_sin_scale = float(getattr(self.position, "cos_sin_scale", lambda: 1.0)())
         self.prepared = bool(self.vd != self.hd or self.qk_norm or self.out_gate or self.hd % 16
                              or self.cos_sin_scale != 1.0)
-        self.conv_path = bool(self.taps or self.unit_norm or getattr(self.position, "interleaved", False))
-        self.variant = dict(chunk=self.chunk, softcap=self.softcap, sink=self.sink)
-        self.plain_scores = not (self.chunk or self.softcap or self.sink)    # what the fused decode kernel computes
+        self.neighbours = bool(getattr(self.position, "interleaved", False))
+        self.whole_conv = self.whole_path and bool(self.taps or self.neighbours or self.values_are_keys)
+        self.conv_path = bool(self.taps or self.unit_norm or self.neighbours) and not self.whole_path
+        self.variant = dict(chunk=self.chunk, softcap=self.softcap, sink=self.sink, keep=self.keep_first)
+        # what the fused decode kernel computes
+        self.plain_scores = not (self.chunk or self.softcap or self.sink or self.keep_first)
+        if self.keep_first < 0:
+            raise ValueError("keep_first must not be negative")
         if self.whole_path:
-            if (self.conv_path or self.out_gate or self.bias or self.sink or not self.own_kv or self.cos_sin_scale != 1.0
+            if self.whole_conv and self.rotate_values:
+                raise ValueError("rotated values go with neither a convolution, pairs (2i, 2i + 1) nor values that are the keys")
+            if self.values_are_keys and self.vd != self.hd:
+                raise ValueError(f"values that are the keys have their size: value_dim {self.vd}, head_dim {self.hd}")
+            if (self.unit_norm or self.out_gate or self.bias or self.sink or not self.own_kv or self.cos_sin_scale != 1.0
                     or (self.qk_norm and not self.whole_norm)):
-                raise ValueError("whole-projection norm, rotated values and sigmoid weights go with none of: convolution, "
-                                 "unit norm, pairs (2i, 2i + 1), output gate, biases, sink, another layer's cache, "
-                                 "scaled cos and sin, a per-head q/k norm")
+                raise ValueError("whole-projection norm, rotated values, sigmoid weights and values that are the keys go "
+                                 "with none of: unit norm, output gate, biases, sink, another layer's cache, scaled cos "
+                                 "and sin, a per-head q/k norm")
             if self.rotate_values and self.vd % 2:
                 raise ValueError("rotated values need an even value size")
             if not (0 < self.hd <= 256 and 0 < self.vd <= 256):
@@ -138,7 +157,7 @@ class GQAttention(Part):
             if not (0 < self.hd <= 256 and 0 < self.vd <= 256):
                 raise ValueError(f"head sizes {self.hd} / {self.vd}: the attention kernels take up to 256")
             self.prepared = False
-        elif (self.chunk or self.softcap or self.sink) and not self.prepared and not self.whole_path:
+        elif (self.chunk or self.softcap or self.sink or self.keep_first) and not self.prepared and not self.whole_path:
             self.prepared = True          # the path whose every step takes the kernels with these options
         if self.prepared:
             if not self.own_kv:
@@ -159,7 +178,8 @@ class GQAttention(Part):
         }
         if self.own_kv:
             t[n["k"]] = TensorSpec((self.nkv * self.hd, self.hidden))
-            t[n["v"]] = TensorSpec((self.nkv * self.vd, self.hidden))
+            if not self.values_are_keys:
+                t[n["v"]] = TensorSpec((self.nkv * self.vd, self.hidden))
         if self.bias:
             t[n["q_bias"]] = TensorSpec((self.nh * self.hd,), vector=True)
             if self.own_kv:
@@ -177,17 +197,18 @@ class GQAttention(Part):
         if self.taps:
             t[n["q_conv"]] = TensorSpec((self.nh * self.hd, self.taps))
             t[n["k_conv"]] = TensorSpec((self.nkv * self.hd, self.taps))
-            t[n["v_conv"]] = TensorSpec((self.nkv * self.vd, self.taps))
+            if not self.values_are_keys:
+                t[n["v_conv"]] = TensorSpec((self.nkv * self.vd, self.taps))
         t.update(self.position.tensors())
         return t
 
     def kv_request(self):
         # (chunks: no query looks further back than its chunk's start, so a ring of one chunk is enough)
-        return KVRequest(self.nkv, self.width, self.window if not self.chunk else self.chunk)
+        return KVRequest(self.nkv, self.width, self.window if not self.chunk else self.chunk, keep=self.keep_first)
 
     @property
     def channels(self):
-        return (self.nh + self.nkv) * self.hd + self.nkv * self.vd
+        return (self.nh + self.nkv) * self.hd + (0 if self.values_are_keys else self.nkv * self.vd)
 
     def describe(self):
         d = f"GQA({self.nh} q / {self.nkv} kv heads, head_dim={self.hd}{', bias' if self.bias else ''})"
@@ -202,7 +223,9 @@ class GQAttention(Part):
         if self.out_gate:
             d += ", sigmoid output gate"
         if self.taps:
-            d += f", convolution of {self.taps} taps on q, k, v"
+            d += f", convolution of {self.taps} taps on " + ("q, k" if self.values_are_keys else "q, k, v")
+        if self.values_are_keys:
+            d += ", values are the convolved keys"
         d += f", {self.position.describe()}"
         if self.unit_norm:
             d += ", q/k unit RMS after the rotation"
@@ -213,7 +236,7 @@ class GQAttention(Part):
         if self.chunk:
             d += f", chunks of {self.chunk}"
         if self.window:
-            d += f", window {self.window}"
+            d += f", window {self.window}" + (f" and the first {self.keep_first}" if self.keep_first else "")
         if not self.own_kv:
             d += ", reads another layer's cache"
         return d
@@ -230,7 +253,7 @@ class GQAttention(Part):
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
         n = self.names
-        roles = ["q", "k", "v"] if self.own_kv else ["q"]
+        roles = (["q", "k"] if self.values_are_keys else ["q", "k", "v"]) if self.own_kv else ["q"]
         ws = [tensors[n[r]] for r in roles]
         if self.out_gate:
             ws.append(tensors[n["gate"]])        # the gate's rows ride in the same product
@@ -247,7 +270,7 @@ class GQAttention(Part):
         self.taps_w = None
         if self.taps:
             # [taps, channels]: a tap's factors for all channels side by side
-            self.taps_w = torch.cat([tensors[n[r + "_conv"]].to(torch.float32) for r in ("q", "k", "v")], dim=0).t().contiguous()
+            self.taps_w = torch.cat([tensors[n[r + "_conv"]].to(torch.float32) for r in roles], dim=0).t().contiguous()
         self.q_norm_w = self.k_norm_w = None
         if self.qk_norm:
             self.q_norm_w = tensors[n["q_norm"]].to(torch.float32).contiguous()
@@ -328,8 +351,8 @@ class GQAttention(Part):
             core.conv_state_update(proj, state, batch, taps=self.taps, channels=self.channels)
         return self._attend_prepared(rt, batch, cache_view, q, k_new, v_new, ctx, None, early)
 
-    def _forward_whole(self, rt, h, batch, cache_view):
-        """Projection -> norm over the whole of q and of k, rotation of q and k, rotation of the values,
+    def _forward_whole(self, rt, h, batch, cache_view, state):
+        """Projection (-> convolution over time) -> norm over the whole of q and of k, rotation of q and k, rotation of the values,
         split and append -> attention over records of width D -> the output turned back and packed ->
         output projection."""
         T, D, nh, nkv = batch.num_tokens, self.width, self.nh, self.nkv
@@ -341,6 +364,15 @@ class GQAttention(Part):
         if getattr(batch, "has_padding", False) and not batch.all_decode:
             ctx.zero_()
         early = batch.all_decode or batch.all_fresh
+        if self.whole_conv:
+            moved = core.whole_conv_prepare(proj, batch, nh=nh, nkv=nkv, d=self.hd, dv=self.vd, width=D, q=q, k=k_new, v=v_new,
+                                            taps_w=self.taps_w, state=state, q_norm=self.q_norm_w, k_norm=self.k_norm_w,
+                                            eps=float(self.qk_norm["eps"]) if self.qk_norm else 0.0, freq=table, rot=rot,
+                                            neighbours=self.neighbours, values_are_keys=self.values_are_keys,
+                                            commit=cache_view if early else None, status=rt.status)
+            if not moved:
+                core.conv_state_update(proj, state, batch, taps=self.taps, channels=self.channels)
+            return self._attend_prepared(rt, batch, cache_view, q, k_new, v_new, ctx, None, early)
         core.whole_prepare(proj, batch, nh=nh, nkv=nkv, d=self.hd, dv=self.vd, width=D, q=q, k=k_new, v=v_new,
                            q_norm=self.q_norm_w, k_norm=self.k_norm_w, eps=float(self.qk_norm["eps"]) if self.qk_norm else 0.0,
                            freq=table, rot=rot, vfreq=self.vfreq, commit=cache_view if early else None, status=rt.status)
@@ -390,7 +422,7 @@ class GQAttention(Part):
         if self.conv_path:
             return self._forward_conv(rt, h, batch, cache_view, state)
         if self.whole_path:
-            return self._forward_whole(rt, h, batch, cache_view)
+            return self._forward_whole(rt, h, batch, cache_view, state)
         if self.prepared:
             return self._forward_prepared(rt, h, batch, cache_view)
         T = batch.num_tokens

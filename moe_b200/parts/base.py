@@ -12,6 +12,7 @@ Interfaces by category
   join      remember(rt, x0); forward(rt, x, pending) -> x: mixes the stream with the embedding output
   position  rotary_table() -> (inv_freq, rotary_dim) or None;  apply(rt, qkv32, layout, positions)
   mixer     forward(rt, h: Activations, batch, cache_view, state) -> delta [T, hidden] float32
+            optional: forward_lazy(the same) -> delta or LazyDelta
             kv_request() -> KVRequest | None;  state_request() -> StateRequest | None
   ffn       forward(rt, h: Activations, batch) -> delta [T, hidden] float32;  wants32: bool
             optional: forward_lazy(rt, h, batch) -> delta or LazyDelta;
@@ -45,14 +46,28 @@ class LazyDelta:
 class PostNormDelta(LazyDelta):
     """A sublayer's output that still has to pass a norm of its own before it joins the stream (a
     block with norms after its sublayers).  Its kind is ``"post_" + norm.kind``; a norm that names that
-    kind forms ``norm(tensor)`` inside its own kernel, in front of the residual sum."""
+    kind forms ``norm(tensor)`` inside its own kernel, in front of the residual sum.  ``tensor`` may itself be a
+    delta not computed yet where that norm's kernel takes it (``ScaledSumDelta``, routed experts' outputs)."""
 
     def __init__(self, tensor: torch.Tensor, norm):
         self.tensor, self.norm = tensor, norm
         self.kind = "post_" + norm.kind
 
     def materialize(self, rt) -> torch.Tensor:
-        return self.norm.normed32(rt, self.tensor)
+        t = self.tensor
+        return self.norm.normed32(rt, t.materialize(rt) if isinstance(t, LazyDelta) else t)
+
+
+class ScaledSumDelta(LazyDelta):
+    """a * sa + b * sb with two constant factors: the outputs of two mixers side by side."""
+
+    kind = "scaled_sum"
+
+    def __init__(self, a, sa: float, b, sb: float):
+        self.a, self.sa, self.b, self.sb = a, float(sa), b, float(sb)
+
+    def materialize(self, rt) -> torch.Tensor:
+        return (self.a * self.sa).add_(self.b, alpha=self.sb)
 
 
 class ScaledPairDelta(LazyDelta):

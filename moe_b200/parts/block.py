@@ -10,7 +10,8 @@ norm) may be absent: x += mixer(norm1(x)) is then the whole layer.
 "Sandwich": a norm before AND after each sublayer, and the feed-forward optional:
     x += post1(mixer(norm1(x)));  x += post2(ffn(norm2(x)))
 A sublayer's output is handed on together with its post-norm (``PostNormDelta``), so the next norm
-before a sublayer may form post-norm, residual sum and its own norm in one kernel.
+before a sublayer may form post-norm, residual sum and its own norm in one kernel.  With the part "none" as
+``norm1`` and ``norm2`` the sublayers read the stream itself: x += post1(mixer(x)); x += post2(ffn(x)).
 
 "Parallel": ONE norm, whose output both sublayers read, and one residual sum; each sublayer's output
 may be multiplied by a per-channel factor first, and the feed-forward is optional:
@@ -89,12 +90,16 @@ class SandwichBlock:
     def forward(self, rt, x, pending, batch, cache_view, state):
         h = self.norm1.forward(rt, x, delta=delta_for(self.norm1, pending, rt),
                                want32=getattr(self.mixer, "wants32", False))
-        pending = PostNormDelta(self.mixer.forward(rt, h, batch, cache_view, state), self.post1)
+        # (an output may come back unsummed or uncombined where the post-norm's kernel forms it)
+        run = getattr(self.mixer, "forward_lazy", self.mixer.forward) if self.post1.kind == "rmsnorm" else self.mixer.forward
+        pending = PostNormDelta(run(rt, h, batch, cache_view, state), self.post1)
         if self.ffn is None:
             return x, pending
+        run = getattr(self.ffn, "forward_lazy", self.ffn.forward) if self.post2.kind == "rmsnorm" else self.ffn.forward
+        kw = {"want16": getattr(self.ffn, "wants16", True)} if self.norm2.kind == "none" else {}
         h = self.norm2.forward(rt, x, delta=delta_for(self.norm2, pending, rt),
-                               want32=getattr(self.ffn, "wants32", False))
-        return x, PostNormDelta(self.ffn.forward(rt, h, batch), self.post2)
+                               want32=getattr(self.ffn, "wants32", False), **kw)
+        return x, PostNormDelta(run(rt, h, batch), self.post2)
 
 
 class ParallelBlock:

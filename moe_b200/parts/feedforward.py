@@ -125,6 +125,8 @@ class CombineDelta(LazyDelta):
     kind = "expert_combine"
 
     def __init__(self, y, pos_of_pair, topk_w, top_k, shared, shared_gate, tokens, hidden):
+        if topk_w is None:               # the weights are in the outputs already: a plain sum
+            self.kind = "expert_sum"
         self.y, self.pos_of_pair, self.topk_w, self.top_k = y, pos_of_pair, topk_w, top_k
         self.shared, self.shared_gate, self.tokens, self.hidden = shared, shared_gate, tokens, hidden
 
@@ -163,9 +165,18 @@ class RoutedExperts(Part):
         # one with weight 1 / top_k
         self.table = str(p.get("router", "softmax")) == "table"
         self.vocab = int(p.get("vocab_size", 0) or 0)
+        # how a logit becomes a score: "softmax" over all experts, or each one's own "sigmoid"
+        self.score = str(p.get("score", "softmax"))
+        # a pick's weight multiplies what the expert reads, not what it returns
+        self.weight_input = bool(p.get("weight_input", False))
+        if self.score not in ("softmax", "sigmoid"):
+            raise ValueError(f"router score '{self.score}' is neither softmax nor sigmoid")
+        if self.weight_input and self.shared_size:
+            raise ValueError("weights on the experts' input go with no shared expert")
+        self.wants16 = not self.weight_input       # (the rows the experts read are then made from the 32-bit input)
         if self.table and (self.vocab <= 0 or p.get("groups") or self.router_bias or p.get("shared_gate")):
             raise ValueError("routing by a table needs the vocabulary's size and takes no router options")
-        if self.table:
+        if self.table and not self.weight_input:
             self.wants32 = False
         # {"count": g, "keep": m}: the experts form g equal groups of neighbours, a group's score is its
         # best expert's, and only experts of the m best groups may be picked
@@ -175,7 +186,7 @@ class RoutedExperts(Part):
             self.groups = self.keep = 0                          # every group kept: no limit at all
         elif self.E % self.groups or self.keep < 1 or self.k > self.keep * (self.E // self.groups):
             raise ValueError("router groups: the count must divide the experts, and the kept groups must hold top_k experts")
-        self._grp = dict(groups=self.groups, keep=self.keep)
+        self._grp = dict(groups=self.groups, keep=self.keep, score=self.score)
         if not 0 < self.k <= self.E:
             raise ValueError("top_k must lie in 1..num_experts")
         # Set to a list to record every routing decision as (expert ids [T, k], weights [T, k]);
@@ -240,7 +251,8 @@ class RoutedExperts(Part):
 
     def describe(self):
         return (f"{self.E} experts of {self.size}, top-{self.k}, "
-                + ("named by a table over token ids, equal weights" if self.table else "softmax gate")
+                + ("named by a table over token ids, equal weights" if self.table else f"{self.score} gate")
+                + (", weights on the input" if self.weight_input else "")
                 + (" with bias" if self.router_bias else "")
                 + (f", within the best {self.keep} of {self.groups} groups" if self.groups else "")
                 + (", renormalised" if self.norm_topk else "")
@@ -360,7 +372,7 @@ class RoutedExperts(Part):
         tokens, norm, router and dispatch are one launch.  None if the sizes or the kind of norm do
         not allow it (the block then runs the norm itself and calls ``forward``)."""
         rms = getattr(norm, "rms_params", None)          # the norm says whether it can be run by a neighbour
-        if rms is None or x.shape[0] > self.fused_norm_tokens or self.E > 256 or self.b_router is not None or self.table:
+        if rms is None or x.shape[0] > self.fused_norm_tokens or self.E > 256 or self.b_router is not None or self.table or self.weight_input:
             return None
         norm_w, norm_eps = rms()
         routed = core.norm_route(x, delta, norm_w, norm_eps, self.w_router, self.k, self.norm_topk, self.scale,
@@ -392,7 +404,8 @@ class RoutedExperts(Part):
             topk_idx, topk_w, sg, offsets, sorted_token, pos_of_pair, xs = core.route_dispatch(
                 h.f32, self.w_router, self.k, self.norm_topk, self.scale, shared_gate_w=self.w_sgate,
                 seq_of_token=getattr(batch, "seq_of_token", None),
-                gather=h.act if h.act.dtype == torch.bfloat16 and T <= 16 else None, status=rt.status,
+                gather=h.act if h.act.dtype == torch.bfloat16 and T <= 16 and not self.weight_input else None,
+                status=rt.status,
                 bias=self.b_router, **self._grp)
             # (more tokens: the gather by that one block would take longer than a launch of its own)
         else:
@@ -417,6 +430,14 @@ class RoutedExperts(Part):
             xs = None
         if self.trace is not None:
             self.trace.append((topk_idx.clone(), topk_w.clone()))
+        if self.weight_input:
+            # what expert e reads for a token is w x: formed from the 32-bit row and rounded once, in expert order
+            if xs is None:
+                xs = rt.empty((P, self.hidden))
+                core.weighted_rows(h.f32, pos_of_pair, topk_w, self.k, xs, rt.status)
+            act = grouped_swiglu_linear(rt, xs, self.w_gu, offsets, None, P)
+            y = grouped_linear(rt, act, self.w_down, offsets, P, early_offsets=True)
+            return CombineDelta(y, pos_of_pair, None, self.k, None, None, T, self.hidden)
         act = grouped_swiglu_linear(rt, h.act, self.w_gu, offsets, sorted_token, P, gathered=xs)
         # (the offsets were written before the product above: the second product may start on its weights early)
         y = grouped_linear(rt, act, self.w_down, offsets, P, early_offsets=True)

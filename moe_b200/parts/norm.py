@@ -15,7 +15,8 @@ from .base import Activations, LazyDelta, Part, TensorSpec, register_part
 class RMSNorm(Part):
     category, kind = "norm", "rmsnorm"
     graph_safe = True
-    lazy_kinds = ("expert_combine", "scaled_pair")      # deltas this norm forms inside its own kernel
+    # deltas this norm forms inside its own kernel
+    lazy_kinds = ("expert_combine", "scaled_pair", "post_rmsnorm")
     default_names = {"weight": "weight"}
 
     def __init__(self, spec):
@@ -24,12 +25,16 @@ class RMSNorm(Part):
         self.eps = float(self.params["eps"])
         # a weight stored around zero: the factor is offset + w (the sum is formed once, in 32-bit, when bound)
         self.offset = float(self.params.get("offset", 0.0) or 0.0)
+        # a constant factor on the output, folded into the weight (a norm on a sublayer's output whose sum with the
+        # stream carries a factor)
+        self.scale = float(self.params.get("scale", 1.0))
 
     def tensors(self):
         return {self.names["weight"]: TensorSpec((self.size,), init="zeros" if self.offset else "ones", vector=True)}
 
     def describe(self):
-        return f"RMSNorm eps {self.eps:g}" + (f", weight {self.offset:g} + w" if self.offset else "")
+        return (f"RMSNorm eps {self.eps:g}" + (f", weight {self.offset:g} + w" if self.offset else "")
+                + (f", output x {self.scale:g}" if self.scale != 1.0 else ""))
 
     def rms_params(self):
         """(weight, eps): what a neighbour needs to run this norm inside a kernel of its own (a
@@ -42,6 +47,8 @@ class RMSNorm(Part):
         self.weight = tensors[self.names["weight"]].to(torch.float32).contiguous()
         if self.offset:
             self.weight = (self.weight + self.offset).contiguous()
+        if self.scale != 1.0:
+            self.weight = (self.weight * self.scale).contiguous()
 
     def normed32(self, rt, t):
         out = rt.empty(t.shape, torch.float32)
@@ -89,6 +96,9 @@ class RMSNorm(Part):
             core.rmsnorm_scaled(x, delta.a, delta.sa, b, delta.sb, self.weight, self.eps, rows=rows, out32=out32,
                                 out16=out16, write_back=write_back, status=rt.status, combine=combine)
             return Activations(act=out16 if rt.is_bf16 else out32, f32=out32)
+        if isinstance(delta, LazyDelta) and delta.kind == "post_rmsnorm":
+            post_norm(rt, x, delta, norm=(self.weight, self.eps), rows=rows, out32=out32, out16=out16, write_back=write_back)
+            return Activations(act=out16 if rt.is_bf16 else out32, f32=out32)
         if isinstance(delta, LazyDelta):
             if delta.kind != "expert_combine" or not core.rmsnorm_combine(
                     x, delta, self.weight, self.eps, rows=rows, out32=out32, out16=out16, write_back=write_back,
@@ -99,6 +109,58 @@ class RMSNorm(Part):
         core.rmsnorm(x, self.weight, self.eps, delta=delta, rows=rows, out32=out32, out16=out16,
                      write_back=write_back, status=rt.status)
         return Activations(act=out16 if rt.is_bf16 else out32, f32=out32)
+
+
+def post_norm(rt, x, delta, **kw):
+    """``core.post_norm`` of what a ``PostNormDelta`` of an RMS norm carries: a tensor, two mixers' outputs with a factor
+    each, or routed experts' outputs before their sum."""
+    t = delta.tensor
+    if isinstance(t, LazyDelta) and t.kind == "scaled_sum":
+        kw.update(a=t.a, sa=t.sa, b=t.b, sb=t.sb)
+    elif isinstance(t, LazyDelta) and t.kind in ("expert_combine", "expert_sum") and t.shared_gate is None:
+        kw.update(combine=(t.y, t.pos_of_pair, t.topk_w, t.top_k, t.shared))
+    else:
+        kw.update(a=t.materialize(rt) if isinstance(t, LazyDelta) else t)
+    core.post_norm(x, post=delta.norm.rms_params(), status=rt.status, **kw)
+
+
+class NoNorm(Part):
+    """A sublayer that reads the stream as it is: the place of a norm in front of it.  What is pending still joins the
+    stream here, with its own norm in the same kernel where it has one (``PostNormDelta``).  The 32-bit result is the
+    stream itself."""
+
+    category, kind = "norm", "none"
+    graph_safe = True
+    lazy_kinds = ("post_rmsnorm",)
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.size = int(self.params["size"])
+
+    def describe(self):
+        return "no norm"
+
+    def normed32(self, rt, t):
+        return t
+
+    def forward(self, rt, x, delta=None, rows=None, want32=False, write_back=True, want16=True) -> Activations:
+        """``want16``: False where nobody reads the rounded rows."""
+        n = x.shape[0] if rows is None else rows.numel()
+        own = rows is None and write_back                  # the stream itself is the 32-bit result
+        out16 = rt.empty((n, self.size), torch.bfloat16) if rt.is_bf16 and want16 else None
+        out32 = rt.empty((n, self.size), torch.float32) if not own and (want32 or not rt.is_bf16) else None
+        kw = dict(rows=rows, out32=out32, out16=out16, write_back=write_back)
+        if isinstance(delta, LazyDelta) and delta.kind == "post_rmsnorm":
+            post_norm(rt, x, delta, **kw)
+        else:
+            if delta is not None:
+                if not own:
+                    raise ValueError("no norm: a plain delta joins the whole stream")
+                core.add_inplace(x, delta.materialize(rt) if isinstance(delta, LazyDelta) else delta)
+            if out16 is not None or out32 is not None:
+                core.post_norm(x, status=rt.status, **kw)
+        f32 = x if own else out32
+        return Activations(act=out16 if rt.is_bf16 and want16 else f32, f32=f32)
 
 
 class LayerNorm(Part):
@@ -240,3 +302,4 @@ register_part("scale", "channel_scale", ChannelScale)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "layernorm", LayerNorm)
 register_part("norm", "dyt", DynamicTanh)
+register_part("norm", "none", NoNorm)

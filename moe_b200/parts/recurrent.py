@@ -25,7 +25,7 @@ import torch
 from ..cache.kv import StateRequest
 from ..ops import core
 from ..ops.linear import grouped_linear, linear
-from .base import Part, TensorSpec, register_part
+from .base import LazyDelta, Part, ScaledSumDelta, TensorSpec, register_part
 
 _STREAMS = ("r", "k", "v", "g", "w")
 
@@ -333,23 +333,192 @@ class DeltaMixer(Part):
         self.norm_w = tensors[n["norm"]].to(torch.float32).repeat(self.nh).contiguous()
         self.wo = tensors[n["o"]].contiguous()
 
+    gate_fn = "silu"
+
+    def _gates(self, rt, h, proj):
+        """(the output gate's logits, the channels' decay logits or None)"""
+        return proj[:, self.gate_at:self.gate_at + self.inner], None
+
     def forward(self, rt, h, batch, cache_view, state):
         T, C, I = batch.num_tokens, self.channels, self.inner
         proj = linear(rt, h.act, self.w_in)                       # float32 [T, q | k | v | gate | b | a]
+        gate, a_rows = self._gates(rt, h, proj)
+        decay = torch.empty((T, self.nh * self.d), dtype=torch.float32, device=proj.device) if a_rows is not None else None
         sizes = dict(heads=self.nh, kv_heads=self.nkv, d=self.d, dv=self.dv)
         qkv = torch.empty((T, C), dtype=torch.float32, device=proj.device)
         step = torch.empty((T, 2 * self.nh), dtype=torch.float32, device=proj.device)
         core.delta_prepare(proj, self.taps_w, self.a_log, self.dt_bias, state, batch, qkv, step, b_at=self.b_at,
-                           a_at=self.a_at, eps=self.UNIT_EPS, q_scale=self.d ** -0.5, **sizes)
+                           a_at=self.a_at, eps=self.UNIT_EPS, q_scale=self.d ** -0.5, a_rows=a_rows, decay=decay, **sizes)
         if self.taps > 1 and not batch.all_decode:
             core.conv_state_update(proj, state, batch, taps=self.taps, channels=C)
-        gate = proj[:, self.gate_at:self.gate_at + I]
         y = rt.empty((T, I))
-        at = dict(offset=self._state_at(), **sizes)
-        if not (batch.all_decode and core.delta_step(qkv, step, state, gate, self.norm_w, self.eps, batch, y, **at)):
+        at = dict(offset=self._state_at(), decay=decay, **sizes)
+        if not (batch.all_decode and core.delta_step(qkv, step, state, gate, self.norm_w, self.eps, batch, y,
+                                                     gate_fn=self.gate_fn, **at)):
             o = torch.empty((T, I), dtype=torch.float32, device=proj.device)
             core.delta_scan(qkv, step, state, batch, o, **at)
-            core.wkv_finish(o, gate, self.norm_w, self.eps, batch, y, heads=self.nh, d=self.dv)
+            core.wkv_finish(o, gate, self.norm_w, self.eps, batch, y, heads=self.nh, d=self.dv, gate_fn=self.gate_fn)
+        return linear(rt, y, self.wo)
+
+
+class ChannelDeltaMixer(DeltaMixer):
+    """The gated delta rule with one decay a value head AND key channel, and a sigmoid gate:
+
+        g = exp(-exp(A_log_h) softplus(Wa2 (Wa1 n) + dt_bias))          heads x d numbers, each for its row of S
+        out = Wo ((o / rms(o over each head)) * norm_weight * sigmoid(Wg2 (Wg1 n)))
+
+    and the rest as in ``DeltaMixer``.  The ranks of the two narrow projections come from the tensors' shapes.  Both pairs
+    are two products: [Wa1; Wg1] on n (whose result the bfloat16 path rounds, as the input of the next product), then Wa2
+    and Wg2 as the blocks of one block-diagonal matrix."""
+
+    kind = "channel_delta"
+    gate_fn = "sigmoid"
+    default_names = {"q": "q", "k": "k", "v": "v", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv", "b": "b",
+                     "a1": "a1", "a2": "a2", "g1": "g1", "g2": "g2", "a_log": "A_log", "dt_bias": "dt_bias", "norm": "norm",
+                     "o": "o"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.ranks = self.params.get("ranks")          # (decay's, gate's); None: read from the tensors' shapes when bound
+
+    def _tensors(self, ra, rg):
+        n, W = self.names, self.hidden
+        return {
+            n["q"]: TensorSpec((self.qk, W)), n["k"]: TensorSpec((self.qk, W)), n["v"]: TensorSpec((self.inner, W)),
+            n["q_conv"]: TensorSpec((self.qk, self.taps)), n["k_conv"]: TensorSpec((self.qk, self.taps)),
+            n["v_conv"]: TensorSpec((self.inner, self.taps)),
+            n["b"]: TensorSpec((self.nh, W)),
+            n["a1"]: TensorSpec((ra, W)), n["a2"]: TensorSpec((self.nh * self.d, ra)),
+            n["g1"]: TensorSpec((rg, W)), n["g2"]: TensorSpec((self.inner, rg)),
+            n["a_log"]: TensorSpec((self.nh,), init="zeros", vector=True),
+            n["dt_bias"]: TensorSpec((self.nh * self.d,), init="zeros", vector=True),
+            n["norm"]: TensorSpec((self.dv,), init="ones", vector=True),
+            n["o"]: TensorSpec((W, self.inner)),
+        }
+
+    def tensors(self):
+        return self._tensors(*(self.ranks or (16, 16)))
+
+    def tensors_in(self, has):
+        return self.tensors() if self.ranks else self._tensors(-1, -1)
+
+    def describe(self):
+        return super().describe().replace("gated delta rule", "gated delta rule with a decay a channel")
+
+    def bind(self, tensors, rt):
+        Part.bind(self, tensors, rt)
+        n = self.names
+        ws = [tensors[n[r]] for r in ("q", "k", "v", "b")]
+        dt = ws[0].dtype if all(w.dtype == ws[0].dtype for w in ws) else torch.float32
+        dev = ws[0].device
+        ws.append(torch.zeros((-sum(w.shape[0] for w in ws) % 8, self.hidden), dtype=dt, device=dev))
+        self.w_in = torch.cat([w.to(dt) for w in ws], dim=0).contiguous()
+        self.gate_at = self.a_at = 0                   # (the gate and the decays have a product of their own)
+        self.b_at = self.channels
+        a1, a2, g1, g2 = (tensors[n[r]] for r in ("a1", "a2", "g1", "g2"))
+        if a1.shape[0] != a2.shape[1] or g1.shape[0] != g2.shape[1]:
+            raise ValueError("channel_delta: a pair of narrow projections disagrees on its inner width")
+        ra, rg = int(a1.shape[0]), int(g1.shape[0])
+        self.ranks = (ra, rg)
+        wide = -(-(ra + rg) // 8) * 8
+        ldt = a1.dtype if a1.dtype == a2.dtype == g1.dtype == g2.dtype else torch.float32
+        self.w_low1 = torch.zeros((wide, self.hidden), dtype=ldt, device=dev)
+        self.w_low1[:ra], self.w_low1[ra:ra + rg] = a1.to(ldt), g1.to(ldt)
+        hd = self.nh * self.d
+        self.w_low2 = torch.zeros((hd + self.inner, wide), dtype=ldt, device=dev)
+        self.w_low2[:hd, :ra], self.w_low2[hd:, ra:ra + rg] = a2.to(ldt), g2.to(ldt)
+        self.taps_w = torch.cat([tensors[n[r + "_conv"]].to(torch.float32) for r in ("q", "k", "v")], dim=0).t().contiguous()
+        self.a_log = tensors[n["a_log"]].to(torch.float32).contiguous()
+        self.dt_bias = tensors[n["dt_bias"]].to(torch.float32).contiguous()
+        self.norm_w = tensors[n["norm"]].to(torch.float32).repeat(self.nh).contiguous()
+        self.wo = tensors[n["o"]].contiguous()
+
+    def _gates(self, rt, h, proj):
+        low = linear(rt, h.act, self.w_low1, out_dtype=rt.compute_dtype)
+        both = linear(rt, low, self.w_low2)                       # float32 [T, decays' logits | gate's logits]
+        hd = self.nh * self.d
+        return both[:, hd:], both[:, :hd]
+
+
+class MLSTMMixer(Part):
+    """An exponentially gated matrix memory (mLSTM).
+
+    With n_t the layer's input and H heads, keys of d and values of dv:
+        q = Wq n * d^(-1/2),  k = Wk n,  v = Wv n
+        i = cap tanh((Wi n + bi) / cap),  f = logsigmoid(cap tanh((Wf n + bf) / cap))           log gates, one a head
+    per head, with S [d, dv], z [d] and a running maximum m, all zero at the start:
+        m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T,  z likewise with k alone;  m <- m'
+        o = S^T q / (max(|z . q|, e^(-m)) + 1e-6)
+    and out = Wo ((o / rms(o over each head)) * norm_weight * sigmoid(Wg n)), a norm weight of all heads' size.
+
+    What a sequence carries is of fixed size, 32-bit: S, z (as often as csrc/mlstm.cu asks for) and m of every head.
+    Everything but the projections is 32-bit arithmetic in both dtypes.  A step of one token a sequence is one product,
+    ``mlstm_step`` (gates, recurrence, head norm and gate) and one product."""
+
+    category, kind = "mixer", "mlstm"
+    graph_safe = True
+    default_names = {"q": "q", "k": "k", "v": "v", "gate": "g", "i": "i", "i_bias": "i.b", "f": "f", "f_bias": "f.b",
+                     "norm": "norm", "o": "o"}
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.hidden = int(p["hidden_size"])
+        self.nh, self.d, self.dv = int(p["num_heads"]), int(p["head_dim"]), int(p["value_dim"])
+        self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
+        if not (0 < self.d <= 256 and self.dv > 0 and self.nh > 0 and self.cap > 0):
+            raise ValueError(f"mlstm: heads of {self.d}, gate cap {self.cap}; the kernels take keys of up to 256, a positive cap")
+        self.inner = self.nh * self.dv
+
+    def tensors(self):
+        n, W, K = self.names, self.hidden, self.nh * self.d
+        return {
+            n["q"]: TensorSpec((K, W)), n["k"]: TensorSpec((K, W)), n["v"]: TensorSpec((self.inner, W)),
+            n["gate"]: TensorSpec((self.inner, W)),
+            n["i"]: TensorSpec((self.nh, W)), n["i_bias"]: TensorSpec((self.nh,), init="zeros", vector=True),
+            n["f"]: TensorSpec((self.nh, W)), n["f_bias"]: TensorSpec((self.nh,), init="zeros", vector=True),
+            n["norm"]: TensorSpec((self.inner,), init="ones", vector=True),
+            n["o"]: TensorSpec((W, self.inner)),
+        }
+
+    def describe(self):
+        return (f"mLSTM ({self.nh} heads, keys of {self.d}, values of {self.dv}, state {self.d}x{self.dv} a head, log gates capped "
+                f"at {self.cap:g})")
+
+    def kv_request(self):
+        return None
+
+    def state_request(self):
+        return StateRequest((core.mlstm_state_floats(self.nh, self.d, self.dv),), torch.float32)
+
+    def bind(self, tensors, rt):
+        super().bind(tensors, rt)
+        n = self.names
+        roles = ("q", "k", "v", "gate", "i", "f")
+        ws = [tensors[n[r]] for r in roles]
+        dt = ws[0].dtype if all(w.dtype == ws[0].dtype for w in ws) else torch.float32
+        self.at, rows = {}, 0
+        for r, w in zip(roles, ws):
+            self.at[r] = rows
+            rows += w.shape[0]
+        ws.append(torch.zeros((-rows % 8, self.hidden), dtype=dt, device=ws[0].device))
+        self.w_in = torch.cat([w.to(dt) for w in ws], dim=0).contiguous()
+        self.i_bias = tensors[n["i_bias"]].to(torch.float32).contiguous()
+        self.f_bias = tensors[n["f_bias"]].to(torch.float32).contiguous()
+        self.norm_w = tensors[n["norm"]].to(torch.float32).contiguous()
+        self.wo = tensors[n["o"]].contiguous()
+
+    def forward(self, rt, h, batch, cache_view, state):
+        T, I = batch.num_tokens, self.inner
+        proj = linear(rt, h.act, self.w_in)                       # float32 [T, q | k | v | gate | i | f]
+        gate = proj[:, self.at["gate"]:self.at["gate"] + I]
+        args = (proj, self.at, self.i_bias, self.f_bias, self.cap, self.d ** -0.5, state)
+        sizes = dict(heads=self.nh, d=self.d, dv=self.dv)
+        y = rt.empty((T, I))
+        if not (batch.all_decode and core.mlstm_step(*args, gate, self.norm_w, self.eps, batch, y, **sizes)):
+            o = torch.empty((T, I), dtype=torch.float32, device=proj.device)
+            core.mlstm_scan(*args, batch, o, **sizes)
+            core.wkv_finish(o, gate, self.norm_w, self.eps, batch, y, heads=self.nh, d=self.dv, gate_fn="sigmoid")
         return linear(rt, y, self.wo)
 
 
@@ -382,7 +551,8 @@ class SideBySideMixer(Part):
     a weight of its own, and the result is half their sum:
         out = (rmsnorm(left(n)) * w_left + rmsnorm(right(n)) * w_right) / 2
     ``left`` and ``right`` are mixers of any registered kind ({"kind", "params"}); their tensors live
-    under ``left.`` / ``right.``.  At most one of them may keep keys and values in pages; state of fixed
+    under ``left.`` / ``right.``.  With ``scales`` = (sl, sr) there are no norms: out = left(n) sl + right(n) sr, handed on
+    unsummed by ``forward_lazy`` (``ScaledSumDelta``).  At most one of them may keep keys and values in pages; state of fixed
     size of both lies side by side in one row a sequence."""
 
     category, kind = "mixer", "side_by_side"
@@ -395,7 +565,8 @@ class SideBySideMixer(Part):
         super().__init__(spec)
         p = self.params
         self.hidden = int(p["hidden_size"])
-        self.eps = float(p["eps"])
+        self.scales = p.get("scales")
+        self.eps = float(p["eps"]) if self.scales is None else 0.0
         self.subs = []
         for side in ("left", "right"):
             sub = p[side]
@@ -414,6 +585,8 @@ class SideBySideMixer(Part):
             for local, ts in fn(m, prefix).items():
                 t[prefix + local] = ts
         n = self.names
+        if self.scales is not None:
+            return t
         t[n["left_out"]] = TensorSpec((self.hidden,), init="ones", vector=True)
         t[n["right_out"]] = TensorSpec((self.hidden,), init="ones", vector=True)
         return t
@@ -425,10 +598,12 @@ class SideBySideMixer(Part):
         return self._sub_tensors(lambda m, prefix: m.tensors_in(lambda local: has(prefix + local)))
 
     def describe(self):
-        return "half the sum of two normed mixers: " + " | ".join(m.describe() for _, m in self.subs)
+        how = ("half the sum of two normed mixers: " if self.scales is None
+               else f"two mixers, {self.scales[0]:g} left + {self.scales[1]:g} right: ")
+        return how + " | ".join(m.describe() for _, m in self.subs)
 
     def step_elements(self, num_tokens):
-        return float(sum(m.step_elements(num_tokens) for _, m in self.subs) + 2 * self.hidden)
+        return float(sum(m.step_elements(num_tokens) for _, m in self.subs) + (2 * self.hidden if self.scales is None else 0))
 
     def kv_request(self):
         for _, m in self.subs:
@@ -445,25 +620,35 @@ class SideBySideMixer(Part):
             if r is not None:
                 if r.dtype != torch.float32 or len(r.shape) != 1:
                     raise ValueError("side_by_side: the mixers' state must be rows of 32-bit floats")
-                n += r.shape[0]
+                n += self._room(r)
         return StateRequest((n,), torch.float32)
+
+    @staticmethod
+    def _room(r) -> int:
+        return -(-r.shape[0] // 4) * 4              # (rows of whole 16-byte units)
 
     def bind(self, tensors, rt):
         super().bind(tensors, rt)
         for prefix, m in self.subs:
             names = [k[len(prefix):] for k in tensors if k.startswith(prefix) and k not in self.names.values()]
             m.bind(_SubTensors(tensors, prefix, names), rt)
+        if self.scales is not None:
+            return
         self.w_left = tensors[self.names["left_out"]].to(torch.float32).contiguous()
         self.w_right = tensors[self.names["right_out"]].to(torch.float32).contiguous()
 
     def forward(self, rt, h, batch, cache_view, state):
+        out = self.forward_lazy(rt, h, batch, cache_view, state)
+        return out.materialize(rt) if isinstance(out, LazyDelta) else out
+
+    def forward_lazy(self, rt, h, batch, cache_view, state):
         """The right mixer runs on a second stream beside the left one (inside a captured step: a fork
         and a join); MOE_B200_SIDE_BY_SIDE_STREAMS=0 runs them one after the other."""
         states, at = [], 0
         for _, m in self.subs:
             r = m.state_request()
             states.append(state[:, at:at + r.shape[0]] if r is not None else None)
-            at += r.shape[0] if r is not None else 0
+            at += self._room(r) if r is not None else 0
         views = [cache_view if m.kv_request() is not None else None for _, m in self.subs]
         (_, left), (_, right) = self.subs
         if self.beside and h.act.is_cuda:
@@ -478,6 +663,8 @@ class SideBySideMixer(Part):
         else:
             a = left.forward(rt, h, batch, views[0], states[0])
             b = right.forward(rt, h, batch, views[1], states[1])
+        if self.scales is not None:
+            return ScaledSumDelta(a, self.scales[0], b, self.scales[1])
         out = torch.empty_like(a)
         core.pair_norm_mean(a, self.w_left, b, self.w_right, self.eps, out)
         return out
@@ -485,4 +672,6 @@ class SideBySideMixer(Part):
 
 register_part("mixer", "ssd", SSDMixer)
 register_part("mixer", "delta", DeltaMixer)
+register_part("mixer", "channel_delta", ChannelDeltaMixer)
+register_part("mixer", "mlstm", MLSTMMixer)
 register_part("mixer", "side_by_side", SideBySideMixer)

@@ -104,6 +104,47 @@ class YarnRotary(RotaryEncoding):
         return 0.1 * math.log(self.factor) + 1.0
 
 
+class BandScaledRotary(RotaryEncoding):
+    """Rotary encoding whose frequencies are scaled by bands of wavelength l = 2 pi / f against an original context
+    length: l < original / high keeps f, l > original / low turns at f / factor, and between the two, with
+    s = (original / l - low) / (high - low), at (1 - s) f / factor + s f.  cos and sin carry no factor.  The table is
+    formed in float64 and rounded to float32 once."""
+
+    kind = "rotary_bands"
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        p = self.params
+        self.factor, self.original = float(p["factor"]), float(p["original"])
+        self.low, self.high = float(p["low"]), float(p["high"])
+        if min(self.factor, self.original, self.low, self.high) <= 0 or self.theta <= 0 or self.high < self.low:
+            raise ValueError("rotary_bands: factor, original, low and high must be positive, and low at most high")
+
+    def frequencies(self) -> torch.Tensor:
+        out = []
+        for i in range(self.rotary_dim // 2):
+            f = self.theta ** (-2.0 * i / self.rotary_dim)
+            length = 2.0 * math.pi / f
+            if length < self.original / self.high:
+                out.append(f)
+            elif length > self.original / self.low:
+                out.append(f / self.factor)
+            elif self.high == self.low:
+                out.append(f)
+            else:
+                s = (self.original / length - self.low) / (self.high - self.low)
+                out.append((1.0 - s) * f / self.factor + s * f)
+        return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+
+    def bind(self, tensors, rt):
+        Part.bind(self, tensors, rt)
+        self.inv_freq = self.frequencies().to(rt.device)
+
+    def describe(self):
+        return (f"rope theta {self.theta:.0f} on {self.rotary_dim} dims, bands {self.low:g} - {self.high:g} of {self.original:g} "
+                f"x{self.factor:g}" + (", pairs (2i, 2i+1)" if self.interleaved else ""))
+
+
 class NoPositionEncoding(Part):
     category, kind = "position", "none"
 
@@ -122,4 +163,5 @@ class NoPositionEncoding(Part):
 
 register_part("position", "rotary", RotaryEncoding)
 register_part("position", "rotary_yarn", YarnRotary)
+register_part("position", "rotary_bands", BandScaledRotary)
 register_part("position", "none", NoPositionEncoding)
