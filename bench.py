@@ -1609,6 +1609,212 @@ def run_ditazen(args):
     return 0
 
 
+# Kulanex at sizes that resemble a real model's layers, and beside each the library's closest model at equal
+# size: Divadra with as many layers, parallel layers (attention of the same heads in chunks of the window's size beside
+# a recurrent mixer with a state of the same size) where Kulanex has them, state-space layers with as many heads, values
+# and state rows where it has delta layers, and as many experts of the same size, of which a token takes as many.
+KULANEX_SHAPES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, window=1024, keep=16, rot=64, taps=4, m_heads=16, m_dim=64, m_vdim=128,
+                  cap=15.0, d_heads=16, d_kv=16, d_dim=128, d_vdim=128, conv=4, rank=128, experts=16, top=2, expert_ff=1408,
+                  order=("channel_delta", "parallel", "channel_delta", "parallel"), vocab=32768),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, window=2048, keep=16, rot=64, taps=4, m_heads=16, m_dim=128, m_vdim=256,
+                  cap=15.0, d_heads=32, d_kv=32, d_dim=128, d_vdim=128, conv=4, rank=128, experts=16, top=2, expert_ff=1408,
+                  order=("channel_delta", "parallel"), vocab=32768),
+}
+
+
+def kulanex_config(sh):
+    par = {"left": {"heads": sh["heads"], "kv_heads": sh["kv_heads"], "dim": sh["dim"], "vdim": sh["dim"], "conv": sh["taps"],
+                    "scale": sh["dim"] ** -0.5, "mask": {"size": sh["window"], "keep_first": sh["keep"]},
+                    "rot": {"dims": sh["rot"], "base": 1e6, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}},
+           "right": {"heads": sh["m_heads"], "dim": sh["m_dim"], "vdim": sh["m_vdim"], "gate_cap": sh["cap"]},
+           "left_scale": 0.5, "right_scale": 0.5}
+    delta = {"heads": sh["d_heads"], "kv_heads": sh["d_kv"], "dim": sh["d_dim"], "vdim": sh["d_vdim"], "conv": sh["conv"]}
+    moe = {"kind": "moe", "router": {"experts": sh["experts"], "top": sh["top"]}, "expert": {"ff": sh["expert_ff"]}}
+    return {"architecture": "Kulanex", "vocab": sh["vocab"], "width": sh["width"], "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "layers": [{"type": t, "mixer": par if t == "parallel" else delta, "mlp": moe} for t in sh["order"]]}
+
+
+def kulanex_divadra_config(sh):
+    left = {"heads": sh["heads"], "kv_heads": sh["kv_heads"], "dim": sh["dim"], "vdim": sh["dim"], "scale": sh["dim"] ** -0.5,
+            "mask": {"size": sh["window"]}, "rot": {"dims": sh["rot"], "base": 1e6}}
+    # (a recurrent state of dim x dim a head, as many numbers in all as the memory's dim x vdim)
+    wd = 128
+    par = {"left": left, "right": {"heads": sh["m_heads"] * sh["m_dim"] * sh["m_vdim"] // (wd * wd), "dim": wd}}
+    ssd = {"heads": sh["d_heads"], "vdim": sh["d_vdim"], "state": sh["d_dim"], "groups": sh["d_kv"], "norm_groups": sh["d_heads"],
+           "conv": sh["conv"]}
+    moe = {"kind": "moe", "router": {"experts": sh["experts"], "top": sh["top"]}, "expert": {"ff": sh["expert_ff"]}}
+    return {"architecture": "Divadra", "vocab": sh["vocab"], "width": sh["width"], "norm": {"eps": 1e-5}, "canon": {"taps": sh["taps"]},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 40503, "mul_cur": 65599}},
+            "layers": [{"type": t, "mixer": par, "mlp": moe} if t == "parallel" else {"type": "mamba2", "mixer": ssd, "mlp": moe}
+                       for t in sh["order"]]}
+
+
+def kulanex_kernels(sh, pk):
+    """The new design's own kernels beside the like kernels of the library's other models, each alone at 8,192
+    tokens of 4 sequences (what a call reads and writes exceeds L2), as fractions of the measured copy bandwidth
+    (attention and recurrences: of the measured bf16 peak, counting the products the mechanism needs); then one token of
+    64 sequences (the attention at a context of 2,048; replayed from a CUDA graph where a kernel is shorter than the
+    host's work to launch it)."""
+    import torch
+
+    from moe_b200.cache.kv import KVCache, KVRequest
+    from moe_b200.ops import core, tc
+
+    sys.path.insert(0, os.path.join(ROOT, "tests"))
+    import gpu_util as G
+
+    dev, bf = "cuda:0", torch.bfloat16
+    B, n = 4, 2048
+    T, W = B * n, sh["width"]
+    H, kv, d, rot, taps, win, keep = (sh[k] for k in ("heads", "kv_heads", "dim", "rot", "taps", "window", "keep"))
+    status = core.new_status(dev)
+    r = lambda *s: torch.randn(*s, device=dev)
+    out = {}
+
+    def row(name, ms, nbytes=None, flops=None):
+        e = {"us": round(ms * 1e3, 1)}
+        if nbytes:
+            e["of_copy_peak"] = round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3)
+        if flops:
+            e["tflops"] = round(flops / ms / 1e9, 1)
+            e["of_bf16_peak"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 4)
+        out[name] = e
+
+    batch = G.make_batch(dev, list(range(1, B + 1)), [0] * B, [n] * B)
+    b1 = G.make_batch(dev, [1], [0], [n])
+    one = G.make_batch(dev, list(range(1, 65)), [n] * 64, [1] * 64)
+    # ---- norms with the residual sum --------------------------------------------------------------------
+    x, a, b, w = r(T, W), r(T, W) / 100, r(T, W) / 100, r(W)
+    o16 = torch.empty((T, W), dtype=bf, device=dev)
+    nb = T * W * (4 + 4 + 4 + 2)
+    row("post_norm (norm of an output + sum)", _median_ms(lambda: core.post_norm(x, a=a, post=(w, 1e-5), out16=o16, status=status)), nb)
+    row("post_norm (two outputs)", _median_ms(lambda: core.post_norm(x, a=a, sa=0.5, b=b, sb=0.5, post=(w, 1e-5), out16=o16, status=status)),
+        nb + 4 * T * W)
+    top = sh["top"]
+    e_, pos = r(T * top, W) / 100, torch.randperm(T * top, device=dev).to(torch.int32)
+    tw_ = torch.rand(T * top, device=dev)
+    row("post_norm (experts' outputs)", _median_ms(lambda: core.post_norm(x, combine=(e_, pos, None, top, None), post=(w, 1e-5), out16=o16,
+                                                                         status=status)), nb + 4 * T * W * (top - 1))
+    row("like: rmsnorm_scaled (two outputs + sum + norm)", _median_ms(lambda: core.rmsnorm_scaled(
+        x, a, w, b, w, w, 1e-5, out16=o16, status=status)), nb + 4 * T * W)
+    row("like: rmsnorm_scaled (an output, experts' outputs)", _median_ms(lambda: core.rmsnorm_scaled(
+        x, a, w, None, w, w, 1e-5, out16=o16, status=status, combine=(e_, pos, tw_, top, None))), nb + 4 * T * W * top)
+    # ---- between projection and attention ----------------------------------------------------------------
+    freq = torch.rand(rot // 2, device=dev)
+    q, k, v = (torch.empty((T, m, d), dtype=bf, device=dev) for m in (H, kv, kv))
+    ch = (H + kv) * d
+    proj, tw, qn, kn = r(T, ch), r(taps, ch), r(H * d), r(kv * d)
+    st = torch.zeros((66, (taps - 1) * (ch + kv * d)), device=dev)
+    rec = (H + 2 * kv) * d * 2
+    sizes = dict(nh=H, nkv=kv, d=d, dv=d, width=d, q=q, k=k, v=v, freq=freq, rot=rot, status=status)
+    row("whole_conv_prepare (convolution, whole norm, rotation, values from the keys)", _median_ms(lambda: core.whole_conv_prepare(
+        proj, batch, taps_w=tw, state=st, q_norm=qn, k_norm=kn, eps=1e-5, neighbours=True, values_are_keys=True, **sizes)), T * (ch * 4 + rec))
+    projv = r(T, ch + kv * d)
+    row("like: whole_prepare (whole norm, rotation)", _median_ms(lambda: core.whole_prepare(
+        projv, batch, q_norm=qn, k_norm=kn, eps=1e-5, **sizes)), T * ((ch + kv * d) * 4 + rec))
+    twv = r(taps, ch + kv * d)
+    row("like: conv_heads_prepare (convolution, rotation, unit norm)", _median_ms(lambda: core.conv_heads_prepare(
+        projv, batch, taps_w=twv, state=st, eps=1e-5, unit_norm=True, **sizes)), T * ((ch + kv * d) * 4 + rec))
+    # ---- attention of whole prompts -----------------------------------------------------------------------
+    seen = sum(min(p + 1, win) for p in range(n)) * B
+    more = sum(min(max(0, p + 1 - win), keep) for p in range(n)) * B
+    q.normal_(), k.normal_(), v.normal_()
+    ctx = torch.empty((T, H, d), dtype=bf, device=dev)
+    att = lambda **kw: _median_ms(lambda: tc.attention_prefill(q, k, v, batch, ctx, nh=H, nkv=kv, hd=d, scale=d ** -0.5, status=status, **kw))
+    row("tcgen05 attention, window and kept positions", att(window=win, keep=keep), flops=4.0 * (seen + more) * H * d)
+    row("like: tcgen05 attention, window", att(window=win), flops=4.0 * seen * H * d)
+    # ---- the delta mixer ----------------------------------------------------------------------------------
+    dh, dk, dd, dv, ct = sh["d_heads"], sh["d_kv"], sh["d_dim"], sh["d_vdim"], sh["conv"]
+    dch, inner = 2 * dk * dd + dh * dv, dh * dv
+    dproj, both = r(T, dch + 2 * dh), r(T, dh * dd + inner)
+    size = dict(heads=dh, kv_heads=dk, d=dd, dv=dv)
+    off = (ct - 1) * dch
+    state = torch.zeros((66, off + dh * dd * dv), device=dev)
+    dtw, alog, dtb, dtc = r(ct, dch), r(dh) - 1, r(dh) - 1, r(dh * dd) - 1
+    qkv, stp, dec = torch.empty((T, dch), device=dev), torch.empty((T, 2 * dh), device=dev), torch.empty((T, dh * dd), device=dev)
+    kw = dict(b_at=dch, a_at=dch + dh, eps=1e-6, q_scale=dd ** -0.5, **size)
+    chan = lambda b_: core.delta_prepare(dproj, dtw, alog, dtc, state, b_, qkv, stp, a_rows=both[:, :dh * dd], decay=dec, **kw)
+    row("delta_prepare with decays of a channel", _median_ms(lambda: chan(batch)), T * (dch * 8 + dh * dd * 8 + dh * 8))
+    row("like: delta_prepare", _median_ms(lambda: core.delta_prepare(dproj, dtw, alog, dtb, state, batch, qkv, stp, **kw)), T * (dch * 8 + dh * 16))
+    o = torch.empty((T, inner), device=dev)
+    macs = 3.0 * inner * dd                               # the recurrence's multiply-adds a token
+    scan = lambda b_, m, **k2: _median_ms(lambda: core.delta_scan(qkv[:m], stp[:m], state, b_, o[:m], offset=off, **size, **k2))
+    chan(batch)
+    row("delta_scan, decays of a channel (4 sequences of 2,048 tokens)", scan(batch, T, decay=dec), T * (dch + inner + dh * dd) * 4, flops=2.0 * T * macs)
+    row("delta_scan, decays of a channel (one sequence)", scan(b1, n, decay=dec[:n]), n * (dch + inner + dh * dd) * 4, flops=2.0 * n * macs)
+    core.delta_prepare(dproj, dtw, alog, dtb, state, batch, qkv, stp, **kw)
+    row("like: delta_scan (4 sequences of 2,048 tokens)", scan(batch, T), T * (dch + inner) * 4, flops=2.0 * T * macs)
+    row("like: delta_scan (one sequence)", scan(b1, n), n * (dch + inner) * 4, flops=2.0 * n * macs)
+    y, gate, nw = torch.empty((T, inner), dtype=bf, device=dev), both[:, dh * dd:], r(inner)
+    fin = lambda fn: _median_ms(lambda: core.wkv_finish(o, gate, nw, 1e-5, batch, y, heads=dh, d=dv, gate_fn=fn))
+    row("wkv_finish (head norm + sigmoid gate)", fin("sigmoid"), T * inner * 10)
+    row("like: wkv_finish (head norm + silu gate)", fin("silu"), T * inner * 10)
+    step = lambda **k2: _graph_ms(lambda: core.delta_step(qkv[:64], stp[:64], state, gate[:64], nw, 1e-5, one, y[:64], offset=off, **size, **k2))
+    row("delta_step, decays of a channel (one token of 64 sequences)", step(decay=dec[:64], gate_fn="sigmoid"), 64 * inner * dd * 8)
+    row("like: delta_step (one token of 64 sequences)", step(), 64 * inner * dd * 8)
+    # ---- the exponentially gated memory -------------------------------------------------------------------
+    mh, md, mv = sh["m_heads"], sh["m_dim"], sh["m_vdim"]
+    mi = mh * mv
+    at = {"q": 0, "k": mh * md, "v": 2 * mh * md, "gate": 2 * mh * md + mi, "i": 2 * mh * md + 2 * mi, "f": 2 * mh * md + 2 * mi + mh}
+    mproj, ib, fb = r(T, at["f"] + mh), r(mh), r(mh) + 2
+    mst = torch.zeros((66, -(-core.mlstm_state_floats(mh, md, mv) // 4) * 4), device=dev)
+    mo, ms_ = torch.empty((T, mi), device=dev), dict(heads=mh, d=md, dv=mv)
+    margs = lambda m: (mproj[:m], at, ib, fb, sh["cap"], md ** -0.5, mst)
+    mm = 2.0 * mi * md                                    # the write and the read, a token
+    mscan = lambda b_, m: _median_ms(lambda: core.mlstm_scan(*margs(m), b_, mo[:m], **ms_))
+    row("mlstm_scan (4 sequences of 2,048 tokens)", mscan(batch, T), T * (2 * mh * md + 2 * mi) * 4, flops=2.0 * T * mm)
+    row("mlstm_scan (one sequence)", mscan(b1, n), n * (2 * mh * md + 2 * mi) * 4, flops=2.0 * n * mm)
+    xbc, dtr, dtm, am, dsk = r(T, mi + 2 * mh * md), r(T, mh), r(mh) - 1, r(mh) - 1, r(mh)
+    sst = torch.zeros((66, mh * md * mv), device=dev)
+    ssd = lambda b_, m: core.ssd_scan(xbc[:m], dtr[:m], dtm, am, dsk, sst, b_, mo[:m], heads=mh, groups=mh, n=md, dv=mv)
+    row("like: ssd_scan (4 sequences of 2,048 tokens)", _median_ms(lambda: ssd(batch, T)), T * (2 * mh * md + 2 * mi) * 4, flops=2.0 * T * mm)
+    row("like: ssd_scan (one sequence)", _median_ms(lambda: ssd(b1, n)), n * (2 * mh * md + 2 * mi) * 4, flops=2.0 * n * mm)
+    my, mg, mw = torch.empty((64, mi), dtype=bf, device=dev), mproj[:64, at["gate"]:at["gate"] + mi], r(mi)
+    row("mlstm_step (one token of 64 sequences)", _graph_ms(lambda: core.mlstm_step(*margs(64), mg, mw, 1e-5, one, my, **ms_)), 64 * mi * md * 8)
+    row("like: ssd_scan (one token of 64 sequences)", _graph_ms(lambda: ssd(one, 64)), 64 * mi * md * 8)
+    # ---- the rows the experts read ------------------------------------------------------------------------
+    xs = torch.empty((T * top, W), dtype=bf, device=dev)
+    row("weighted_rows", _median_ms(lambda: core.weighted_rows(x, pos, tw_, top, xs, status)), T * W * (4 + 2 * top))
+    rows_ = (pos % T).contiguous()
+    row("like: gather_rows", _median_ms(lambda: tc.gather_rows(o16, rows_, T * top, status)), T * W * (2 + 2 * top))
+    # ---- one token of 64 sequences at a context of 2,048 -------------------------------------------------------
+    S, ctxlen = 64, 2048
+
+    def decode_case(keep_):
+        cache = KVCache({0: KVRequest(kv, d, win, keep=keep_)}, {0: None}, max_tokens=S * (ctxlen + 64), max_slots=S + 1, dtype=bf, device=dev)
+        cache.groups[0].storage.normal_()
+        slots = [cache.acquire() for _ in range(S)]
+        for s_ in slots:
+            G.give_pages(cache, s_, ctxlen + 1)
+        step_ = G.make_batch(dev, slots, [ctxlen] * S, [1] * S)
+        q_, o_ = torch.randn(S, H, d, device=dev).to(bf), torch.empty((S, H * d), dtype=bf, device=dev)
+        ms = _graph_ms(lambda: core.attention_decode(q_, cache.view(0), step_, o_, nh=H, window=win, keep=keep_, scale=0.1, status=status))
+        return ms, S * min(ctxlen + 1, win + keep_) * kv * d * 4
+
+    row("decode attention, window and kept positions", *decode_case(keep))
+    row("like: decode attention, window", *decode_case(0))
+    core.check_status(status)
+    return out
+
+
+def run_kulanex(args):
+    """``--workload kulanex``: prefill and decode of the Kulanex design at two sizes, the closest existing
+    model at equal size beside it, and the new kernels beside their counterparts.  One JSON line per
+    shape; not the benchmark record."""
+    pk = peaks()
+    for name in [args.shape] if args.shape in KULANEX_SHAPES else list(KULANEX_SHAPES):
+        sh = KULANEX_SHAPES[name]
+        clocks = ClockSampler()
+        clocks.start()
+        res = {"workload": "kulanex", "shape": name, "sizes": sh, "dtype": "bfloat16", "data": "synthetic, random weights",
+               "peaks": pk, "kulanex": _model_rates(kulanex_config(sh), args), "divadra": _model_rates(kulanex_divadra_config(sh), args)}
+        res["clocks"] = clocks.stop()
+        res["kernels_at_8192_tokens"] = kulanex_kernels(sh, pk)
+        print(json.dumps(res), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1622,12 +1828,12 @@ def main():
     ap.add_argument("--batch", type=int, default=8, help="with --profile-step decode: sequences in the batch")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="with --profile-step: the path whose kernels are wanted")
-    ap.add_argument("--shape", choices=["a2.7b", "57b"] + sorted(set(SUPEVIK_SHAPES) | set(FOGAPEL_SHAPES) | set(ZOSIPEL_SHAPES) | set(DIVADRA_SHAPES) | set(DITAZEN_SHAPES)), default="a2.7b",
-                    help="with --sweep: the layer sizes; with --workload supevik, fogapel, zosipel, divadra or ditazen: one of its shapes (default: all)")
+    ap.add_argument("--shape", choices=["a2.7b", "57b"] + sorted(set(SUPEVIK_SHAPES) | set(FOGAPEL_SHAPES) | set(ZOSIPEL_SHAPES) | set(DIVADRA_SHAPES) | set(DITAZEN_SHAPES) | set(KULANEX_SHAPES)), default="a2.7b",
+                    help="with --sweep: the layer sizes; with --workload supevik, fogapel, zosipel, divadra, ditazen or kulanex: one of its shapes (default: all)")
     ap.add_argument("--prompt-len", type=int, default=0, help="with --sweep: tokens in each prompt (default 512)")
-    ap.add_argument("--workload", choices=["fp32-32k", "long-prompt", "supevik", "fogapel", "zosipel", "divadra", "ditazen"], default=None,
+    ap.add_argument("--workload", choices=["fp32-32k", "long-prompt", "supevik", "fogapel", "zosipel", "divadra", "ditazen", "kulanex"], default=None,
                     help="fp32-32k: the true 32-bit path at a context of 32,768; long-prompt: one bfloat16 prompt of "
-                         "--prompt-len tokens [32768] run in pieces; supevik, fogapel, zosipel, divadra, ditazen: that design at two sizes beside "
+                         "--prompt-len tokens [32768] run in pieces; supevik, fogapel, zosipel, divadra, ditazen, kulanex: that design at two sizes beside "
                          "the closest model at equal size (each prints its own line, no benchmark record)")
     ap.add_argument("--unequal", action="store_true", help="with --sweep: prompts of unequal lengths, 256 to 2,048 tokens")
     ap.add_argument("--sweep", default=None, help="comma-separated batch sizes: print decode throughput for each "
@@ -1657,6 +1863,8 @@ def main():
         return run_divadra(args)
     if args.workload == "ditazen":
         return run_ditazen(args)
+    if args.workload == "kulanex":
+        return run_kulanex(args)
     return run_ours(args)
 
 

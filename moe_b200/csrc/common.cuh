@@ -168,6 +168,24 @@ __device__ __forceinline__ float attn_denominator(float m, float l, int sink, fl
     return sink == ATTN_SIGMOID ? expf(-m) : sink ? l + expf(sv - m) : l;
 }
 
+// SMs of the current device (a scan's launch asks whether its blocks fill them).
+inline int scan_sms() {
+    static int n = 0;
+    if (!n) {
+        int dev = 0;
+        if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess) n = 148;
+    }
+    return n;
+}
+
+// Dynamic shared memory for a scan of `blocks` blocks that need `need` bytes each: where every block could have an SM
+// of its own, more than half an SM's, so that no two share one (placed beside other kernels' blocks they would, and
+// a scan is as slow as its most crowded SM).
+inline size_t scan_smem(size_t need, long long blocks) {
+    const size_t alone = 116 * 1024;
+    return blocks <= scan_sms() && need < alone ? alone : need;
+}
+
 static inline int launch_status() { return (int)cudaGetLastError(); }
 
 // ---- programmatic dependent launch ------------------------------------------------------

@@ -283,13 +283,15 @@ delta_step_kernel(const DeltaSeq p, const float* __restrict__ gate, long long ld
 // one token at a time the products with S are eight independent sums instead of two with an update between
 // them, their sums over the threads are formed together, and the state is multiplied by a decay once.
 //
-// grid (ceil(dv / 32), heads, sequences), 128 threads: thread (kp = tid % 16, cg = tid / 16) holds four neighbouring
-// columns of rows 4 kp ... 4 kp + 3 of every 64 rows of S in registers (rows beyond d stay zero; the sixteen
-// threads' reads of a token's k and q are then neighbours in shared memory).  A run of sixteen tokens is staged
+// grid (ceil(dv / COLS), heads, sequences), 128 threads: thread (kp = tid % KP, cg = tid / KP) holds four neighbouring
+// columns of rows 4 kp ... 4 kp + 3 of every 4 KP rows of S in registers (rows beyond d stay zero; the KP
+// threads' reads of a token's k and q are then neighbours in shared memory).  KP = 16 (32 columns a block) or, where those
+// blocks would leave SMs idle, 32 (16 columns a block, half as many rows a thread).  A run of sixteen tokens is staged
 // in shared memory as [k | q | the block's columns of v] a token (cp.async, two buffers; rows beyond the
 // sequence's last token are zeros with beta 0 and decay 1: they change nothing); warp w forms the scalars of the
 // run's group w.  Within a run the groups follow one another without a block barrier.
-constexpr int DG = 4, DRUN = 16, DKP = 16, DCG = 8, DCOLS = 4 * DCG, DTHREADS = DKP * DCG;
+constexpr int DG = 4, DRUN = 16, DTHREADS = 128;
+__host__ __device__ constexpr int dcols(int kp) { return 4 * (DTHREADS / kp); }
 
 __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes, bool on) {
     const unsigned at = (unsigned)__cvta_generic_to_shared(dst);
@@ -301,14 +303,14 @@ __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes
 }
 
 // VEC: rows of q, k and v start on 16-byte boundaries and hold whole 16-byte units.
-template <int RPT, bool CH>
+template <int RPT, int KP, bool CH>
 __host__ __device__ constexpr size_t delta_scan_floats() {
-    return (size_t)2 * DRUN * ((CH ? 3 : 2) * RPT * DKP + DCOLS) + 4 * DRUN + 4 * 32 + DG * DCOLS + (CH ? 4 * RPT * DKP : 0);
+    return (size_t)2 * DRUN * ((CH ? 3 : 2) * RPT * KP + dcols(KP)) + 4 * DRUN + 4 * 32 + DG * dcols(KP) + (CH ? 4 * RPT * KP : 0);
 }
-template <int RPT, bool VEC, bool CH>
+template <int RPT, int KP, bool VEC, bool CH>
 __global__ void __launch_bounds__(DTHREADS, RPT <= 8 ? (CH && RPT == 8 ? 3 : 4) : 2)
 delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
-    constexpr int NP = RPT * DKP;
+    constexpr int NP = RPT * KP, DCOLS = dcols(KP);
     constexpr int V_AT = (CH ? 3 : 2) * NP;                   // a token's row: k, q, CH: its decays, then v
     constexpr int ROWLEN = V_AT + DCOLS;
     extern __shared__ __align__(16) float sm[];               // [2][DRUN][ROWLEN] | steps [2][2][DRUN] | scalars [4][32] | u [DG][DCOLS]
@@ -316,7 +318,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     float* s_coef = s_step + 4 * DRUN;
     float* s_u = s_coef + 4 * 32;
     float* s_g4 = s_u + DG * DCOLS;
-    const int tid = threadIdx.x, kp = tid % DKP, cg = tid / DKP, lane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, kp = tid % KP, cg = tid / KP, lane = tid & 31, warp = tid >> 5;
     const int h = blockIdx.y, s = blockIdx.z, g = h / (p.H / p.G), d = p.d, dv = p.dv;
     const int c0 = blockIdx.x * DCOLS, col = c0 + cg * 4;
     for (int i = tid; i < 2 * DRUN * ROWLEN; i += DTHREADS) sm[i] = 0.f;         // columns that no copy writes stay zero
@@ -329,7 +331,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     float sreg[RPT][4];
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
-        const int n = (m / 4) * 64 + kp * 4 + m % 4;
+        const int n = (m / 4) * 4 * KP + kp * 4 + m % 4;
         if (vec_state && n < d && col < dv) {
             const float4 t4 = *reinterpret_cast<const float4*>(S + (size_t)n * dv + col);
             sreg[m][0] = t4.x, sreg[m][1] = t4.y, sreg[m][2] = t4.z, sreg[m][3] = t4.w;
@@ -482,8 +484,8 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             for (int m0 = 0; m0 < RPT; m0 += 4) {
 #pragma unroll
                 for (int i = 0; i < DG; i++) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + m0 * DKP);
-                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0 * DKP);
+                    const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + m0 * KP);
+                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0 * KP);
                     kr[i][m0] = k4.x, kr[i][m0 + 1] = k4.y, kr[i][m0 + 2] = k4.z, kr[i][m0 + 3] = k4.w;
                     const float qi[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
@@ -495,7 +497,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
                         }
                 }
             }
-            // Sums over the sixteen threads of a column group.  On the way every thread drops what another one
+            // Sums over the threads of a column group.  On the way every thread drops what another one
             // carries on: bits 0 and 1 of kp pick the column, bit 2 the product with the keys or the queries.
             float r2[2 * DG][2], r1[2 * DG], rr[DG];
 #pragma unroll
@@ -512,6 +514,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             for (int i = 0; i < DG; i++) {
                 rr[i] = (b2 ? r1[DG + i] : r1[i]) + __shfl_xor_sync(0xffffffffu, b2 ? r1[i] : r1[DG + i], 4);
                 rr[i] += __shfl_xor_sync(0xffffffffu, rr[i], 8);
+                if (KP == 32) rr[i] += __shfl_xor_sync(0xffffffffu, rr[i], 16);
             }
             float cf[32];
 #pragma unroll
@@ -528,12 +531,12 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             u[3] = cf[3] * vrow[3 * ROWLEN] - cf[7] * rr[3] - cf[19] * u[0] - cf[20] * u[1] - cf[21] * u[2];
 #pragma unroll
             for (int i = 0; i < DG; i++) {
-                if (!b2 && !b3) s_u[i * DCOLS + cg * 4 + my_col] = cf[12 + i] * u[i];
+                if (!b2 && !b3 && kp < 16) s_u[i * DCOLS + cg * 4 + my_col] = cf[12 + i] * u[i];
                 const float other = __shfl_xor_sync(0xffffffffu, u[i], 4);
                 u[i] = b2 ? other : u[i];
             }
-            __syncwarp();                             // a column group's sixteen threads lie in one warp
-            if (b2 && !b3 && col + my_col < dv) {
+            __syncwarp();                             // a column group's threads lie in one warp
+            if (b2 && !b3 && kp < 16 && col + my_col < dv) {
                 const float out[DG] = {cf[8] * rr[0] + cf[22] * u[0], cf[9] * rr[1] + cf[23] * u[0] + cf[24] * u[1],
                                        cf[10] * rr[2] + cf[25] * u[0] + cf[26] * u[1] + cf[27] * u[2],
                                        cf[11] * rr[3] + cf[28] * u[0] + cf[29] * u[1] + cf[30] * u[2] + cf[31] * u[3]};
@@ -552,7 +555,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
             if (CH) {                                 // the decays and the keys of the update, row by row
 #pragma unroll
                 for (int m0 = 0; m0 < RPT; m0 += 4) {
-                    const float4 g4 = *reinterpret_cast<const float4*>(s_g4 + gr * NP + kp * 4 + m0 * DKP);
+                    const float4 g4 = *reinterpret_cast<const float4*>(s_g4 + gr * NP + kp * 4 + m0 * KP);
                     const float gm[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
                     for (int z = 0; z < 4; z++)
@@ -560,7 +563,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
                         for (int c = 0; c < 4; c++) sreg[m0 + z][c] *= gm[z];
 #pragma unroll
                     for (int i = 0; i < DG; i++) {
-                        const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + 2 * NP + m0 * DKP);
+                        const float4 k4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + 2 * NP + m0 * KP);
                         const float km[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
                         for (int z = 0; z < 4; z++)
@@ -582,7 +585,7 @@ delta_scan_kernel(const DeltaSeq p, float* __restrict__ o) {
     }
 #pragma unroll
     for (int m = 0; m < RPT; m++) {
-        const int n = (m / 4) * 64 + kp * 4 + m % 4;
+        const int n = (m / 4) * 4 * KP + kp * 4 + m % 4;
         if (n >= d) continue;
         if (vec_state && col < dv) {
             *reinterpret_cast<float4*>(S + (size_t)n * dv + col) = make_float4(sreg[m][0], sreg[m][1], sreg[m][2], sreg[m][3]);
@@ -683,32 +686,39 @@ MOE_API int moe_delta_scan(const float* qkv, const float* step, float* state, lo
         state_pitch < (long long)H * d * dv || H > 65535 || num_seqs > 65535)
         return (int)cudaErrorInvalidValue;
     const DeltaSeq p{qkv, step, state, state_pitch, cu_seqlens, slots, H, G, d, dv, decay};
-    const dim3 grid((dv + DCOLS - 1) / DCOLS, H, num_seqs);
+    // few blocks: the narrow form puts twice as many on the SMs
+    const bool narrow = d > 64 && (long long)((dv + dcols(16) - 1) / dcols(16)) * H * num_seqs * 2 <= scan_sms();
+    const int cols = dcols(narrow ? 32 : 16);
+    const dim3 grid((dv + cols - 1) / cols, H, num_seqs);
     const bool vec = d % 4 == 0 && dv % 4 == 0 && aligned16(qkv) && aligned16(decay);
     // An ordinary launch: blocks that are placed while the kernel before still occupies some SMs end up several to
     // an SM beside empty ones, and a scan is as slow as its most crowded SM.
-#define SCAN_V(RPT_, V_, C_)                                                                                           \
+#define SCAN_V(RPT_, KP_, V_, C_)                                                                                      \
     do {                                                                                                               \
-        constexpr size_t smem = delta_scan_floats<RPT_, C_>() * sizeof(float);                                         \
+        const size_t smem = scan_smem(delta_scan_floats<RPT_, KP_, C_>() * sizeof(float), (long long)grid.x * grid.y * grid.z); \
         if (smem > 48 * 1024) {                                                                                        \
-            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, V_, C_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPT_, KP_, V_, C_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                       \
         }                                                                                                              \
-        delta_scan_kernel<RPT_, V_, C_><<<grid, DTHREADS, smem, stream>>>(p, o);                                       \
+        delta_scan_kernel<RPT_, KP_, V_, C_><<<grid, DTHREADS, smem, stream>>>(p, o);                                  \
         return launch_status();                                                                                        \
     } while (0)
-#define SCAN(RPT_)                                                                                                     \
+#define SCAN(RPT_, KP_)                                                                                                \
     do {                                                                                                               \
         if (decay) {                                                                                                   \
-            if (vec) SCAN_V(RPT_, true, true);                                                                         \
-            SCAN_V(RPT_, false, true);                                                                                 \
+            if (vec) SCAN_V(RPT_, KP_, true, true);                                                                    \
+            SCAN_V(RPT_, KP_, false, true);                                                                            \
         }                                                                                                              \
-        if (vec) SCAN_V(RPT_, true, false);                                                                            \
-        SCAN_V(RPT_, false, false);                                                                                    \
+        if (vec) SCAN_V(RPT_, KP_, true, false);                                                                       \
+        SCAN_V(RPT_, KP_, false, false);                                                                               \
     } while (0)
-    if (d <= 64) SCAN(4);
-    if (d <= 128) SCAN(8);
-    SCAN(16);
+    if (d <= 64) SCAN(4, 16);
+    if (narrow) {
+        if (d <= 128) SCAN(4, 32);
+        SCAN(8, 32);
+    }
+    if (d <= 128) SCAN(8, 16);
+    SCAN(16, 16);
 #undef SCAN
 #undef SCAN_V
 }

@@ -6,8 +6,8 @@
 //   m' = max(lf + m, li);  a = e^(lf + m - m');  b = e^(li - m');  m <- m'
 //   S <- a S + b k v^T;  n <- a n + b k;  o = S^T q / (max(|n . q|, e^(-m)) + 1e-6)
 //
-//   mlstm_gates   a, b and e^(-m) of every token, and the sequences' m moved on: a warp a (head, sequence), 32 tokens
-//                 at a time (the pairs (lf, li) compose as m -> max(lf + m, li), an associative operation).
+//   mlstm_gates   a, b and e^(-m) of every token, and the sequences' m moved on: a block a (head, sequence), a token a
+//                 thread (the pairs (lf, li) compose as m -> max(lf + m, li), an associative operation).
 //   mlstm_scan    several tokens a sequence, four at a time, state and normaliser in registers.
 //   mlstm_step    one token a sequence: gates, recurrence with the state read once and written once, and the output's
 //                 norm and gate behind it, a block a (head, sequence).
@@ -34,47 +34,54 @@ struct MemSeq {
     float* steps;              // [T, 3 H]: a, b, e^(-m)
     int H, d, dv;
     float cap, q_scale;
-    int copies;                // of n, one for every 32 columns of S: blocks that share a head have one of their own each
+    int copies;                // of n, one for every 16 columns of S: blocks that share a head have ones of their own
     __device__ __forceinline__ size_t n_at(int copy, int h) const { return (size_t)H * d * dv + ((size_t)copy * H + h) * d; }
     __device__ __forceinline__ size_t m_at(int h) const { return (size_t)H * d * (dv + copies) + h; }
 };
 
-constexpr int GATE_WARPS = 4;
-
-// grid (ceil(H / 4), sequences)
-__global__ void __launch_bounds__(GATE_WARPS * 32)
+// grid (H, sequences); any whole number of warps: a chunk of as many tokens as threads at a time
+__global__ void __launch_bounds__(1024)
 mlstm_gates_kernel(const MemSeq p) {
+    __shared__ float wf[32], wi[32];                  // a warp's tokens as one pair
     pdl_sync();
-    const int lane = threadIdx.x & 31, h = blockIdx.x * GATE_WARPS + (threadIdx.x >> 5), s = blockIdx.y;
-    if (h >= p.H) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5, h = blockIdx.x, s = blockIdx.y;
     const int tok0 = p.cu_seqlens[s], cnt = p.cu_seqlens[s + 1] - tok0;
     if (cnt <= 0) return;
     float* m_at = p.state + (size_t)p.slots[s] * p.state_pitch + p.m_at(h);
     const float ib = p.i_bias[h], fb = p.f_bias[h];
     float m = *m_at;
-    for (int t0 = 0; t0 < cnt; t0 += 32) {
-        const bool on = t0 + lane < cnt;
-        const float* row = p.proj + (size_t)(tok0 + min(t0 + lane, cnt - 1)) * p.ld;
+    for (int t0 = 0; t0 < cnt; t0 += blockDim.x) {
+        const int t = t0 + threadIdx.x;
+        const bool on = t < cnt;                      // (places beyond the last token leave m as it is)
+        const float* row = p.proj + (size_t)(tok0 + min(t, cnt - 1)) * p.ld;
         const float li = on ? log_in(row[p.i_at + h] + ib, p.cap) : -INFINITY;
         const float lf = on ? log_keep(row[p.f_at + h] + fb, p.cap) : 0.f;
-        float cf = lf, ci = li;                       // the tokens up to this one as one pair
+        float cf = lf, ci = li;                       // the warp's tokens up to this one as one pair
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
             const float pf = __shfl_up_sync(0xffffffffu, cf, o), pi = __shfl_up_sync(0xffffffffu, ci, o);
             if (lane >= o) ci = fmaxf(cf + pi, ci), cf += pf;
         }
-        const float after = fmaxf(cf + m, ci);
-        float before = __shfl_up_sync(0xffffffffu, after, 1);
-        if (lane == 0) before = m;
+        if (lane == 31) wf[warp] = cf, wi[warp] = ci;
+        __syncthreads();
+        float before = m, mine = m;                   // m in front of the warp, and at the end of the chunk
+        for (int w = 0; w < warps; w++) {
+            if (w == warp) mine = before;
+            before = fmaxf(wf[w] + before, wi[w]);
+        }
+        m = before;
+        const float after = fmaxf(cf + mine, ci);
+        before = __shfl_up_sync(0xffffffffu, after, 1);
+        if (lane == 0) before = mine;
         if (on) {
-            float* out = p.steps + (size_t)(tok0 + t0 + lane) * 3 * p.H + h;
+            float* out = p.steps + (size_t)(tok0 + t) * 3 * p.H + h;
             out[0] = expf(fminf(lf + before - after, 0.f));
             out[p.H] = expf(fminf(li - after, 0.f));
             out[2 * p.H] = expf(-after);
         }
-        m = __shfl_sync(0xffffffffu, after, 31);      // (places beyond the last token leave it as it is)
+        __syncthreads();                              // the pairs are read before the next chunk's are written
     }
-    if (lane == 0) *m_at = m;
+    if (threadIdx.x == 0) *m_at = m;
 }
 
 // ---- one token a sequence --------------------------------------------------------------------------
@@ -169,12 +176,14 @@ mlstm_step_kernel(const MemSeq p, const float* __restrict__ gate, long long ldg,
 //     S <- A_4 S + sum_j P_4j b_j k_j v_j^T,                          n <- A_4 n + sum_j P_4j b_j k_j
 // which is the recurrence written out.  The normaliser n is one more column of S whose value is always 1.
 //
-// grid (ceil(dv / 32), heads, sequences), 128 threads: thread (kp = tid % 16, cg = tid / 16) holds four neighbouring
-// columns of rows 4 kp ... 4 kp + 3 of every 64 rows of S in registers, and the same rows of n (every column group
-// for itself).  A run of sixteen tokens is staged in shared memory as [k | q | the block's columns of v] a token
+// grid (ceil(dv / COLS), heads, sequences), 128 threads: thread (kp = tid % KP, cg = tid / KP) holds four neighbouring
+// columns of rows 4 kp ... 4 kp + 3 of every 4 KP rows of S in registers, and the same rows of n (every column group
+// for itself).  KP = 16 (32 columns a block) or, where those blocks would leave SMs idle, 32 (16 columns a block, half as
+// many rows a thread).  A run of sixteen tokens is staged in shared memory as [k | q | the block's columns of v] a token
 // (cp.async, two buffers; places beyond the sequence's last token are zeros with a = 1, b = 0); warp w forms the
 // scalars of the run's group w.  Within a run the groups follow one another without a block barrier.
-constexpr int MG = 4, MRUN = 16, MKP = 16, MCG = 8, MCOLS = 4 * MCG, MTHREADS = MKP * MCG;
+constexpr int MG = 4, MRUN = 16, MTHREADS = 128, COPY_COLS = 16;
+__host__ __device__ constexpr int mcols(int kp) { return 4 * (MTHREADS / kp); }
 constexpr int MCOEF = 36;      // a group's scalars: [0, 16) c_ij of token i in row i, [16, 20) A_i, [20, 24) P_4j b_j, [24, 28) e^(-m_i)
 
 __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes, bool on) {
@@ -186,44 +195,104 @@ __device__ __forceinline__ void cp_zfill(float* dst, const float* src, int bytes
         asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(at), "l"(src), "r"(n) : "memory");
 }
 
-template <int RPT>
+template <int RPT, int KP>
 __host__ __device__ constexpr size_t mlstm_scan_floats() {
-    return (size_t)2 * MRUN * (2 * RPT * MKP + MCOLS) + 2 * 3 * MRUN + 4 * MCOEF;
+    return (size_t)2 * MRUN * (2 * RPT * KP + mcols(KP)) + 2 * 3 * MRUN + 4 * MCOEF;
 }
 
 // VEC: rows of q, k and v start on 16-byte boundaries and hold whole 16-byte units.
-template <int RPT, bool VEC>
-__global__ void __launch_bounds__(MTHREADS, RPT <= 8 ? 4 : 2)
-mlstm_scan_kernel(const MemSeq p, float* __restrict__ o) {
-    constexpr int NP = RPT * MKP;
+// Few, long sequences leave SMs idle and the chain over the tokens long: a sequence's tokens may be cut into segments
+// that run side by side (a is one number a head and token, so a segment's effect on what follows is its own end from a
+// zero start and the product of its a):
+//   phase 1  every segment but a sequence's last: its end and that product into a workspace, no outputs; the first one
+//            also copies the sequence's state there
+//   phase 2  every segment: its start from that copy and the ends before it, then the recurrence with outputs; the last
+//            segment that holds tokens writes the state back
+// which changes the order of additions, nothing else.
+struct MemSegments {
+    int segs, seg_len;       // segments a sequence (1: none of this), tokens a segment (a multiple of the staged run)
+    float* ends;             // [sequence][segs] planes of `pitch` floats, S then n as in the state; the last one: the copy
+    long long pitch;
+    float* products;         // [sequence][segs][H]
+};
+
+// PHASE (0: the whole sequence in one go; 1, 2: see above) is known when compiled.
+template <int RPT, int KP, bool VEC, int PHASE>
+__global__ void __launch_bounds__(MTHREADS, RPT == 4 ? 4 : RPT == 8 ? 3 : 1)
+mlstm_scan_kernel(const MemSeq p, float* __restrict__ o, const MemSegments sg) {
+    constexpr int NP = RPT * KP, MCOLS = mcols(KP);
     constexpr int ROWLEN = 2 * NP + MCOLS;
     extern __shared__ __align__(16) float sm[];               // [2][MRUN][ROWLEN] | scalars [4][MCOEF] | steps [2][3][MRUN]
     float* s_coef = sm + 2 * MRUN * ROWLEN;
     float* s_step = s_coef + 4 * MCOEF;
-    const int tid = threadIdx.x, kp = tid % MKP, cg = tid / MKP, lane = tid & 31, warp = tid >> 5;
-    const int h = blockIdx.y, s = blockIdx.z, d = p.d, dv = p.dv;
+    const int tid = threadIdx.x, kp = tid % KP, cg = tid / KP, lane = tid & 31, warp = tid >> 5;
+    const int h = blockIdx.y, s = PHASE ? blockIdx.z / sg.segs : blockIdx.z, seg = PHASE ? blockIdx.z % sg.segs : 0, d = p.d, dv = p.dv;
     const int c0 = blockIdx.x * MCOLS, col = c0 + cg * 4;
     for (int i = tid; i < 2 * MRUN * ROWLEN; i += MTHREADS) sm[i] = 0.f;         // columns that no copy writes stay zero
-    const int tok0 = p.cu_seqlens[s], cnt = p.cu_seqlens[s + 1] - tok0;
+    const int seq_cnt = p.cu_seqlens[s + 1] - p.cu_seqlens[s];
+    const int tok0 = p.cu_seqlens[s] + (PHASE ? seg * sg.seg_len : 0);
+    const int cnt = PHASE ? min(sg.seg_len, seq_cnt - seg * sg.seg_len) : seq_cnt;
     if (cnt <= 0) return;
+    const bool last_seg = !PHASE || (seg + 1) * sg.seg_len >= seq_cnt;            // the last one that holds tokens
+    if (PHASE == 1 && last_seg && seg > 0) return;                              // nothing comes after it
     const int ncols = min(MCOLS, dv - c0);
+    const size_t s_off = (size_t)h * d * dv, n_off = p.n_at(blockIdx.x * (MCOLS / COPY_COLS), h);
     float* state = p.state + (size_t)p.slots[s] * p.state_pitch;
-    float* S = state + (size_t)h * d * dv;
-    float* N = state + p.n_at(blockIdx.x, h);
-    const bool vec_state = dv % 4 == 0 && ((uintptr_t)S) % 16 == 0;
+    float* planes = PHASE ? sg.ends + (size_t)s * sg.segs * sg.pitch : nullptr;
+    const bool vec_state = dv % 4 == 0 && ((uintptr_t)(state + s_off)) % 16 == 0;
     float sreg[RPT][4], nreg[RPT];
+    // this thread's part of S and n from the plane `from`, times `keep` what it holds plus it
+    auto load = [&](const float* from, float keep) {
 #pragma unroll
-    for (int m = 0; m < RPT; m++) {
-        const int n = (m / 4) * 64 + kp * 4 + m % 4;
-        nreg[m] = n < d ? N[n] : 0.f;
-        if (vec_state && n < d && col < dv) {
-            const float4 t4 = *reinterpret_cast<const float4*>(S + (size_t)n * dv + col);
-            sreg[m][0] = t4.x, sreg[m][1] = t4.y, sreg[m][2] = t4.z, sreg[m][3] = t4.w;
-        } else {
+        for (int m = 0; m < RPT; m++) {
+            const int n = (m / 4) * 4 * KP + kp * 4 + m % 4;
+            if (n >= d) continue;
+            nreg[m] = fmaf(keep, nreg[m], from[n_off + n]);
+            const float* row = from + s_off + (size_t)n * dv + col;
+            if (vec_state && col < dv) {
+                const float4 t4 = *reinterpret_cast<const float4*>(row);
+                sreg[m][0] = fmaf(keep, sreg[m][0], t4.x), sreg[m][1] = fmaf(keep, sreg[m][1], t4.y);
+                sreg[m][2] = fmaf(keep, sreg[m][2], t4.z), sreg[m][3] = fmaf(keep, sreg[m][3], t4.w);
+            } else {
 #pragma unroll
-            for (int c = 0; c < 4; c++) sreg[m][c] = (n < d && col + c < dv) ? S[(size_t)n * dv + col + c] : 0.f;
+                for (int c = 0; c < 4; c++)
+                    if (col + c < dv) sreg[m][c] = fmaf(keep, sreg[m][c], row[c]);
+            }
         }
+    };
+    auto store = [&](float* to) {
+#pragma unroll
+        for (int m = 0; m < RPT; m++) {
+            const int n = (m / 4) * 4 * KP + kp * 4 + m % 4;
+            if (n >= d) continue;
+            float* row = to + s_off + (size_t)n * dv + col;
+            if (vec_state && col < dv) {
+                *reinterpret_cast<float4*>(row) = make_float4(sreg[m][0], sreg[m][1], sreg[m][2], sreg[m][3]);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; c++)
+                    if (col + c < dv) row[c] = sreg[m][c];
+            }
+            if (cg < MCOLS / COPY_COLS && blockIdx.x * (MCOLS / COPY_COLS) + cg < p.copies) to[n_off + (size_t)cg * p.H * d + n] = nreg[m];
+        }
+    };
+    auto clear = [&]() {
+#pragma unroll
+        for (int m = 0; m < RPT; m++) nreg[m] = sreg[m][0] = sreg[m][1] = sreg[m][2] = sreg[m][3] = 0.f;
+    };
+    clear();
+    if (PHASE == 0) load(state, 0.f);
+    if (PHASE == 1 && seg == 0) {
+        load(state, 0.f);
+        store(planes + (size_t)(sg.segs - 1) * sg.pitch);
+        if (last_seg) return;
+        clear();
     }
+    if (PHASE == 2) {
+        load(planes + (size_t)(sg.segs - 1) * sg.pitch, 0.f);
+        for (int q = 0; q < seg; q++) load(planes + (size_t)q * sg.pitch, sg.products[((size_t)s * sg.segs + q) * p.H + h]);
+    }
+    float product = 1.f;
     const float* base = p.proj + (size_t)tok0 * p.ld;
     const float* sbase = p.steps + (size_t)tok0 * 3 * p.H + h;
     const int k_at = p.k_at + h * d, q_at = p.q_at + h * d, v_at = p.v_at + h * dv + c0;
@@ -325,6 +394,7 @@ mlstm_scan_kernel(const MemSeq p, float* __restrict__ o) {
             const float* cf = s_coef + gr * MCOEF;
             const float* vgr = run + gr * MG * ROWLEN + 2 * NP + cg * 4;
             float hq[MG][4], hn[MG];
+            if (PHASE == 1) product *= cf[28];
 #pragma unroll
             for (int i = 0; i < MG; i++) {
                 hn[i] = 0.f;
@@ -343,8 +413,8 @@ mlstm_scan_kernel(const MemSeq p, float* __restrict__ o) {
 #pragma unroll
             for (int m0 = 0; m0 < RPT; m0 += 4) {
 #pragma unroll
-                for (int i = 0; i < MG; i++) {
-                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0 * MKP);
+                for (int i = 0; i < (PHASE == 1 ? 0 : MG); i++) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(row + i * ROWLEN + NP + m0 * KP);
                     const float qi[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
                     for (int z = 0; z < 4; z++) {
@@ -361,7 +431,7 @@ mlstm_scan_kernel(const MemSeq p, float* __restrict__ o) {
                 }
 #pragma unroll
                 for (int j = 0; j < MG; j++) {
-                    const float4 k4 = *reinterpret_cast<const float4*>(row + j * ROWLEN + m0 * MKP);
+                    const float4 k4 = *reinterpret_cast<const float4*>(row + j * ROWLEN + m0 * KP);
                     const float kj[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
                     for (int z = 0; z < 4; z++) {
@@ -371,47 +441,43 @@ mlstm_scan_kernel(const MemSeq p, float* __restrict__ o) {
                     }
                 }
             }
-            // Sums over the sixteen threads of a column group; on the way every thread drops what another one carries
-            // on: bits 0 and 1 of kp pick the column, bits 2 and 3 the token.
-            float r2[MG][2], r1[MG], t2[2], n2[2];
+            if constexpr (PHASE != 1) {               // (phase 1: the end alone)
+                // Sums over the threads of a column group; on the way every thread drops what another one carries
+                // on: bits 0 and 1 of kp pick the column, bits 2 and 3 the token.
+                float r2[MG][2], r1[MG], t2[2], n2[2];
 #pragma unroll
-            for (int i = 0; i < MG; i++)
+                for (int i = 0; i < MG; i++)
 #pragma unroll
-                for (int c = 0; c < 2; c++)
-                    r2[i][c] = (b0 ? hq[i][2 + c] : hq[i][c]) + __shfl_xor_sync(0xffffffffu, b0 ? hq[i][c] : hq[i][2 + c], 1);
+                    for (int c = 0; c < 2; c++)
+                        r2[i][c] = (b0 ? hq[i][2 + c] : hq[i][c]) + __shfl_xor_sync(0xffffffffu, b0 ? hq[i][c] : hq[i][2 + c], 1);
 #pragma unroll
-            for (int i = 0; i < MG; i++)
-                r1[i] = (b1 ? r2[i][1] : r2[i][0]) + __shfl_xor_sync(0xffffffffu, b1 ? r2[i][0] : r2[i][1], 2);
+                for (int i = 0; i < MG; i++)
+                    r1[i] = (b1 ? r2[i][1] : r2[i][0]) + __shfl_xor_sync(0xffffffffu, b1 ? r2[i][0] : r2[i][1], 2);
 #pragma unroll
-            for (int i = 0; i < 2; i++) {
-                t2[i] = (b2 ? r1[2 + i] : r1[i]) + __shfl_xor_sync(0xffffffffu, b2 ? r1[i] : r1[2 + i], 4);
-                n2[i] = (b2 ? hn[2 + i] : hn[i]) + __shfl_xor_sync(0xffffffffu, b2 ? hn[i] : hn[2 + i], 4);
+                for (int i = 0; i < 2; i++) {
+                    t2[i] = (b2 ? r1[2 + i] : r1[i]) + __shfl_xor_sync(0xffffffffu, b2 ? r1[i] : r1[2 + i], 4);
+                    n2[i] = (b2 ? hn[2 + i] : hn[i]) + __shfl_xor_sync(0xffffffffu, b2 ? hn[i] : hn[2 + i], 4);
+                }
+                float read = (b3 ? t2[1] : t2[0]) + __shfl_xor_sync(0xffffffffu, b3 ? t2[0] : t2[1], 8);
+                float size = (b3 ? n2[1] : n2[0]) + __shfl_xor_sync(0xffffffffu, b3 ? n2[0] : n2[1], 8);
+                if (KP == 32) read += __shfl_xor_sync(0xffffffffu, read, 16), size += __shfl_xor_sync(0xffffffffu, size, 16);
+                size += __shfl_xor_sync(0xffffffffu, size, 1);
+                size += __shfl_xor_sync(0xffffffffu, size, 2);
+                const float4 c4 = *reinterpret_cast<const float4*>(cf + 4 * my_tok);
+                const float ai = cf[16 + my_tok];
+                read = ai * read + c4.x * vgr[my_col] + c4.y * vgr[ROWLEN + my_col] + c4.z * vgr[2 * ROWLEN + my_col] + c4.w * vgr[3 * ROWLEN + my_col];
+                size = ai * size + c4.x + c4.y + c4.z + c4.w;
+                const int t = t0 + gr * MG + my_tok;
+                if (kp < 16 && t < cnt && col + my_col < dv)
+                    o[(size_t)(tok0 + t) * p.H * dv + (size_t)h * dv + col + my_col] = read / (fmaxf(fabsf(size), cf[24 + my_tok]) + READ_EPS);
             }
-            float read = (b3 ? t2[1] : t2[0]) + __shfl_xor_sync(0xffffffffu, b3 ? t2[0] : t2[1], 8);
-            float size = (b3 ? n2[1] : n2[0]) + __shfl_xor_sync(0xffffffffu, b3 ? n2[0] : n2[1], 8);
-            size += __shfl_xor_sync(0xffffffffu, size, 1);
-            size += __shfl_xor_sync(0xffffffffu, size, 2);
-            const float4 c4 = *reinterpret_cast<const float4*>(cf + 4 * my_tok);
-            const float ai = cf[16 + my_tok];
-            read = ai * read + c4.x * vgr[my_col] + c4.y * vgr[ROWLEN + my_col] + c4.z * vgr[2 * ROWLEN + my_col] + c4.w * vgr[3 * ROWLEN + my_col];
-            size = ai * size + c4.x + c4.y + c4.z + c4.w;
-            const int t = t0 + gr * MG + my_tok;
-            if (t < cnt && col + my_col < dv)
-                o[(size_t)(tok0 + t) * p.H * dv + (size_t)h * dv + col + my_col] = read / (fmaxf(fabsf(size), cf[24 + my_tok]) + READ_EPS);
         }
     }
-#pragma unroll
-    for (int m = 0; m < RPT; m++) {
-        const int n = (m / 4) * 64 + kp * 4 + m % 4;
-        if (n >= d) continue;
-        if (vec_state && col < dv) {
-            *reinterpret_cast<float4*>(S + (size_t)n * dv + col) = make_float4(sreg[m][0], sreg[m][1], sreg[m][2], sreg[m][3]);
-        } else {
-#pragma unroll
-            for (int c = 0; c < 4; c++)
-                if (col + c < dv) S[(size_t)n * dv + col + c] = sreg[m][c];
-        }
-        if (cg == 0) N[n] = nreg[m];
+    if (PHASE == 1) {
+        store(planes + (size_t)seg * sg.pitch);
+        if (tid == 0 && blockIdx.x == 0) sg.products[((size_t)s * sg.segs + seg) * p.H + h] = product;
+    } else if (last_seg) {
+        store(state);
     }
 }
 
@@ -421,7 +487,7 @@ bool aligned16(const void* p) { return (uintptr_t)p % 16 == 0; }
 
 // How a slot's state is laid out, in floats: S [heads][d][dv] | n [copies][heads][d] | m [heads]; the size in all.
 MOE_API long long moe_mlstm_state_floats(int H, int d, int dv) {
-    return (long long)H * d * (dv + (dv + MCOLS - 1) / MCOLS) + H;
+    return (long long)H * d * (dv + (dv + COPY_COLS - 1) / COPY_COLS) + H;
 }
 
 static int mlstm_bad(const float* proj, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at, const float* i_bias,
@@ -435,45 +501,67 @@ static int mlstm_bad(const float* proj, long long ld, int q_at, int k_at, int v_
 }
 
 // proj: [T, ld] 32-bit with the columns of q (H * d), k (H * d), v (H * dv) and the gates' logits (H each) from the places
-// given; i_bias, f_bias: [H]; state: moe_mlstm_state_floats floats a slot from the pointer given; steps: [T, 3 H] scratch,
-// filled here; o: [T, H * dv] 32-bit (rows of no sequence are left alone).
+// given; i_bias, f_bias: [H]; state: moe_mlstm_state_floats floats a slot from the pointer given; longest: the most tokens a
+// sequence brings (0: unknown); segs, seg_len, ends, pitch, products: MemSegments; steps: [T, 3 H] scratch, filled here; o: [T, H * dv] 32-bit (rows of no sequence are left alone).
 MOE_API int moe_mlstm_scan(const float* proj, long long ld, int q_at, int k_at, int v_at, int i_at, int f_at,
                            const float* i_bias, const float* f_bias, float cap, float q_scale, float* state,
                            long long state_pitch, const int* cu_seqlens, const int* slots, int num_seqs, int H, int d,
-                           int dv, float* steps, float* o, cudaStream_t stream) {
+                           int dv, float* steps, float* o, int longest, int segs,
+                           int seg_len, float* ends, long long pitch, float* products, cudaStream_t stream) {
     if (num_seqs <= 0) return 0;
     if (!steps || !o || num_seqs > 65535 ||
         mlstm_bad(proj, ld, q_at, k_at, v_at, i_at, f_at, i_bias, f_bias, state, state_pitch, cu_seqlens, slots, H, d, dv, cap))
         return (int)cudaErrorInvalidValue;
-    const int copies = (dv + MCOLS - 1) / MCOLS;
+    if (segs < 1 || (segs > 1 && (!ends || !products || seg_len <= 0 || seg_len % MRUN || pitch < moe_mlstm_state_floats(H, d, dv) - H ||
+                                  pitch % 4 || (long long)num_seqs * segs > 65535)))
+        return (int)cudaErrorInvalidValue;
+    const int copies = (dv + COPY_COLS - 1) / COPY_COLS;
     const MemSeq p{proj, ld, q_at, k_at, v_at, i_at, f_at, i_bias, f_bias, state, state_pitch, cu_seqlens, slots, steps,
                    H, d, dv, cap, q_scale, copies};
-    int code = launch_pdl(mlstm_gates_kernel, dim3((H + GATE_WARPS - 1) / GATE_WARPS, num_seqs), dim3(GATE_WARPS * 32), 0, stream, p);
+    const int threads = longest > 0 && longest < 1024 ? (longest + 31) / 32 * 32 : 1024;
+    int code = launch_pdl(mlstm_gates_kernel, dim3(H, num_seqs), dim3(threads), 0, stream, p);
     if (code) return code;
-    const dim3 grid(copies, H, num_seqs);
+    // few blocks: the narrow form puts twice as many on the SMs
+    const bool narrow = d > 64 && (long long)((dv + mcols(16) - 1) / mcols(16)) * H * num_seqs * segs * 2 <= scan_sms();
+    const int cols = mcols(narrow ? 32 : 16);
+    const dim3 grid((dv + cols - 1) / cols, H, num_seqs * segs);
+    const MemSegments sg{segs, seg_len, ends, pitch, products};
     const bool vec = d % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && q_at % 4 == 0 && k_at % 4 == 0 && v_at % 4 == 0 && aligned16(proj);
     // (an ordinary launch: blocks placed while the kernel before still holds some SMs would be several to an SM beside
     // empty ones, and a scan is as slow as its most crowded SM)
-#define SCAN_V(RPT_, V_)                                                                                               \
+#define SCAN_P(RPT_, KP_, V_, PH_)                                                                                     \
     do {                                                                                                               \
-        constexpr size_t smem = mlstm_scan_floats<RPT_>() * sizeof(float);                                             \
+        const size_t smem = scan_smem(mlstm_scan_floats<RPT_, KP_>() * sizeof(float), (long long)grid.x * grid.y * grid.z); \
         if (smem > 48 * 1024) {                                                                                        \
-            cudaError_t e = cudaFuncSetAttribute(mlstm_scan_kernel<RPT_, V_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(mlstm_scan_kernel<RPT_, KP_, V_, PH_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e;                                                                       \
         }                                                                                                              \
-        mlstm_scan_kernel<RPT_, V_><<<grid, MTHREADS, smem, stream>>>(p, o);                                           \
-        return launch_status();                                                                                        \
+        mlstm_scan_kernel<RPT_, KP_, V_, PH_><<<grid, MTHREADS, smem, stream>>>(p, o, sg);                             \
+        if (PH_ != 1) return launch_status();                                                                          \
     } while (0)
-#define SCAN(RPT_)                                                                                                     \
+#define SCAN_V(RPT_, KP_, V_)                                                                                          \
     do {                                                                                                               \
-        if (vec) SCAN_V(RPT_, true);                                                                                   \
-        SCAN_V(RPT_, false);                                                                                           \
+        if (segs > 1) {                                                                                                \
+            SCAN_P(RPT_, KP_, V_, 1);                                                                                  \
+            SCAN_P(RPT_, KP_, V_, 2);                                                                                  \
+        }                                                                                                              \
+        SCAN_P(RPT_, KP_, V_, 0);                                                                                      \
     } while (0)
-    if (d <= 64) SCAN(4);
-    if (d <= 128) SCAN(8);
-    SCAN(16);
+#define SCAN(RPT_, KP_)                                                                                                \
+    do {                                                                                                               \
+        if (vec) SCAN_V(RPT_, KP_, true);                                                                              \
+        SCAN_V(RPT_, KP_, false);                                                                                      \
+    } while (0)
+    if (d <= 64) SCAN(4, 16);
+    if (narrow) {
+        if (d <= 128) SCAN(4, 32);
+        SCAN(8, 32);
+    }
+    if (d <= 128) SCAN(8, 16);
+    SCAN(16, 16);
 #undef SCAN
 #undef SCAN_V
+#undef SCAN_P
 }
 
 // One token a sequence: gates, recurrence, head norm (norm_w [H * dv]) and gate (gate: [T, H * dv] 32-bit logits, rows of
@@ -493,7 +581,7 @@ MOE_API int moe_mlstm_step(const float* proj, long long ld, int q_at, int k_at, 
     const size_t smem = ((size_t)2 * ((d + 3) & ~3) + dv + (size_t)kp * dv) * sizeof(float);
     if (units > 32 || smem > 48 * 1024) return -1;
     const MemSeq p{proj, ld, q_at, k_at, v_at, i_at, f_at, i_bias, f_bias, state, state_pitch, cu_seqlens, slots, nullptr,
-                   H, d, dv, cap, q_scale, (dv + MCOLS - 1) / MCOLS};
+                   H, d, dv, cap, q_scale, (dv + COPY_COLS - 1) / COPY_COLS};
 #define STEP(OT_, U_)                                                                                                  \
     return launch_pdl(mlstm_step_kernel<OT_, U_>, dim3(H, num_seqs), dim3(256), smem, stream, p, gate, ldg, norm_w, norm_eps, \
                       seq_of_token, num_tokens, gate_fn, (OT_*)out)

@@ -588,6 +588,13 @@ struct NormRouteParams {
     int vec_ok;
     int cluster;              // 1: the tokens' blocks are one cluster (at most 8 tokens), see the kernel
     int groups, keep;         // experts picked within the best `keep` of `groups` groups (0: no groups)
+    // A norm on what is pending instead of a norm in front of the router (post_w not null; norm_w is then not read):
+    // x += rms(delta sa + delta_b sb) post_w, and the router reads the stream itself.
+    const float* delta_b;     // or null
+    float sa, sb;
+    const float* post_w;
+    float post_eps;
+    int weight_input;         // the gathered rows are multiplied by their pick's weight
 };
 
 template <typename WT>
@@ -606,7 +613,7 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
              off += (size_t)p.num_tokens * blockDim.x * line)
             prefetch_l2((const char*)p.wr + off);
         for (size_t off = threadIdx.x * line; off < (size_t)H * sizeof(float); off += blockDim.x * line)
-            prefetch_l2((const char*)p.norm_w + off);
+            prefetch_l2((const char*)(p.post_w ? p.post_w : p.norm_w) + off);
         if (p.wsg)
             for (size_t off = threadIdx.x * line; off < (size_t)H * sizeof(WT); off += blockDim.x * line)
                 prefetch_l2((const char*)p.wsg + off);
@@ -625,22 +632,39 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
     float* xr = p.x + (size_t)t * H;
     const float* dr = p.delta ? p.delta + (size_t)t * H : nullptr;
     float ss = 0.f;
-    for (int j = threadIdx.x; j < H; j += blockDim.x) {
-        float v = xr[j];
-        if (dr) {
-            v += dr[j];
-            xr[j] = v;
+    if (p.post_w) {
+        const float* br = p.delta_b ? p.delta_b + (size_t)t * H : nullptr;
+        for (int j = threadIdx.x; j < H; j += blockDim.x) {
+            float y = p.sa * dr[j];
+            if (br) y = fmaf(p.sb, br[j], y);
+            row[j] = y;
+            ss = fmaf(y, y, ss);
         }
-        row[j] = v;
-        ss += v * v;
-    }
-    ss = block_sum(ss, red);
-    const float rs = 1.0f / sqrtf(ss / (float)H + p.eps);
-    for (int j = threadIdx.x; j < H; j += blockDim.x) {
-        const float y = row[j] * rs * p.norm_w[j];
-        row[j] = y;
-        if (p.out32) p.out32[(size_t)t * H + j] = y;
-        if (p.out16) p.out16[(size_t)t * H + j] = __float2bfloat16_rn(y);
+        ss = block_sum(ss, red);
+        const float rs = 1.0f / sqrtf(ss / (float)H + p.post_eps);
+        for (int j = threadIdx.x; j < H; j += blockDim.x) {
+            const float v = fmaf(row[j] * rs, p.post_w[j], xr[j]);
+            xr[j] = v;
+            row[j] = v;
+        }
+    } else {
+        for (int j = threadIdx.x; j < H; j += blockDim.x) {
+            float v = xr[j];
+            if (dr) {
+                v += dr[j];
+                xr[j] = v;
+            }
+            row[j] = v;
+            ss += v * v;
+        }
+        ss = block_sum(ss, red);
+        const float rs = 1.0f / sqrtf(ss / (float)H + p.eps);
+        for (int j = threadIdx.x; j < H; j += blockDim.x) {
+            const float y = row[j] * rs * p.norm_w[j];
+            row[j] = y;
+            if (p.out32) p.out32[(size_t)t * H + j] = y;
+            if (p.out16) p.out16[(size_t)t * H + j] = __float2bfloat16_rn(y);
+        }
     }
     __syncthreads();
 
@@ -748,8 +772,9 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
                 const int q = sorted[t * p.top_k + j];
                 if (q < 0) continue;
                 __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.xs) + (size_t)q * H;
+                const float f = p.weight_input ? p.topk_w[(size_t)t * p.top_k + j] : 1.0f;
                 for (int c = threadIdx.x * 2; c < H; c += blockDim.x * 2)
-                    *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(row[c], row[c + 1]);
+                    *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(f * row[c], f * row[c + 1]);
             }
         }
         cl_sync();      // no block leaves while another may still read its picks
@@ -833,16 +858,19 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
 MOE_API void moe_set_norm_route_cluster(int enabled) { g_norm_route_cluster = enabled ? 1 : 0; }
 
 // The norm before a routed feed-forward, the router and the dispatch of a step of few tokens, one
-// launch (see norm_route_kernel).  Returns -1, with nothing launched, for sizes it does not take
+// launch (see norm_route_kernel).  With post_w: the norm of what is pending, delta sa + delta_b sb, in front of its sum
+// with the stream, which the router then reads as it is (up to 8 tokens); weight_input: see NormRouteParams.  Returns -1, with nothing launched, for sizes it does not take
 // (more than 64 tokens, 256 experts or 4096 (token, expert) pairs, or a row too long for shared
 // memory): the caller then runs the separate kernels.
 MOE_API int moe_norm_route(float* x, const float* delta, const float* norm_w, float eps, int hidden, int num_tokens,
                            float* out32, void* out16, const void* wr, const void* wsg, int w_dt, int num_experts,
                            int top_k, int norm_topk, float scale, const int* seq_of_token, int* topk_idx,
                            float* topk_w, float* shared_gate, int* offsets, int* sorted_token, int* pos_of_pair,
-                           void* xs, int* ticket, int* status, int groups, int keep, cudaStream_t stream) {
+                           void* xs, int* ticket, int* status, int groups, int keep, const float* delta_b, float sa,
+                           float sb, const float* post_w, float post_eps, int weight_input, cudaStream_t stream) {
     if (num_tokens <= 0) return 0;
-    if (top_k <= 0 || top_k > num_experts || hidden <= 0 || !ticket || (wsg && !shared_gate) || (xs && !out16))
+    if (top_k <= 0 || top_k > num_experts || hidden <= 0 || !ticket || (wsg && !shared_gate) || (xs && !out16 && !post_w) ||
+        (post_w ? !delta : !norm_w) || ((delta_b || weight_input) && !post_w))
         return (int)cudaErrorInvalidValue;
     if (groups > 1 && (num_experts % groups || keep < 1 || keep > groups || top_k > keep * (num_experts / groups)))
         return (int)cudaErrorInvalidValue;
@@ -856,6 +884,7 @@ MOE_API int moe_norm_route(float* x, const float* delta, const float* norm_w, fl
     p.offsets = offsets, p.sorted_token = sorted_token, p.pos_of_pair = pos_of_pair;
     p.xs = (uint4*)xs, p.row_units = hidden * 2 / 16, p.ticket = ticket, p.status = status;
     p.groups = groups, p.keep = keep;
+    p.delta_b = delta_b, p.sa = sa, p.sb = sb, p.post_w = post_w, p.post_eps = post_eps, p.weight_input = weight_input;
     if (xs && ((hidden * 2) % 16 || (uintptr_t)xs % 16 || (uintptr_t)out16 % 16)) return -1;
     const size_t elt = w_dt == DT_F32 ? 4 : 2;
     p.vec_ok = (hidden % 8 == 0) && ((uintptr_t)wr % 16 == 0) && (!wsg || (uintptr_t)wsg % 16 == 0) &&
@@ -870,6 +899,7 @@ MOE_API int moe_norm_route(float* x, const float* delta, const float* norm_w, fl
     }
     // up to 8 tokens: one cluster, no ticket, no second reading of what other blocks wrote
     p.cluster = (num_tokens <= 8 && top_k <= 64 && hidden % 2 == 0 && g_norm_route_cluster) ? 1 : 0;
+    if (post_w && !p.cluster) return -1;                     // (the ticket form gathers normed rows only)
     if (p.cluster) return launch_pdl_cluster(kernel, dim3(1, 1, num_tokens), 1024, smem, stream, num_tokens, p);
     return launch_pdl(kernel, num_tokens, 1024, smem, stream, p);
 }

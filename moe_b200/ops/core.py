@@ -69,7 +69,7 @@ def lib():
             "moe_wkv_finish": [P, P, LL, P, F, P, I, I, I, I, P, I, P],
             "moe_rmsnorm_scaled": [P, P, P, P, P, P, P, P, P, I, I, I, F, I, P, P, P, P, I, P, P, P, P],
             "moe_attention_decode_fused": [P, P, I, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, I, F, I, P, I, I, P, P],
-            "moe_norm_route": [P, P, P, F, I, I, P, P, P, P, I, I, I, I, F, P, P, P, P, P, P, P, P, P, P, I, I, P],
+            "moe_norm_route": [P, P, P, F, I, I, P, P, P, P, I, I, I, I, F, P, P, P, P, P, P, P, P, P, P, I, I, P, F, F, P, F, I, P],
             "moe_align": [P, I, I, I, P, P, P, P, P],
             "moe_swiglu": [P, P, I, LL, I, I, F, P],
             "moe_combine": [P, P, P, I, P, P, P, I, I, P],
@@ -92,7 +92,7 @@ def lib():
             "moe_delta_prepare": [P, LL, I, I, P, I, P, LL, P, P, P, P, P, I, I, I, I, I, F, F, I, P, P, P, LL, P, P],
             "moe_delta_step": [P, P, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P, I, P],
             "moe_delta_scan": [P, P, P, LL, P, P, I, I, I, I, I, P, P, P],
-            "moe_mlstm_scan": [P, LL, I, I, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, P, P, P],
+            "moe_mlstm_scan": [P, LL, I, I, I, I, I, P, P, F, F, P, LL, P, P, I, I, I, I, P, P, I, I, I, P, LL, P, P],
             "moe_mlstm_step": [P, LL, I, I, I, I, I, P, P, F, F, P, LL, P, LL, P, F, P, P, P, I, I, I, I, I, I, P, I, P],
             "moe_post_norm": [P, P, F, P, F, P, P, P, I, P, P, F, P, F, P, P, P, I, I, I, I, P, P],
             "moe_weighted_rows": [P, P, P, I, I, I, I, P, I, P, P],
@@ -379,7 +379,7 @@ def heads_prepare(proj, pos, seq_of_token, *, nh, nkv, d, dv, width, q, k, v, q_
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("heads_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, sl, tb = view.k, view.v, batch.seq_end, batch.slots, g.table
-        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
+        ts, ring, ps, npg, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_heads_prepare(_p(proj), proj.stride(0), _p(pos), _p(seq_of_token), _p(q_norm), _p(k_norm), float(eps),
                                 _p(freq) if rot else None, int(rot), float(mscale), T, nh, nkv, d, dv, width, _p(q),
                                 _p(k), _p(v), q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(sl), _p(tb), ts, ring, ps, npg, pin,
@@ -553,7 +553,7 @@ def conv_heads_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, taps_w=No
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("conv_heads_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, tb = commit.k, commit.v, batch.seq_end, g.table
-        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
+        ts, ring, ps, npg, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_conv_heads_prepare(_p(proj), proj.stride(0), _p(taps_w), taps, _p(state),
                                      state.stride(0) if state is not None else 0, _p(batch.pos), _p(batch.seq_of_token),
                                      _p(batch.cu_seqlens), _p(batch.slots), float(eps), 1 if unit_norm else 0,
@@ -1154,19 +1154,31 @@ def rope_commit(qkv, pos, inv_freq, nh, nkv, hd, rot, q, view, batch, status):
 
 
 def norm_route(x, delta, norm_w, eps, w_router, top_k, norm_topk, scale, *, bf16, shared_gate_w=None,
-               seq_of_token=None, status=None, groups=0, keep=0, score="softmax"):
+               seq_of_token=None, status=None, groups=0, keep=0, score="softmax", post=None, sa=1.0, delta_b=None, sb=1.0,
+               weight_input=False):
     """Few tokens: ``x += delta``, RMS norm, router logits, pick, table inversion and gather of the
     normalised bfloat16 rows in ONE launch.  Returns None (nothing launched) for sizes the kernel
     does not take, else (out32 or None, out16 or None, topk_idx, topk_w, shared_gate, offsets,
-    sorted_token, pos_of_pair, gathered or None)."""
-    _chk(x, "x", torch.float32, 2), _chk(norm_w, "norm weight", torch.float32, 1), _chk(w_router, "router weight", dims=2)
+    sorted_token, pos_of_pair, gathered or None).
+
+    With ``post`` = (weight, eps) (``norm_w`` None; up to 8 tokens) what is pending passes an RMS norm of its own before the
+    sum, x += rms(delta sa + delta_b sb) weight, and the router reads the stream itself (out32 and out16 are None);
+    ``weight_input``: the gathered rows are the stream's times their pick's weight."""
+    _chk(x, "x", torch.float32, 2), _chk(w_router, "router weight", dims=2)
     T, H = x.shape
     E = w_router.shape[0]
-    if T > 64 or E > 256 or T * top_k > 4096 or norm_w.numel() != H or w_router.shape[1] != H:
+    nw = norm_w if post is None else post[0]
+    _chk(nw, "norm weight", torch.float32, 1)
+    for t in (delta, delta_b):
+        if t is not None:
+            _chk(t, "delta", torch.float32, 2)
+            if t.shape != x.shape:
+                raise KernelError("norm_route: the delta's shape")
+    if T > 64 or E > 256 or T * top_k > 4096 or nw.numel() != H or w_router.shape[1] != H or (post is not None and T > 8):
         return None
     dev = x.device
-    out16 = torch.empty((T, H), dtype=torch.bfloat16, device=dev) if bf16 else None
-    out32 = None if bf16 else torch.empty((T, H), dtype=torch.float32, device=dev)
+    out16 = torch.empty((T, H), dtype=torch.bfloat16, device=dev) if bf16 and post is None else None
+    out32 = None if bf16 or post is not None else torch.empty((T, H), dtype=torch.float32, device=dev)
     P_ = T * top_k
     topk_idx = torch.empty((T, top_k), dtype=torch.int32, device=dev)
     topk_w = torch.empty((T, top_k), dtype=torch.float32, device=dev)
@@ -1179,7 +1191,8 @@ def norm_route(x, delta, norm_w, eps, w_router, top_k, norm_topk, scale, *, bf16
     code = lib().moe_norm_route(_p(x), _p(delta), _p(norm_w), float(eps), H, T, _p(out32), _p(out16), _p(w_router),
                                 _p(shared_gate_w), _dt(w_router), E, top_k, _route_flags(norm_topk, score), float(scale),
                                 _p(seq_of_token), _p(topk_idx), _p(topk_w), _p(sg), _p(offsets), _p(sorted_token),
-                                _p(pos_of_pair), _p(xs), _p(ticket), _p(status), int(groups), int(keep), _stream())
+                                _p(pos_of_pair), _p(xs), _p(ticket), _p(status), int(groups), int(keep), _p(delta_b), float(sa), float(sb),
+                                _p(post[0]) if post else None, float(post[1]) if post else 0.0, 1 if weight_input else 0, _stream())
     if code == -1:
         return None
     _ok(code, "norm_route")
@@ -1257,7 +1270,7 @@ def whole_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, q_norm=None, k
         if k.dtype != g.dtype or g.num_kv_heads != nkv or g.head_dim != width:
             raise KernelError("whole_prepare: the cache layer differs from the keys in dtype or shape")
         kc, vc, se, sl, tb = commit.k, commit.v, batch.seq_end, batch.slots, g.table
-        ts, ring, ps, npg, pin, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
+        ts, ring, ps, npg, pin = g.table.stride(0), g.ring, g.page_size, g.num_pages, g.pinned
     _ok(lib().moe_whole_prepare(_p(proj), proj.stride(0), _p(batch.pos), _p(batch.seq_of_token), _p(q_norm), _p(k_norm),
                                 float(eps), _p(freq) if rot else None, int(rot), _p(vfreq), T, nh, nkv, d, dv, width,
                                 _p(q), _p(k), _p(v), q.stride(0), k.stride(0), _dt(q), _p(kc), _p(vc), _p(se), _p(sl),
@@ -1431,7 +1444,7 @@ def table_route(table, batch, top_k, num_experts, topk_idx, topk_w, status):
 
 
 def scan_segments(batch, blocks_per_sequence: int, device) -> int:
-    """Into how many segments a sequence's tokens are cut for ``ssd_scan`` and ``wkv_scan``: one where the launch fills
+    """Into how many segments a sequence's tokens are cut for ``ssd_scan``, ``wkv_scan`` and ``mlstm_scan``: one where the launch fills
     the GPU anyway or the sequences are short; else enough to fill it, of at least 128 tokens each, eight
     at most.  (``MOE_B200_SCAN_SEGMENTS``: 0 this rule, n > 0 that many.)"""
     forced = int(os.environ.get("MOE_B200_SCAN_SEGMENTS", "0"))
@@ -1571,9 +1584,9 @@ def delta_scan(qkv, step, state, batch, o, *, heads, kv_heads, d, dv, offset=0, 
 
 
 def mlstm_state_floats(heads, d, dv) -> int:
-    """Floats of a sequence's state (csrc/mlstm.cu): the memory, its normaliser (once for every 32 columns of the
+    """Floats of a sequence's state (csrc/mlstm.cu): the memory, its normaliser (once for every 16 columns of the
     memory) and the running maximum of every head."""
-    return heads * d * (dv + -(-dv // 32)) + heads
+    return heads * d * (dv + -(-dv // 16)) + heads
 
 
 def _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, heads, d, dv):
@@ -1587,18 +1600,31 @@ def _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, he
             float(q_scale), st, state.stride(0))
 
 
-def mlstm_scan(proj, at, i_bias, f_bias, cap, q_scale, state, batch, o, *, heads, d, dv, offset=0):
+def mlstm_scan(proj, at, i_bias, f_bias, cap, q_scale, state, batch, o, *, heads, d, dv, offset=0, segments=None):
     """Several tokens a sequence of the exponentially gated memory (csrc/mlstm.cu) on 32-bit projection rows whose columns
     of q, k, v and of the gates' logits i and f start at ``at``; queries are multiplied by ``q_scale``; ``state`` rows hold
-    ``mlstm_state_floats`` floats from ``offset``; o: float32 [T, heads * dv]."""
+    ``mlstm_state_floats`` floats from ``offset``; o: float32 [T, heads * dv].  ``segments``: into how many pieces that run
+    side by side every sequence's tokens are cut (None: ``scan_segments`` decides)."""
     _chk(o, "o", torch.float32, 2)
     T = proj.shape[0]
     if tuple(o.shape) != (T, heads * dv):
         raise KernelError("mlstm_scan: shapes")
     args = _mlstm_args(proj, at, i_bias, f_bias, cap, q_scale, state, offset, batch, heads, d, dv)
     steps = torch.empty((T, 3 * heads), dtype=torch.float32, device=o.device)
+    longest = int(getattr(batch, "max_new", 0) or 0)
+    if segments is None:
+        segs = scan_segments(batch, heads * -(-dv // 32), o.device)
+        segs = 1 if segs == 2 else segs        # (two halves, the first one run twice, take as long as one whole)
+    else:
+        segs = int(segments)
+    seg_len, pitch, ends, products = 0, 0, None, None
+    if segs > 1:
+        seg_len = -(-(-(-(longest or T) // segs)) // 16) * 16
+        pitch = -(-mlstm_state_floats(heads, d, dv) // 4) * 4
+        ends = torch.empty((batch.num_seqs, segs, pitch), dtype=torch.float32, device=o.device)
+        products = torch.empty((batch.num_seqs, segs, heads), dtype=torch.float32, device=o.device)
     _ok(lib().moe_mlstm_scan(*args, _p(batch.cu_seqlens), _p(batch.slots), batch.num_seqs, heads, d, dv, _p(steps), _p(o),
-                             _stream()), "mlstm_scan")
+                             longest, segs, seg_len, _p(ends), pitch, _p(products), _stream()), "mlstm_scan")
 
 
 def mlstm_step(proj, at, i_bias, f_bias, cap, q_scale, state, gate, norm_w, norm_eps, batch, out, *, heads, d, dv, offset=0,

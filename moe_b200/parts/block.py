@@ -95,6 +95,12 @@ class SandwichBlock:
         pending = PostNormDelta(run(rt, h, batch, cache_view, state), self.post1)
         if self.ffn is None:
             return x, pending
+        prenorm = getattr(self.ffn, "forward_prenorm", None)
+        if prenorm is not None and self.norm2.kind == "none" and self.post2.kind == "rmsnorm":
+            # few tokens: the feed-forward may take post-norm and sum along with its own first kernel
+            out = prenorm(rt, x, pending, self.norm2, batch)
+            if out is not None:
+                return x, PostNormDelta(out, self.post2)
         run = getattr(self.ffn, "forward_lazy", self.ffn.forward) if self.post2.kind == "rmsnorm" else self.ffn.forward
         kw = {"want16": getattr(self.ffn, "wants16", True)} if self.norm2.kind == "none" else {}
         h = self.norm2.forward(rt, x, delta=delta_for(self.norm2, pending, rt),

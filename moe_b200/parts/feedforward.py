@@ -371,8 +371,21 @@ class RoutedExperts(Part):
         """The block's offer to take the norm before this feed-forward along: for a step of few
         tokens, norm, router and dispatch are one launch.  None if the sizes or the kind of norm do
         not allow it (the block then runs the norm itself and calls ``forward``)."""
+        if x.shape[0] > self.fused_norm_tokens or self.E > 256 or self.b_router is not None or self.table:
+            return None
+        if norm.kind == "none" and self.weight_input and isinstance(delta, LazyDelta) and delta.kind == "post_rmsnorm":
+            # what is pending has a norm of its own and this feed-forward reads the stream itself
+            t, kw = delta.tensor, {}
+            if isinstance(t, LazyDelta) and t.kind == "scaled_sum":
+                t, kw = t.a, dict(sa=t.sa, delta_b=t.b, sb=t.sb)
+            if isinstance(t, LazyDelta):
+                return None
+            routed = core.norm_route(x, t, None, 0.0, self.w_router, self.k, self.norm_topk, self.scale, bf16=rt.is_bf16,
+                                     seq_of_token=getattr(batch, "seq_of_token", None), status=rt.status,
+                                     post=delta.norm.rms_params(), weight_input=True, **kw, **self._grp)
+            return None if routed is None else self._run(rt, Activations(act=x, f32=x), batch, routed[2:])
         rms = getattr(norm, "rms_params", None)          # the norm says whether it can be run by a neighbour
-        if rms is None or x.shape[0] > self.fused_norm_tokens or self.E > 256 or self.b_router is not None or self.table or self.weight_input:
+        if rms is None or self.weight_input:
             return None
         norm_w, norm_eps = rms()
         routed = core.norm_route(x, delta, norm_w, norm_eps, self.w_router, self.k, self.norm_topk, self.scale,

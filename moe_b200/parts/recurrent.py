@@ -335,14 +335,14 @@ class DeltaMixer(Part):
 
     gate_fn = "silu"
 
-    def _gates(self, rt, h, proj):
-        """(the output gate's logits, the channels' decay logits or None)"""
-        return proj[:, self.gate_at:self.gate_at + self.inner], None
+    def _project(self, rt, h):
+        """(float32 [T, q | k | v | ...], the output gate's logits, the channels' decay logits or None)"""
+        proj = linear(rt, h.act, self.w_in)                       # [q | k | v | gate | b | a]
+        return proj, proj[:, self.gate_at:self.gate_at + self.inner], None
 
     def forward(self, rt, h, batch, cache_view, state):
         T, C, I = batch.num_tokens, self.channels, self.inner
-        proj = linear(rt, h.act, self.w_in)                       # float32 [T, q | k | v | gate | b | a]
-        gate, a_rows = self._gates(rt, h, proj)
+        proj, gate, a_rows = self._project(rt, h)
         decay = torch.empty((T, self.nh * self.d), dtype=torch.float32, device=proj.device) if a_rows is not None else None
         sizes = dict(heads=self.nh, kv_heads=self.nkv, d=self.d, dv=self.dv)
         qkv = torch.empty((T, C), dtype=torch.float32, device=proj.device)
@@ -379,6 +379,7 @@ class ChannelDeltaMixer(DeltaMixer):
 
     def __init__(self, spec):
         super().__init__(spec)
+        self.beside = os.environ.get("MOE_B200_NARROW_BESIDE", "1") != "0"
         self.ranks = self.params.get("ranks")          # (decay's, gate's); None: read from the tensors' shapes when bound
 
     def _tensors(self, ra, rg):
@@ -433,11 +434,26 @@ class ChannelDeltaMixer(DeltaMixer):
         self.norm_w = tensors[n["norm"]].to(torch.float32).repeat(self.nh).contiguous()
         self.wo = tensors[n["o"]].contiguous()
 
-    def _gates(self, rt, h, proj):
+    def _low(self, rt, h):
         low = linear(rt, h.act, self.w_low1, out_dtype=rt.compute_dtype)
-        both = linear(rt, low, self.w_low2)                       # float32 [T, decays' logits | gate's logits]
+        return linear(rt, low, self.w_low2)                       # float32 [T, decays' logits | gate's logits]
+
+    def _project(self, rt, h):
+        """The two narrow products run on a side stream beside the wide one (inside a captured step: a fork and a join);
+        MOE_B200_NARROW_BESIDE=0 runs them after it."""
+        if self.beside and h.act.is_cuda:
+            main = torch.cuda.current_stream()
+            side = rt.side_stream(3)
+            side.wait_stream(main)
+            with torch.cuda.stream(side):
+                both = self._low(rt, h)
+            proj = linear(rt, h.act, self.w_in)                   # float32 [T, q | k | v | b]
+            main.wait_stream(side)
+            both.record_stream(main)
+        else:
+            proj, both = linear(rt, h.act, self.w_in), self._low(rt, h)
         hd = self.nh * self.d
-        return both[:, hd:], both[:, :hd]
+        return proj, both[:, hd:], both[:, :hd]
 
 
 class MLSTMMixer(Part):

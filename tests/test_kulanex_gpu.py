@@ -504,13 +504,42 @@ def test_exponentially_gated_memory_over_steps(H, d, dv, cap, gain):
         ref = plain.unit_rms(o, eps).reshape(n, -1) * norm_w.double() * torch.sigmoid(gates[s].double())
         close(torch.cat(outs[s]), ref, 1e-3)
         have = state[s + 1, off:].double().cpu()
-        copies = -(-dv // 32)
+        copies = -(-dv // 16)
         m = have[H * d * (dv + copies):H * d * (dv + copies) + H]
         close(m, mu, 1e-5)
         close(have[:H * d * dv].view(H, d, dv) * torch.exp(m - mu)[:, None, None], S, 1e-4)
         for c in range(copies):
             close(have[H * d * (dv + c):H * d * (dv + c + 1)].view(H, d) * torch.exp(m - mu)[:, None], z, 1e-4)
     assert float(state[0].abs().max()) == 0.0 and float(state[3].abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("segments", [2, 3, 8])
+@pytest.mark.parametrize("H,d,dv", [(4, 16, 24), (2, 96, 64), (3, 10, 7), (1, 200, 40)])
+def test_memory_in_segments_that_run_side_by_side(H, d, dv, segments):
+    """Three sequences of unequal lengths (one so short that it lies in the first segment) that go on from a state, cut into
+    segments: outputs and state as in one go."""
+    from moe_b200.ops import core
+
+    g = torch.Generator().manual_seed(H * 7 + d)
+    width = -(-(H * (dv + 2 * d + 2)) // 4) * 4
+    at = {"q": 0, "k": H * d, "v": 2 * H * d, "i": H * (2 * d + dv), "f": H * (2 * d + dv + 1)}
+    counts = [403, 9, 260]
+    proj = torch.randn(sum(counts), width, generator=g)
+    proj[:, at["i"]:at["i"] + 2 * H] *= 4.0
+    size = -(-core.mlstm_state_floats(H, d, dv) // 4) * 4
+    ib, fb = torch.randn(H, generator=g), torch.randn(H, generator=g) + 1.0
+    batch = G.make_batch(DEV, [1, 2, 3], [0, 0, 0], counts)
+    res = []
+    for n in (1, segments):
+        state = torch.zeros((5, size), device=DEV)
+        for _ in range(2):                                   # (the second time from what the first left)
+            o = torch.empty((sum(counts), H * dv), device=DEV)
+            core.mlstm_scan(dev(proj), at, dev(ib), dev(fb), 6.0, d ** -0.5, state, batch, o, heads=H, d=d, dv=dv, segments=n)
+        res.append((o.double().cpu(), state.double().cpu()))
+    scale = float(res[0][0].abs().max())
+    assert float((res[0][0] - res[1][0]).abs().max()) < 2e-4 * scale
+    assert float((res[0][1] - res[1][1]).abs().max()) < 2e-4 * float(res[0][1].abs().max())
+    assert float(res[1][1][0].abs().max()) == float(res[1][1][4].abs().max()) == 0.0
 
 
 def test_a_strong_input_is_remembered_and_a_weak_one_after_it_is_not():
@@ -567,6 +596,48 @@ def test_sigmoid_scores_multiply_what_the_experts_read(T, W, E, top, ff, dtype):
     assert torch.equal(idx.long().cpu().sort(-1).values, picks.sort(-1).values)
     close(weight, torch.gather(score, 1, idx.long().cpu()), 1e-5)
     close(got, plain.experts_ff(w64, "f", {"router": {"experts": E, "top": top}}, x.double()), 2e-2 if dtype == "bfloat16" else 1e-5)
+
+
+@pytest.mark.parametrize("T", [1, 3, 8])
+@pytest.mark.parametrize("W,E,top", [(64, 5, 2), (48, 3, 3), (2048, 16, 2), (136, 1, 1), (4096, 40, 8)])
+@pytest.mark.parametrize("two", [False, True])
+def test_few_tokens_norm_sum_router_and_weighted_rows_in_one_launch(T, W, E, top, two):
+    """x += rms(y) w, scores, picks, the experts' order and the rows they read, against the plain formulas; a row of no
+    sequence gets no expert."""
+    from moe_b200.ops import core
+
+    g = torch.Generator().manual_seed(W + T)
+    x, a, b = (torch.randn(T, W, generator=g) for _ in range(3))
+    pw, eps = 0.5 * (1 + 0.3 * torch.randn(W, generator=g)), 1e-5
+    wr = (2 * torch.randn(E, W, generator=g) / math.sqrt(W)).to(torch.bfloat16)
+    seq = torch.zeros(T, dtype=torch.int32)
+    if T > 1:
+        seq[1] = -1
+    xs_, st = dev(x), core.new_status(DEV)
+    kw = dict(sa=0.7, delta_b=dev(b), sb=-0.4) if two else {}
+    got = core.norm_route(xs_, dev(a), None, 0.0, wr.to(DEV), top, False, 1.0, bf16=True, seq_of_token=seq.to(DEV), status=st,
+                          score="sigmoid", post=(dev(pw), eps), weight_input=True, **kw)
+    core.check_status(st)
+    o32, o16, idx, wt, _, offsets, sorted_token, place, rows = got
+    assert o32 is None and o16 is None
+    y = 0.7 * a.double() - 0.4 * b.double() if two else a.double()
+    new = x.double() + plain.unit_rms(y, eps) * pw.double()
+    close(xs_, new, 5e-6)
+    score = torch.sigmoid(new @ wr.double().T)
+    live = [t for t in range(T) if seq[t] >= 0]
+    idx, wt, place, rows = idx.long().cpu(), wt.double().cpu(), place.view(T, top).cpu(), rows.double().cpu()
+    for t in range(T):
+        if t not in live:
+            assert idx[t].tolist() == [-1] * top and place[t].tolist() == [-1] * top
+            continue
+        best = torch.topk(score[t], top).indices
+        assert sorted(idx[t].tolist()) == sorted(best.tolist())
+        close(wt[t], score[t, idx[t]], 1e-5)
+        for j in range(top):
+            p = int(place[t, j])
+            assert int(offsets[idx[t, j]]) <= p < int(offsets[idx[t, j] + 1]) and int(sorted_token[p]) == t
+            close(rows[p], score[t, idx[t, j]] * new[t], 1e-2)
+    assert int(offsets[E]) == len(live) * top
 
 
 def test_scores_of_large_logits_stay_finite():
