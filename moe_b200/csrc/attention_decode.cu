@@ -143,8 +143,9 @@ __device__ __forceinline__ void rotated_chunk(const float* __restrict__ src, int
     }
 }
 
-// LPR: lanes per key row (row bytes / 16); GH: query heads handled together.
-template <typename T, int LPR, int GH, bool FUSED>
+// LPR: lanes per key row (row bytes / 16); GH: query heads handled together; KEEP: AttnVariant::keep may be set (a form of
+// its own, so that the others carry nothing of it).
+template <typename T, int LPR, int GH, bool FUSED, bool KEEP>
 __global__ void __launch_bounds__(WARPS * 32, (GH == 1 && LPR <= 16) ? 4 : 1)
 attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                         float* __restrict__ partial, const int* __restrict__ seq_of_token,
@@ -185,7 +186,8 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
     // tiles of 32 positions, aligned to 32: the keys of a tile are contiguous in one page
     // (kept first positions: their tiles come first, then those of the window; attn_seen turns a tile's number
     // in that order into its place)
-    const int tile_lo = lo / 32, kept_tiles = min((av.keep + 31) / 32, tile_lo), pinned = attn_pinned(av);
+    const int keep = KEEP ? av.keep : 0;
+    const int tile_lo = lo / 32, kept_tiles = min((keep + 31) / 32, tile_lo), pinned = KEEP ? attn_pinned(av) : 0;
     const int n_tiles = kept_tiles + p / 32 + 1 - tile_lo;
     const int tps = (n_tiles + nsplit - 1) / nsplit;
     const int tb = split * tps, te = min(n_tiles, tb + tps);
@@ -251,7 +253,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
             for (int i = 0; i < NI; i++) raw[i] = *reinterpret_cast<const uint4*>(kt + (size_t)i * RPI * HD);
             const int my_row = sub * RPI + rgrp;          // the row whose score this lane ends up with
             const int my_j = j0 + my_row;
-            const bool valid = (my_j >= lo || my_j < av.keep) && my_j <= hi;
+            const bool valid = (my_j >= lo || (KEEP && my_j < keep)) && my_j <= hi;
             float sc[GH];
 #pragma unroll
             for (int g = 0; g < GH; g++) {
@@ -301,7 +303,7 @@ attn_decode_fast_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, 
                     // rows out of sight may hold anything: they are skipped, not multiplied by zero
                     const int j = j0 + i * RPI + rgrp;
                     const float pi = __shfl_sync(0xffffffffu, pr, lane - sub + i);   // holder of row (i, rgrp)
-                    if ((j >= lo || j < av.keep) && j <= hi) {
+                    if ((j >= lo || (KEEP && j < keep)) && j <= hi) {
                         float vc[EPC];
                         Chunk<T>::unpack(raw[i], vc);
 #pragma unroll
@@ -901,11 +903,15 @@ int launch(const void* q, const void* k_cache, const void* v_cache, void* out, f
         grid.y = (unsigned)(nkv * ((group + GH - 1) / GH));                                                       \
         if (grid.y > 65535) return (int)cudaErrorInvalidValue;                                                    \
         if (fused)                                                                                                \
-            rc = launch_pdl(attn_decode_fast_kernel<T, LPR, GH, true>, grid, WARPS * 32, 0, stream, (const T*)q,  \
+            rc = launch_pdl(attn_decode_fast_kernel<T, LPR, GH, true, false>, grid, WARPS * 32, 0, stream, (const T*)q,  \
+                            (const T*)k_cache, (const T*)v_cache, partial, seq_of_token, pos, slots, tables,      \
+                            table_stride, ring, page_size, num_pages, nh, nkv, window, scale, status, fa, budget, av); \
+        else if (av.keep > 0)                                                                                     \
+            rc = launch_pdl(attn_decode_fast_kernel<T, LPR, GH, false, true>, grid, WARPS * 32, 0, stream, (const T*)q, \
                             (const T*)k_cache, (const T*)v_cache, partial, seq_of_token, pos, slots, tables,      \
                             table_stride, ring, page_size, num_pages, nh, nkv, window, scale, status, fa, budget, av); \
         else                                                                                                      \
-            rc = launch_pdl(attn_decode_fast_kernel<T, LPR, GH, false>, grid, WARPS * 32, 0, stream, (const T*)q, \
+            rc = launch_pdl(attn_decode_fast_kernel<T, LPR, GH, false, false>, grid, WARPS * 32, 0, stream, (const T*)q, \
                             (const T*)k_cache, (const T*)v_cache, partial, seq_of_token, pos, slots, tables,      \
                             table_stride, ring, page_size, num_pages, nh, nkv, window, scale, status, fa, budget, av); \
     } while (0)

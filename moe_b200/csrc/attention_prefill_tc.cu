@@ -201,7 +201,8 @@ struct PackedOut {
     int ld;
 };
 
-template <int HD, bool SHARED>
+// KEEP: AttnVariant::keep may be set (a form of its own: in every tile's mask its comparison costs the others a tenth).
+template <int HD, bool SHARED, bool KEEP>
 __global__ void __launch_bounds__(320, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmKc,
@@ -256,12 +257,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     // Kept first positions (AttnVariant::keep) that lie in front of the window: `kc` tiles of the cache and `kl` of
     // the step's own tokens.  The tiles' order: kept cached, cached, kept own, own; a kept tile is never one
     // of the window's.
-    const int kc = min((min(av.keep, start) + KT - 1) / KT, nc > 0 ? kt_lo : INT_MAX);
-    const int kl = min((max(0, av.keep - start) + KT - 1) / KT, t_lo);
+    const int keep = KEEP ? av.keep : 0;
+    const int kc = KEEP ? min((min(keep, start) + KT - 1) / KT, nc > 0 ? kt_lo : INT_MAX) : 0;
+    const int kl = KEEP ? min((max(0, keep - start) + KT - 1) / KT, t_lo) : 0;
     const int n_cached = kc + nc;
     const int n_tiles = n_cached + kl + q_last / KT - t_lo + 1;
     // where tile `it` starts: a multiple of KT, an absolute position for a cached tile, a token of the step else
     auto tile_at = [&](int it) {
+        if (!KEEP) return (it < n_cached ? kt_lo + it : t_lo + it - n_cached) * KT;
         return it < n_cached ? (it < kc ? it : kt_lo + it - kc) * KT : (it - n_cached < kl ? it - n_cached : t_lo + it - n_cached - kl) * KT;
     };
 
@@ -315,7 +318,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             bool ok = true;
             int nk = 0, nv = 0;                         // tiles whose keys / values have been requested
             const int* table = n_cached > 0 ? tables + (size_t)slots[seq] * table_stride : nullptr;
-            const int pinned = attn_pinned(av);
+            const int pinned = KEEP ? attn_pinned(av) : 0;
             int page_row[2][2];                         // of a cache tile's two pages: first row in the cache seen
                                                         // as rows of one head's keys, [page][kv head][64] of them
             auto find_pages = [&](int it) {
@@ -325,7 +328,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                     if (page < 0 || page >= num_pages) {
                         // only a page that holds a key some row needs is an error; the half of a tile
                         // beyond the sequence's cached tokens just has to be finite, and every page is
-                        if (a < start && (a + 63 >= lo_pos || a < av.keep)) atomicOr(status, ST_BAD_PAGE);
+                        if (a < start && (a + 63 >= lo_pos || (KEEP && a < keep))) atomicOr(status, ST_BAD_PAGE);
                         page = 0;
                     }
                     page_row[it & 1][h] = (page * nkv + kvh) * 64;
@@ -468,10 +471,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             // a tile strictly below the diagonal, inside the window and inside the sequence needs no mask
             const bool full = j0 + KT - 1 <= start + q0 && j0 + KT <= jmax &&
                               (av.chunk > 0 ? j0 >= attn_lo(start + q0 + QT - 1, 0, av.chunk)
-                                            : (window <= 0 || j0 >= start + q0 + QT - window || j0 + KT <= av.keep));
+                                            : (window <= 0 || j0 >= start + q0 + QT - window || (KEEP && j0 + KT <= keep)));
             auto tile_softmax = [&](auto masked_tag) -> bool {
                 constexpr bool MASKED = decltype(masked_tag)::value;
-                auto visible = [&](int j) { return j <= prow && j < jmax && (j >= lo_row || j < av.keep); };
+                auto visible = [&](int j) { return j <= prow && j < jmax && (j >= lo_row || (KEEP && j < keep)); };
                 float m_new = m, alpha = 1.f;
                 if (!sigmoid_w) {
                 // pass 1: the maximum of the half row (of the raw scores: the scale is positive)
@@ -676,22 +679,27 @@ struct CacheArgs {
     int table_stride, ring, num_pages;
 };
 
-template <int HD, bool SHARED>
-int launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CacheArgs& c, void* out,
+template <int HD, bool SHARED, bool KEEP>
+int launch_form(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CacheArgs& c, void* out,
            const int* cu_seqlens, int num_seqs, int num_tokens, int nh, int nkv, int window, float scale, int* status,
            const AttnVariant av, const PackedOut po, cudaStream_t stream) {
     constexpr int TILE_BYTES = (HD / 64) * 128 * 128;
     const int smem = (SHARED ? (HD <= 128 ? 4 : 3) : 5) * TILE_BYTES + 1024 + 192;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, SHARED, KEEP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(((num_tokens + QT - 1) / QT + num_seqs) * nh);
-    return launch_pdl(attn_prefill_tc_kernel<HD, SHARED>, grid, 320, (size_t)smem, stream, tmQ, tmK, tmV, c.tmK, c.tmV,
+    return launch_pdl(attn_prefill_tc_kernel<HD, SHARED, KEEP>, grid, 320, (size_t)smem, stream, tmQ, tmK, tmV, c.tmK, c.tmV,
                       (__nv_bfloat16*)out, cu_seqlens, c.seq_start, c.slots, c.tables, c.table_stride, c.ring,
                       c.num_pages, num_seqs, nh, nkv, window, scale * 1.4426950408889634f, status, av, po);
+}
+
+template <int HD, bool SHARED, typename... Args>
+int launch(const AttnVariant& av, Args&... args) {
+    return av.keep > 0 ? launch_form<HD, SHARED, true>(args...) : launch_form<HD, SHARED, false>(args...);
 }
 
 int run(const void* q, const void* k, const void* v, CacheArgs& c, void* out, const int* cu_seqlens, int num_seqs,
@@ -703,7 +711,7 @@ int run(const void* q, const void* k, const void* v, CacheArgs& c, void* out, co
         return -1;
     if (!c.seq_start) c.tmK = tmK, c.tmV = tmV;         // never used: no tile comes from the cache
 #define RUN(HD_, S_)                                                                                                   \
-    return launch<HD_, S_>(tmQ, tmK, tmV, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, window, scale, status, av, po, stream)
+    return launch<HD_, S_>(av, tmQ, tmK, tmV, c, out, cu_seqlens, num_seqs, num_tokens, nh, nkv, window, scale, status, av, po, stream)
     if (shared) {
         if (hd == 64) RUN(64, true);
         if (hd == 128) RUN(128, true);

@@ -597,7 +597,8 @@ struct NormRouteParams {
     int weight_input;         // the gathered rows are multiplied by their pick's weight
 };
 
-template <typename WT>
+// POST: post_w and what goes with it (a form of its own, so that the other carries nothing of it).
+template <typename WT, bool POST>
 __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams p) {
     extern __shared__ __align__(16) float nr_smem[];
     __shared__ float red[32];
@@ -613,7 +614,7 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
              off += (size_t)p.num_tokens * blockDim.x * line)
             prefetch_l2((const char*)p.wr + off);
         for (size_t off = threadIdx.x * line; off < (size_t)H * sizeof(float); off += blockDim.x * line)
-            prefetch_l2((const char*)(p.post_w ? p.post_w : p.norm_w) + off);
+            prefetch_l2((const char*)(POST ? p.post_w : p.norm_w) + off);
         if (p.wsg)
             for (size_t off = threadIdx.x * line; off < (size_t)H * sizeof(WT); off += blockDim.x * line)
                 prefetch_l2((const char*)p.wsg + off);
@@ -632,7 +633,7 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
     float* xr = p.x + (size_t)t * H;
     const float* dr = p.delta ? p.delta + (size_t)t * H : nullptr;
     float ss = 0.f;
-    if (p.post_w) {
+    if (POST) {
         const float* br = p.delta_b ? p.delta_b + (size_t)t * H : nullptr;
         for (int j = threadIdx.x; j < H; j += blockDim.x) {
             float y = p.sa * dr[j];
@@ -772,7 +773,7 @@ __global__ void __launch_bounds__(1024) norm_route_kernel(const NormRouteParams 
                 const int q = sorted[t * p.top_k + j];
                 if (q < 0) continue;
                 __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.xs) + (size_t)q * H;
-                const float f = p.weight_input ? p.topk_w[(size_t)t * p.top_k + j] : 1.0f;
+                const float f = (POST && p.weight_input) ? p.topk_w[(size_t)t * p.top_k + j] : 1.0f;
                 for (int c = threadIdx.x * 2; c < H; c += blockDim.x * 2)
                     *reinterpret_cast<__nv_bfloat162*>(dst + c) = __floats2bfloat162_rn(f * row[c], f * row[c + 1]);
             }
@@ -892,7 +893,8 @@ MOE_API int moe_norm_route(float* x, const float* delta, const float* norm_w, fl
     const size_t smem = ((size_t)((hidden + 3) & ~3) + p.rows + num_experts + top_k) * sizeof(float) +
                         ((size_t)2 * pairs + 2 * num_experts) * sizeof(int);
     if (smem > 200 * 1024) return -1;
-    auto kernel = w_dt == DT_F32 ? norm_route_kernel<float> : norm_route_kernel<__nv_bfloat16>;
+    auto kernel = post_w ? (w_dt == DT_F32 ? norm_route_kernel<float, true> : norm_route_kernel<__nv_bfloat16, true>)
+                         : (w_dt == DT_F32 ? norm_route_kernel<float, false> : norm_route_kernel<__nv_bfloat16, false>);
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
