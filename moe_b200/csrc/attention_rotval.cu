@@ -17,7 +17,7 @@
 //                   sequence's state, the last taps - 1 projected rows, and are zero before position 0), then the
 //                   norms over the whole of q and of k, then the rotation, of pairs (2i, 2i + 1) or (i, i + rot/2).
 //                   Values have rows of their own in the projection and pass the convolution too, or ARE the
-//                   keys as they leave the convolution, before norm and rotation.  In a step of one token a
+//                   convolved keys, neither normed nor turned.  In a step of one token a
 //                   sequence the same launch moves the convolution's state on.
 // Convolution, norm, angles and rotations are 32-bit; only the stores round to the activation dtype.
 #include "common.cuh"

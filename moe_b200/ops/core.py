@@ -1284,7 +1284,7 @@ def whole_conv_prepare(proj, batch, *, nh, nkv, d, dv, width, q, k, v, taps_w=No
     sequence, which come from the step or from ``state`` ([slots + 1, >= (taps - 1) * channels]); then the norms over the
     whole of q and of k, the rotation of the first ``rot`` dimensions of every query and key head (``neighbours``: of
     pairs (2i, 2i + 1)), the split and optionally the append to the cache layer ``commit``.  ``values_are_keys``: the values
-    are the keys as they leave the convolution, and the projection has no rows for them.  Returns True if it has also
+    are the convolved keys, and the projection has no rows for them.  Returns True if it has also
     moved the convolution's state on (a step of one token a sequence); else the caller runs ``conv_state_update``."""
     _chk(proj, "proj", torch.float32, 2)
     T = proj.shape[0]

@@ -50,7 +50,7 @@ A third prepared path, whose kernel ``whole_prepare`` stands in the same place, 
               (tensor role ``head_bias``), and the weights are not normalised over the keys.
 
 With the norm over the whole projection (``qk_norm`` ``whole``), the convolution, a rotation of pairs (2i, 2i + 1) and
-  values_are_keys  the value of a position is its key as it leaves the convolution, before norm and rotation;
+  values_are_keys  a position's value is its convolved key, neither normed nor turned;
               there is no value projection
 go together; the kernel is then ``whole_conv_prepare``.
 

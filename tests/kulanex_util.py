@@ -69,10 +69,10 @@ CONFIGS = {
         layer(parallel(8, 1, 16, 3, 8, scaling=None, size=130, keep=2, scale=1.2, rheads=2, rdim=8, rvdim=8, ls=1.0, rs=0.2), 0)]),
     # records of 64 and 128 on the tensor-core kernels, eight heads on a record, states of 64 x 128 and 32 x 64, a
     # wider model with more experts
-    "wide": dict(vocab=203, width=128, eps=1e-5, mult=0.5, ranks=(16, 24), layers=[
+    "wide": dict(vocab=203, width=128, eps=1e-5, mult=0.45, ranks=(16, 24), layers=[
         layer(delta(4, 4, 64, 128, 4), 12, 2, 64),
-        layer(parallel(8, 8, 64, 4, 32, size=150, keep=9, rheads=4, rdim=32, rvdim=64), 8, 1, 64),
-        layer(parallel(8, 1, 96, 4, 48, base=1e6, scaling=(4.0, 1.0, 4.0, 256), size=40, keep=130, rheads=2, rdim=64, rvdim=32), 8, 4, 32)]),
+        layer(parallel(8, 8, 64, 4, 32, size=150, keep=9, rheads=4, rdim=32, rvdim=64), 9, 1, 72),
+        layer(parallel(8, 1, 80, 5, 40, base=2e5, scaling=(3.0, 1.0, 5.0, 256), size=44, keep=130, rheads=2, rdim=64, rvdim=32), 10, 4, 32)]),
     # heads of more than 128 numbers on both sides, a delta state of 200 x 72
     "large": dict(vocab=90, width=96, eps=1e-5, mult=0.5, ranks=(20, 12), layers=[
         layer(parallel(2, 1, 160, 3, 64, size=100, keep=4, rheads=2, rdim=136, rvdim=40), 3, 1, 64),

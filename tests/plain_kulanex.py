@@ -117,7 +117,7 @@ def seen_mask(T, size, keep_first):
 
 
 def window_attention(w, p, m, x, eps):
-    """Queries and keys pass a short convolution; the values are the keys as they leave it; then queries and
+    """Queries and keys pass a short convolution; the values are those convolved keys; then queries and
     keys are normed over the whole projection and turned by their positions."""
     T = x.shape[0]
     H, G, d = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])

@@ -175,7 +175,7 @@ def test_norm_of_a_sublayer_s_output_in_front_of_the_sum(W, source, then):
 def test_convolution_whole_norm_rotation_and_records_over_steps(bf16, nh, nkv, d, taps, rot, neighbours, shared):
     """Two sequences of unequal lengths over steps that bring fewer rows than the convolution has taps, the last two of one
     token each (in which the kernel moves the state on itself): records of queries, keys and values, and the state.
-    ``shared``: the values are the keys as they leave the convolution."""
+    ``shared``: the values are the convolved keys, neither normed nor turned."""
     from moe_b200.cache import KVCache, KVRequest
     from moe_b200.ops import core
     from moe_b200.parts.attention import record_width
